@@ -2,6 +2,7 @@
 
     serve | engine | status | stop     the launcher (serving/launch.py): one engine rank per GPU + the HTTP front end
     front                              the OpenAI-compatible front end alone (serving/openai_server.py)
+    replay                             replay a trace of token ids step by step (serving/session.py; also bin/trace_run)
     build                              compile the CUDA kernels and the C++ runtime in-tree
     bench-gemm | bench-decode | bench-prefill | bench-mx | bench-fused | bench-http | profile-round
                                        kernel and serving microbenchmarks
@@ -19,6 +20,7 @@ import runpy
 import sys
 
 MODULES = {
+    "replay": "spark_engine_b200.serving.session",
     "front": "spark_engine_b200.serving.openai_server",
     "build": "spark_engine_b200.build",
     "bench-gemm": "spark_engine_b200.ops.bench_gemm",

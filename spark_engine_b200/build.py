@@ -1,6 +1,7 @@
 """In-tree build of the native libraries (no JIT cache: the built .so files travel with the source tree).
 
   libspark_kernels.so : every .cu under csrc/kernels, compiled for sm_100a only
+  libspark_kernels_<family>.so : the part of it one model family needs (`kernel_library`)
   _runtime*.so        : C++ host runtime (KV pool, scheduler core, prefix-cache I/O, ...) as a pybind11 module
 
 Usage: `python -m spark_engine_b200.build [--force]`.
@@ -36,10 +37,27 @@ def _run(cmd):
     return r.stdout + r.stderr
 
 
-def build_kernels(force=False, verbose=False) -> str:
+# kernel sources of families that need only part of the library
+FAMILY_SOURCES = {"vabunex": ("block_rows", "elementwise", "gemm", "gemm_simt", "gemv", "latent", "linear_state", "mla")}
+
+
+def kernel_library(family: str) -> str:
+    """Path of a kernel library that serves `family`, built if need be: the complete one when it is up to date, else one of
+    the family's own sources (a first start compiles no more than the model needs; the objects are shared)."""
+    build_runtime()
+    full = os.path.join(LIBDIR, "libspark_kernels.so")
+    srcs = glob.glob(os.path.join(CSRC, "kernels", "*.cu*")) + glob.glob(os.path.join(CSRC, "common", "*.cuh"))
+    if not _newer(srcs, full) or family not in FAMILY_SOURCES:
+        return full if not _newer(srcs, full) else build_kernels()
+    return build_kernels(family=family)
+
+
+def build_kernels(force=False, verbose=False, family=None) -> str:
     os.makedirs(LIBDIR, exist_ok=True)
-    out = os.path.join(LIBDIR, "libspark_kernels.so")
+    out = os.path.join(LIBDIR, "libspark_kernels.so" if family is None else f"libspark_kernels_{family}.so")
     cus = sorted(glob.glob(os.path.join(CSRC, "kernels", "*.cu")))
+    if family is not None:
+        cus = [c for c in cus if os.path.basename(c)[:-3] in FAMILY_SOURCES[family]]
     headers = glob.glob(os.path.join(CSRC, "**", "*.cuh"), recursive=True) + glob.glob(os.path.join(CSRC, "**", "*.h"), recursive=True)
     objs, jobs = [], []
     for cu in cus:
@@ -51,7 +69,7 @@ def build_kernels(force=False, verbose=False) -> str:
         for log in ex.map(_run, jobs):
             if verbose and log:
                 print(log)
-    if jobs or not os.path.exists(out):
+    if jobs or _newer(objs, out):
         _run([NVCC, "-shared", "-o", out] + objs + ["-lcudart"])
     return out
 

@@ -66,9 +66,17 @@ class KvBacking:
 
 
 class KvManager:
+    """Leases of the model's KV rows: contiguous regions, or page lists for models whose caches are paged."""
+
     def __init__(self, model, granule: int = 256):
         self.model = model
-        self.pool = rt().KvPool(model.kv_tokens, granule)
+        self.paged = getattr(model, "page", 0) > 0
+        if self.paged:
+            self.pool = rt().PagePool(model.kv_tokens, model.page)
+            for s in range(model.n_slots):                # nothing is leased yet
+                model.set_pages(s, [])
+        else:
+            self.pool = rt().KvPool(model.kv_tokens, granule)
         self.lease: Dict[int, int] = {}           # slot -> lease id
         self.backing = getattr(model, "kv_backing", None)
 
@@ -97,13 +105,15 @@ class KvManager:
             self.pool.release(v)
             if owner is not None:
                 del self.lease[owner]
+                if self.paged:
+                    self.model.set_pages(owner, [])
                 self.model.reset_slot(owner)
             lid = self.pool.acquire(tokens)
         l = self.pool.get(lid)
         self.lease[slot] = lid
         self.pool.pin(lid, True)
         self._back()                                  # the rows exist before anything may address them
-        self.model.set_kv_region(slot, l.base, l.cap)
+        self._publish(slot, l)
         return True
 
     def grow(self, slot: int, tokens: int) -> bool:
@@ -112,8 +122,14 @@ class KvManager:
             return False
         l = self.pool.get(lid)
         self._back()
-        self.model.set_kv_region(slot, l.base, l.cap)
+        self._publish(slot, l)
         return True
+
+    def _publish(self, slot: int, l):
+        if self.paged:
+            self.model.set_pages(slot, l.pages)
+        else:
+            self.model.set_kv_region(slot, l.base, l.cap)
 
     def idle(self, slot: int):
         """The sequence finished: keep its rows for prefix reuse but allow eviction."""
@@ -126,6 +142,8 @@ class KvManager:
         lid = self.lease.pop(slot, None)
         if lid is not None:
             self.pool.release(lid)
+            if self.paged:
+                self.model.set_pages(slot, [])
             self._back()
 
     def stats(self) -> dict:

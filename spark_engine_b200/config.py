@@ -84,9 +84,59 @@ class MoeConfig:
 
 
 @dataclass
+class LightningConfig:
+    """Linear attention with one constant decay per head (no softmax, no delta rule)."""
+    n_heads: int = 2
+    head_dim: int = 32
+    v_dim: int = 32
+    decay: List[float] = field(default_factory=lambda: [0.9, 0.99])
+
+
+@dataclass
+class WkvConfig:
+    """Token-shifted recurrence with a learned decay per token and key channel and a bonus for the current token."""
+    n_heads: int = 2
+    head_dim: int = 32
+    decay_rank: int = 16
+
+
+@dataclass
+class LatentConfig:
+    """Dense causal attention over cached latents, low-rank queries, one shared rotated key part, per-head output gate."""
+    n_heads: int = 2
+    head_dim: int = 32            # unrotated query / key dimensions per head
+    v_dim: int = 32
+    q_rank: int = 64
+    kv_rank: int = 48
+    rope_dim: int = 16
+    rope_theta: float = 1e4
+    rope_interleaved: bool = True
+    scale: float = 0.125
+
+
+MIXER_CONFIGS = {"lightning": LightningConfig, "wkv": WkvConfig, "latent": LatentConfig}
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a model whose layers carry their own sizes."""
+    kind: str = "lightning"       # key of MIXER_CONFIGS
+    mixer: object = None
+    ffn: int = 0                  # width of the dense feed-forward (0 = none)
+
+
+@dataclass
+class LoopConfig:
+    """Layers start .. stop-1 run `times` times in a row with the same weights, every pass with its own cache / state."""
+    start: int = 0
+    stop: int = 0
+    times: int = 1
+
+
+@dataclass
 class ModelConfig:
     name: str = "tiny-hybrid"
-    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4
+    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex
     n_layers: int = 4
     layer_types: List[str] = field(default_factory=lambda: ["gdn", "gdn", "gdn", "attn"])
     hidden: int = 256
@@ -112,6 +162,18 @@ class ModelConfig:
     kv_dtype: str = "bf16"        # bf16 | fp8
     kv_quant_on_cpu: bool = False  # the CPU runner keeps fp32 caches; set to model the packed FP8 latent rows there too
 
+    layer_specs: List[LayerSpec] = field(default_factory=list)   # per-layer sizes (vabunex); else the shared configs above
+    loop: Optional[LoopConfig] = None
+    norm_one_plus: bool = False   # norm weights are stored around zero
+    embed_scale: float = 1.0
+
+    def layer_runs(self) -> List[int]:
+        """Weight layer of every layer run, in order."""
+        lp = self.loop
+        if lp is None:
+            return list(range(self.n_layers))
+        return [*range(lp.start), *(list(range(lp.start, lp.stop)) * lp.times), *range(lp.stop, self.n_layers)]
+
     def to_json(self) -> str:
         return json.dumps(dataclasses.asdict(self), indent=1)
 
@@ -122,12 +184,20 @@ class ModelConfig:
                          ("mla", MlaConfig), ("moe", MoeConfig)):
             if key in d and isinstance(d[key], dict):
                 d[key] = cls(**d[key])
+        if isinstance(d.get("loop"), dict):
+            d["loop"] = LoopConfig(**d["loop"])
+        d["layer_specs"] = [x if isinstance(x, LayerSpec) else
+                            LayerSpec(x["kind"], MIXER_CONFIGS[x["kind"]](**x["mixer"]), x["ffn"]) for x in d.get("layer_specs", [])]
         return ModelConfig(**d)
 
     @staticmethod
     def from_json(path: str) -> "ModelConfig":
         with open(path) as f:
-            return ModelConfig.from_dict(json.load(f))
+            d = json.load(f)
+        if "architecture" in d:                 # a checkpoint's own configuration: the registry reads it
+            from .models.registry import architecture
+            return architecture(d).read_config(d)
+        return ModelConfig.from_dict(d)
 
 
 def _pattern(n_layers: int, period: int, a: str, b: str) -> List[str]:
@@ -183,6 +253,22 @@ def ds4_style(n_layers: int = 40, weight_format: str = "mx") -> ModelConfig:
         weight_format=weight_format, kv_dtype="fp8")
 
 
+def vabunex_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 5632, vocab: int = 65536) -> ModelConfig:
+    """Vabunex at the layer sizes of a small real model: one latent-attention, two lightning and one wkv layer per period,
+    the first period run twice."""
+    kinds = [("latent", "lightning", "lightning", "wkv")[i % 4] for i in range(n_layers)]
+    heads = hidden // 128
+    mixers = {"latent": LatentConfig(n_heads=heads, head_dim=128, v_dim=128, q_rank=768, kv_rank=512, rope_dim=64,
+                                     rope_theta=5e4, scale=192 ** -0.5),
+              "lightning": LightningConfig(n_heads=heads, head_dim=128, v_dim=128,
+                                           decay=[1.0 - 2.0 ** (-1 - 8 * h / heads) for h in range(heads)]),
+              "wkv": WkvConfig(n_heads=hidden // 64, head_dim=64, decay_rank=64)}
+    return ModelConfig(name="vabunex-style", family="vabunex", n_layers=n_layers, layer_types=kinds, hidden=hidden, vocab=vocab,
+                       norm_eps=1e-5, layer_specs=[LayerSpec(k, dataclasses.replace(mixers[k]), ffn) for k in kinds],
+                       loop=LoopConfig(0, min(4, n_layers), 2), norm_one_plus=True, embed_scale=float(hidden) ** 0.5,
+                       weight_format="dense")
+
+
 def scaled_down(cfg: ModelConfig, hidden: int = 256, n_layers: int = 4, vocab: int = 1024) -> ModelConfig:
     """Same layer types, small dimensions: the CPU test shape of a large config."""
     c = dataclasses.replace(cfg)
@@ -224,6 +310,7 @@ class EngineConfig:
     """Engine switches (CLI `--flag`, JSON file, `SPARK_<NAME>` environment fallback)."""
     model: str = "tiny-hybrid"
     numerics: str = "deterministic"      # deterministic | fast (multimem hardware reductions)
+    dtype: str = "bfloat16"              # activations and dense weights on the device: bfloat16 | float32 (vabunex only)
     tp: int = 1
     ep: int = 1
     max_seqs: int = 8
@@ -270,7 +357,7 @@ class EngineConfig:
     def signature(self) -> str:
         """Flag signature: captured graphs are keyed on it so a changed switch forces a
         re-capture (reference: spec_probe.rs:316-327)."""
-        keys = ("numerics", "tp", "ep", "comm", "spec", "spec_depth", "cuda_graphs")
+        keys = ("numerics", "dtype", "tp", "ep", "comm", "spec", "spec_depth", "cuda_graphs")
         return "|".join(f"{k}={getattr(self, k)}" for k in keys)
 
 
@@ -279,6 +366,7 @@ PRESETS = {
     "qwen3next-style": qwen3next_style,
     "glm-style": glm_style,
     "ds4-style": ds4_style,
+    "vabunex-style": vabunex_style,
 }
 
 

@@ -12,13 +12,23 @@
 // FP8 cache rows (lat_fp8): [kv_lora e4m3 | 4 fp32 tile scales (tiles of kv_lora / max(1, kv_lora / 128)) | rope bf16],
 // 656 bytes instead of 1152 for 512 + 64; the decode kernel copies the packed row into the tail of its bf16 tile row and
 // a warp expands it in place.
-// The visible tokens of a row come from the top-k pool selection (sparse_select.cu) or are 0..pos.
+// The visible tokens of a row come from the top-k pool selection (sparse_select.cu) or are 0..pos.  Cache rows are a
+// contiguous region per sequence (row_kv), or 64-token pages of a shared pool (MlaPages; a split is one page).  SPLITP
+// carries the softmax weights as two-term bf16 sums into the second product (fp32 weights to 2^-17).
 // Reference: engine-rs/shim/latent.cu (sparse_latent*, latent_tc16*, merge_latent), ds41_attn.cu:90-424,
 // engine-rs/src/mla_latent.rs:36-38,196-248, dsa.rs:127-230; FP8 rows: latent.cu:25-47.
 #include <cuda_fp8.h>
 #include "../common/ptx.cuh"
 
 namespace spark {
+
+constexpr int MLA_PAGE = 64;        // tokens per page of a paged latent cache
+struct MlaPages {
+  const int* table;                 // [slots][ld] page ids (nullptr: contiguous regions)
+  int ld;
+  const int* row_slot;              // [plan rows]
+  const int* rows;                  // optional: plan row of each query row of this launch
+};
 
 struct MlaDims {
   int q_lora, kv_lora, rope, idx_dim, idx_heads, pool;
@@ -175,7 +185,7 @@ __device__ __forceinline__ void mla_mma(float (&c)[4], const uint32_t (&a)[4], u
 
 // grid (R, ceil(nsplit / spc)); 256 threads; a CTA walks `spc` consecutive splits.  HM = 16-head MMA tiles (H <= 16*HM).  KW = kv_lora + rope (multiple of 16),
 // L = kv_lora (multiple of 16).
-template <int HM>
+template <int HM, bool SPLITP>
 __global__ void __launch_bounds__(256)
 mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
                   const __nv_bfloat16* __restrict__ lat,         // [tokens, KW]
@@ -184,7 +194,7 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
                   float* __restrict__ part_ml,                   // [R, H, nsplit, 2]
                   int H, int KW, int L, float scale, int nsplit, int spc,
                   const int* __restrict__ row_pos0, const int* __restrict__ row_j, const int* __restrict__ anc,
-                  int lat_fp8) {
+                  int lat_fp8, MlaPages pg) {
   extern __shared__ __align__(16) uint8_t smem_mla[];
   const int LDK = KW + 8;
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_mla);          // [HM*16][LDK]
@@ -192,15 +202,18 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
   float* Ss = reinterpret_cast<float*>(Ls + MLA_TS * LDK);                  // [HM*16][65]
   __nv_bfloat16* Ps = reinterpret_cast<__nv_bfloat16*>(Ss + HM * 16 * 65);  // [HM*16][72]
   __shared__ int stok[MLA_TS];
-  const int r = blockIdx.x;
+  __nv_bfloat16* Pl = Ps + HM * 16 * 72;                                    // SPLITP: low parts of the weights
+  const int r = blockIdx.x;                                                // query row of this launch
+  const int pr = pg.rows ? pg.rows[r] : r;                                 // its row of the plan
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   // tree rows (anc given, no selection): the committed context [0, first in-flight slot) plus the in-flight slots
   // of the row's ancestors and its own, bit j of anc[r] = node j of the sequence is visible
   const bool tree = anc != nullptr;
   const int tp0 = tree ? row_pos0[r] : 0;
   const unsigned amask = tree ? static_cast<unsigned>(anc[r]) : 0u;
-  const int n_ctx = sel ? sel_n[r] : (tree ? tp0 + row_j[r] + 1 : pos[r] + 1);
-  const long long base = row_kv[r];
+  const int n_ctx = sel ? sel_n[r] : (tree ? tp0 + row_j[r] + 1 : pos[pr] + 1);
+  long long base = pg.table ? 0 : row_kv[r];
+  const int* pages = pg.table ? pg.table + static_cast<size_t>(pg.row_slot[pr]) * pg.ld : nullptr;
   const int VPR = KW >> 3;
   // the row's queries (all heads) are staged once and serve every split this CTA walks through
   for (int i = tid; i < HM * 16 * VPR; i += 256) {
@@ -219,6 +232,7 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
     continue;
   }
   const int nt = min(MLA_TS, n_ctx - t0);
+  if (pages != nullptr) base = static_cast<long long>(max(pages[t0 / MLA_PAGE], 0)) * MLA_PAGE - t0;     // a split is one page
   __syncthreads();                                             // the previous split's tiles are no longer read
   if (tid < MLA_TS) stok[tid] = tid < nt ? (sel ? sel[static_cast<size_t>(r) * sel_ld + t0 + tid] : t0 + tid) : -1;
   __syncthreads();
@@ -319,6 +333,10 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
     const float l = warp_sum(e0 + e1);
     Ps[h * 72 + lane] = __float2bfloat16(e0);
     Ps[h * 72 + lane + 32] = __float2bfloat16(e1);
+    if (SPLITP) {
+      Pl[h * 72 + lane] = __float2bfloat16(e0 - __bfloat162float(__float2bfloat16(e0)));
+      Pl[h * 72 + lane + 32] = __float2bfloat16(e1 - __bfloat162float(__float2bfloat16(e1)));
+    }
     if (lane == 0 && h < H) {
       part_ml[(pb + static_cast<size_t>(h) * nsplit) * 2] = m;
       part_ml[(pb + static_cast<size_t>(h) * nsplit) * 2 + 1] = l;
@@ -342,6 +360,11 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
         mla_ldsm4(a, Ps + (m * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * 72 + kk * 16 + (lane >> 4) * 8);
         mla_mma(o[m][0], a, b[0], b[1]);
         mla_mma(o[m][1], a, b[2], b[3]);
+        if (SPLITP) {
+          mla_ldsm4(a, Pl + (m * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * 72 + kk * 16 + (lane >> 4) * 8);
+          mla_mma(o[m][0], a, b[0], b[1]);
+          mla_mma(o[m][1], a, b[2], b[3]);
+        }
       }
     }
 #pragma unroll
@@ -367,7 +390,9 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
 // round of a few rows still fills the SMs (one head per CTA), while a prefill chunk keeps one CTA per row.
 __global__ void __launch_bounds__(256)
 mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int nsplit, const float* __restrict__ sink,
-                 int H, int L, int hpc, __nv_bfloat16* __restrict__ out) {
+                 int H, int L, int hpc, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gate, int ldg,
+                 const int* __restrict__ rows) {
+  // gate (optional): one logit per head in the row's gate columns, the head's output is scaled by its sigmoid
   extern __shared__ float wts[];                        // [hpc][nsplit]: exp(m_s - M) / l
   const int r = blockIdx.x, h0 = blockIdx.y * hpc;
   const int nh = min(hpc, H - h0);
@@ -381,7 +406,8 @@ mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ par
       const float m = part_ml[(pb + s) * 2];
       if (m != -INFINITY) l += __expf(m - M) * part_ml[(pb + s) * 2 + 1];
     }
-    const float inv = 1.f / l;
+    float inv = 1.f / l;
+    if (gate) inv /= 1.f + expf(-__bfloat162float(gate[static_cast<size_t>(rows ? rows[r] : r) * ldg + h]));
     for (int s = 0; s < nsplit; ++s) {
       const float m = part_ml[(pb + s) * 2];
       wts[hl * nsplit + s] = m != -INFINITY ? __expf(m - M) * inv : 0.f;
@@ -439,35 +465,69 @@ extern "C" int spark_mla_qrope(const void* qb, int ldq, int R, int H, int D, int
   return spark_launch_rc(__func__);
 }
 
-// part_o: fp32 [R, H, nsplit, L]; part_ml: fp32 [R, H, nsplit, 2]; out: bf16 [R, H, L].
-extern "C" int spark_mla_attn(const void* q_full, const void* lat, const int* pos, const long long* row_kv, const int* sel,
-                              const int* sel_n, int sel_ld, float* part_o, float* part_ml, int nsplit, const float* sink,
-                              int R, int H, int kv_lora, int rope, float scale, void* out, cudaStream_t s,
-                              const int* row_pos0, const int* row_j, const int* anc, int lat_fp8) {
+namespace spark {
+
+template <int HM, bool SPLITP>
+static int launch_mla_decode(dim3 grid, int smem, cudaStream_t s, const void* q_full, const void* lat, const int* pos, const long long* row_kv,
+                             const int* sel, const int* sel_n, int sel_ld, float* part_o, float* part_ml, int H, int KW, int L,
+                             float scale, int nsplit, int spc, const int* row_pos0, const int* row_j, const int* anc, int lat_fp8,
+                             MlaPages pg) {
+  auto kern = mla_decode_kernel<HM, SPLITP>;
+  static bool done = false;
+  if (!done) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); done = true; }
+  kern<<<grid, 256, smem, s>>>((const __nv_bfloat16*)q_full, (const __nv_bfloat16*)lat, pos, row_kv, sel, sel_n, sel_ld, part_o,
+                               part_ml, H, KW, L, scale, nsplit, spc, row_pos0, row_j, anc, lat_fp8, pg);
+  return 0;
+}
+
+static int mla_attn(const void* q_full, const void* lat, const int* pos, const long long* row_kv, const int* sel,
+                    const int* sel_n, int sel_ld, float* part_o, float* part_ml, int nsplit, const float* sink,
+                    int R, int H, int kv_lora, int rope, float scale, void* out, cudaStream_t s, const int* row_pos0,
+                    const int* row_j, const int* anc, int lat_fp8, MlaPages pg, bool splitp, const void* gate, int ldg) {
   if (R <= 0) return 0;
   const int KW = kv_lora + rope;
   if (lat_fp8 && !mla_fp8_ok(kv_lora, rope)) return -5;
   if (H > 64 || (KW & 15) || (kv_lora & 15) || nsplit <= 0) return -5;
   if (anc && (sel || !row_pos0 || !row_j)) return -5;          // tree rows read a dense context
   const int HM = H <= 16 ? 1 : (H <= 32 ? 2 : 4);
-  const int smem = (HM * 16 + MLA_TS) * (KW + 8) * 2 + HM * 16 * 65 * 4 + HM * 16 * 72 * 2;
+  const int smem = (HM * 16 + MLA_TS) * (KW + 8) * 2 + HM * 16 * 65 * 4 + HM * 16 * 72 * 2 * (splitp ? 2 : 1);
   if (smem > 200 * 1024) return -6;
-  void (*kern)(const __nv_bfloat16*, const __nv_bfloat16*, const int*, const long long*, const int*, const int*, int, float*,
-               float*, int, int, int, float, int, int, const int*, const int*, const int*, int) = HM == 1 ? mla_decode_kernel<1> : (HM == 2 ? mla_decode_kernel<2> : mla_decode_kernel<4>);
-  static bool done[3] = {false, false, false};
-  const int id = HM == 1 ? 0 : (HM == 2 ? 1 : 2);
-  if (!done[id]) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); done[id] = true; }
   // few rows (decode): one split per CTA for parallelism; many rows (prefill): a CTA per row walks all its splits
   const int spc = R >= 128 ? nsplit : (R >= 32 ? 4 : 1);
-  kern<<<dim3(R, (nsplit + spc - 1) / spc), 256, smem, s>>>((const __nv_bfloat16*)q_full, (const __nv_bfloat16*)lat, pos, row_kv,
-                                                            sel, sel_n, sel_ld, part_o, part_ml, H, KW, kv_lora, scale, nsplit, spc,
-                                                            row_pos0, row_j, anc, lat_fp8);
-  if (H * nsplit * 4 > 48 * 1024) return -6;
+  const dim3 grid(R, (nsplit + spc - 1) / spc);
+#define SPARK_MLA_DEC(HMV, SPV)                                                                                            \
+  launch_mla_decode<HMV, SPV>(grid, smem, s, q_full, lat, pos, row_kv, sel, sel_n, sel_ld, part_o, part_ml, H, KW, kv_lora, \
+                              scale, nsplit, spc, row_pos0, row_j, anc, lat_fp8, pg)
+  if (splitp) { if (HM == 1) SPARK_MLA_DEC(1, true); else if (HM == 2) SPARK_MLA_DEC(2, true); else SPARK_MLA_DEC(4, true); }
+  else { if (HM == 1) SPARK_MLA_DEC(1, false); else if (HM == 2) SPARK_MLA_DEC(2, false); else SPARK_MLA_DEC(4, false); }
+#undef SPARK_MLA_DEC
   int hpc = H;                                          // heads per merge CTA: enough CTAs for two per SM when rows are few
-  while (hpc > 1 && R * ((H + hpc - 1) / hpc) < 296) hpc = (hpc + 1) / 2;
+  while (hpc > 1 && (R * ((H + hpc - 1) / hpc) < 296 || hpc * nsplit * 4 > 48 * 1024)) hpc = (hpc + 1) / 2;
+  if (hpc * nsplit * 4 > 48 * 1024) return -6;
   const int L4 = kv_lora >> 2;
   const int mthreads = hpc * L4 >= 256 ? 256 : ((hpc * L4 + 31) / 32 * 32);
   mla_merge_kernel<<<dim3(R, (H + hpc - 1) / hpc), mthreads, hpc * nsplit * 4, s>>>(part_o, part_ml, nsplit, sink, H, kv_lora, hpc,
-                                                                                  (__nv_bfloat16*)out);
-  return spark_launch_rc(__func__);
+                                                                                  (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, ldg,
+                                                                                  pg.rows);
+  return spark_launch_rc("spark_mla_attn");
+}
+
+}  // namespace spark
+
+// part_o: fp32 [R, H, nsplit, L]; part_ml: fp32 [R, H, nsplit, 2]; out: bf16 [R, H, L].
+extern "C" int spark_mla_attn(const void* q_full, const void* lat, const int* pos, const long long* row_kv, const int* sel,
+                              const int* sel_n, int sel_ld, float* part_o, float* part_ml, int nsplit, const float* sink,
+                              int R, int H, int kv_lora, int rope, float scale, void* out, cudaStream_t s,
+                              const int* row_pos0, const int* row_j, const int* anc, int lat_fp8) {
+  return mla_attn(q_full, lat, pos, row_kv, sel, sel_n, sel_ld, part_o, part_ml, nsplit, sink, R, H, kv_lora, rope, scale, out, s,
+                  row_pos0, row_j, anc, lat_fp8, MlaPages{nullptr, 0, nullptr, nullptr}, false, nullptr, 0);
+}
+
+// Rows over a paged latent cache (dense causal context), fp32-grade softmax weights, optional per-head sigmoid gate.
+// Query row i of the launch is plan row rows[i] (rows == nullptr: i); pos and row_slot are indexed by plan row.
+extern "C" int spark_mla_attn_paged(const void* q_full, const void* lat, const int* pos, const int* rows, const int* row_slot,
+                                    const int* page_table, int page_ld, float* part_o, float* part_ml, int nsplit, int R, int H,
+                                    int kv_lora, int rope, float scale, const void* gate, int ldg, void* out, cudaStream_t s) {
+  return mla_attn(q_full, lat, pos, nullptr, nullptr, nullptr, 0, part_o, part_ml, nsplit, nullptr, R, H, kv_lora, rope, scale, out,
+                  s, nullptr, nullptr, nullptr, 0, MlaPages{page_table, page_ld, row_slot, rows}, true, gate, ldg);
 }

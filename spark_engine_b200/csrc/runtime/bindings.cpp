@@ -31,6 +31,16 @@ PYBIND11_MODULE(_runtime, m) {
       .def("active_tokens", &KvPool::active_tokens).def("total", &KvPool::total).def("granule", &KvPool::granule)
       .def("bytes_per_token", &KvPool::bytes_per_token);
 
+  py::class_<PageLease>(m, "PageLease").def_readonly("id", &PageLease::id).def_readonly("pages", &PageLease::pages)
+      .def_readonly("cap", &PageLease::cap).def_readonly("used", &PageLease::used).def_readonly("pinned", &PageLease::pinned);
+  py::class_<PagePool>(m, "PagePool").def(py::init<int64_t, int64_t>())
+      .def("acquire", &PagePool::acquire).def("grow", &PagePool::grow).def("release", &PagePool::release)
+      .def("touch", &PagePool::touch).def("pin", &PagePool::pin).def("set_used", &PagePool::set_used)
+      .def("get", &PagePool::get, py::return_value_policy::copy).def("lru_victim", &PagePool::lru_victim)
+      .def("total", &PagePool::total).def("granule", &PagePool::granule).def("free_tokens", &PagePool::free_tokens)
+      .def("largest_free_run", &PagePool::largest_free_run).def("allocated_tokens", &PagePool::allocated_tokens)
+      .def("active_tokens", &PagePool::active_tokens);
+
   py::class_<PcacheEntry>(m, "PcacheEntry").def_readonly("key", &PcacheEntry::key).def_readonly("tokens", &PcacheEntry::tokens)
       .def_readonly("bytes", &PcacheEntry::bytes);
   py::class_<Pcache>(m, "Pcache").def(py::init<const std::string&, const std::string&, int64_t, bool>(), py::arg("root"), py::arg("identity"), py::arg("byte_budget"), py::arg("direct_io") = true)

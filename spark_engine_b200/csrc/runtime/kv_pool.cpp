@@ -84,4 +84,57 @@ int64_t KvPool::bytes_per_token(const std::vector<ArrayLayout>& arrays, int laye
   return static_cast<int64_t>(b * layers + 0.5);
 }
 
+// ------------------------------------------------------------------------------------------------ pages
+PagePool::PagePool(int64_t total_tokens, int64_t page) : page_(page) {
+  if (page <= 0 || total_tokens < page) throw std::invalid_argument("PagePool: bad size");
+  const int64_t n = total_tokens / page;
+  total_ = n * page;
+  for (int64_t i = n - 1; i >= 0; --i) free_.push_back(static_cast<int32_t>(i));
+}
+
+int PagePool::acquire(int64_t tokens) {
+  PageLease l;
+  l.id = next_id_;
+  l.last_use = clock_ + 1;
+  leases_[l.id] = l;
+  if (!grow(l.id, std::max<int64_t>(tokens, 1))) { leases_.erase(l.id); return -1; }
+  ++clock_;
+  return next_id_++;
+}
+
+bool PagePool::grow(int id, int64_t tokens) {
+  auto it = leases_.find(id);
+  if (it == leases_.end()) return false;
+  PageLease& l = it->second;
+  const int64_t need = (tokens + page_ - 1) / page_ - static_cast<int64_t>(l.pages.size());
+  if (need <= 0) return true;
+  if (need > static_cast<int64_t>(free_.size())) return false;
+  for (int64_t i = 0; i < need; ++i) { l.pages.push_back(free_.back()); free_.pop_back(); }
+  l.cap = static_cast<int64_t>(l.pages.size()) * page_;
+  return true;
+}
+
+void PagePool::release(int id) {
+  auto it = leases_.find(id);
+  if (it == leases_.end()) return;
+  for (int32_t p : it->second.pages) free_.push_back(p);
+  leases_.erase(it);
+}
+
+void PagePool::touch(int id) { auto it = leases_.find(id); if (it != leases_.end()) it->second.last_use = ++clock_; }
+void PagePool::pin(int id, bool on) { auto it = leases_.find(id); if (it != leases_.end()) it->second.pinned = on; }
+void PagePool::set_used(int id, int64_t used) {
+  auto it = leases_.find(id);
+  if (it == leases_.end()) return;
+  if (used > it->second.cap) throw std::out_of_range("sequence capacity exceeded");
+  it->second.used = used;
+}
+const PageLease* PagePool::get(int id) const { auto it = leases_.find(id); return it == leases_.end() ? nullptr : &it->second; }
+int PagePool::lru_victim() const {
+  int best = -1; uint64_t stamp = ~0ull;
+  for (auto& kv : leases_) if (!kv.second.pinned && kv.second.last_use < stamp) { stamp = kv.second.last_use; best = kv.first; }
+  return best;
+}
+int64_t PagePool::active_tokens() const { int64_t s = 0; for (auto& kv : leases_) s += kv.second.used; return s; }
+
 }  // namespace spark_rt

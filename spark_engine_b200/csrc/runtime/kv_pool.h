@@ -59,4 +59,41 @@ class KvPool {
   uint64_t clock_ = 0;
 };
 
+// Page pool: the same leases over fixed-size pages instead of one contiguous run per sequence.  A lease grows by any free
+// pages, so a pool that is exactly as large as what its sequences hold never fails by fragmentation; a sequence's rows
+// are found through its page list (models whose cache kernels take a page table).
+struct PageLease {
+  int id = -1;
+  std::vector<int32_t> pages;
+  int64_t cap = 0, used = 0;
+  uint64_t last_use = 0;
+  bool pinned = false;
+};
+
+class PagePool {
+ public:
+  PagePool(int64_t total_tokens, int64_t page);
+  int acquire(int64_t tokens);                // lease id or -1 (nothing changes on failure)
+  bool grow(int id, int64_t tokens);
+  void release(int id);                       // pages go back; the one given back last is handed out next
+  void touch(int id);
+  void pin(int id, bool on);
+  void set_used(int id, int64_t used);
+  const PageLease* get(int id) const;
+  int lru_victim() const;
+  int64_t total() const { return total_; }
+  int64_t granule() const { return page_; }
+  int64_t free_tokens() const { return static_cast<int64_t>(free_.size()) * page_; }
+  int64_t largest_free_run() const { return free_tokens(); }
+  int64_t allocated_tokens() const { return total_ - free_tokens(); }
+  int64_t active_tokens() const;
+
+ private:
+  int64_t total_, page_;
+  std::vector<int32_t> free_;
+  std::map<int, PageLease> leases_;
+  int next_id_ = 0;
+  uint64_t clock_ = 0;
+};
+
 }  // namespace spark_rt

@@ -165,6 +165,12 @@ def build_random_model(cfg: ModelConfig, device="cuda", seed: int = 0, tp=(0, 1)
     rank's shard is generated (heads, experts by id, vocabulary rows of lm_head); replicated tensors come from a
     generator that is seeded identically on every rank."""
     rank, world = tp
+    from .registry import family
+    fam = family(cfg)
+    if fam is not None:
+        if world > 1:
+            raise ValueError(f"{cfg.family} models are not sharded over ranks")
+        return fam.random_weights(cfg, device, seed)
     from ..parallel.tp import local_config
     lcfg = local_config(cfg, world) if world > 1 else cfg
     it = _DevInit(device, seed, cfg.weight_format, cfg.exl3_bits, rank=rank)
@@ -219,7 +225,11 @@ def decode_step_bytes(W, cfg: ModelConfig, rows: int) -> int:
             return sum(nbytes(v) for v in x.values())
         return 0
     total = nbytes(W["lm_head"]) + nbytes(W["final_norm"]) + rows * cfg.hidden * 2
-    for lw in W["layers"]:
+    for i in cfg.layer_runs():
+        lw = W["layers"][i]
+        if "post_norm" not in lw:                # parallel block: one norm, everything dense (prompts' up-projection not read)
+            total += nbytes(lw["in_norm"]) + sum(nbytes(t) for k, t in lw["mix"].items() if k != "kv_up")
+            continue
         total += nbytes(lw["mix"]) + nbytes(lw["in_norm"]) + nbytes(lw["post_norm"])
         m = lw["mlp"]
         if "dense_gu" in m:

@@ -154,9 +154,14 @@ def _mapped_tensor(st, name: str) -> torch.Tensor:
     return t.view(dt).view(*info.shape)
 
 
+def mapped_tensors(path: str) -> Dict[str, torch.Tensor]:
+    """Every tensor of one safetensors file as zero-copy host tensors by name."""
+    st = rt().SafeTensors(path)
+    return {n: _mapped_tensor(st, n) for n in st.names()}
+
+
 def load_config(directory: str) -> ModelConfig:
-    with open(os.path.join(directory, "config.json")) as f:
-        return ModelConfig.from_dict(json.load(f))
+    return ModelConfig.from_json(os.path.join(directory, "config.json"))
 
 
 def _to_device(x, device, pinned: bool):
@@ -194,11 +199,20 @@ def _streamed_tensor(st, name: str, device) -> torch.Tensor:
 
 
 def load_checkpoint(directory: str, device="cpu", tp: Tuple[int, int] = (0, 1), pinned: bool = True,
-                    cfg: Optional[ModelConfig] = None, stream: Optional[bool] = None):
+                    cfg: Optional[ModelConfig] = None, stream: Optional[bool] = None, dtype=None):
     """-> (cfg, W) with W this rank's shard on `device`.  `stream` (default: SPARK_LOAD_STREAM=1): an unsharded load (one
     rank, or a directory written by `write_rank_shards`) reads every tensor straight to the device through the threaded
-    loader instead of mapping the files."""
+    loader instead of mapping the files.  `dtype`: dense weights of architectures with their own checkpoint format
+    (default: fp32 on the CPU, bf16 on the device)."""
     cfg = cfg or load_config(directory)
+    if not os.path.exists(os.path.join(directory, INDEX)):      # an architecture with its own tensor names (models/registry.py)
+        from .registry import family
+        fam = family(cfg)
+        if fam is None:
+            raise FileNotFoundError(f"{directory} has no {INDEX}")
+        if tp[1] > 1:
+            raise ValueError(f"{cfg.family} checkpoints are not sharded over ranks")
+        return cfg, fam.load_weights(directory, cfg, device, dtype or (torch.float32 if str(device) == "cpu" else torch.bfloat16))
     with open(os.path.join(directory, INDEX)) as f:
         idx = json.load(f)
     rank, world = tp

@@ -642,9 +642,15 @@ class Model:
         self.lcfg = tp.local_config(cfg) if tp is not None else cfg      # per-rank head counts
         self.n_slots, self.kv_tokens = n_slots, kv_tokens
         per = slot_tokens or kv_tokens // n_slots
+        self.page = 0                        # > 0: caches are pages of this many tokens, found through `page_table`
+        if cfg.layer_specs:
+            self._init_pages(per)
+        elif dtype == torch.float32 and self.device.type == "cuda":
+            raise ValueError(f"{cfg.family} models have no 32-bit kernels")
         # with a growable backing no region exists until a KvManager leases (and backs) one
-        self.seqs = [SeqInfo(i * per, per) if kv_backing is None else SeqInfo(0, 0) for i in range(n_slots)]
-        self.layers = self._build_layers(W["layers"])
+        if not self.page:
+            self.seqs = [SeqInfo(i * per, per) if kv_backing is None else SeqInfo(0, 0) for i in range(n_slots)]
+        self.layers = self._build_layers([W["layers"][i] for i in cfg.layer_runs()])
         self.mtp_layers = self._build_layers(W["mtp"]["layers"]) if "mtp" in W else []
         self.hidden_out = None
         # a hashed n-gram table that stays on the host is read through asynchronous gathers into a pinned ring
@@ -658,6 +664,12 @@ class Model:
 
     def _build_layers(self, lws):
         out = []
+        if self.cfg.layer_specs:
+            from .parallel_mixers import build_parallel_mixer
+            for lw, i in zip(lws, self.cfg.layer_runs()):       # every run of a layer has its own cache or state
+                out.append((lw, build_parallel_mixer(self.cfg, self.cfg.layer_specs[i], lw["mix"], self.n_slots, self.n_pages,
+                                                     self.page, self.page_table, self.device, self.dtype), None))
+            return out
         for lw in lws:
             kind = lw["type"]
             if kind == "gdn":
@@ -685,12 +697,40 @@ class Model:
     def set_kv_region(self, slot: int, base: int, cap: int):
         self.seqs[slot].kv_base, self.seqs[slot].kv_cap = base, cap
 
+    # -- paged caches (models with per-layer specs) -------------------------------------------
+    def _init_pages(self, per: int):
+        """Pool of 64-token pages shared by the slots; until a `KvManager` takes over, slot i owns a fixed run of pages."""
+        if self.kv_backing is not None or self.tp is not None:
+            raise ValueError("paged models run on one GPU with a dense pool")
+        self.page = 64
+        pages = -(-per // self.page)
+        self.n_pages = max(pages * self.n_slots if per * self.n_slots >= self.kv_tokens else 1, -(-self.kv_tokens // self.page))
+        self.kv_tokens = self.n_pages * self.page
+        self.page_table = torch.full((self.n_slots, self.n_pages), -1, dtype=torch.int32, device=self.device)
+        self.seqs = [SeqInfo(0, 0) for _ in range(self.n_slots)]
+        for i in range(self.n_slots):
+            self.set_pages(i, list(range(i * pages, min((i + 1) * pages, self.n_pages))))
+
+    def set_pages(self, slot: int, pages: List[int]):
+        """The pages of a slot in position order (entries past them are -1: the kernels never write there)."""
+        row = torch.full((self.n_pages,), -1, dtype=torch.int32)
+        row[: len(pages)] = torch.tensor(pages, dtype=torch.int32)
+        self.page_table[slot].copy_(row)
+        self.seqs[slot].kv_base, self.seqs[slot].kv_cap = 0, len(pages) * self.page
+
+    def _token_rows(self, slot: int, n: int) -> torch.Tensor:
+        t = torch.arange(n, device=self.device)
+        return self.page_table[slot, t // self.page].long() * self.page + t % self.page
+
     # -- forward ----------------------------------------------------------------------------
     def _block(self, lw, mix, mlp, X, pend, plan, commit):
         """One decoder block.  `pend` is the previous block's MLP output, still to be added to the residual
         (under tensor parallelism it is this rank's partial sum): the add, the all-reduce and this block's
         first RMSNorm happen in one fused op.  Returns (X, new pending output)."""
         cfg, tp = self.cfg, self.tp
+        if cfg.layer_specs:                  # parallel block: `mix` holds the feed-forward too
+            h, X, h32 = ops.add_norm_rows(pend, X, lw["in_norm"], cfg.norm_eps, cfg.norm_one_plus, self.dtype, mix.wants_f32_rows)
+            return X, mix.forward(h, plan, self.seqs, commit, h32=h32)
         if cfg.hc_kind == "none":
             # decode rounds on the device: the MoE combine is deferred into the next residual update (one launch for
             # combine + add + norm; under tensor parallelism the combine happens inside the all-reduce push)
@@ -736,7 +776,7 @@ class Model:
             X[salted.to(X.device)] = 0
             X = inject_rows(X, plan.ids, plan.mm_rows)
         else:
-            X = ops.embed(W["embed"], plan.ids, self.dtype)
+            X = ops.embed(W["embed"], plan.ids, self.dtype, cfg.embed_scale)
         if cfg.hc_kind != "none":
             X = X.unsqueeze(1).repeat(1, cfg.hc_streams, 1).contiguous()
         self._ids_for_ngram = plan
@@ -756,6 +796,8 @@ class Model:
             X = hf if hf is not None else hn
         elif cfg.hc_kind == "mhc":
             X, hn = ops.mhc_final(X, pend, W["final_norm"], cfg.norm_eps, self.tp)
+        elif cfg.layer_specs:
+            hn, X, _ = ops.add_norm_rows(pend, X, W["final_norm"], cfg.norm_eps, cfg.norm_one_plus, self.dtype)
         else:
             hn, X = ops.add_rmsnorm(pend, X, W["final_norm"], cfg.norm_eps, self.tp)
         if self.tp is not None and getattr(self.tp, "rows_sharded", False):
@@ -767,6 +809,8 @@ class Model:
                 self.seqs[s.slot].length = s.pos0 + s.n
         if plan.logit_rows.shape[0] != hn.shape[0]:
             hn = hn[plan.logit_rows]
+        if hn.shape[0] == 0:                 # a step whose logits nobody asked for
+            return torch.empty(0, cfg.vocab, dtype=torch.float32, device=hn.device)
         return ops.lm_head(hn, W["lm_head"])
 
     def greedy(self, logits: torch.Tensor) -> torch.Tensor:
@@ -828,6 +872,8 @@ class Model:
         block; latent attention: top-k pools x pool), or None when no layer selects.  Up to here dense visibility of the
         committed context (what tree-verification rows use) equals what a decode row sees."""
         lim = None
+        if self.cfg.layer_specs:             # recurrent parallel blocks verify chains only
+            return 0
         for _, mix, _ in self.layers:
             c = getattr(mix, "c", None)
             if isinstance(mix, AttnMixer) and c.sparse_topk_blocks:
@@ -880,8 +926,10 @@ class Model:
         for _, mix, _ in self.layers + self.mtp_layers:
             d = {}
             for name, t in mix.state_tensors().items():
-                if name in ("S", "tail"):
+                if name in ("S", "tail", "carried"):
                     d[name] = t[slot].clone()
+                elif self.page:
+                    d[name] = t.view(-1, t.shape[-1])[self._token_rows(slot, si.length)]
                 elif name in ("ik_pool", "pool"):
                     blk = self.cfg.attn.block if name == "ik_pool" else self.cfg.mla.pool
                     d[name] = t[si.kv_base // blk: si.kv_base // blk + si.length // blk + 1].clone()
@@ -896,8 +944,10 @@ class Model:
         assert n <= si.kv_cap, "sequence capacity exceeded"
         for (_, mix, _), d in zip(self.layers + self.mtp_layers, snap["layers"]):
             for name, t in mix.state_tensors().items():
-                if name in ("S", "tail"):
+                if name in ("S", "tail", "carried"):
                     t[slot] = d[name]
+                elif self.page:
+                    t.view(-1, t.shape[-1])[self._token_rows(slot, n)] = d[name]
                 elif name in ("ik_pool", "pool"):
                     blk = self.cfg.attn.block if name == "ik_pool" else self.cfg.mla.pool
                     t[si.kv_base // blk: si.kv_base // blk + d[name].shape[0]] = d[name]

@@ -163,6 +163,9 @@ def layer_weights(cfg: ModelConfig, i: int, it: _Init, kind: str = None) -> dict
 
 def init_weights(cfg: ModelConfig, seed: int = 0, std: float = 0.02) -> dict:
     """Dense fp32 weights on CPU, N(0, std), deterministic in `seed`."""
+    from .registry import family
+    if family(cfg) is not None:                  # families with their own layout and scales
+        return family(cfg).random_weights(cfg, "cpu", seed, torch.float32)
     it = _Init(seed, std)
     W = {"embed": it.mat(cfg.vocab, cfg.hidden), "final_norm": it.ones(cfg.hidden),
          "lm_head": it.mat(cfg.vocab, cfg.hidden),
@@ -202,7 +205,7 @@ def count_params(W) -> int:
     return n
 
 
-FP32_KEYS = {"conv", "ape", "norm", "scale", "base", "f_b", "g_b"}
+FP32_KEYS = {"conv", "ape", "norm", "scale", "base", "f_b", "g_b", "mu", "u"}
 
 
 def to_device(W, device, dtype=torch.bfloat16):

@@ -30,6 +30,12 @@ def cuda_ops():
     return _cuda_ops
 
 
+def block_ops():
+    """The parallel-block bindings."""
+    from . import parallel_block
+    return parallel_block
+
+
 def use_kernels(t: torch.Tensor) -> bool:
     return t.is_cuda and not _FALLBACK
 
@@ -41,11 +47,14 @@ def set_fallback(on: bool):
 
 
 # ----------------------------------------------------------------------------- basic ops
-def embed(table: torch.Tensor, ids: torch.Tensor, dtype) -> torch.Tensor:
-    """Token embedding rows.  On the device the residual stream is fp32 (activations bf16)."""
+def embed(table: torch.Tensor, ids: torch.Tensor, dtype, scale: float = 1.0) -> torch.Tensor:
+    """Token embedding rows (times `scale`).  On the device the residual stream is fp32 (activations bf16)."""
     if use_kernels(table):
+        if scale != 1.0 or table.dtype == torch.float32:
+            return block_ops().embed_scaled(table, ids.to(torch.int32), scale)
         return cuda_ops().embed(table, ids.to(torch.int32))
-    return table[ids].to(dtype)
+    x = table[ids].to(dtype)
+    return x * scale if scale != 1.0 else x
 
 
 def to_tensor(x):
@@ -100,8 +109,10 @@ def lm_head(h, w) -> torch.Tensor:
     return linear(h, w).float()
 
 
-def linear(x: torch.Tensor, w) -> torch.Tensor:
-    """y = x @ W^T for a dense `[N,K]` tensor or a quantised weight object."""
+def linear(x: torch.Tensor, w, out_f32: bool = False) -> torch.Tensor:
+    """y = x @ W^T for a dense `[N,K]` tensor or a quantised weight object (`out_f32`: dense weights only)."""
+    if out_f32:
+        return cuda_ops().dense_linear(x, w, out_f32=True) if use_kernels(x) else (x @ w.to(x.dtype).t()).float()
     if isinstance(w, QuantWeight):
         if use_kernels(x):
             return cuda_ops().quant_linear(x, w)
@@ -330,3 +341,105 @@ def ngram_embed(model, X, plan, w):
     d = (key * L.rms(X.float(), w["norm_q"].float(), cfg.norm_eps)).sum(-1, keepdim=True) / math.sqrt(X.shape[-1])
     gate = torch.sigmoid(torch.sign(d) * torch.sqrt(d.abs().clamp_min(cfg.norm_eps)))
     return (X.float() + gate * val).to(X.dtype)
+
+
+# ----------------------------------------------------------------------------- parallel block
+def add_norm_rows(delta, res, w, eps, one_plus: bool, dtype, want_f32: bool = False):
+    """res' = res + delta (delta may be None); returns (h = RMSNorm(res') * (w or 1 + w) in `dtype`, res', fp32 h if asked)."""
+    if use_kernels(res):
+        return block_ops().add_norm_rows(delta, res, w, eps, one_plus, dtype, want_f32)
+    if delta is not None:
+        res = res + delta
+    h = L.rms(res.float(), w.float(), eps, one_plus)
+    return h.to(dtype), res, h
+
+
+def gelu_tanh(x):
+    return F.gelu(x.float(), approximate="tanh")
+
+
+def gate_concat(o, n, group, w, eps, gate, kind, ff, width_ff, off, width, dtype, out=None):
+    """Input row of a parallel block's output product: [ group-RMSNorm(o) * w * gate(g), padded to `off` | gelu(ff gate) *
+    (ff up) ].  group 0 = no norm, kind = sigmoid | silu | None (no gate); o None = the mixer part is in `out` already."""
+    src = o if o is not None else out
+    if use_kernels(src):
+        return block_ops().gate_concat(o, n, group, w, eps, gate, kind, ff, width_ff, off, width, dtype, out)
+    R = src.shape[0]
+    if out is None:
+        out = torch.zeros(R, width, dtype=dtype)
+    if o is not None:
+        x = o.float()
+        if group:
+            x = x.view(R, n // group, group)
+            x = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)).reshape(R, n)
+        if w is not None:
+            x = x * w
+        if kind is not None:
+            x = x * (torch.sigmoid(gate.float()) if kind == "sigmoid" else F.silu(gate.float()))
+        out[:, :n] = x.to(dtype)
+    if ff is not None:
+        up = width - off
+        out[:, off: off + width_ff] = (gelu_tanh(ff[:, :width_ff]) * ff[:, up: up + width_ff].float()).to(dtype)
+    return out
+
+
+def token_shift(h32, carried, mu, plan, dtype):
+    """[n, R, H]: for each mu row the mix h + (h' - h) mu of a row and its predecessor (the carried row of the slot for the
+    first row of a segment)."""
+    if use_kernels(h32):
+        return block_ops().token_shift(h32, carried, mu, plan, dtype)
+    prev = torch.empty_like(h32)
+    for s in plan.segs:
+        prev[s.r0] = carried[s.slot]
+        prev[s.r0 + 1: s.r0 + s.n] = h32[s.r0: s.r0 + s.n - 1]
+    return (h32 + (prev - h32) * mu.unsqueeze(1)).to(dtype)
+
+
+def linear_stack(xs, w):
+    """n independent products [n, R, K] x [n, N, K] -> [n, R, N]."""
+    if use_kernels(xs):
+        return block_ops().linear_stack(xs, w)
+    return torch.einsum("nrk,nok->nro", xs, w.to(xs.dtype))
+
+
+def channel_decay(z, w2, w0, n: int):
+    """log decay -exp(w2 tanh(z) + w0) [R, n] in fp32."""
+    if use_kernels(z):
+        return block_ops().channel_decay(z, w2, w0, n)
+    return -torch.exp(torch.tanh(z.float()) @ w2.float().t() + w0)
+
+
+def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=None, u=None, h32=None, carried=None,
+                 n_rows=None):
+    """Decayed linear attention (constant decay per head, or decay per channel and token with a bonus for the current
+    token): o fp32 [R, H * V]; the slots' states advance when `commit` (by n_rows[i] rows of segment i if given)."""
+    if use_kernels(q):
+        return block_ops().linear_state(q, k, v, H, D, V, S, plan, commit, act, log2a, logw, u, h32, carried, n_rows)
+    R = q.shape[0]
+    q, k, v = q.float().view(R, H, D), k.float().view(R, H, D), v.float().view(R, H, V)
+    if act:
+        q, k, v = F.silu(q), F.silu(k), F.silu(v)
+    o = q.new_zeros(R, H, V)
+    a = torch.exp2(log2a).view(H, 1, 1) if log2a is not None else None
+    for i, s in enumerate(plan.segs):
+        St = S[s.slot]
+        n = s.n if n_rows is None else min(s.n, int(n_rows[i]))
+        for r in range(s.r0, s.r0 + n):
+            kv = k[r].unsqueeze(-1) * v[r].unsqueeze(-2)
+            if a is not None:
+                St = a * St + kv
+                o[r] = torch.einsum("hd,hdv->hv", q[r], St)
+            else:
+                o[r] = torch.einsum("hd,hdv->hv", q[r], St + u.view(H, D, 1) * kv)
+                St = torch.exp(logw[r]).view(H, D, 1) * St + kv
+        if commit and n:
+            S[s.slot] = St
+            if carried is not None:
+                carried[s.slot] = h32[s.r0 + n - 1]
+    return o.view(R, H * V)
+
+
+def latent_mixer(mixer, proj, plan, cat):
+    if use_kernels(proj):
+        return block_ops().latent_mixer(mixer, proj, plan, cat)
+    return None

@@ -26,6 +26,7 @@ _SIGS = {
     "spark_gemm_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "spark_gemm_bf16_swiglu": [vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp],
     "spark_gemm_grouped_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, i32, f32, i32, vp, vp],
+    "spark_gemm_simt": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, i32, i32, vp],
     "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, f32, i32, vp],
     "spark_gemv_bf16_items": [vp, i32, i64, vp, i64, i32, vp, i32, i64, i32, i32, i32, i32, vp, i32, vp],
     "spark_add_rmsnorm": [vp, i32, vp, vp, vp, i32, i32, f32, i32, vp],
@@ -227,13 +228,14 @@ def _as_bf16(x):
     return x if x.dtype == torch.bfloat16 else x.to(torch.bfloat16)
 
 
-def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out_f32: bool = False, fmt: int = 1) -> torch.Tensor:
+def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out_f32: bool = False, fmt: int = 1, out=None) -> torch.Tensor:
     """C[M,N] = A[M,K] B[N,K]^T on tcgen05.  fmt 1 = bf16 operands, 0 = fp16 operands."""
     M, K = a.shape
     N = b.shape[0]
     assert a.stride(1) == 1 and b.stride(1) == 1 and K % 8 == 0
-    c = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=a.device)
-    rc = lib().spark_gemm_bf16(P(a), P(b), P(c), M, N, K, a.stride(0), b.stride(0), N, int(out_f32), fmt,
+    c = out if out is not None else torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=a.device)
+    out_f32 = c.dtype == torch.float32
+    rc = lib().spark_gemm_bf16(P(a), P(b), P(c), M, N, K, a.stride(0), b.stride(0), c.stride(0), int(out_f32), fmt,
                                P(status_word(a.device)), stream())
     check(rc, "spark_gemm_bf16")
     return c
@@ -272,14 +274,37 @@ def gemv_bf16_items(x, ldx, x_item_stride, w, expert_stride, ldw, y, ldy, y_item
     return y
 
 
-def dense_linear(x: torch.Tensor, w: torch.Tensor, out_f32: bool = False) -> torch.Tensor:
-    if w.dtype != torch.bfloat16:
-        raise TypeError("dense weights must be bf16 on the device")
+def gemv_rows(K: int) -> int:
+    """Rows one GEMV launch takes at contraction length K (a power of two: the staged rows fill shared memory)."""
+    r = 16
+    while r > 1 and r * K * 2 > 200 * 1024:
+        r //= 2
+    return r
+
+
+def gemm_simt(a, lda, sa, b, ldb, sb, c, ldc, sc, batch, M, N, K):
+    """Batched C = A B^T on the FP32 units (32-bit mode, unaligned bf16 shapes).  Strides in elements."""
+    rc = lib().spark_gemm_simt(P(a), lda, sa, P(b), ldb, sb, P(c), ldc, sc, batch, M, N, K, int(b.dtype == torch.float32),
+                               int(c.dtype == torch.float32), stream())
+    check(rc, "spark_gemm_simt")
+    return c
+
+
+def dense_linear(x: torch.Tensor, w: torch.Tensor, out_f32: bool = False, out=None) -> torch.Tensor:
+    if w.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError("dense weights must be bf16 (or fp32 in the 32-bit mode) on the device")
+    R, (N, K) = x.shape[0], w.shape
+    if w.dtype == torch.float32 or K % 8:                  # 32-bit mode; contraction lengths the vector kernels cannot address
+        x = x.to(w.dtype).contiguous()
+        if out is None:
+            out = torch.empty(R, N, dtype=torch.float32 if out_f32 else w.dtype, device=x.device)
+        return gemm_simt(x, x.stride(0), 0, w, w.stride(0), 0, out, out.stride(0), 0, 1, R, N, K)
     x = _as_bf16(x)
-    R = x.shape[0]
-    if R <= 16:
-        return gemv_bf16(x.contiguous(), w, out_f32=out_f32)
-    return gemm_bf16(x.contiguous(), w, out_f32)
+    if x.stride(1) != 1 or x.stride(0) % 8 or x.data_ptr() % 16:
+        x = x.contiguous()
+    if R <= 16 and R <= gemv_rows(K):
+        return gemv_bf16(x, w, out_f32=out_f32, out=out)
+    return gemm_bf16(x, w, out_f32, out=out)
 
 
 # ----------------------------------------------------------------------------- EXL3

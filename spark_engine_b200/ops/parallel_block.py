@@ -1,0 +1,306 @@
+"""CUDA implementations of the parallel-block ops (`csrc/kernels/block_rows.cu`, `linear_state.cu`, `latent.cu`, `mla.cu`):
+row ops around the block, the two decayed linear recurrences, latent attention over a paged cache.  bf16 and fp32
+activations; what the mechanisms keep in fp32 (residual, norms, states, decays, scores, softmax weights) is fp32 in both."""
+from __future__ import annotations
+
+import torch
+
+from . import cuda as cu
+from .cuda import P, check, f32, i32, i64, lib, scratch, status_word, stream, vp
+
+_LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32]
+cu._SIGS.update({
+    "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, i32, vp, vp],
+    "spark_add_norm_rows": [vp, vp, vp, vp, vp, i32, i32, f32, i32, i32, vp],
+    "spark_token_shift": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, vp],
+    "spark_channel_decay": [vp, i32, vp, i32, i32, vp, vp, i32, i32, i32, vp],
+    "spark_neg_exp_bias": [vp, vp, i32, i32, vp],
+    "spark_tanh_split": [vp, i32, vp, i32, i32, vp],
+    "spark_gate_concat": [vp, i32, i32, i32, vp, f32, vp, i32, i32, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp],
+    "spark_linear_seq": _LIN + [i32, i32, vp],
+    "spark_linear_chunked": _LIN + [i32, vp, i32, vp, vp, vp, vp],
+    "spark_latent_prep": [vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp, i32, vp, vp,
+                          i32, vp, vp],
+    "spark_latent_qrope": [vp, i32, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp, i32, i32, vp],
+    "spark_latent_gather": [vp, i32, vp, i32, i32, vp, i32, vp, vp],
+    "spark_latent_rows": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
+    "spark_latent_prefill": [vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
+    "spark_mla_attn_paged": [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
+})
+cu._KERNELS_PER_CALL.update({"spark_linear_chunked": 3, "spark_mla_attn_paged": 2})
+
+CHUNK_MIN_ROWS = 32          # segments of at least this many rows take the chunked / flash kernels
+LC = 64                      # rows per chunk of the chunked recurrences
+
+
+def _is32(dtype) -> int:
+    return int(dtype == torch.float32)
+
+
+# ----------------------------------------------------------------------------- rows
+def embed_scaled(table, ids32, scale: float):
+    R, H = ids32.shape[0], table.shape[1]
+    cu.dbg.check_index("embed token ids", ids32, 0, table.shape[0])
+    out = torch.empty(R, H, dtype=torch.float32, device=table.device)
+    check(lib().spark_embed_scaled(P(table), P(ids32), P(out), R, H, table.shape[0], float(scale), _is32(table.dtype),
+                                   P(status_word(table.device)), stream()), "spark_embed_scaled")
+    return out
+
+
+def add_norm_rows(delta, res, w, eps, one_plus, dtype, want_f32):
+    """res (fp32, in place) += delta (fp32); returns (h in `dtype`, res, fp32 copy of h or None)."""
+    R, H = res.shape
+    assert res.dtype == torch.float32 and res.is_contiguous()
+    if delta is not None:
+        delta = delta.float().contiguous()
+    h = torch.empty(R, H, dtype=dtype, device=res.device)
+    h32 = h if dtype == torch.float32 else (torch.empty(R, H, dtype=torch.float32, device=res.device) if want_f32 else None)
+    check(lib().spark_add_norm_rows(P(delta), P(res), P(w), P(h), P(h32) if h32 is not h else None, R, H, float(eps), int(one_plus),
+                                    _is32(dtype), stream()), "spark_add_norm_rows")
+    return h, res, h32
+
+
+def token_shift(h32, carried, mu, plan, dtype):
+    d = cu._plan_dev(plan, h32.device)
+    R, H = h32.shape
+    n = mu.shape[0]
+    out = torch.empty(n, R, H, dtype=dtype, device=h32.device)
+    check(lib().spark_token_shift(P(h32), P(carried), P(d["row_slot"]), P(d["row_j"]), P(mu), n, P(out), R, H, _is32(dtype), stream()),
+          "spark_token_shift")
+    return out
+
+
+def channel_decay(z, w2, w0, n: int):
+    """z [R, rank] fp32 -> log decay -exp(w2 tanh(z) + w0) [R, n] fp32."""
+    R, r = z.shape
+    if w2.dtype == torch.bfloat16 and R >= 64 and 2 * r % 8 == 0:
+        # prompts: tanh as a two-term bf16 sum against [w2 | w2], one tensor-core product
+        t = torch.empty(R, 2 * r, dtype=torch.bfloat16, device=z.device)
+        check(lib().spark_tanh_split(P(z), z.stride(0), P(t), R, r, stream()), "spark_tanh_split")
+        out = cu.dense_linear(t, _doubled(w2), out_f32=True)
+        check(lib().spark_neg_exp_bias(P(out), P(w0), R, n, stream()), "spark_neg_exp_bias")
+        return out
+    out = torch.empty(R, n, dtype=torch.float32, device=z.device)
+    check(lib().spark_channel_decay(P(z), z.stride(0), P(w2), w2.stride(0), r, P(w0), P(out), R, n, _is32(w2.dtype), stream()),
+          "spark_channel_decay")
+    return out
+
+
+_twice = {}
+
+
+def _doubled(w):
+    key = (w.data_ptr(), tuple(w.shape))
+    hit = _twice.get(key)
+    if hit is None or hit[0]() is not w:
+        import weakref
+        hit = (weakref.ref(w), torch.cat((w, w), 1).contiguous())
+        _twice[key] = hit
+    return hit[1]
+
+
+GATES = {None: 0, "sigmoid": 1, "silu": 2}
+
+
+def gate_concat(o, n, group, w, eps, gate, kind, ff, F, off, width, dtype, out=None, gate_div=1):
+    """[ group-norm(o) * w * gate | gelu(ff gate) * ff up ] -> [R, width]; `ff` = [gate | up] columns (up at width - off)."""
+    src = o if o is not None else ff
+    R = src.shape[0]
+    if out is None:
+        out = torch.empty(R, width, dtype=dtype, device=src.device)
+    check(lib().spark_gate_concat(P(o), 0 if o is None else o.stride(0), n, group, P(w), float(eps), P(gate),
+                                  0 if gate is None else gate.stride(0), GATES[kind], gate_div, P(ff), 0 if ff is None else ff.stride(0),
+                                  width - off, F, P(out), width, off, R, _is32(dtype), stream()), "spark_gate_concat")
+    return out
+
+
+def linear_stack(xs, w):
+    """xs [n, R, K], w [n, N, K] -> [n, R, N]: n independent products of equal shape."""
+    n, R, K = xs.shape
+    N = w.shape[1]
+    dev = xs.device
+    if w.dtype == torch.float32 or K % 8:
+        y = torch.empty(n, R, N, dtype=xs.dtype, device=dev)
+        return cu.gemm_simt(xs, K, R * K, w, K, N * K, y, N, R * N, n, R, N, K)
+    if R <= 16 and cu.gemv_rows(K) >= R:
+        y = torch.empty(n, R, N, dtype=torch.bfloat16, device=dev)
+        return cu.gemv_bf16_items(xs, K, R * K, w, N * K, K, y, N, R * N, n, R, N, K, _iota(n, dev))
+    return torch.stack([cu.dense_linear(xs[i], w[i]) for i in range(n)]) if n == 1 else _stack_gemm(xs, w)
+
+
+def _stack_gemm(xs, w):
+    n, R, _ = xs.shape
+    y = torch.empty(n, R, w.shape[1], dtype=torch.bfloat16, device=xs.device)
+    for i in range(n):
+        cu.dense_linear(xs[i], w[i], out=y[i])
+    return y
+
+
+_iotas = {}
+
+
+def _iota(n, dev):
+    key = (n, str(dev))
+    if key not in _iotas:
+        _iotas[key] = torch.arange(n, dtype=torch.int32, device=dev)
+    return _iotas[key]
+
+
+# ----------------------------------------------------------------------------- recurrences
+def _split(plan, dev):
+    """Segment tables of a committed plan: (short segments, long segments), each (device table, segments)."""
+    d = cu._plan_dev(plan, dev)
+    if "seg_split" not in d:
+        longs = [s for s in plan.segs if s.n >= CHUNK_MIN_ROWS]
+        if not longs:
+            d["seg_split"] = ((d["seg"], plan.segs), (None, []))
+        else:
+            shorts = [s for s in plan.segs if s.n < CHUNK_MIN_ROWS]
+            tab = lambda ss: torch.tensor([[s.slot, s.r0, s.n, s.pos0] for s in ss], dtype=torch.int32).to(dev) if ss else None
+            d["seg_split"] = ((tab(shorts), shorts), (d["seg"] if not shorts else tab(longs), longs))
+    return d["seg_split"]
+
+
+def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=None, u=None, h32=None, carried=None,
+                 n_rows=None):
+    """Decayed linear attention of every segment from its slot's state S [slots, H, D, V]; returns o fp32 [R, H * V].
+    `log2a` [H]: constant decay per head; else `logw` [R, H * D] (log decay) and `u` (bonus), with the token-shift row
+    carried along (h32 rows -> carried [slots, width]).  `n_rows`: device counts of accepted rows (commit)."""
+    dev = q.device
+    d = cu._plan_dev(plan, dev)
+    R = q.shape[0]
+    o = torch.empty(R, H * V, dtype=torch.float32, device=dev)
+    if cu.dbg.CHECK:
+        cu._check_slots("linear_state", plan, S.shape[0])
+    width = h32.shape[1] if h32 is not None else 0
+
+    def args(seg):
+        return (P(q), q.stride(0), P(k), k.stride(0), P(v), v.stride(0), D, V, P(log2a), P(logw), P(u), P(S), P(seg), P(n_rows), P(o),
+                P(h32), P(carried), width, H, D, V, int(commit), int(act))
+    short, longs = (d["seg"], plan.segs), (None, [])
+    if n_rows is None and commit and q.dtype == torch.bfloat16 and D <= 128:
+        short, longs = _split(plan, dev)
+    if short[1]:
+        check(lib().spark_linear_seq(*args(short[0]), len(short[1]), _is32(q.dtype), stream()), "spark_linear_seq")
+    if longs[1]:
+        if "lin_chunks" not in d:
+            chunks, first = [], []
+            for i, sg in enumerate(longs[1]):
+                first.append(len(chunks))
+                chunks += [(i, c) for c in range((sg.n + LC - 1) // LC)]
+            d["lin_chunks"] = (torch.tensor(chunks, dtype=torch.int32).to(dev), torch.tensor(first, dtype=torch.int32).to(dev))
+        chunks, first = d["lin_chunks"]
+        nch = chunks.shape[0]
+        ws_u = scratch("lin_ws_u", nch * H * D * V, torch.float32, dev)
+        ws_d = scratch("lin_ws_d", nch * H * D, torch.float32, dev)
+        check(lib().spark_linear_chunked(*args(longs[0]), len(longs[1]), P(chunks), nch, P(first), P(ws_u), P(ws_d), stream()),
+              "spark_linear_chunked")
+    return o
+
+
+# ----------------------------------------------------------------------------- latent attention
+def _short_long(plan, dev):
+    """Rows of segments below CHUNK_MIN_ROWS as an int32 row list (None = every row) and the table of the other segments
+    with their offsets in the gathered context: (rows or None, count, table [n, 5], segments, gathered rows)."""
+    d = cu._plan_dev(plan, dev)
+    if "latent_split" not in d:
+        longs = [s for s in plan.segs if s.n >= CHUNK_MIN_ROWS]
+        if not longs:
+            d["latent_split"] = (None, plan.rows, None, [], 0)
+        else:
+            rows = [r for s in plan.segs if s.n < CHUNK_MIN_ROWS for r in range(s.r0, s.r0 + s.n)]
+            tab, off = [], 0
+            for s in longs:
+                tab.append([s.slot, s.r0, s.n, s.pos0, off])
+                off += s.pos0 + s.n
+            d["latent_split"] = (torch.tensor(rows, dtype=torch.int32).to(dev) if rows else None, len(rows),
+                                 torch.tensor(tab, dtype=torch.int32).to(dev), longs, off)
+    return d["latent_split"]
+
+
+def _max_ctx(plan, d):
+    if "max_ctx" not in d:
+        d["max_ctx"] = max(s.pos0 + s.n for s in plan.segs)
+    return d["max_ctx"]
+
+
+def _heads_product(x, ldx, xh, w, y, ldy, yh, R):
+    """y[r, h] = x[r, h] w[h]^T over heads: x at r * ldx + h * xh, w [H, N, K], y at r * ldy + h * yh."""
+    H, N, K = w.shape
+    if w.dtype == torch.float32 or R > 64 or K % 8 or xh % 8 or ldx % 8 or x.data_ptr() % 16:
+        return cu.gemm_simt(x, ldx, xh, w, K, N * K, y, ldy, yh, H, R, N, K)
+    step = min(16, cu.gemv_rows(K))
+    for r in range(0, R, step):                         # every head's matrix is streamed once per 16 rows
+        cu.gemv_bf16_items(x[r:], ldx, xh, w, N * K, K, y[r:], ldy, yh, H, min(step, R - r), N, K, _iota(H, x.device))
+    return y
+
+
+def latent_mixer(mx, proj, plan, cat):
+    """Latent attention of every row of `proj` (columns: mx.off), per-head outputs into cat[:, :H * V] (gated)."""
+    c, w, dev, dt = mx.c, mx.w, proj.device, proj.dtype
+    d = cu._plan_dev(plan, dev)
+    R, H, D, V = proj.shape[0], c.n_heads, c.head_dim, c.v_dim
+    Dp, Rp, Vp, Lp, KW = mx.Dp, mx.Rp, mx.Vp, mx.Lp, mx.Lp + mx.Rp
+    pages, pld = mx.pages, mx.pages.shape[1]
+    is32 = _is32(dt)
+    if not hasattr(mx, "_inv"):
+        mx._inv = (c.rope_theta ** (-torch.arange(c.rope_dim // 2, dtype=torch.float64) * 2 / c.rope_dim)).to(dev)
+    cq = torch.empty(R, w["uq"].shape[1], dtype=dt, device=dev)
+    check(lib().spark_latent_prep(P(proj), proj.stride(0), mx.off["dq"], mx.off["lat"], mx.off["rot"], R, c.q_rank, cq.shape[1], c.kv_rank,
+                                  Lp, c.rope_dim, Rp, int(c.rope_interleaved), float(mx.eps), P(w["dq_norm"]), P(w["kv_norm"]), P(mx._inv),
+                                  P(d["pos32"]), P(d["row_slot"]), P(pages), pld, P(cq), P(mx.lat), is32, P(status_word(dev)), stream()),
+          "spark_latent_prep")
+    q = cu.dense_linear(cq, w["uq"])                      # [R, H * (Dp + Rp)]
+    gate = proj[:, mx.off["g"]:]
+    rows, ns, tab, longs, ctx = (None, R, None, [], 0) if is32 else _short_long(plan, dev)
+    if longs and not mx.prefill_ok:
+        rows, ns, longs = None, R, []
+    if ns:
+        qs = q if rows is None else cu.gather_rows(q, rows)
+        o = _latent_absorbed(mx, qs, rows, ns, gate, d, plan, is32)
+        dst = cat if rows is None else torch.empty(ns, H * V, dtype=dt, device=dev)
+        _heads_product(o, H * Lp, Lp, w["uv"], dst, dst.stride(0), V, ns)
+        if rows is not None:
+            cat[:, : H * V].index_copy_(0, rows.long(), dst)
+    if longs:
+        lat = scratch("latent_ctx", ctx * KW, torch.bfloat16, dev)[: ctx * KW].view(ctx, KW)
+        check(lib().spark_latent_gather(P(mx.lat), KW * 2, P(tab), len(longs), max(s.pos0 + s.n for s in longs), P(pages), pld, P(lat),
+                                        stream()), "spark_latent_gather")
+        kv = cu.dense_linear(lat[:, :Lp], w["kv_up"])
+        qr = q[:, Dp:]
+        check(lib().spark_latent_qrope(P(qr), q.stride(0), Dp + Rp, P(qr), q.stride(0), Dp + Rp, R, H, c.rope_dim, Rp,
+                                       int(c.rope_interleaved), P(mx._inv), P(d["pos32"]), None, 0, 0, stream()), "spark_latent_qrope")
+        check(lib().spark_latent_prefill(P(q), q.stride(0), P(kv), kv.stride(0), P(lat), KW, P(tab), len(longs), max(s.n for s in longs),
+                                         H, Dp, Rp, V, Vp, Lp, float(c.scale), P(gate), proj.stride(0), P(cat), cat.stride(0), stream()),
+              "spark_latent_prefill")
+    return cat
+
+
+def _latent_absorbed(mx, q, rows, n, gate, d, plan, is32):
+    """Absorbed attention rows [n, H, Lp] (gated): q [n, H * (Dp + Rp)] before rotation."""
+    c, w, dev = mx.c, mx.w, q.device
+    H, Dp, Rp, Lp = c.n_heads, mx.Dp, mx.Rp, mx.Lp
+    KW = Lp + Rp
+    pages, pld = mx.pages, mx.pages.shape[1]
+    qf = torch.empty(n, H * KW, dtype=q.dtype, device=dev)
+    _heads_product(q, q.stride(0), Dp + Rp, w["uk_t"], qf, H * KW, KW, n)
+    qr, qt = q[:, Dp:], qf[:, Lp:]
+    check(lib().spark_latent_qrope(P(qr), q.stride(0), Dp + Rp, P(qt), H * KW, KW, n, H, c.rope_dim, Rp, int(c.rope_interleaved),
+                                   P(mx._inv), P(d["pos32"]), P(rows), 1, is32, stream()), "spark_latent_qrope")
+    o = torch.empty(n, H * Lp, dtype=q.dtype, device=dev)
+    if is32 or not mx.decode_tc_ok:
+        check(lib().spark_latent_rows(P(qf), P(mx.lat), P(d["pos32"]), P(rows), P(d["row_slot"]), P(pages), pld, n, H, Lp, Rp, float(c.scale),
+                                      P(gate), gate.stride(0), P(o), is32, stream()), "spark_latent_rows")
+        return o
+    nsplit = (_max_ctx(plan, d) + 63) // 64
+    step = n if n <= 16 else 16                            # bounds the partial results of long contexts
+    part_o = scratch("latent_part_o", step * H * nsplit * Lp, torch.float32, dev)
+    part_ml = scratch("latent_part_ml", step * H * nsplit * 2, torch.float32, dev)
+    if rows is None and n > step:
+        rows = _iota(n, dev)
+    for r in range(0, n, step):
+        m = min(step, n - r)
+        check(lib().spark_mla_attn_paged(P(qf[r:]), P(mx.lat), P(d["pos32"]), P(rows[r:]) if rows is not None else None, P(d["row_slot"]),
+                                         P(pages), pld, P(part_o), P(part_ml), nsplit, m, H, Lp, Rp, float(c.scale), P(gate),
+                                         gate.stride(0), P(o[r:]), stream()), "spark_mla_attn_paged")
+    return o

@@ -61,6 +61,17 @@ def rope_neox(x: torch.Tensor, pos: torch.Tensor, rot: int, theta: float, inv: O
     return torch.cat((x1 * cos - x2 * sin, x2 * cos + x1 * sin, rest), -1)
 
 
+def rope_interleaved(x: torch.Tensor, pos: torch.Tensor, rot: int, theta: float):
+    """Rotary with interleaved pairs (2i, 2i + 1) on the first `rot` dims of the last axis; x [T, ..., D], pos [T]."""
+    inv = theta ** (-torch.arange(rot // 2, dtype=torch.float64) * 2 / rot)
+    ang = (pos.to(x.device).double().unsqueeze(1) * inv.to(x.device)).float()
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [rot // 2]
+    cos, sin = ang.cos().view(shape), ang.sin().view(shape)
+    u, v = x[..., 0:rot:2], x[..., 1:rot:2]
+    turned = torch.stack((u * cos - v * sin, v * cos + u * sin), -1).flatten(-2)
+    return torch.cat((turned, x[..., rot:]), -1)
+
+
 def causal_conv(x: torch.Tensor, w: torch.Tensor, dilation: int = 1, tail: Optional[torch.Tensor] = None):
     """Depthwise causal conv over time.  x [T, C]; w [C, k] (w[:, -1] multiplies the current step);
     `tail` [(k-1)*dilation, C] = inputs before x (zeros when None)."""

@@ -22,6 +22,13 @@ from ..models.plan import make_plan
 from .graphs import GraphCache, RoundGraph, ctx_bucket, runtime_signature
 
 
+def compute_dtype(ecfg: EngineConfig, device) -> torch.dtype:
+    """Activation dtype of the runner: fp32 on the CPU, else `EngineConfig.dtype`."""
+    if ecfg.dtype not in ("bfloat16", "float32"):
+        raise ValueError(f"unknown dtype {ecfg.dtype!r} (bfloat16 | float32)")
+    return torch.float32 if str(device) == "cpu" or ecfg.dtype == "float32" else torch.bfloat16
+
+
 @dataclass
 class GenStats:
     prefill_ms: float = 0.0
@@ -36,7 +43,7 @@ class LLMEngine:
     def __init__(self, cfg: ModelConfig, W: dict, ecfg: Optional[EngineConfig] = None, device="cuda",
                  max_seqs: int = 4, kv_tokens_per_seq: int = 4096, tp=None):
         self.cfg, self.ecfg = cfg, ecfg or EngineConfig()
-        dtype = torch.float32 if str(device) == "cpu" else torch.bfloat16
+        dtype = compute_dtype(self.ecfg, device)
         self.model = Model(cfg, W, device=device, dtype=dtype, n_slots=max_seqs,
                            kv_tokens=max_seqs * kv_tokens_per_seq, slot_tokens=kv_tokens_per_seq, tp=tp)
         self.device = self.model.device

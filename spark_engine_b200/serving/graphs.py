@@ -267,7 +267,9 @@ class RoundGraph:
     def _commit_body(self):
         from ..ops import cuda as cu
         for mix, pend in self.pendings:
-            if hasattr(mix.c, "gate_rank"):
+            if hasattr(mix, "commit_rows"):
+                mix.commit_rows(pend[0], self.plan, self.d_acc)
+            elif hasattr(mix.c, "gate_rank"):
                 cu.kda_mixer(mix, pend[0], pend[1], self.plan, True, n_rows=self.d_acc)
             else:
                 cu.gdn_mixer(mix, pend[0], pend[1], self.plan, True, n_rows=self.d_acc)

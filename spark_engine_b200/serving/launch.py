@@ -65,9 +65,13 @@ def _engine_main(a):
     if a.layers:
         cfg.n_layers = a.layers
         cfg.layer_types = cfg.layer_types[: a.layers]
+        cfg.layer_specs = cfg.layer_specs[: a.layers]
+        if cfg.loop is not None:
+            cfg.loop.start, cfg.loop.stop = min(cfg.loop.start, a.layers), min(cfg.loop.stop, a.layers)
     ecfg = EngineConfig.from_env(max_seqs=a.max_seqs, kv_tokens=a.kv_tokens, prefill_chunk=a.prefill_chunk, spec=a.spec,
                                  spec_depth=a.spec_depth, pcache_dir=a.pcache_dir, socket=a.socket, profile=a.profile,
-                                 tp=world, prewarm=a.prewarm)
+                                 tp=world, prewarm=a.prewarm, dtype=a.dtype)
+    dtype = torch.float32 if ecfg.dtype == "float32" else torch.bfloat16
     tp = None
     if dev != "cpu":
         torch.cuda.set_device(local)
@@ -88,20 +92,20 @@ def _engine_main(a):
                           rows_cap=max(1024, min(a.prefill_chunk, 4096)))
     if a.checkpoint:
         from ..models.checkpoint import load_checkpoint
-        _, W = load_checkpoint(a.checkpoint, dev, tp=(rank, world), cfg=cfg)
+        _, W = load_checkpoint(a.checkpoint, dev, tp=(rank, world), cfg=cfg, dtype=None if dev == "cpu" else dtype)
     elif dev == "cpu":
         W = init_weights(cfg, seed=a.seed)
         if world > 1:
             from ..parallel.tp import shard_weights
             W = shard_weights(W, cfg, rank, world)
-    elif cfg.weight_format != "dense" or cfg.hidden > 1024:
+    elif (cfg.weight_format != "dense" or cfg.hidden > 1024) and ecfg.dtype == "bfloat16":
         W = build_random_model(cfg, dev, seed=a.seed, tp=(rank, world))
     else:
         W = init_weights(cfg, seed=a.seed)
         if world > 1:
             from ..parallel.tp import shard_weights
             W = shard_weights(W, cfg, rank, world)
-        W = to_device(W, dev)
+        W = to_device(W, dev, dtype)
     oplog = os.environ.get("SPARK_OPLOG", f"/spark_b200_oplog_{os.getppid()}")
     vision = _vision_tower(a, cfg)
     if world == 1:
@@ -251,6 +255,8 @@ def main():
     ap.add_argument("--ack-timeout-ms", type=int, default=30000, help="op-log deadline between leader and followers")
     ap.add_argument("--layers", type=int, default=0)
     ap.add_argument("--device", default="cuda")
+    ap.add_argument("--dtype", default=None, choices=["bfloat16", "float32"],
+                    help="activations and dense weights on the device (float32: models with 32-bit kernels)")
     ap.add_argument("--socket", default="/tmp/spark-b200.sock")
     ap.add_argument("--host", default="127.0.0.1")
     ap.add_argument("--port", type=int, default=8000)

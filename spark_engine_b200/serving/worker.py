@@ -59,7 +59,8 @@ class EngineServer:
             assert vcfg.out_hidden == cfg.hidden, "the aligner must project to the model's hidden size"
             self.tower = VisionTower(vcfg, vW, device=device, dtype=torch.float32 if str(device) == "cpu" else torch.bfloat16)
         e = self.ecfg
-        dtype = torch.float32 if str(device) == "cpu" else torch.bfloat16
+        from .engine import compute_dtype
+        dtype = compute_dtype(e, device)
         per = max(256, e.kv_tokens // e.max_seqs // 256 * 256)
         backing = None
         if e.kv_backing == "vmm":
