@@ -58,6 +58,8 @@ class BatchSession:
         m = self.model
         items, rows, r = [], [], 0
         for rid, toks, want in entries:
+            if not toks:
+                continue
             for t in toks:
                 if not 0 <= t < self.cfg.vocab:
                     raise ValueError(f"token id {t} is outside the vocabulary of {self.cfg.vocab} entries")
@@ -65,6 +67,8 @@ class BatchSession:
             items.append((slot, list(toks), m.seqs[slot].length))
             rows += [r + w for w in want]
             r += len(toks)
+        if not items:
+            return torch.empty(0, self.cfg.vocab, device=m.device)
         plan = make_plan(items, device=m.device)
         plan.logit_rows = torch.tensor(rows, dtype=torch.long, device=m.device)
         plan.gather_logit_rows = True
