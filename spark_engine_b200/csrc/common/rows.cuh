@@ -25,8 +25,20 @@ __device__ __forceinline__ void stf4(__nv_bfloat16* p, float4 v) {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// Activations that are rounded to bf16 next: hardware exponential and reciprocal (relative error of a few 2^-22).
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
+  return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-x)) : sigmoid_f(x);
+}
+template <typename T> __device__ __forceinline__ float silu_t(float x) {
+  return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : silu_f(x);
+}
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+// gelu_tanh(z) = z * sigmoid(2 sqrt(2/pi) (z + 0.044715 z^3))
+template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
+  return sizeof(T) == 2 ? __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))) : gelu_tanh_f(z);
 }
 
 // Sum over the block in a fixed order; every thread gets the same bits.  sh: >= 32 floats.

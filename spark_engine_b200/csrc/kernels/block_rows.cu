@@ -96,29 +96,40 @@ token_shift_kernel(const float* __restrict__ h, const float* __restrict__ carrie
 // log of the decay exp(-exp(x)), bounded where the decay itself is 0 in fp32 (differences of its running sums stay exact)
 __device__ __forceinline__ float log_decay(float x) { return fmaxf(-expf(x), -105.f); }
 
-// grid (ceil(N / 128), ceil(R / 16)); 128 threads: channel per thread, 16 rows per CTA.
-template <typename TW>
+// grid (ceil(N / 32), ceil(R / RB)); 128 threads: four lanes per channel (eight ranks each in turn), RB rows per CTA.
+// rank is a multiple of 8.
+template <typename TW, int RB>
 __global__ void __launch_bounds__(128)
 channel_decay_kernel(const float* __restrict__ z, int ldz, const TW* __restrict__ w2, int ldw, int rank,
                      const float* __restrict__ w0, float* __restrict__ logw, int R, int N) {
-  extern __shared__ float t[];                               // [rank][16]
+  extern __shared__ float t[];                               // [rank][RB]
+  const int d = blockIdx.x * 32 + (threadIdx.x >> 2), part = threadIdx.x & 3, r0 = blockIdx.y * RB;
   pdl_wait();
-  const int r0 = blockIdx.y * 16, d = blockIdx.x * 128 + threadIdx.x;
-  for (int i = threadIdx.x; i < rank * 16; i += 128) {
-    const int k = i >> 4, r = r0 + (i & 15);
+  for (int i = threadIdx.x; i < rank * RB; i += 128) {
+    const int k = i / RB, r = r0 + i % RB;
     t[i] = r < R ? tanhf(z[static_cast<size_t>(r) * ldz + k]) : 0.f;
   }
   __syncthreads();
-  if (d >= N) return;
-  float acc[16];
+  float acc[RB];
 #pragma unroll
-  for (int r = 0; r < 16; ++r) acc[r] = 0.f;
-  for (int k = 0; k < rank; ++k) {
-    const float w = ldf(w2 + static_cast<size_t>(d) * ldw + k);
+  for (int r = 0; r < RB; ++r) acc[r] = 0.f;
+  if (d < N)
+    for (int k0 = part * 8; k0 < rank; k0 += 32) {
+      const TW* wr = w2 + static_cast<size_t>(d) * ldw + k0;
+      const float4 a = ldf4(wr), b = ldf4(wr + 4);
+      const float w[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
 #pragma unroll
-    for (int r = 0; r < 16; ++r) acc[r] = fmaf(w, t[k * 16 + r], acc[r]);
+      for (int k = 0; k < 8; ++k)
+#pragma unroll
+        for (int r = 0; r < RB; ++r) acc[r] = fmaf(w[k], t[(k0 + k) * RB + r], acc[r]);
+    }
+#pragma unroll
+  for (int r = 0; r < RB; ++r) {
+    float v = acc[r];
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = log_decay(v + w0[d]);
   }
-  for (int r = 0; r < 16 && r0 + r < R; ++r) logw[static_cast<size_t>(r0 + r) * N + d] = log_decay(acc[r] + w0[d]);
 }
 
 // z [R, N] fp32 holds W2 tanh(..) already (prefill: a tensor-core product): z <- -exp(z + w0), in place.
@@ -149,7 +160,8 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 gate_concat_kernel(const float* __restrict__ o, int ldin, int N, int group, const float* __restrict__ w, float eps,
                    const T* __restrict__ gate, int ldg, int gate_kind, int gate_div, const T* __restrict__ ff, int ldff, int up_off,
-                   int F, T* __restrict__ out, int ldo, int off) {
+                   int F, T* __restrict__ out, int ldo, int off, int vec) {
+  // vec: every row start the kernel touches is 4-element aligned and groups are multiples of 4 columns
   __shared__ float sh[32];
   pdl_wait();
   const int r = blockIdx.x;
@@ -157,8 +169,20 @@ gate_concat_kernel(const float* __restrict__ o, int ldin, int N, int group, cons
   if (blockIdx.y > 0) {
     const T* fr = ff + static_cast<size_t>(r) * ldff;
     const int base = (blockIdx.y - 1) * 1024;
+    const int i4 = base + threadIdx.x * 4;
+    if (vec) {                                                // four columns per thread
+      if (i4 >= ldo - off) return;
+      if (i4 + 4 <= F) {
+        const float4 g = ldf4(fr + i4), u = ldf4(fr + up_off + i4);
+        stf4(orow + off + i4, make_float4(gelu_tanh_t<T>(g.x) * u.x, gelu_tanh_t<T>(g.y) * u.y, gelu_tanh_t<T>(g.z) * u.z,
+                                          gelu_tanh_t<T>(g.w) * u.w));
+        return;
+      }
+      for (int i = i4; i < min(i4 + 4, ldo - off); ++i) stf(orow + off + i, i < F ? gelu_tanh_t<T>(ldf(fr + i)) * ldf(fr + up_off + i) : 0.f);
+      return;
+    }
     for (int i = base + threadIdx.x; i < min(base + 1024, ldo - off); i += 256)
-      stf(orow + off + i, i < F ? gelu_tanh_f(ldf(fr + i)) * ldf(fr + up_off + i) : 0.f);
+      stf(orow + off + i, i < F ? gelu_tanh_t<T>(ldf(fr + i)) * ldf(fr + up_off + i) : 0.f);
     return;
   }
   if (o == nullptr) return;
@@ -167,10 +191,35 @@ gate_concat_kernel(const float* __restrict__ o, int ldin, int N, int group, cons
   auto put = [&](int i, float rs) {
     float v = x[i] * rs;
     if (w) v *= w[i];
-    if (gate_kind == 1) v *= sigmoid_f(ldf(gr + i / gate_div));
-    else if (gate_kind == 2) v *= silu_f(ldf(gr + i / gate_div));
+    if (gate_kind == 1) v *= sigmoid_t<T>(ldf(gr + i / gate_div));
+    else if (gate_kind == 2) v *= silu_t<T>(ldf(gr + i / gate_div));
     stf(orow + i, v);
   };
+  if (vec && group > 0 && gate_kind > 0 && w != nullptr) {
+    auto put4 = [&](int i, float4 v, float rs) {
+      const float4 ww = ldf4(w + i), g = ldf4(gr + i);
+      const bool sg = gate_kind == 1;
+      v.x *= rs * ww.x * (sg ? sigmoid_t<T>(g.x) : silu_t<T>(g.x)); v.y *= rs * ww.y * (sg ? sigmoid_t<T>(g.y) : silu_t<T>(g.y));
+      v.z *= rs * ww.z * (sg ? sigmoid_t<T>(g.z) : silu_t<T>(g.z)); v.w *= rs * ww.w * (sg ? sigmoid_t<T>(g.w) : silu_t<T>(g.w));
+      stf4(orow + i, v);
+    };
+    if (group == N) {
+      float ss = 0.f;
+      for (int i = threadIdx.x * 4; i < N; i += 1024) { const float4 v = ldf4(x + i); ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+      const float rs = 1.f / sqrtf(block_sum_all(ss, sh) / N + eps);
+      for (int i = threadIdx.x * 4; i < N; i += 1024) put4(i, ldf4(x + i), rs);
+    } else {
+      const int lane = threadIdx.x & 31;
+      for (int g = threadIdx.x >> 5; g < N / group; g += 8) {
+        float ss = 0.f;
+        for (int i = lane * 4; i < group; i += 128) { const float4 v = ldf4(x + g * group + i); ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+        const float rs = 1.f / sqrtf(warp_sum(ss) / group + eps);
+        for (int i = lane * 4; i < group; i += 128) put4(g * group + i, ldf4(x + g * group + i), rs);
+      }
+    }
+    for (int i = N + threadIdx.x; i < off; i += 256) stf(orow + i, 0.f);
+    return;
+  }
   if (group == N && group > 0) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < N; i += 256) ss = fmaf(x[i], x[i], ss);
@@ -225,9 +274,12 @@ extern "C" int spark_token_shift(const float* h, const float* carried, const int
 extern "C" int spark_channel_decay(const float* z, int ldz, const void* w2, int ldw, int rank, const float* w0, float* logw,
                                    int R, int N, int f32, cudaStream_t s) {
   if (R <= 0) return 0;
-  if (rank <= 0 || rank * 64 > 48 * 1024) return -5;
-  SPARK_BY_TYPE(f32, spark_launch_pdl(channel_decay_kernel<T>, dim3((N + 127) / 128, (R + 15) / 16), dim3(128), rank * 64, s,
-                                      dim3(1, 1, 1), z, ldz, (const T*)w2, ldw, rank, w0, logw, R, N))
+  if (rank <= 0 || (rank & 7) || (ldw & 7) || rank * 64 > 48 * 1024) return -5;
+#define SPARK_CHD(RB)                                                                                                     \
+  spark_launch_pdl(channel_decay_kernel<T, RB>, dim3((N + 31) / 32, (R + RB - 1) / RB), dim3(128), rank * RB * 4, s,      \
+                   dim3(1, 1, 1), z, ldz, (const T*)w2, ldw, rank, w0, logw, R, N)
+  SPARK_BY_TYPE(f32, if (R <= 4) SPARK_CHD(4); else SPARK_CHD(16))
+#undef SPARK_CHD
   return spark_launch_rc(__func__);
 }
 
@@ -250,7 +302,12 @@ extern "C" int spark_gate_concat(const float* o, int ldin, int N, int group, con
   if (R <= 0) return 0;
   if (group > 0 && N % group) return -5;
   const int nff = ff ? (ldo - off + 1023) / 1024 : 0;
+  const uintptr_t a16 = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w);
+  const uintptr_t a8 = reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(ff) | reinterpret_cast<uintptr_t>(out);
+  const int vec = ((a16 | (f32 ? a8 : 0)) & 15) == 0 && (a8 & 7) == 0 && gate_div == 1 &&
+                  ((ldin | N | group | (gate ? ldg : 0) | (ff ? ldff | up_off : 0) | ldo | off) & 3) == 0;
   SPARK_BY_TYPE(f32, spark_launch_pdl(gate_concat_kernel<T>, dim3(R, 1 + nff), dim3(256), 0, s, dim3(1, 1, 1), o, ldin, N, group, w,
-                                      eps, (const T*)gate, ldg, gate_kind, gate_div, (const T*)ff, ldff, up_off, F, (T*)out, ldo, off))
+                                      eps, (const T*)gate, ldg, gate_kind, gate_div, (const T*)ff, ldff, up_off, F, (T*)out, ldo, off,
+                                      vec))
   return spark_launch_rc(__func__);
 }

@@ -190,12 +190,20 @@ gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
   int n0 = rows_of(0, w0, w1);
   pdl_wait();
   if (n0 < N) load(w0, w1, kb);                          // in flight while the rows are staged
+  // rows past R are left as they are: an MMA column only ever reaches its own row's outputs, which are not stored
   const int KV8 = K >> 3;
-  for (int i = threadIdx.x; i < NT * 8 * KV8; i += blockDim.x) {
-    const int r = i / KV8, kv = i - r * KV8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < R) v = *reinterpret_cast<const uint4*>(x + static_cast<size_t>(r) * ldx + kv * 8);
-    *reinterpret_cast<uint4*>(xs + r * lds + kv * 8) = v;
+  for (int i0 = threadIdx.x; i0 < R * KV8; i0 += 4 * GEMV_WARPS * 32) {
+    uint4 v[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = i0 + u * GEMV_WARPS * 32, r = i / KV8;
+      if (i < R * KV8) v[u] = *reinterpret_cast<const uint4*>(x + static_cast<size_t>(r) * ldx + (i - r * KV8) * 8);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = i0 + u * GEMV_WARPS * 32, r = i / KV8;
+      if (i < R * KV8) *reinterpret_cast<uint4*>(xs + r * lds + (i - r * KV8) * 8) = v[u];
+    }
   }
   __syncthreads();
   for (int cg = 0; cg < (KS ? 1 : cpc); ++cg) {
@@ -277,12 +285,14 @@ static int launch_gemv_wide(const void* x, int ldx, const void* W, int ldw, void
 }
 
 // Shapes the wide kernel takes: one item, no activation, no expert tables, K a multiple of 32 and small enough that
-// 16 staged rows fit in shared memory (the choice must not depend on the number of rows: a row's result may not
+// 8 staged rows fit in shared memory (the choice must not depend on the number of rows: a row's result may not
 // change with the batch it is in).
 static bool gemv_wide_ok(int ldx, int ldw, int items, int N, int K, const int* pe, const int* pr, int act) {
   return items == 1 && !pe && !pr && act == 0 && N >= 2048 && (K & 31) == 0 && (ldx & 7) == 0 && (ldw & 7) == 0 &&
-         16 * (K + GEMV_MMA_PAD) * 2 <= 200 * 1024;
+         8 * (K + GEMV_MMA_PAD) * 2 <= 200 * 1024;
 }
+// Contractions too long for 16 staged rows run in groups of 8 rows (a row's chain of MMAs is the same either way).
+static bool gemv_wide_rows16(int K) { return 16 * (K + GEMV_MMA_PAD) * 2 <= 200 * 1024; }
 
 }  // namespace spark
 
@@ -296,6 +306,16 @@ extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long 
   if (K % 8 || rows_per_item > 16) return -5;
   if (gemv_wide_ok(ldx, ldw, items, N, K, pair_expert, pair_row, act) &&
       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) == 0) {
+    if (rows_per_item > 8 && !gemv_wide_rows16(K)) {
+      const size_t es = out_f32 ? 4 : 2;
+      for (int r = 0; r < rows_per_item; r += 8) {
+        const int rc = spark_gemv_bf16(static_cast<const uint8_t*>(x) + static_cast<size_t>(r) * ldx * 2, ldx, W, expert_stride, ldw,
+                                       static_cast<uint8_t*>(y) + static_cast<size_t>(r) * ldy * es, ldy, items,
+                                       rows_per_item - r < 8 ? rows_per_item - r : 8, N, K, pair_expert, pair_row, act, limit, out_f32, s);
+        if (rc) return rc;
+      }
+      return 0;
+    }
     if (rows_per_item <= 8)
       return out_f32 ? launch_gemv_wide<1, float>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s)
                      : launch_gemv_wide<1, __nv_bfloat16>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s);

@@ -142,32 +142,81 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   hi = *reinterpret_cast<const uint32_t*>(&h);
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
+// 2^x on the special-function unit (relative error about 2^-22; 0 for very negative x)
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float LOG2E = 1.4426950408889634f;
 __device__ __forceinline__ void split1(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) {
   hi = __float2bfloat16(x);
   lo = __float2bfloat16(x - __bfloat162float(hi));
 }
 
-// Row tile [LC][ld] of one head: rows past nv and channels past D are zero; SiLU optional.
+// Row tile [LC][lds] of one head by 128 threads: rows past nv and channels past ncol are zero; SiLU optional.  Whole aligned
+// tiles are fetched as a batch of 16-byte loads.  dst rows are 4-byte aligned.
+__device__ __forceinline__ void put_rows8(__nv_bfloat16* dst, const float (&f)[8], int act) {
+#pragma unroll
+  for (int e = 0; e < 8; e += 2) {
+    const float x = act ? silu_t<__nv_bfloat16>(f[e]) : f[e], y = act ? silu_t<__nv_bfloat16>(f[e + 1]) : f[e + 1];
+    *reinterpret_cast<__nv_bfloat162*>(dst + e) = __floats2bfloat162_rn(x, y);
+  }
+}
 template <int COLS>
-__device__ __forceinline__ void load_rows(__nv_bfloat16* dst, int lds, const __nv_bfloat16* src, int ld, int nv, int ncol, int act) {
-  for (int i = threadIdx.x; i < LC * (COLS / 8); i += blockDim.x) {
-    const int r = i / (COLS / 8), c = (i - r * (COLS / 8)) * 8;
+__device__ __forceinline__ void load_rows(__nv_bfloat16* __restrict__ dst, int lds, const __nv_bfloat16* __restrict__ src, int ld,
+                                          int nv, int ncol, int act) {
+  constexpr int PER = LC * (COLS / 8) / 128;                 // 16-byte pieces per thread
+  const bool whole = nv == LC && ncol >= COLS && (ld & 7) == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+  if (whole) {
+    uint4 u[PER];
+#pragma unroll
+    for (int b = 0; b < PER; ++b) {
+      const int i = threadIdx.x + b * 128, r = i / (COLS / 8), c = (i % (COLS / 8)) * 8;
+      u[b] = *reinterpret_cast<const uint4*>(src + static_cast<size_t>(r) * ld + c);
+    }
+#pragma unroll
+    for (int b = 0; b < PER; ++b) {
+      const int i = threadIdx.x + b * 128, r = i / (COLS / 8), c = (i % (COLS / 8)) * 8;
+      const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&u[b]);
+      float f[8];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { const float2 t = __bfloat1622float2(p[e]); f[2 * e] = t.x; f[2 * e + 1] = t.y; }
+      put_rows8(dst + r * lds + c, f, act);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < LC * (COLS / 8); i += 128) {
+    const int r = i / (COLS / 8), c = (i % (COLS / 8)) * 8;
     float f[8];
-    const __nv_bfloat16* p = src + static_cast<size_t>(r) * ld + c;
-    if (r < nv && c + 8 <= ncol && (reinterpret_cast<uintptr_t>(p) & 15) == 0) {
-      const uint4 u = *reinterpret_cast<const uint4*>(p);
-      const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&u);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) { const float2 t = __bfloat1622float2(b[e]); f[2 * e] = t.x; f[2 * e + 1] = t.y; }
-    } else {
+    for (int e = 0; e < 8; ++e) f[e] = (r < nv && c + e < ncol) ? __bfloat162float(src[static_cast<size_t>(r) * ld + c + e]) : 0.f;
+    put_rows8(dst + r * lds + c, f, act);
+  }
+}
+// Log decays [LC][ldg] (base 2) of one head: zero past nv / ncol.
+template <int COLS>
+__device__ __forceinline__ void load_decays(float* __restrict__ G, int ldg, const float* __restrict__ lw, size_t ld, int nv, int ncol) {
+  constexpr int PER = LC * (COLS / 4) / 128;
+  if (nv == LC && ncol >= COLS && (ld & 3) == 0 && (reinterpret_cast<uintptr_t>(lw) & 15) == 0) {
+    float4 u[PER];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] = (r < nv && c + e < ncol) ? __bfloat162float(p[e]) : 0.f;
+    for (int b = 0; b < PER; ++b) {
+      const int i = threadIdx.x + b * 128;
+      u[b] = ldf4(lw + (i / (COLS / 4)) * ld + (i % (COLS / 4)) * 4);
     }
 #pragma unroll
-    for (int e = 0; e < 8; e += 2) {
-      const float x = act ? silu_f(f[e]) : f[e], y = act ? silu_f(f[e + 1]) : f[e + 1];
-      *reinterpret_cast<__nv_bfloat162*>(dst + r * lds + c + e) = __floats2bfloat162_rn(x, y);
+    for (int b = 0; b < PER; ++b) {
+      const int i = threadIdx.x + b * 128;
+      float2* d = reinterpret_cast<float2*>(G + (i / (COLS / 4)) * ldg + (i % (COLS / 4)) * 4);
+      d[0] = make_float2(LOG2E * u[b].x, LOG2E * u[b].y);
+      d[1] = make_float2(LOG2E * u[b].z, LOG2E * u[b].w);
     }
+    return;
+  }
+  for (int i = threadIdx.x; i < LC * COLS; i += 128) {
+    const int r = i / COLS, c = i % COLS;
+    G[r * ldg + c] = (r < nv && c < ncol) ? LOG2E * lw[r * ld + c] : 0.f;
   }
 }
 
@@ -189,29 +238,50 @@ linear_chunk_u_kernel(const __grid_constant__ LinearArgs a, const int* __restric
   const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(a.v) + r0 * a.ldv + h * a.hsv + v0;
   load_rows<LVT>(Vs, LVS, v, a.ldv, nv, a.V - v0, a.act);
   if (MODE == 0) {
+    load_rows<DP>(Kh, LDK, k, a.ldk, nv, a.D, a.act);
+    __syncthreads();
     const float l2 = a.log2a[h];
-    for (int i = tid; i < LC * DP; i += 128) {
-      const int r = i / DP, c = i - r * DP;
-      float x = (r < nv && c < a.D) ? __bfloat162float(k[static_cast<size_t>(r) * a.ldk + c]) : 0.f;
-      if (a.act) x = __bfloat162float(__float2bfloat16(silu_f(x)));
+    for (int i = tid; i < LC * (DP / 2); i += 128) {
+      const int r = i / (DP / 2), c = (i - r * (DP / 2)) * 2;
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Kh + r * LDK + c));
       const int e = nv - 1 - r;
-      x = e > 0 ? x * exp2f(l2 * e) : (e == 0 ? x : 0.f);
-      split1(x, Kh[r * LDK + c], Kl[r * LDK + c]);
+      const float w = e > 0 ? exp2f(l2 * e) : (e == 0 ? 1.f : 0.f);
+      uint32_t hi, lo;
+      split2(x.x * w, x.y * w, hi, lo);
+      *reinterpret_cast<uint32_t*>(Kh + r * LDK + c) = hi;
+      *reinterpret_cast<uint32_t*>(Kl + r * LDK + c) = lo;
     }
   } else {
-    for (int c = tid; c < DP; c += 128) {                                 // suffix sums: G_C - G_j, last row first
-      float g = 0.f;
-      const float* lw = a.logw + r0 * (static_cast<size_t>(a.H) * a.D) + h * a.D + c;
-#pragma unroll 8
-      for (int r = LC - 1; r >= 0; --r) {
-        float x = 0.f;
-        if (r < nv && c < a.D) {
-          x = __bfloat162float(k[static_cast<size_t>(r) * a.ldk + c]) * expf(g);
-          g += lw[static_cast<size_t>(r) * a.H * a.D];
-        }
-        split1(x, Kh[r * LDK + c], Kl[r * LDK + c]);
-      }
-      if (c < a.D && v0 == 0) ws_d[(static_cast<size_t>(ci) * a.H + h) * a.D + c] = expf(g);
+    float* G = reinterpret_cast<float*>(smem_lu + (2 * LC * LDK + LC * LVS) * 2);     // [64][DP] running sums, base 2
+    float* gsum = G + LC * DP;                                                         // [16][DP] of four-row groups
+    load_rows<DP>(Kh, LDK, k, a.ldk, nv, a.D, 0);
+    load_decays<DP>(G, DP, a.logw + r0 * (static_cast<size_t>(a.H) * a.D) + h * a.D, static_cast<size_t>(a.H) * a.D, nv, a.D);
+    __syncthreads();
+    for (int i = tid; i < 16 * DP; i += 128) {                            // four rows at a time, then the 16 group sums
+      const int gr = i / DP, c = i - gr * DP;
+      float s = 0.f;
+#pragma unroll
+      for (int r = 0; r < 4; ++r) { s += G[(gr * 4 + r) * DP + c]; G[(gr * 4 + r) * DP + c] = s; }
+      gsum[i] = s;
+    }
+    __syncthreads();
+    for (int c = tid; c < DP; c += 128) {
+      float s = 0.f;
+#pragma unroll
+      for (int gr = 0; gr < 16; ++gr) { const float x = gsum[gr * DP + c]; gsum[gr * DP + c] = s; s += x; }
+      gsum[16 * DP + c] = s;
+      if (c < a.D && v0 == 0) ws_d[(static_cast<size_t>(ci) * a.H + h) * a.D + c] = ex2(s);
+    }
+    __syncthreads();
+    for (int i = tid; i < LC * (DP / 2); i += 128) {
+      const int r = i / (DP / 2), c = (i - r * (DP / 2)) * 2;
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Kh + r * LDK + c));
+      const float w0 = ex2(gsum[16 * DP + c] - (G[r * DP + c] + gsum[(r >> 2) * DP + c]));
+      const float w1 = ex2(gsum[16 * DP + c + 1] - (G[r * DP + c + 1] + gsum[(r >> 2) * DP + c + 1]));
+      uint32_t hi, lo;
+      split2(x.x * w0, x.y * w1, hi, lo);
+      *reinterpret_cast<uint32_t*>(Kh + r * LDK + c) = hi;
+      *reinterpret_cast<uint32_t*>(Kl + r * LDK + c) = lo;
     }
   }
   __syncthreads();
@@ -239,53 +309,80 @@ linear_chunk_u_kernel(const __grid_constant__ LinearArgs a, const int* __restric
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = mt * 16 + g + (e >> 1) * 8, vv = i * 8 + 2 * t + (e & 1);
-        if (d < a.D && v0 + vv < a.V) U[static_cast<size_t>(d) * a.V + vv] = acc[i][e];
+      for (int e = 0; e < 4; e += 2) {
+        const int d = mt * 16 + g + (e >> 1) * 8, vv = i * 8 + 2 * t;
+        float* p = U + static_cast<size_t>(d) * a.V + vv;
+        if (d < a.D && v0 + vv + 1 < a.V && (a.V & 1) == 0) *reinterpret_cast<float2*>(p) = make_float2(acc[i][e], acc[i][e + 1]);
+        else if (d < a.D) {
+          if (v0 + vv < a.V) p[0] = acc[i][e];
+          if (v0 + vv + 1 < a.V) p[1] = acc[i][e + 1];
+        }
       }
   }
 }
 
-// grid (ceil(D * V / 256), H, nseg); 256 threads: one state element each.
-template <int MODE>
-__global__ void __launch_bounds__(256)
+// grid (ceil(D * V / (128 VEC)), H, nseg); 128 threads: VEC consecutive state elements each (V % VEC == 0).
+template <int MODE, int VEC>
+__global__ void __launch_bounds__(128)
 linear_scan_kernel(const __grid_constant__ LinearArgs a, const int* __restrict__ seg_chunk0, float* __restrict__ ws_u,
                    const float* __restrict__ ws_d) {
-  const int h = blockIdx.y, sg = blockIdx.z, e = blockIdx.x * 256 + threadIdx.x;
+  const int h = blockIdx.y, sg = blockIdx.z, e = (blockIdx.x * 128 + threadIdx.x) * VEC;
   const int DV = a.D * a.V;
   const int slot = a.seg[sg * 4], r0 = a.seg[sg * 4 + 1], n = a.seg[sg * 4 + 2];
   const int nch = (n + LC - 1) / LC;
   if (e < DV) {
+    struct Vec { float v[VEC]; };
+    auto ld = [](const float* p) {
+      Vec x;
+      if (VEC == 4) { const float4 t = ldf4(p); x.v[0] = t.x; x.v[VEC > 1 ? 1 : 0] = t.y; x.v[VEC > 2 ? 2 : 0] = t.z; x.v[VEC > 3 ? 3 : 0] = t.w; }
+      if (VEC == 1) x.v[0] = *p;
+      return x;
+    };
+    auto st = [](float* p, const Vec& x) {
+      if (VEC == 4) stf4(p, make_float4(x.v[0], x.v[VEC > 1 ? 1 : 0], x.v[VEC > 2 ? 2 : 0], x.v[VEC > 3 ? 3 : 0]));
+      else *p = x.v[0];
+    };
     float* Sp = a.S + (static_cast<size_t>(slot) * a.H + h) * DV + e;
-    float s = *Sp;
+    Vec s = ld(Sp);
     const size_t cst = static_cast<size_t>(a.H) * DV;
     float* u = ws_u + (static_cast<size_t>(seg_chunk0[sg]) * a.H + h) * DV + e;
     const float* dd = MODE ? ws_d + (static_cast<size_t>(seg_chunk0[sg]) * a.H + h) * a.D + e / a.V : nullptr;
     const float full = MODE ? 0.f : exp2f(a.log2a[h] * LC);
     const float last = MODE ? 0.f : exp2f(a.log2a[h] * (n - (nch - 1) * LC));
-    for (int c0 = 0; c0 < nch; c0 += 8) {                      // eight chunks of loads in flight
-      float x[8], dc[8];
+    constexpr int PF = 8;                                      // chunks of loads in flight: batch c0 + 8 is fetched while c0 is scanned
+    Vec x[PF], nx[PF];
+    float dc[PF], nd[PF];
+    auto fetch = [&](int c0, Vec (&xx)[PF], float (&dx)[PF]) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int c = c0 + i;
-        x[i] = c < nch ? u[c * cst] : 0.f;
-        dc[i] = MODE ? (c < nch ? dd[static_cast<size_t>(c) * a.H * a.D] : 0.f) : (c == nch - 1 ? last : full);
+      for (int i = 0; i < PF; ++i) {
+        const int c = min(c0 + i, nch - 1);
+        xx[i] = ld(u + c * cst);
+        dx[i] = MODE ? dd[static_cast<size_t>(c) * a.H * a.D] : (c == nch - 1 ? last : full);
       }
+    };
+    fetch(0, x, dc);
+    for (int c0 = 0; c0 < nch; c0 += PF) {
+      if (c0 + PF < nch) fetch(c0 + PF, nx, nd);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        if (c0 + i < nch) { u[(c0 + i) * cst] = s; s = fmaf(dc[i], s, x[i]); }
+      for (int i = 0; i < PF; ++i) {
+        if (c0 + i < nch) {
+          st(u + (c0 + i) * cst, s);
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) s.v[k] = fmaf(dc[i], s.v[k], x[i].v[k]);
+        }
+        x[i] = nx[i]; dc[i] = nd[i];
       }
     }
-    if (a.commit) *Sp = s;
+    if (a.commit) st(Sp, s);
   }
   if (MODE == 1 && a.commit && a.h32 != nullptr && blockIdx.x == 0 && h == 0)
-    for (int i = threadIdx.x; i < a.width; i += 256)
+    for (int i = threadIdx.x; i < a.width; i += 128)
       a.carried[static_cast<size_t>(slot) * a.width + i] = a.h32[(static_cast<size_t>(r0) + n - 1) * a.width + i];
 }
 
 template <int DP, int MODE>
 struct ChunkOSmem {
-  static constexpr int LDK = DP + 8, LDR = DP + 2, LDG = DP + 1;
+  static constexpr int LDK = DP + 8, LDR = DP + 2, LDG = DP + 2;      // pairs of channels, rows spread over the banks
   static constexpr int KHL = MODE ? 2 * LC * LDK * 2 : 2 * LC * LDK * 2;            // MODE 0: Q | K;  MODE 1: K^ high | low
   static constexpr int RAW = MODE ? 2 * LC * LDR * 2 : 0;                             // MODE 1: r, k as they are
   static constexpr int G = MODE ? ((LC * LDG * 4 + 15) / 16 * 16) : 0;
@@ -294,7 +391,7 @@ struct ChunkOSmem {
   static constexpr int TOTAL = KHL + RAW + G + DG + VB + SB;
 };
 
-// grid (chunks, H); 128 threads: warp w owns rows 16w .. 16w + 15 of the chunk.
+// grid (chunks, H, ceil(V / 64)); 128 threads: warp w owns rows 16w .. 16w + 15 of the chunk.
 template <int DP, int MODE>
 __global__ void __launch_bounds__(128)
 linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restrict__ chunks, const float* __restrict__ ws_u) {
@@ -305,12 +402,13 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
   __nv_bfloat16* A1 = A0 + LC * LDK;                                     // MODE 0: K;  MODE 1: K^ low
   __nv_bfloat16* Rr = reinterpret_cast<__nv_bfloat16*>(smem_lo + SM::KHL);
   __nv_bfloat16* Kr = Rr + LC * LDR;
-  float* G = reinterpret_cast<float*>(smem_lo + SM::KHL + SM::RAW);      // inclusive running log decay
+  float* G = reinterpret_cast<float*>(smem_lo + SM::KHL + SM::RAW);      // inclusive running log decay, base 2
   float* Dg = reinterpret_cast<float*>(smem_lo + SM::KHL + SM::RAW + SM::G);   // diagonal 16 x 16 blocks
   __nv_bfloat16* Vs = reinterpret_cast<__nv_bfloat16*>(smem_lo + SM::KHL + SM::RAW + SM::G + SM::DG);
   __nv_bfloat16* Sh = Vs + LC * LVS;                                     // [DP][LVS] state entering the chunk, high / low
   __nv_bfloat16* Sl = Sh + DP * LVS;
-  const int ci = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int ci = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * LVT;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int sg = chunks[2 * ci], t0 = chunks[2 * ci + 1] * LC;
   const int n = a.seg[sg * 4 + 2], nv = min(LC, n - t0);
   const size_t r0 = static_cast<size_t>(a.seg[sg * 4 + 1]) + t0;
@@ -319,29 +417,77 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
   const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(a.v) + r0 * a.ldv + h * a.hsv;
   const float l2 = MODE == 0 ? a.log2a[h] : 0.f;
   const int row_lo = warp * 16 + g, row_hi = row_lo + 8;
+  // the state that entered the chunk (this CTA's value columns) as two-term sums
+  const float* Sin = ws_u + (static_cast<size_t>(ci) * a.H + h) * a.D * a.V;
+  auto load_state = [&]() {
+    auto put = [&](int d, int c, float4 x) {
+      uint32_t h0, l0, h1, l1;
+      split2(x.x, x.y, h0, l0);
+      split2(x.z, x.w, h1, l1);
+      *reinterpret_cast<uint2*>(Sh + d * LVS + c) = make_uint2(h0, h1);
+      *reinterpret_cast<uint2*>(Sl + d * LVS + c) = make_uint2(l0, l1);
+    };
+    constexpr int PER = DP * (LVT / 4) / 128, BT = PER < 8 ? PER : 8;
+    if (a.D == DP && v0 + LVT <= a.V && (a.V & 3) == 0) {
+      for (int b0 = 0; b0 < PER; b0 += BT) {
+        float4 x[BT];
+#pragma unroll
+        for (int b = 0; b < BT; ++b) {
+          const int i = tid + (b0 + b) * 128;
+          x[b] = ldf4(Sin + static_cast<size_t>(i / (LVT / 4)) * a.V + v0 + (i % (LVT / 4)) * 4);
+        }
+#pragma unroll
+        for (int b = 0; b < BT; ++b) { const int i = tid + (b0 + b) * 128; put(i / (LVT / 4), (i % (LVT / 4)) * 4, x[b]); }
+      }
+      return;
+    }
+    for (int i = tid; i < DP * (LVT / 4); i += 128) {
+      const int d = i / (LVT / 4), c = (i % (LVT / 4)) * 4;
+      const float* p = Sin + static_cast<size_t>(d) * a.V + v0 + c;
+      float f[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) f[e] = (d < a.D && v0 + c + e < a.V) ? p[e] : 0.f;
+      put(d, c, make_float4(f[0], f[1], f[2], f[3]));
+    }
+  };
   if (MODE == 0) {
     load_rows<DP>(A0, LDK, q, a.ldq, nv, a.D, a.act);
     load_rows<DP>(A1, LDK, k, a.ldk, nv, a.D, a.act);
+    load_state();
+    load_rows<LVT>(Vs, LVS, v + v0, a.ldv, nv, a.V - v0, a.act);
     __syncthreads();
   } else {
-    for (int i = tid; i < LC * DP; i += 128) {
-      const int r = i / DP, c = i - r * DP;
-      const bool in = r < nv && c < a.D;
-      Rr[r * LDR + c] = in ? q[static_cast<size_t>(r) * a.ldq + c] : __float2bfloat16(0.f);
-      Kr[r * LDR + c] = in ? k[static_cast<size_t>(r) * a.ldk + c] : __float2bfloat16(0.f);
-      G[r * LDG + c] = in ? a.logw[(r0 + r) * (static_cast<size_t>(a.H) * a.D) + h * a.D + c] : 0.f;
+    load_state();
+    load_rows<LVT>(Vs, LVS, v + v0, a.ldv, nv, a.V - v0, a.act);
+    load_rows<DP>(Rr, LDR, q, a.ldq, nv, a.D, 0);
+    load_rows<DP>(Kr, LDR, k, a.ldk, nv, a.D, 0);
+    load_decays<DP>(G, LDG, a.logw + r0 * (static_cast<size_t>(a.H) * a.D) + h * a.D, static_cast<size_t>(a.H) * a.D, nv, a.D);
+    __syncthreads();
+    for (int i = tid; i < 4 * DP; i += 128) {                              // running sums of the 16-row blocks, then across them
+      const int b = i / DP, c = i % DP;
+      float s = 0.f;
+#pragma unroll
+      for (int r = 0; r < 16; ++r) { s += G[(b * 16 + r) * LDG + c]; G[(b * 16 + r) * LDG + c] = s; }
     }
     __syncthreads();
-    for (int c = tid; c < DP; c += 128) {
-      float s = 0.f;
-#pragma unroll 8
-      for (int r = 0; r < LC; ++r) { s += G[r * LDG + c]; G[r * LDG + c] = s; }
+    for (int i = tid; i < 3 * DP; i += 128) {
+      const int b = 1 + i / DP, c = i % DP;
+      float add = 0.f;
+      for (int p = 0; p < b; ++p) add += G[(p * 16 + 15) * LDG + c];
+      Dg[i] = add;                                                           // (scratch until the diagonal blocks are formed)
     }
+    __syncthreads();
+    for (int i = tid; i < 48 * DP; i += 128) { const int r = 16 + i / DP, c = i % DP; G[r * LDG + c] += Dg[(r / 16 - 1) * DP + c]; }
     __syncthreads();
     // keys decayed to the end of their own 16-row block
-    for (int i = tid; i < LC * DP; i += 128) {
-      const int r = i / DP, c = i - r * DP;
-      split1(__bfloat162float(Kr[r * LDR + c]) * expf(G[(r | 15) * LDG + c] - G[r * LDG + c]), A0[r * LDK + c], A1[r * LDK + c]);
+    for (int i = tid; i < LC * (DP / 2); i += 128) {
+      const int r = i / (DP / 2), c = (i - r * (DP / 2)) * 2;
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Kr + r * LDR + c));
+      const float2 e = *reinterpret_cast<const float2*>(G + (r | 15) * LDG + c), f = *reinterpret_cast<const float2*>(G + r * LDG + c);
+      uint32_t hi, lo;
+      split2(x.x * ex2(e.x - f.x), x.y * ex2(e.y - f.y), hi, lo);
+      *reinterpret_cast<uint32_t*>(A0 + r * LDK + c) = hi;
+      *reinterpret_cast<uint32_t*>(A1 + r * LDK + c) = lo;
     }
     // diagonal blocks, pair by pair: i > j decayed from j to i - 1, i == j weighted by the bonus
     for (int p = lane; p < 136; p += 32) {
@@ -354,9 +500,16 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
         for (int c = 0; c < a.D; ++c)
           s = fmaf(__bfloat162float(Rr[ri * LDR + c]) * a.u[h * a.D + c], __bfloat162float(Kr[rj * LDR + c]), s);
       } else {
-        for (int c = 0; c < a.D; ++c)
-          s = fmaf(__bfloat162float(Rr[ri * LDR + c]) * __bfloat162float(Kr[rj * LDR + c]),
-                   expf(G[(ri - 1) * LDG + c] - G[rj * LDG + c]), s);
+        float s1 = 0.f;
+#pragma unroll 4
+        for (int c = 0; c < DP; c += 2) {                                  // (channels past D are zero)
+          const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Rr + ri * LDR + c));
+          const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Kr + rj * LDR + c));
+          const float2 e = *reinterpret_cast<const float2*>(G + (ri - 1) * LDG + c), f = *reinterpret_cast<const float2*>(G + rj * LDG + c);
+          s = fmaf(x.x * y.x, ex2(e.x - f.x), s);
+          s1 = fmaf(x.y * y.y, ex2(e.y - f.y), s1);
+        }
+        s += s1;
       }
       Dg[(warp * 16 + i) * 17 + j] = s;
     }
@@ -367,19 +520,14 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int row = (e & 1) ? row_hi : row_lo, c = ks * 16 + 2 * t + (e >> 1) * 8;
-      float x[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const float E = row > 0 ? G[(row - 1) * LDG + c + i] : 0.f;
-        const float ref = ref_row >= 0 ? G[ref_row * LDG + c + i] : 0.f;
-        x[i] = __bfloat162float(Rr[row * LDR + c + i]) * expf(E - ref);
-      }
-      split2(x[0], x[1], hi[e], lo[e]);
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Rr + row * LDR + c));
+      const float2 E = row > 0 ? *reinterpret_cast<const float2*>(G + (row - 1) * LDG + c) : make_float2(0.f, 0.f);
+      const float2 f = ref_row >= 0 ? *reinterpret_cast<const float2*>(G + ref_row * LDG + c) : make_float2(0.f, 0.f);
+      split2(x.x * ex2(E.x - f.x), x.y * ex2(E.y - f.y), hi[e], lo[e]);
     }
   };
   // ---- weights of the keys of this chunk as MMA operands: two-term sums, key blocks 0 .. warp
   uint32_t ph[4][4], pl[4][4];
-  const float p_lo_rows = 0.f; (void)p_lo_rows;
 #pragma unroll
   for (int kb = 0; kb < 4; ++kb) {
 #pragma unroll
@@ -426,15 +574,7 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
     split2(s[1][0], s[1][1], ph[kb][2], pl[kb][2]); split2(s[1][2], s[1][3], ph[kb][3], pl[kb][3]);
   }
   const float dec_lo = MODE == 0 ? exp2f(l2 * (row_lo + 1)) : 1.f, dec_hi = MODE == 0 ? exp2f(l2 * (row_hi + 1)) : 1.f;
-  const float* Sin = ws_u + (static_cast<size_t>(ci) * a.H + h) * a.D * a.V;
-  for (int v0 = 0; v0 < a.V; v0 += LVT) {
-    if (v0) __syncthreads();
-    load_rows<LVT>(Vs, LVS, v + v0, a.ldv, nv, a.V - v0, a.act);
-    for (int i = tid; i < DP * LVT; i += 128) {
-      const int d = i / LVT, c = i - d * LVT;
-      split1((d < a.D && v0 + c < a.V) ? Sin[static_cast<size_t>(d) * a.V + v0 + c] : 0.f, Sh[d * LVS + c], Sl[d * LVS + c]);
-    }
-    __syncthreads();
+  {
     float o[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
@@ -474,9 +614,14 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int row = (e >> 1) ? row_hi : row_lo, c = v0 + i * 8 + 2 * t + (e & 1);
-        if (row < nv && c < a.V) a.o[(r0 + row) * (static_cast<size_t>(a.H) * a.V) + h * a.V + c] = o[i][e];
+      for (int e = 0; e < 4; e += 2) {
+        const int row = e ? row_hi : row_lo, c = v0 + i * 8 + 2 * t;
+        float* p = a.o + (r0 + row) * (static_cast<size_t>(a.H) * a.V) + h * a.V + c;
+        if (row < nv && c + 1 < a.V && (a.V & 1) == 0) *reinterpret_cast<float2*>(p) = make_float2(o[i][e], o[i][e + 1]);
+        else if (row < nv) {
+          if (c < a.V) p[0] = o[i][e];
+          if (c + 1 < a.V) p[1] = o[i][e + 1];
+        }
       }
   }
 }
@@ -486,7 +631,7 @@ static int launch_chunked(const LinearArgs& a, const int* chunks, int n_chunks, 
                           cudaStream_t s) {
   auto ku = linear_chunk_u_kernel<DP, MODE>;
   auto ko = linear_chunk_o_kernel<DP, MODE>;
-  constexpr int SU = (2 * LC * (DP + 8) + LC * LVS) * 2, SO = ChunkOSmem<DP, MODE>::TOTAL;
+  constexpr int SU = (2 * LC * (DP + 8) + LC * LVS) * 2 + (MODE ? (LC + 17) * DP * 4 : 0), SO = ChunkOSmem<DP, MODE>::TOTAL;
   static bool done = false;
   if (!done) {
     cudaFuncSetAttribute(ku, cudaFuncAttributeMaxDynamicSharedMemorySize, SU);
@@ -494,8 +639,9 @@ static int launch_chunked(const LinearArgs& a, const int* chunks, int n_chunks, 
     done = true;
   }
   ku<<<dim3(n_chunks, a.H, (a.V + LVT - 1) / LVT), 128, SU, s>>>(a, chunks, ws_u, ws_d);
-  linear_scan_kernel<MODE><<<dim3((a.D * a.V + 255) / 256, a.H, nseg), 256, 0, s>>>(a, chunk0, ws_u, ws_d);
-  ko<<<dim3(n_chunks, a.H), 128, SO, s>>>(a, chunks, ws_u);
+  if (a.V % 4 == 0) linear_scan_kernel<MODE, 4><<<dim3((a.D * a.V + 511) / 512, a.H, nseg), 128, 0, s>>>(a, chunk0, ws_u, ws_d);
+  else linear_scan_kernel<MODE, 1><<<dim3((a.D * a.V + 127) / 128, a.H, nseg), 128, 0, s>>>(a, chunk0, ws_u, ws_d);
+  ko<<<dim3(n_chunks, a.H, (a.V + LVT - 1) / LVT), 128, SO, s>>>(a, chunks, ws_u);
   return spark_launch_rc("spark_linear_chunked");
 }
 
