@@ -192,15 +192,15 @@ gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
   if (n0 < N) load(w0, w1, kb);                          // in flight while the rows are staged
   // rows past R are left as they are: an MMA column only ever reaches its own row's outputs, which are not stored
   const int KV8 = K >> 3;
-  for (int i0 = threadIdx.x; i0 < R * KV8; i0 += 4 * GEMV_WARPS * 32) {
-    uint4 v[4];
+  for (int i0 = threadIdx.x; i0 < R * KV8; i0 += 2 * GEMV_WARPS * 32) {
+    uint4 v[2];
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
+    for (int u = 0; u < 2; ++u) {
       const int i = i0 + u * GEMV_WARPS * 32, r = i / KV8;
       if (i < R * KV8) v[u] = *reinterpret_cast<const uint4*>(x + static_cast<size_t>(r) * ldx + (i - r * KV8) * 8);
     }
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
+    for (int u = 0; u < 2; ++u) {
       const int i = i0 + u * GEMV_WARPS * 32, r = i / KV8;
       if (i < R * KV8) *reinterpret_cast<uint4*>(xs + r * lds + (i - r * KV8) * 8) = v[u];
     }
@@ -256,6 +256,90 @@ gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
   pdl_trigger();
 }
 
+// Contractions too long for 16 staged rows: K in segments of `kseg` 32-wide chunks, the rows of a segment staged in turn;
+// 16 weight rows per CTA, the 8 warps split every segment and keep their accumulators over all of them.  Segments depend on K
+// only, so a row's result does not change with the batch it is in.
+template <int NT, typename TO>
+__global__ void __launch_bounds__(GEMV_WARPS * 32, NT == 1 ? 2 : 1)
+gemv_long_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W, int ldw,
+                     TO* __restrict__ y, int ldy, int R, int N, int K, int kseg) {
+  extern __shared__ __align__(16) uint8_t smem_gemv[];
+  __shared__ float red[GEMV_WARPS][NT * 4][32];
+  __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem_gemv);     // [NT * 8][kseg * 32 + GEMV_MMA_PAD]
+  const int lds = kseg * 32 + GEMV_MMA_PAD;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int KC = K >> 5, n0 = blockIdx.x * 16;
+  constexpr int BATCH = 8;
+  const uint4* w0 = reinterpret_cast<const uint4*>(W + static_cast<size_t>(min(n0 + g, N - 1)) * ldw) + t;
+  const uint4* w1 = reinterpret_cast<const uint4*>(W + static_cast<size_t>(min(n0 + g + 8, N - 1)) * ldw) + t;
+  uint4 ra[BATCH], rb[BATCH];
+  float acc[NT][4];
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt) { acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f; }
+  pdl_wait();
+  for (int s0 = 0; s0 < KC; s0 += kseg) {
+    const int sn = min(kseg, KC - s0), per = (sn + GEMV_WARPS - 1) / GEMV_WARPS;
+    const int kb = s0 + min(sn, warp * per), ke = s0 + min(sn, warp * per + per);
+    auto load = [&](int kc0) {
+#pragma unroll
+      for (int u = 0; u < BATCH; ++u) {
+        const bool in = kc0 + u < ke;
+        ra[u] = in ? __ldg(w0 + (kc0 + u) * 4) : make_uint4(0u, 0u, 0u, 0u);
+        rb[u] = in ? __ldg(w1 + (kc0 + u) * 4) : make_uint4(0u, 0u, 0u, 0u);
+      }
+    };
+    load(kb);                                            // in flight while the segment's rows are staged
+    if (s0) __syncthreads();
+    const int KV8 = sn * 4;
+    for (int i = threadIdx.x; i < R * KV8; i += GEMV_WARPS * 32) {
+      const int r = i / KV8, kv = i - r * KV8;
+      *reinterpret_cast<uint4*>(xs + r * lds + kv * 8) =
+          *reinterpret_cast<const uint4*>(x + static_cast<size_t>(r) * ldx + s0 * 32 + kv * 8);
+    }
+    __syncthreads();
+    for (int kc0 = kb; kc0 < ke; kc0 += BATCH) {
+      if (kc0 != kb) load(kc0);
+#pragma unroll
+      for (int u = 0; u < BATCH; ++u) {
+        if (kc0 + u < ke) {
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) {
+            const uint4 xb = *reinterpret_cast<const uint4*>(xs + (nt * 8 + g) * lds + (kc0 + u - s0) * 32 + t * 8);
+            gemv_mma16816(acc[nt], ra[u].x, rb[u].x, ra[u].y, rb[u].y, xb.x, xb.y);
+            gemv_mma16816(acc[nt], ra[u].z, rb[u].z, ra[u].w, rb[u].w, xb.z, xb.w);
+          }
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) red[warp][nt * 4 + j][lane] = acc[nt][j];
+  __syncthreads();
+  for (int i = threadIdx.x; i < NT * 4 * 32; i += blockDim.x) {
+    const int slot = i >> 5, ln = i & 31, nt = slot >> 2, j = slot & 3;
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < GEMV_WARPS; ++w) v += red[w][slot][ln];
+    const int r = nt * 8 + 2 * (ln & 3) + (j & 1), n = n0 + (ln >> 2) + (j >> 1) * 8;
+    if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(v);
+  }
+  pdl_trigger();
+}
+
+template <int NT, typename TO>
+static int launch_gemv_long(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K, cudaStream_t s) {
+  auto kern = gemv_long_mma_kernel<NT, TO>;
+  const int KC = K >> 5, nseg = (KC + 127) / 128, kseg = (KC + nseg - 1) / nseg;      // <= 128 chunks: 16 rows in 131 KB
+  const int smem = NT * 8 * (kseg * 32 + GEMV_MMA_PAD) * 2;
+  static bool set = false;
+  if (!set) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); set = true; }
+  const cudaError_t err = spark_launch_pdl(kern, dim3((N + 15) / 16), dim3(GEMV_WARPS * 32), smem, s, dim3(1, 1, 1),
+                                           (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)y, ldy, rows, N, K, kseg);
+  return err == cudaSuccess ? 0 : -4;
+}
+
 template <int NT, typename TO, bool KS>
 static int launch_gemv_wide_as(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K,
                                cudaStream_t s) {
@@ -275,24 +359,25 @@ static int launch_gemv_wide_as(const void* x, int ldx, const void* W, int ldw, v
   return err == cudaSuccess ? 0 : -4;
 }
 
+static bool gemv_wide_rows16(int K) { return 16 * (K + GEMV_MMA_PAD) * 2 <= 200 * 1024; }
+
 // Fewer than 8 x 148 tiles of 16 weight rows: split K over the warps of a CTA instead of giving every warp its own tile
 // (depends on N only, so a row's result does not change with the batch it is in).
 template <int NT, typename TO>
 static int launch_gemv_wide(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K,
                             cudaStream_t s) {
+  if (!gemv_wide_rows16(K)) return launch_gemv_long<NT, TO>(x, ldx, W, ldw, y, ldy, rows, N, K, s);
   return (N + 15) / 16 < 8 * 148 ? launch_gemv_wide_as<NT, TO, true>(x, ldx, W, ldw, y, ldy, rows, N, K, s)
                                  : launch_gemv_wide_as<NT, TO, false>(x, ldx, W, ldw, y, ldy, rows, N, K, s);
 }
 
-// Shapes the wide kernel takes: one item, no activation, no expert tables, K a multiple of 32 and small enough that
-// 8 staged rows fit in shared memory (the choice must not depend on the number of rows: a row's result may not
-// change with the batch it is in).
+// Shapes the wide kernels take: one item, no activation, no expert tables, K a multiple of 32.  The choice (and the one
+// between whole and segmented staging) must not depend on the number of rows: a row's result may not change with the
+// batch it is in.
 static bool gemv_wide_ok(int ldx, int ldw, int items, int N, int K, const int* pe, const int* pr, int act) {
   return items == 1 && !pe && !pr && act == 0 && N >= 2048 && (K & 31) == 0 && (ldx & 7) == 0 && (ldw & 7) == 0 &&
-         8 * (K + GEMV_MMA_PAD) * 2 <= 200 * 1024;
+         K <= 1 << 20;
 }
-// Contractions too long for 16 staged rows run in groups of 8 rows (a row's chain of MMAs is the same either way).
-static bool gemv_wide_rows16(int K) { return 16 * (K + GEMV_MMA_PAD) * 2 <= 200 * 1024; }
 
 }  // namespace spark
 
@@ -306,16 +391,6 @@ extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long 
   if (K % 8 || rows_per_item > 16) return -5;
   if (gemv_wide_ok(ldx, ldw, items, N, K, pair_expert, pair_row, act) &&
       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) == 0) {
-    if (rows_per_item > 8 && !gemv_wide_rows16(K)) {
-      const size_t es = out_f32 ? 4 : 2;
-      for (int r = 0; r < rows_per_item; r += 8) {
-        const int rc = spark_gemv_bf16(static_cast<const uint8_t*>(x) + static_cast<size_t>(r) * ldx * 2, ldx, W, expert_stride, ldw,
-                                       static_cast<uint8_t*>(y) + static_cast<size_t>(r) * ldy * es, ldy, items,
-                                       rows_per_item - r < 8 ? rows_per_item - r : 8, N, K, pair_expert, pair_row, act, limit, out_f32, s);
-        if (rc) return rc;
-      }
-      return 0;
-    }
     if (rows_per_item <= 8)
       return out_f32 ? launch_gemv_wide<1, float>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s)
                      : launch_gemv_wide<1, __nv_bfloat16>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s);

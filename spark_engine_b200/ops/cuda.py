@@ -274,9 +274,12 @@ def gemv_bf16_items(x, ldx, x_item_stride, w, expert_stride, ldw, y, ldy, y_item
     return y
 
 
-def gemv_rows(K: int) -> int:
-    """Rows one GEMV launch takes at contraction length K (a power of two: the staged rows fill shared memory)."""
+def gemv_rows(K: int, N: int = 0) -> int:
+    """Rows one GEMV launch takes at contraction length K (a power of two: the staged rows fill shared memory; projections of
+    2048 rows and more are staged in segments)."""
     r = 16
+    if N >= 2048 and K % 32 == 0:
+        return r
     while r > 1 and r * K * 2 > 200 * 1024:
         r //= 2
     return r
@@ -302,7 +305,7 @@ def dense_linear(x: torch.Tensor, w: torch.Tensor, out_f32: bool = False, out=No
     x = _as_bf16(x)
     if x.stride(1) != 1 or x.stride(0) % 8 or x.data_ptr() % 16:
         x = x.contiguous()
-    if R <= 16 and R <= gemv_rows(K):
+    if R <= 16 and R <= gemv_rows(K, N):
         return gemv_bf16(x, w, out_f32=out_f32, out=out)
     return gemm_bf16(x, w, out_f32, out=out)
 

@@ -171,6 +171,19 @@ def test_simt_product_shapes():
         assert torch.allclose(got, ref, atol=2e-5 * K ** 0.5)
 
 
+@pytest.mark.parametrize("N,K", [(2048, 6400), (2056, 10272), (4100, 7680)])
+def test_long_contractions_of_decode_rows(N, K):
+    """Output products of wide feed-forwards: rows staged in segments; one row's bits do not depend on the others."""
+    from spark_engine_b200.ops import cuda as cu
+    g = torch.Generator().manual_seed(1)
+    x, w = torch.randn(16, K, generator=g).bfloat16().cuda(), (torch.randn(N, K, generator=g) * K ** -0.5).bfloat16().cuda()
+    ref = x.double() @ w.double().T
+    full = cu.dense_linear(x, w, out_f32=True)
+    assert (full.double() - ref).abs().max() < 1e-4
+    for r in (1, 3, 8, 9):
+        assert torch.equal(cu.dense_linear(x[:r], w, out_f32=True), full[:r])
+
+
 def test_rows_do_not_depend_on_the_batch():
     """The same decode rows alone, and beside other sequences whose pages and slots differ: bitwise equal."""
     cfg, T = _setup(MIXED)
