@@ -172,7 +172,7 @@ def main():
         from spark_engine_b200.serving import bench_design
         if args.design != "vabunex":
             raise SystemExit(f"unknown --design {args.design!r} (vabunex)")
-        return bench_design.run(args)
+        return bench_design.run(args, ClockSampler(0))
 
     import torch
     import torch.distributed as dist

@@ -254,18 +254,18 @@ def ds4_style(n_layers: int = 40, weight_format: str = "mx") -> ModelConfig:
 
 
 def vabunex_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 5632, vocab: int = 65536) -> ModelConfig:
-    """Vabunex at the layer sizes of a small real model: one latent-attention, two lightning and one wkv layer per period,
-    the first period run twice."""
-    kinds = [("latent", "lightning", "lightning", "wkv")[i % 4] for i in range(n_layers)]
+    """Vabunex at the layer sizes of a small real model: two lightning, one wkv and one latent-attention layer per period of
+    four, the second period run twice."""
+    kinds = [("lightning", "wkv", "lightning", "latent")[i % 4] for i in range(n_layers)]
     heads = hidden // 128
     mixers = {"latent": LatentConfig(n_heads=heads, head_dim=128, v_dim=128, q_rank=768, kv_rank=512, rope_dim=64,
-                                     rope_theta=5e4, scale=192 ** -0.5),
+                                     rope_theta=1e6, scale=192 ** -0.5),
               "lightning": LightningConfig(n_heads=heads, head_dim=128, v_dim=128,
                                            decay=[1.0 - 2.0 ** (-1 - 8 * h / heads) for h in range(heads)]),
               "wkv": WkvConfig(n_heads=hidden // 64, head_dim=64, decay_rank=64)}
     return ModelConfig(name="vabunex-style", family="vabunex", n_layers=n_layers, layer_types=kinds, hidden=hidden, vocab=vocab,
                        norm_eps=1e-5, layer_specs=[LayerSpec(k, dataclasses.replace(mixers[k]), ffn) for k in kinds],
-                       loop=LoopConfig(0, min(4, n_layers), 2), norm_one_plus=True, embed_scale=float(hidden) ** 0.5,
+                       loop=LoopConfig(min(4, n_layers), min(8, n_layers), 2), norm_one_plus=True, embed_scale=float(hidden) ** 0.5,
                        weight_format="dense")
 
 

@@ -87,6 +87,8 @@ class WkvMixer(_ParallelMixer):
         c = self.c
         self.n = c.n_heads * c.head_dim
         self.S = torch.zeros(n_slots, c.n_heads, c.head_dim, c.head_dim, device=device, dtype=torch.float32)
+        # prompts multiply a two-term bf16 sum of the rank activations: [w2 | w2]
+        self.w2x2 = torch.cat((w["w2"], w["w2"]), 1).contiguous() if dtype == torch.bfloat16 else None
         self.carried = torch.zeros(n_slots, cfg.hidden, device=device, dtype=torch.float32)     # the previous token's row
 
     def reset(self, slot: int):
@@ -102,7 +104,7 @@ class WkvMixer(_ParallelMixer):
         w = self.w
         mix = ops.token_shift(h32, self.carried, w["mu"], plan, self.dtype)              # r k v g w
         rkvg = ops.linear_stack(mix[:4], w["rkvg"])
-        logw = ops.channel_decay(ops.linear(mix[4], w["w1"], out_f32=True), w["w2"], w["w0"], self.n)
+        logw = ops.channel_decay(ops.linear(mix[4], w["w1"], out_f32=True), w["w2"], w["w0"], self.n, self.w2x2)
         o = self._state(rkvg, logw, h32, plan, commit)
         self.pending = None if commit else ((rkvg, logw, h32), plan)
         ff = ops.linear(h, w["ff"]) if self.F else None

@@ -402,10 +402,10 @@ def linear_stack(xs, w):
     return torch.einsum("nrk,nok->nro", xs, w.to(xs.dtype))
 
 
-def channel_decay(z, w2, w0, n: int):
+def channel_decay(z, w2, w0, n: int, w2x2=None):
     """log decay -exp(w2 tanh(z) + w0) [R, n] in fp32."""
     if use_kernels(z):
-        return block_ops().channel_decay(z, w2, w0, n)
+        return block_ops().channel_decay(z, w2, w0, n, w2x2)
     return -torch.exp(torch.tanh(z.float()) @ w2.float().t() + w0)
 
 

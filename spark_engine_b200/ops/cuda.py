@@ -77,9 +77,31 @@ _SIGS = {
     "spark_exl3_had_rows": [vp, i32, vp, vp, i32, i32, i32, i32, vp, vp, i64],
 }
 
+# parallel blocks (ops/parallel_block.py)
+_LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32]
+_SIGS.update({
+    "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, i32, vp, vp],
+    "spark_add_norm_rows": [vp, vp, vp, vp, vp, i32, i32, f32, i32, i32, vp],
+    "spark_token_shift": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, vp],
+    "spark_channel_decay": [vp, i32, vp, i32, i32, vp, vp, i32, i32, i32, vp],
+    "spark_neg_exp_bias": [vp, vp, i32, i32, vp],
+    "spark_tanh_split": [vp, i32, vp, i32, i32, vp],
+    "spark_gate_concat": [vp, i32, i32, i32, vp, f32, vp, i32, i32, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp],
+    "spark_linear_seq": _LIN + [i32, i32, vp],
+    "spark_linear_chunked": _LIN + [i32, vp, i32, vp, vp, vp, vp],
+    "spark_latent_prep": [vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp, i32, vp, vp,
+                          i32, vp, vp],
+    "spark_latent_qrope": [vp, i32, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp, i32, i32, vp],
+    "spark_latent_gather": [vp, i32, vp, i32, i32, vp, i32, vp, vp],
+    "spark_latent_rows": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
+    "spark_latent_prefill": [vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
+    "spark_mla_attn_paged": [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
+})
+
 
 # kernels launched by one call of each entry point (for the launch counter)
-_KERNELS_PER_CALL = {"spark_attn_decode": 2, "spark_moe_sort": 3, "spark_argmax": 2, "spark_hc_gated_site": 2}
+_KERNELS_PER_CALL = {"spark_attn_decode": 2, "spark_moe_sort": 3, "spark_argmax": 2, "spark_hc_gated_site": 2,
+                     "spark_linear_chunked": 3, "spark_mla_attn_paged": 2}
 _launches = 0
 
 

@@ -6,28 +6,7 @@ from __future__ import annotations
 import torch
 
 from . import cuda as cu
-from .cuda import P, check, f32, i32, i64, lib, scratch, status_word, stream, vp
-
-_LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32]
-cu._SIGS.update({
-    "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, i32, vp, vp],
-    "spark_add_norm_rows": [vp, vp, vp, vp, vp, i32, i32, f32, i32, i32, vp],
-    "spark_token_shift": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, vp],
-    "spark_channel_decay": [vp, i32, vp, i32, i32, vp, vp, i32, i32, i32, vp],
-    "spark_neg_exp_bias": [vp, vp, i32, i32, vp],
-    "spark_tanh_split": [vp, i32, vp, i32, i32, vp],
-    "spark_gate_concat": [vp, i32, i32, i32, vp, f32, vp, i32, i32, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp],
-    "spark_linear_seq": _LIN + [i32, i32, vp],
-    "spark_linear_chunked": _LIN + [i32, vp, i32, vp, vp, vp, vp],
-    "spark_latent_prep": [vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp, i32, vp, vp,
-                          i32, vp, vp],
-    "spark_latent_qrope": [vp, i32, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp, i32, i32, vp],
-    "spark_latent_gather": [vp, i32, vp, i32, i32, vp, i32, vp, vp],
-    "spark_latent_rows": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
-    "spark_latent_prefill": [vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
-    "spark_mla_attn_paged": [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
-})
-cu._KERNELS_PER_CALL.update({"spark_linear_chunked": 3, "spark_mla_attn_paged": 2})
+from .cuda import P, check, lib, scratch, status_word, stream
 
 CHUNK_MIN_ROWS = 32          # segments of at least this many rows take the chunked / flash kernels
 LC = 64                      # rows per chunk of the chunked recurrences
@@ -70,33 +49,20 @@ def token_shift(h32, carried, mu, plan, dtype):
     return out
 
 
-def channel_decay(z, w2, w0, n: int):
-    """z [R, rank] fp32 -> log decay -exp(w2 tanh(z) + w0) [R, n] fp32."""
+def channel_decay(z, w2, w0, n: int, w2x2=None):
+    """z [R, rank] fp32 -> log decay -exp(w2 tanh(z) + w0) [R, n] fp32.  `w2x2`: [w2 | w2] in bf16."""
     R, r = z.shape
-    if w2.dtype == torch.bfloat16 and R >= 64 and 2 * r % 8 == 0:
+    if w2x2 is not None and R >= 64:
         # prompts: tanh as a two-term bf16 sum against [w2 | w2], one tensor-core product
         t = torch.empty(R, 2 * r, dtype=torch.bfloat16, device=z.device)
         check(lib().spark_tanh_split(P(z), z.stride(0), P(t), R, r, stream()), "spark_tanh_split")
-        out = cu.dense_linear(t, _doubled(w2), out_f32=True)
+        out = cu.dense_linear(t, w2x2, out_f32=True)
         check(lib().spark_neg_exp_bias(P(out), P(w0), R, n, stream()), "spark_neg_exp_bias")
         return out
     out = torch.empty(R, n, dtype=torch.float32, device=z.device)
     check(lib().spark_channel_decay(P(z), z.stride(0), P(w2), w2.stride(0), r, P(w0), P(out), R, n, _is32(w2.dtype), stream()),
           "spark_channel_decay")
     return out
-
-
-_twice = {}
-
-
-def _doubled(w):
-    key = (w.data_ptr(), tuple(w.shape))
-    hit = _twice.get(key)
-    if hit is None or hit[0]() is not w:
-        import weakref
-        hit = (weakref.ref(w), torch.cat((w, w), 1).contiguous())
-        _twice[key] = hit
-    return hit[1]
 
 
 GATES = {None: 0, "sigmoid": 1, "silu": 2}

@@ -178,13 +178,14 @@ def kernel_figures(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: 
     return out
 
 
-def run(args) -> int:
+def run(args, clocks) -> int:
     here = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
     try:
         with open(os.path.join(here, "MEASURED_PEAKS.json")) as f:
             peaks = json.load(f)
     except OSError:
         peaks = {}
+    clocks.start()
     sizes = {}
     for name, (hidden, ffn) in SIZES.items():
         cv = vabunex_config(hidden, ffn)
@@ -197,6 +198,7 @@ def run(args) -> int:
     out = {"metric": "vabunex prefill / decode throughput beside the closest existing family at equal size", "design": "vabunex",
            "closest": "KDA + latent attention (GLM-style layer types), sequential pre-norm blocks, dense feed-forward, bf16",
            "dtype": "bf16", "data": "synthetic", "sizes": sizes, "kernels": kernel_figures(peaks),
+           "clocks": clocks.stop(),
            "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")}}
     print(json.dumps(out))
     return 0

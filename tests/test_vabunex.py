@@ -278,7 +278,7 @@ def test_snapshot_moves_a_sequence_to_another_slot():
 def test_switches():
     from spark_engine_b200.config import get_model_config
     mc = get_model_config("vabunex-style", n_layers=5)
-    assert mc.layer_runs() == [0, 1, 2, 3, 0, 1, 2, 3, 4] and mc.layer_specs[3].kind == "wkv"
+    assert mc.layer_runs() == [0, 1, 2, 3, 4, 4] and mc.layer_specs[1].kind == "wkv"
     assert dataclasses.replace(mc).layer_specs
     with pytest.raises(ValueError):
         LLMEngine(mc, {}, EngineConfig(dtype="float8"), device="cuda")
