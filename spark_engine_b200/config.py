@@ -75,12 +75,18 @@ class MoeConfig:
     ffn: int = 128
     n_shared: int = 1
     shared_ffn: int = 0           # 0 -> ffn * n_shared
-    router: str = "softmax"       # softmax | sigmoid_bias | sqrt_softplus
+    router: str = "softmax"       # softmax | sigmoid_bias | sqrt_softplus | softmax_bias (bias: added to the choice scores only)
     route_scale: float = 1.0
     shared_gate: bool = False     # sigmoid(x . w_sg) on the shared expert
     swiglu_limit: float = 0.0     # clamp-SwiGLU limit (0 = off)
     dense_layers: int = 0         # first N layers use a dense MLP of width dense_ffn
     dense_ffn: int = 0
+    act: str = "swiglu"           # swiglu (gate and up matrices) | relu2 (squared relu of a single up matrix)
+    n_identity: int = 0           # router outputs behind the experts' whose "expert" returns its input
+
+    @property
+    def n_routes(self) -> int:
+        return self.n_experts + self.n_identity
 
 
 @dataclass
@@ -114,7 +120,23 @@ class LatentConfig:
     scale: float = 0.125
 
 
-MIXER_CONFIGS = {"lightning": LightningConfig, "wkv": WkvConfig, "latent": LatentConfig}
+@dataclass
+class PagedGqaConfig:
+    """Grouped-query softmax attention over a paged cache, without rotation: short convolutions on q, k and v, soft-capped
+    scores, a learned bias per distance bucket and head, chunked visibility, a sink in the denominator."""
+    n_heads: int = 4
+    n_kv_heads: int = 2
+    head_dim: int = 32
+    v_dim: int = 32
+    conv_k: int = 4               # taps of the causal convolutions (1: the current token only)
+    scale: float = 0.125
+    softcap: float = 0.0          # 0: none
+    bias_buckets: int = 32        # rows of the bias table
+    bias_max: int = 1024          # distance from which on the last row is used
+    chunk: int = 0                # tokens see their own aligned chunk of the sequence (0: everything before them)
+
+
+MIXER_CONFIGS = {"lightning": LightningConfig, "wkv": WkvConfig, "latent": LatentConfig, "gqa": PagedGqaConfig}
 
 
 @dataclass
@@ -123,6 +145,7 @@ class LayerSpec:
     kind: str = "lightning"       # key of MIXER_CONFIGS
     mixer: object = None
     ffn: int = 0                  # width of the dense feed-forward (0 = none)
+    moe: Optional[MoeConfig] = None   # experts instead of the dense feed-forward
 
 
 @dataclass
@@ -136,7 +159,7 @@ class LoopConfig:
 @dataclass
 class ModelConfig:
     name: str = "tiny-hybrid"
-    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex
+    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex | debisun
     n_layers: int = 4
     layer_types: List[str] = field(default_factory=lambda: ["gdn", "gdn", "gdn", "attn"])
     hidden: int = 256
@@ -162,10 +185,13 @@ class ModelConfig:
     kv_dtype: str = "bf16"        # bf16 | fp8
     kv_quant_on_cpu: bool = False  # the CPU runner keeps fp32 caches; set to model the packed FP8 latent rows there too
 
-    layer_specs: List[LayerSpec] = field(default_factory=list)   # per-layer sizes (vabunex); else the shared configs above
+    layer_specs: List[LayerSpec] = field(default_factory=list)   # per-layer sizes; else the shared configs above
     loop: Optional[LoopConfig] = None
+    block: str = "parallel"       # models with layer_specs: parallel (one norm, mixer + feed-forward) | sequential (pre-norm each)
+    norm_kind: str = "rms"        # models with layer_specs: rms | layer (weight and bias)
     norm_one_plus: bool = False   # norm weights are stored around zero
     embed_scale: float = 1.0
+    side_dim: int = 0             # width of the per-layer token input (0 = none)
 
     def layer_runs(self) -> List[int]:
         """Weight layer of every layer run, in order."""
@@ -186,8 +212,10 @@ class ModelConfig:
                 d[key] = cls(**d[key])
         if isinstance(d.get("loop"), dict):
             d["loop"] = LoopConfig(**d["loop"])
+        moe = lambda m: MoeConfig(**m) if isinstance(m, dict) else m
         d["layer_specs"] = [x if isinstance(x, LayerSpec) else
-                            LayerSpec(x["kind"], MIXER_CONFIGS[x["kind"]](**x["mixer"]), x["ffn"]) for x in d.get("layer_specs", [])]
+                            LayerSpec(x["kind"], MIXER_CONFIGS[x["kind"]](**x["mixer"]), x["ffn"], moe(x.get("moe")))
+                            for x in d.get("layer_specs", [])]
         return ModelConfig(**d)
 
     @staticmethod
@@ -269,6 +297,22 @@ def vabunex_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 5632, vocab
                        weight_format="dense")
 
 
+def debisun_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 8192, vocab: int = 65536, experts: int = 64, top: int = 4,
+                  chunk: int = 2048) -> ModelConfig:
+    """Debisun at the layer sizes of a small real model: a dense first layer, then experts (a quarter as wide, plus identity
+    experts and a shared one), heads of 128 with four queries per key / value head."""
+    heads = hidden // 128
+    mixer = PagedGqaConfig(n_heads=heads, n_kv_heads=max(1, heads // 4), head_dim=128, v_dim=128, conv_k=4, scale=128 ** -0.5,
+                           softcap=50.0, bias_buckets=32, bias_max=1024, chunk=chunk)
+    moe = MoeConfig(n_experts=experts, n_identity=experts // 4, top_k=top, ffn=ffn // 4, n_shared=1, shared_ffn=ffn // 4,
+                    router="softmax_bias", route_scale=1.5, shared_gate=True, act="relu2")
+    specs = [LayerSpec("gqa", dataclasses.replace(mixer), 0 if i else ffn, dataclasses.replace(moe) if i else None)
+             for i in range(n_layers)]
+    return ModelConfig(name="debisun-style", family="debisun", n_layers=n_layers, layer_types=["gqa"] * n_layers, hidden=hidden,
+                       vocab=vocab, norm_eps=1e-5, layer_specs=specs, block="sequential", norm_kind="layer", side_dim=hidden // 16,
+                       weight_format="dense")
+
+
 def scaled_down(cfg: ModelConfig, hidden: int = 256, n_layers: int = 4, vocab: int = 1024) -> ModelConfig:
     """Same layer types, small dimensions: the CPU test shape of a large config."""
     c = dataclasses.replace(cfg)
@@ -310,7 +354,7 @@ class EngineConfig:
     """Engine switches (CLI `--flag`, JSON file, `SPARK_<NAME>` environment fallback)."""
     model: str = "tiny-hybrid"
     numerics: str = "deterministic"      # deterministic | fast (multimem hardware reductions)
-    dtype: str = "bfloat16"              # activations and dense weights on the device: bfloat16 | float32 (vabunex only)
+    dtype: str = "bfloat16"              # activations and dense weights on the device: bfloat16 | float32 (models with layer_specs)
     tp: int = 1
     ep: int = 1
     max_seqs: int = 8
@@ -367,6 +411,7 @@ PRESETS = {
     "glm-style": glm_style,
     "ds4-style": ds4_style,
     "vabunex-style": vabunex_style,
+    "debisun-style": debisun_style,
 }
 
 

@@ -1,0 +1,29 @@
+// Activation applied to a product's fp32 accumulators before they are stored (GEMV, tcgen05 GEMM and FP32-unit GEMM share it).
+//   1  squared relu
+//   2  gelu_tanh(v) * table[ids[row]][off + col]: a row of an embedding table gated by the product (columns from `n` on, and
+//      ids outside the table, give 0)
+#pragma once
+#include "rows.cuh"
+
+namespace spark {
+
+struct OutAct {
+  int kind;
+  int ld, off, n, rows, f32;        // the table: row stride, first column, valid columns, rows, element type
+  const void* table;
+  const int* ids;
+};
+
+__device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.f); return v * v; }
+
+__device__ __forceinline__ float out_act(const OutAct& a, float v, int row, int col) {
+  if (a.kind == 0) return v;
+  if (a.kind == 1) return relu2_f(v);
+  const int id = a.ids[row];
+  if (col >= a.n || id < 0 || id >= a.rows) return 0.f;
+  const size_t i = static_cast<size_t>(id) * a.ld + a.off + col;
+  const float e = a.f32 ? static_cast<const float*>(a.table)[i] : __bfloat162float(static_cast<const __nv_bfloat16*>(a.table)[i]);
+  return gelu_tanh_f(v) * e;
+}
+
+}  // namespace spark

@@ -1,8 +1,9 @@
-// Row kernels of the parallel block (one norm feeds a mixer and a feed-forward, both outputs are added together), for
-// bf16 and fp32 activations.  The residual stream, norms, token-shift state and decays are fp32 in both.
+// Row kernels of the models whose layers carry their own sizes, for bf16 and fp32 activations.  The residual stream, norms,
+// token-shift state and decays are fp32 in both.
 //
 //   embed_scaled      x = table[id] * scale
-//   add_norm_rows     res += delta;  h = RMSNorm(res) * (w or 1 + w), optionally a second fp32 copy of h
+//   row_update        res += an update (plain rows or the slots of a routed feed-forward; per-channel scale, or RMS-normed);
+//                     h = norm of the new residual (RMS, layer norm, or the residual itself), optionally an fp32 copy of h
 //   token_shift       five mixes h + (h' - h) mu_s of the current and the previous row of the sequence
 //   channel_decay     log decay  -exp(W2 tanh(z) + w0)  per channel, fp32 throughout
 //   gate_concat       [ group-RMSNorm(o) * w * gate(g) | gelu(gate) * up ]: the input row of the block's single output
@@ -23,47 +24,163 @@ embed_scaled_kernel(const TW* __restrict__ table, const int* __restrict__ ids, f
     out[static_cast<size_t>(r) * H + i] = ok ? ldf(table + static_cast<size_t>(id) * H + i) * scale : 0.f;
 }
 
-template <typename TO>
-__global__ void __launch_bounds__(256)
-add_norm_rows_kernel(const float* __restrict__ delta, float* __restrict__ res, const float* __restrict__ w,
-                     TO* __restrict__ out, float* __restrict__ out32, int H, float eps, int one_plus) {
+struct RowUpdate {
+  float* res;                                   // [R, H], in place
+  // the update: `delta` rows, or sum over slots of wts * y (expert outputs) + sg * shared + self_w * self_x, or nothing
+  const float* delta;
+  const float* y; const int* inv; const float* wts; const int* ids;      // pair p's row of y: inv[p] (inv null: p); ids[p] < 0: none
+  const float* shared; const float* sg; const float* self_w; const void* self_x;
+  const float* scale;                           // [H] (null: 1)
+  const float* post_w;                          // [H]: the update is RMS-normed with this weight (null: it is not)
+  // the new rows
+  const float* w; const float* b;
+  void* out; float* out32;
+  int H, slots, norm, one_plus;                 // norm: 0 none, 1 RMS (w or 1 + w), 2 layer norm (w, b)
+  float eps, post_eps;
+};
+
+// One CTA per row.  NV > 0: every thread keeps NV groups of four channels in registers (blockDim * 4 * NV >= H, H % 4 == 0,
+// 16-byte aligned rows); NV == 0: any width, values are read again.
+template <typename T, int NV>
+__global__ void __launch_bounds__(NV <= 2 ? 1024 : 256)
+row_update_kernel(const __grid_constant__ RowUpdate a) {
   __shared__ float sh[32];
   pdl_wait();
-  const size_t row = static_cast<size_t>(blockIdx.x) * H;
-  float* x = res + row;
-  const bool vec = (H & 3) == 0;
-  float ss = 0.f;
-  if (vec) {
-    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
-      float4 v = ldf4(x + i);
-      if (delta != nullptr) {
-        const float4 d = ldf4(delta + row + i);
-        v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
-        stf4(x + i, v);
+  const int r = blockIdx.x, H = a.H, t = threadIdx.x, nt = blockDim.x;
+  const size_t row = static_cast<size_t>(r) * H;
+  float* x = a.res + row;
+  const bool has = a.delta != nullptr || a.y != nullptr;
+  const float sg = a.shared ? (a.sg ? a.sg[r] : 1.f) : 0.f, own = a.self_w ? a.self_w[r] : 0.f;
+  const T* sx = static_cast<const T*>(a.self_x) + (a.self_w ? row : 0);
+  T* out = static_cast<T*>(a.out) + row;
+  const float one = a.one_plus ? 1.f : 0.f;
+  if constexpr (NV > 0) {
+    float4 v[NV], u[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (t + k * nt) * 4;
+      u[k] = v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i >= H) continue;
+      v[k] = ldf4(x + i);
+      if (a.delta) u[k] = ldf4(a.delta + row + i);
+      else if (a.y) {
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s0 = 0; s0 < a.slots; s0 += 4) {           // four slots' rows in flight, added in slot order
+          float4 p[4]; float w[4];
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            const int pi = r * a.slots + s0 + q;
+            const bool live = s0 + q < a.slots && a.ids[pi] >= 0;
+            w[q] = live ? a.wts[pi] : 0.f;
+            p[q] = live ? __ldcg(reinterpret_cast<const float4*>(a.y + static_cast<size_t>(a.inv ? a.inv[pi] : pi) * H + i))
+                        : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            s.x = fmaf(w[q], p[q].x, s.x); s.y = fmaf(w[q], p[q].y, s.y); s.z = fmaf(w[q], p[q].z, s.z); s.w = fmaf(w[q], p[q].w, s.w);
+          }
+        }
+        if (own != 0.f) {
+          const float4 p = ldf4(sx + i);
+          s.x = fmaf(own, p.x, s.x); s.y = fmaf(own, p.y, s.y); s.z = fmaf(own, p.z, s.z); s.w = fmaf(own, p.w, s.w);
+        }
+        if (a.shared) {
+          const float4 p = ldf4(a.shared + row + i);
+          s.x = fmaf(sg, p.x, s.x); s.y = fmaf(sg, p.y, s.y); s.z = fmaf(sg, p.z, s.z); s.w = fmaf(sg, p.w, s.w);
+        }
+        u[k] = s;
       }
-      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;
+    }
+    const float ps = a.post_w ? 1.f / sqrtf(block_sum_all(ss, sh) / H + a.post_eps) : 1.f;
+    float sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (t + k * nt) * 4;
+      if (i >= H) continue;
+      if (has) {
+        float4 m = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (a.scale) m = ldf4(a.scale + i);
+        if (a.post_w) { const float4 p = ldf4(a.post_w + i); m.x *= ps * p.x; m.y *= ps * p.y; m.z *= ps * p.z; m.w *= ps * p.w; }
+        v[k].x += u[k].x * m.x; v[k].y += u[k].y * m.y; v[k].z += u[k].z * m.z; v[k].w += u[k].w * m.w;
+        stf4(x + i, v[k]);
+      }
+      sum += a.norm == 2 ? v[k].x + v[k].y + v[k].z + v[k].w : v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+    float mean = 0.f, rs = 1.f;
+    if (a.norm) {
+      sum = block_sum_all(sum, sh) / H;
+      if (a.norm == 2) {
+        mean = sum;
+        float q = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+          if ((t + k * nt) * 4 >= H) continue;
+          const float dx = v[k].x - mean, dy = v[k].y - mean, dz = v[k].z - mean, dw = v[k].w - mean;
+          q += dx * dx + dy * dy + dz * dz + dw * dw;
+        }
+        sum = block_sum_all(q, sh) / H;
+      }
+      rs = 1.f / sqrtf(sum + a.eps);
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (t + k * nt) * 4;
+      if (i >= H) continue;
+      float4 y = v[k];
+      if (a.norm) {
+        const float4 g = ldf4(a.w + i);
+        y = make_float4((y.x - mean) * rs * (one + g.x), (y.y - mean) * rs * (one + g.y), (y.z - mean) * rs * (one + g.z),
+                        (y.w - mean) * rs * (one + g.w));
+        if (a.norm == 2) { const float4 b = ldf4(a.b + i); y.x += b.x; y.y += b.y; y.z += b.z; y.w += b.w; }
+      }
+      if (a.out) stf4(out + i, y);
+      if (a.out32) stf4(a.out32 + row + i, y);
     }
   } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    auto update = [&](int i) {
+      if (a.delta) return a.delta[row + i];
+      float s = 0.f;
+      for (int k = 0; k < a.slots; ++k) {
+        const int pi = r * a.slots + k;
+        if (a.ids[pi] >= 0) s = fmaf(a.wts[pi], a.y[static_cast<size_t>(a.inv ? a.inv[pi] : pi) * H + i], s);
+      }
+      if (own != 0.f) s = fmaf(own, ldf(sx + i), s);
+      if (a.shared) s = fmaf(sg, a.shared[row + i], s);
+      return s;
+    };
+    float ps = 1.f;
+    if (has && a.post_w) {
+      float ss = 0.f;
+      for (int i = t; i < H; i += nt) { const float u = update(i); ss = fmaf(u, u, ss); }
+      ps = 1.f / sqrtf(block_sum_all(ss, sh) / H + a.post_eps);
+    }
+    float sum = 0.f;
+    for (int i = t; i < H; i += nt) {
       float v = x[i];
-      if (delta != nullptr) { v += delta[row + i]; x[i] = v; }
-      ss += v * v;
+      if (has) {
+        v += update(i) * (a.scale ? a.scale[i] : 1.f) * (a.post_w ? ps * a.post_w[i] : 1.f);
+        x[i] = v;
+      }
+      sum += a.norm == 2 ? v : v * v;
     }
-  }
-  const float rs = 1.f / sqrtf(block_sum_all(ss, sh) / H + eps);
-  const float one = one_plus ? 1.f : 0.f;
-  if (vec) {
-    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
-      const float4 v = ldf4(x + i), g = ldf4(w + i);
-      const float4 y = make_float4(v.x * rs * (one + g.x), v.y * rs * (one + g.y), v.z * rs * (one + g.z), v.w * rs * (one + g.w));
-      if (out != nullptr) stf4(out + row + i, y);
-      if (out32 != nullptr) stf4(out32 + row + i, y);
+    float mean = 0.f, rs = 1.f;
+    if (a.norm) {
+      sum = block_sum_all(sum, sh) / H;
+      if (a.norm == 2) {
+        mean = sum;
+        float q = 0.f;
+        for (int i = t; i < H; i += nt) { const float d = x[i] - mean; q = fmaf(d, d, q); }
+        sum = block_sum_all(q, sh) / H;
+      }
+      rs = 1.f / sqrtf(sum + a.eps);
     }
-  } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float y = x[i] * rs * (one + w[i]);
-      if (out != nullptr) stf(out + row + i, y);
-      if (out32 != nullptr) out32[row + i] = y;
+    for (int i = t; i < H; i += nt) {
+      float y = x[i];
+      if (a.norm) y = (y - mean) * rs * (one + a.w[i]) + (a.norm == 2 ? a.b[i] : 0.f);
+      if (a.out) stf(out + i, y);
+      if (a.out32) a.out32[row + i] = y;
     }
   }
 }
@@ -255,11 +372,25 @@ extern "C" int spark_embed_scaled(const void* table, const int* ids, float* out,
   return spark_launch_rc(__func__);
 }
 
-extern "C" int spark_add_norm_rows(const float* delta, float* res, const float* w, void* out, float* out32, int R, int H,
-                                   float eps, int one_plus, int f32, cudaStream_t s) {
+extern "C" int spark_row_update(const RowUpdate* u, int R, int f32, cudaStream_t s) {
   if (R <= 0) return 0;
-  SPARK_BY_TYPE(f32, spark_launch_pdl(add_norm_rows_kernel<T>, dim3(R), dim3(256), 0, s, dim3(1, 1, 1), delta, res, w, (T*)out,
-                                      out32, H, eps, one_plus))
+  if (u->y && (u->slots <= 0 || !u->wts || !u->ids)) return -5;
+  if ((u->norm && !u->w) || (u->norm == 2 && !u->b) || (u->self_w && !u->self_x)) return -5;
+  const uintptr_t al = reinterpret_cast<uintptr_t>(u->res) | reinterpret_cast<uintptr_t>(u->delta) | reinterpret_cast<uintptr_t>(u->y) |
+                       reinterpret_cast<uintptr_t>(u->shared) | reinterpret_cast<uintptr_t>(u->self_x) | reinterpret_cast<uintptr_t>(u->scale) |
+                       reinterpret_cast<uintptr_t>(u->post_w) | reinterpret_cast<uintptr_t>(u->w) | reinterpret_cast<uintptr_t>(u->b) |
+                       reinterpret_cast<uintptr_t>(u->out) | reinterpret_cast<uintptr_t>(u->out32);
+  const int groups = u->H / 4, warps = (groups + 31) / 32 * 32;
+  int th = warps < 256 ? warps : 256;                       // many rows: 256 threads each; few rows: up to 1024
+  if (R < 148 && groups <= 2048) th = warps < 1024 ? warps : 1024;
+  const int nv = th > 0 ? (groups + th - 1) / th : 0;
+#define SPARK_ROWUP(NV) SPARK_BY_TYPE(f32, spark_launch_pdl(row_update_kernel<T, NV>, dim3(R), dim3(NV ? th : (u->H >= 4096 ? 1024 : 256)), 0, s, dim3(1, 1, 1), *u))
+  if ((u->H & 3) || (al & 15) || nv > 8) { SPARK_ROWUP(0) }
+  else if (nv <= 1) { SPARK_ROWUP(1) }
+  else if (nv <= 2) { SPARK_ROWUP(2) }
+  else if (nv <= 4) { SPARK_ROWUP(4) }
+  else { SPARK_ROWUP(8) }
+#undef SPARK_ROWUP
   return spark_launch_rc(__func__);
 }
 

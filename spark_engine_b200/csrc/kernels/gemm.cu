@@ -84,6 +84,25 @@ extern "C" int spark_gemm_bf16(const void* A, const void* B, void* C, int M, int
   return launch<128, EpiStoreBf16, false>(tA, tB, g, EpiStoreBf16{(__nv_bfloat16*)C, ldc, N}, grid, stream);
 }
 
+// The same product with an activation on the accumulators (squared relu, or a token row gated by the product), bf16 C.
+extern "C" int spark_gemm_bf16_act(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc,
+                                   const OutAct* act, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  CUtensorMap tA, tB;
+  int r = make_tmap_bf16(&tA, A, M, K, lda, 128);
+  if (r) return r;
+  r = make_tmap_bf16(&tB, B, N, K, ldb, 128);
+  if (r) return r;
+  GemmArgs g{};
+  g.M = M; g.N = N; g.K = K; g.status = status; g.ab_fmt = 1;
+  const int mt = (M + GEMM_BM - 1) / GEMM_BM, bn = N > 128 && mt * ((N + 255) / 256) >= num_sms() ? 256 : 128;
+  g.num_n_tiles = (N + bn - 1) / bn; g.num_tiles = mt * g.num_n_tiles;
+  const int grid = g.num_tiles < num_sms() ? g.num_tiles : num_sms();
+  const EpiActBf16 epi{(__nv_bfloat16*)C, ldc, N, *act};
+  return bn == 256 ? launch<256, EpiActBf16, false>(tA, tB, g, epi, grid, stream)
+                   : launch<128, EpiActBf16, false>(tA, tB, g, epi, grid, stream);
+}
+
 // SwiGLU-fused: C[M,F] = act(A B_gate^T) * (A B_up^T) with B = [gate rows (F) | up rows (F)], F % 128 == 0.
 extern "C" int spark_gemm_bf16_swiglu(const void* A, const void* B, void* C, int M, int F, int K, int lda, int ldb,
                                       int ldc, float limit, int* status, cudaStream_t stream) {
@@ -105,6 +124,7 @@ extern "C" int spark_gemm_bf16_swiglu(const void* A, const void* B, void* C, int
 // expert order; tile_list[i] = {a_row0, row_end, expert, 0}; *tile_count m-tiles are valid.
 //   mode 0: C[rows, N] fp32 = A B_e^T          (down projection; combine sums slots later)
 //   mode 1: C[rows, F] bf16 = swiglu(A B_e^T)  (B_e = [gate | up], N = F)
+//   mode 2: C[rows, N] bf16 = max(A B_e^T, 0)^2
 extern "C" int spark_gemm_grouped_bf16(const void* A, const void* B, void* C, int total_rows, int N, int K,
                                        int lda, int ldb, int ldc, int n_experts, int b_rows_per_expert,
                                        const void* tile_list, const int* tile_count, int max_m_tiles, int mode,
@@ -123,6 +143,17 @@ extern "C" int spark_gemm_grouped_bf16(const void* A, const void* B, void* C, in
     if (N % 128) return -5;
     g.gate_up_F = N; g.num_n_tiles = N / 128; g.num_tiles = max_m_tiles * g.num_n_tiles;
     return launch<256, EpiSwigluBf16, true>(tA, tB, g, EpiSwigluBf16{(__nv_bfloat16*)C, ldc, N, limit}, num_sms(), stream);
+  }
+  if (mode == 2) {
+    OutAct a{};
+    a.kind = 1;
+    const EpiActBf16 epi{(__nv_bfloat16*)C, ldc, N, a};
+    if (N % 256 == 0) {
+      g.num_n_tiles = N / 256; g.num_tiles = max_m_tiles * g.num_n_tiles;
+      return launch<256, EpiActBf16, true>(tA, tB, g, epi, num_sms(), stream);
+    }
+    g.num_n_tiles = (N + 127) / 128; g.num_tiles = max_m_tiles * g.num_n_tiles;
+    return launch<128, EpiActBf16, true>(tA, tB, g, epi, num_sms(), stream);
   }
   if (N % 256 == 0) {
     g.num_n_tiles = N / 256; g.num_tiles = max_m_tiles * g.num_n_tiles;

@@ -13,6 +13,7 @@
 // its mma.sync grouped GEMMs (engine-rs/shim/moe_exl3.cuh:521-1233); none of those has a tcgen05 path.
 #pragma once
 #include "../common/comm.cuh"
+#include "../common/out_act.cuh"
 
 namespace spark {
 
@@ -298,6 +299,25 @@ struct EpiSwigluBf16 {
   __device__ __forceinline__ void operator()(const TileCoord& tc, int row, int col, const float (&v)[32]) const {
     EpiStoreBf16 st{C, ldc, N};
     st(tc, row, col, v);
+  }
+};
+
+// Plain product with an activation on the accumulators -> bf16 (out_act.cuh).
+struct EpiActBf16 {
+  static constexpr bool kWarpTile = false;
+  __nv_bfloat16* C; int ldc; int N; OutAct a;
+  __device__ __forceinline__ void cta_done(int) const {}
+  __device__ __forceinline__ float act(float g, float u) const { return g; }
+  __device__ __forceinline__ void operator()(const TileCoord& tc, int row, int col, const float (&v)[32]) const {
+    float y[32];
+    if (a.kind == 1) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) y[i] = relu2_f(v[i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) y[i] = out_act(a, v[i], row, col + i);
+    }
+    EpiStoreBf16{C, ldc, N}(tc, row, col, y);
   }
 };
 

@@ -6,7 +6,7 @@
 // The `item` dimension (blockIdx.y) turns it into the MoE decode GEMV: item i multiplies its own
 // activation row by expert pair_expert[i]'s matrix.
 // Replaces engine-rs/shim/gemv.cu:8-72, qwen_f16.cu:14-258, dataflow.cu:772 bf16w_rows.
-#include "../common/decode.cuh"
+#include "../common/out_act.cuh"
 
 namespace spark {
 
@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(GEMV_WARPS * 32)
 gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W,
                  long long expert_stride, int ldw, TO* __restrict__ y, int ldy, int rows_per_item, int N, int K,
                  const int* __restrict__ pair_expert, const int* __restrict__ pair_row, int act, float limit,
-                 long long x_item_stride, long long y_item_stride, int cpc) {
+                 long long x_item_stride, long long y_item_stride, int cpc, const OutAct oact) {
   extern __shared__ __align__(16) uint8_t smem_gemv[];
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem_gemv);     // [RB][K]
   const int item = blockIdx.y;
@@ -109,8 +109,8 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
     for (int r = 0; r < RB; ++r) {
       if (r < R) {
         TO* yr = y + static_cast<size_t>(yr0 + r) * ldy;
-        yr[n0] = static_cast<TO>(acc0[r]);
-        if (two) yr[n0 + 1] = static_cast<TO>(acc1[r]);
+        yr[n0] = static_cast<TO>(out_act(oact, acc0[r], r, n0));
+        if (two) yr[n0 + 1] = static_cast<TO>(out_act(oact, acc1[r], r, n0 + 1));
       }
     }
   }
@@ -119,7 +119,7 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
 
 template <int RB, typename TO>
 static int launch_gemv(const void* x, int ldx, const void* W, long long es, int ldw, void* y, int ldy, int items,
-                       int rows, int N, int K, const int* pe, const int* pr, int act, float limit, cudaStream_t s,
+                       int rows, int N, int K, const int* pe, const int* pr, int act, float limit, const OutAct& oact, cudaStream_t s,
                        long long xis = 0, long long yis = 0) {
   auto kern = gemv_bf16_kernel<RB, TO>;
   const int smem = RB * K * 2;
@@ -135,7 +135,7 @@ static int launch_gemv(const void* x, int ldx, const void* W, long long es, int 
   dim3 grid((groups + cpc - 1) / cpc, items);
   const cudaError_t err = spark_launch_pdl(kern, grid, dim3(GEMV_WARPS * 32), smem, s, dim3(1, 1, 1),
                                            (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, es, ldw, (TO*)y, ldy, rows, N, K,
-                                           pe, pr, act, limit, xis, yis, cpc);
+                                           pe, pr, act, limit, xis, yis, cpc, oact);
   return err == cudaSuccess ? 0 : -4;
 }
 
@@ -161,7 +161,7 @@ __device__ __forceinline__ void gemv_mma16816(float (&c)[4], uint32_t a0, uint32
 template <int NT, typename TO, bool KS>
 __global__ void __launch_bounds__(GEMV_WARPS * 32, NT == 1 ? 3 : 2)      // <= 85 registers: three CTAs of loads in flight per SM
 gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W, int ldw,
-                     TO* __restrict__ y, int ldy, int R, int N, int K, int cpc) {
+                     TO* __restrict__ y, int ldy, int R, int N, int K, int cpc, const OutAct oact) {
   extern __shared__ __align__(16) uint8_t smem_gemv[];
   __shared__ float red[KS ? GEMV_WARPS : 1][NT * 4][32];
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem_gemv);     // [NT * 8][K + GEMV_MMA_PAD]
@@ -239,7 +239,7 @@ gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
 #pragma unroll
         for (int w = 0; w < GEMV_WARPS; ++w) v += red[w][slot][ln];
         const int r = nt * 8 + 2 * (ln & 3) + (j & 1), n = n0 + (ln >> 2) + (j >> 1) * 8;
-        if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(v);
+        if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(out_act(oact, v, r, n));
       }
     } else {
       // accumulator (g, t): weight rows n0 + g and n0 + g + 8, activation rows nt * 8 + 2t and + 1
@@ -248,7 +248,7 @@ gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int r = nt * 8 + 2 * t + (j & 1), n = n0 + g + (j >> 1) * 8;
-          if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(acc[nt][j]);
+          if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(out_act(oact, acc[nt][j], r, n));
         }
       }
     }
@@ -262,7 +262,7 @@ gemv_wide_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
 template <int NT, typename TO>
 __global__ void __launch_bounds__(GEMV_WARPS * 32, NT == 1 ? 2 : 1)
 gemv_long_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W, int ldw,
-                     TO* __restrict__ y, int ldy, int R, int N, int K, int kseg) {
+                     TO* __restrict__ y, int ldy, int R, int N, int K, int kseg, const OutAct oact) {
   extern __shared__ __align__(16) uint8_t smem_gemv[];
   __shared__ float red[GEMV_WARPS][NT * 4][32];
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem_gemv);     // [NT * 8][kseg * 32 + GEMV_MMA_PAD]
@@ -323,26 +323,27 @@ gemv_long_mma_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bf
 #pragma unroll
     for (int w = 0; w < GEMV_WARPS; ++w) v += red[w][slot][ln];
     const int r = nt * 8 + 2 * (ln & 3) + (j & 1), n = n0 + (ln >> 2) + (j >> 1) * 8;
-    if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(v);
+    if (r < R && n < N) y[static_cast<size_t>(r) * ldy + n] = static_cast<TO>(out_act(oact, v, r, n));
   }
   pdl_trigger();
 }
 
 template <int NT, typename TO>
-static int launch_gemv_long(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K, cudaStream_t s) {
+static int launch_gemv_long(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K, const OutAct& oact,
+                            cudaStream_t s) {
   auto kern = gemv_long_mma_kernel<NT, TO>;
   const int KC = K >> 5, nseg = (KC + 127) / 128, kseg = (KC + nseg - 1) / nseg;      // <= 128 chunks: 16 rows in 131 KB
   const int smem = NT * 8 * (kseg * 32 + GEMV_MMA_PAD) * 2;
   static bool set = false;
   if (!set) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); set = true; }
   const cudaError_t err = spark_launch_pdl(kern, dim3((N + 15) / 16), dim3(GEMV_WARPS * 32), smem, s, dim3(1, 1, 1),
-                                           (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)y, ldy, rows, N, K, kseg);
+                                           (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)y, ldy, rows, N, K, kseg, oact);
   return err == cudaSuccess ? 0 : -4;
 }
 
 template <int NT, typename TO, bool KS>
 static int launch_gemv_wide_as(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K,
-                               cudaStream_t s) {
+                               const OutAct& oact, cudaStream_t s) {
   auto kern = gemv_wide_mma_kernel<NT, TO, KS>;
   const int smem = NT * 8 * (K + GEMV_MMA_PAD) * 2;
   if (smem > 200 * 1024) return -6;
@@ -355,7 +356,7 @@ static int launch_gemv_wide_as(const void* x, int ldx, const void* W, int ldw, v
   if (cpc < 1) cpc = 1;
   dim3 grid((groups + cpc - 1) / cpc);
   const cudaError_t err = spark_launch_pdl(kern, grid, dim3(GEMV_WARPS * 32), smem, s, dim3(1, 1, 1),
-                                           (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)y, ldy, rows, N, K, cpc);
+                                           (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)y, ldy, rows, N, K, cpc, oact);
   return err == cudaSuccess ? 0 : -4;
 }
 
@@ -365,10 +366,10 @@ static bool gemv_wide_rows16(int K) { return 16 * (K + GEMV_MMA_PAD) * 2 <= 200 
 // (depends on N only, so a row's result does not change with the batch it is in).
 template <int NT, typename TO>
 static int launch_gemv_wide(const void* x, int ldx, const void* W, int ldw, void* y, int ldy, int rows, int N, int K,
-                            cudaStream_t s) {
-  if (!gemv_wide_rows16(K)) return launch_gemv_long<NT, TO>(x, ldx, W, ldw, y, ldy, rows, N, K, s);
-  return (N + 15) / 16 < 8 * 148 ? launch_gemv_wide_as<NT, TO, true>(x, ldx, W, ldw, y, ldy, rows, N, K, s)
-                                 : launch_gemv_wide_as<NT, TO, false>(x, ldx, W, ldw, y, ldy, rows, N, K, s);
+                            const OutAct& oact, cudaStream_t s) {
+  if (!gemv_wide_rows16(K)) return launch_gemv_long<NT, TO>(x, ldx, W, ldw, y, ldy, rows, N, K, oact, s);
+  return (N + 15) / 16 < 8 * 148 ? launch_gemv_wide_as<NT, TO, true>(x, ldx, W, ldw, y, ldy, rows, N, K, oact, s)
+                                 : launch_gemv_wide_as<NT, TO, false>(x, ldx, W, ldw, y, ldy, rows, N, K, oact, s);
 }
 
 // Shapes the wide kernels take: one item, no activation, no expert tables, K a multiple of 32.  The choice (and the one
@@ -386,23 +387,24 @@ using namespace spark;
 // items x rows_per_item rows; K % 8 == 0; out_f32 selects fp32 or bf16 output.
 extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long expert_stride, int ldw, void* y, int ldy,
                                int items, int rows_per_item, int N, int K, const int* pair_expert, const int* pair_row,
-                               int act, float limit, int out_f32, cudaStream_t s) {
+                               int act, float limit, int out_f32, const OutAct* out, cudaStream_t s) {
   if (items <= 0 || rows_per_item <= 0) return 0;
+  const OutAct oact = out ? *out : OutAct{};
   if (K % 8 || rows_per_item > 16) return -5;
   if (gemv_wide_ok(ldx, ldw, items, N, K, pair_expert, pair_row, act) &&
       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15) == 0) {
     if (rows_per_item <= 8)
-      return out_f32 ? launch_gemv_wide<1, float>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s)
-                     : launch_gemv_wide<1, __nv_bfloat16>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s);
-    return out_f32 ? launch_gemv_wide<2, float>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s)
-                   : launch_gemv_wide<2, __nv_bfloat16>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, s);
+      return out_f32 ? launch_gemv_wide<1, float>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, oact, s)
+                     : launch_gemv_wide<1, __nv_bfloat16>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, oact, s);
+    return out_f32 ? launch_gemv_wide<2, float>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, oact, s)
+                   : launch_gemv_wide<2, __nv_bfloat16>(x, ldx, W, ldw, y, ldy, rows_per_item, N, K, oact, s);
   }
 #define SPARK_GEMV_CASE(RB)                                                                                          \
   if (rows_per_item <= RB)                                                                                           \
     return out_f32 ? launch_gemv<RB, float>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N, K,       \
-                                            pair_expert, pair_row, act, limit, s)                                    \
+                                            pair_expert, pair_row, act, limit, oact, s)                                    \
                    : launch_gemv<RB, __nv_bfloat16>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N,  \
-                                                    K, pair_expert, pair_row, act, limit, s);
+                                                    K, pair_expert, pair_row, act, limit, oact, s);
   SPARK_GEMV_CASE(1)
   SPARK_GEMV_CASE(2)
   SPARK_GEMV_CASE(4)
@@ -424,9 +426,9 @@ extern "C" int spark_gemv_bf16_items(const void* x, int ldx, long long x_item_st
 #define SPARK_GEMV_ITEMS(RB)                                                                                         \
   if (rows_per_item <= RB)                                                                                           \
     return out_f32 ? launch_gemv<RB, float>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N, K,       \
-                                            pair_expert, nullptr, 0, 0.f, s, x_item_stride, y_item_stride)           \
+                                            pair_expert, nullptr, 0, 0.f, OutAct{}, s, x_item_stride, y_item_stride)           \
                    : launch_gemv<RB, __nv_bfloat16>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N,  \
-                                                    K, pair_expert, nullptr, 0, 0.f, s, x_item_stride, y_item_stride);
+                                                    K, pair_expert, nullptr, 0, 0.f, OutAct{}, s, x_item_stride, y_item_stride);
   SPARK_GEMV_ITEMS(1)
   SPARK_GEMV_ITEMS(2)
   SPARK_GEMV_ITEMS(4)

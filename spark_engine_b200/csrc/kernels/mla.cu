@@ -18,7 +18,7 @@
 // Reference: engine-rs/shim/latent.cu (sparse_latent*, latent_tc16*, merge_latent), ds41_attn.cu:90-424,
 // engine-rs/src/mla_latent.rs:36-38,196-248, dsa.rs:127-230; FP8 rows: latent.cu:25-47.
 #include <cuda_fp8.h>
-#include "../common/ptx.cuh"
+#include "../common/split_merge.cuh"
 
 namespace spark {
 
@@ -384,77 +384,6 @@ mla_decode_kernel(const __nv_bfloat16* __restrict__ q_full,      // [R, H, KW]
   asm volatile("cp.async.wait_all;" ::: "memory");               // the query copy, if every split was empty
 }
 
-// grid (R, ceil(H / hpc)); 256 threads.  Splits merged in ascending order; `sink` (per head, optional) joins the
-// denominator.  A CTA owns `hpc` heads of one row: the per-head weights of the splits are computed once into shared
-// memory, then the threads sweep the hpc x L outputs with 16-byte loads.  The launcher picks hpc so that a decode
-// round of a few rows still fills the SMs (one head per CTA), while a prefill chunk keeps one CTA per row.
-__global__ void __launch_bounds__(256)
-mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int nsplit, const float* __restrict__ sink,
-                 int H, int L, int hpc, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gate, int ldg,
-                 const int* __restrict__ rows) {
-  // gate (optional): one logit per head in the row's gate columns, the head's output is scaled by its sigmoid
-  // The statistics of a head's splits are reduced by one warp (split s in lane s % 32, so empty trailing splits do not
-  // change a bit of the result).
-  extern __shared__ float wts[];                        // [hpc][nsplit]: exp(m_s - M) / l
-  __shared__ int live_s;                                // splits that hold visible tokens
-  if (threadIdx.x == 0) live_s = 0;
-  __syncthreads();
-  const int r = blockIdx.x, h0 = blockIdx.y * hpc;
-  const int nh = min(hpc, H - h0);
-  const int lane = threadIdx.x & 31;
-  for (int hl = threadIdx.x >> 5; hl < nh; hl += blockDim.x >> 5) {
-    const int h = h0 + hl;
-    const float2* ml = reinterpret_cast<const float2*>(part_ml) + (static_cast<size_t>(r) * H + h) * nsplit;
-    float M = sink ? sink[h] : -INFINITY;
-    int live = 0;
-    for (int s = lane; s < nsplit; s += 32) {
-      const float m = ml[s].x;
-      M = fmaxf(M, m);
-      if (m != -INFINITY) live = s + 1;
-    }
-    M = warp_max(M);
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) live = max(live, __shfl_xor_sync(0xffffffffu, live, o));
-    float l = 0.f;
-    for (int s = lane; s < live; s += 32) {
-      const float2 v = ml[s];
-      if (v.x != -INFINITY) l += __expf(v.x - M) * v.y;
-    }
-    l = warp_sum(l) + (sink ? __expf(sink[h] - M) : 0.f);
-    float inv = 1.f / l;
-    if (gate) inv /= 1.f + expf(-__bfloat162float(gate[static_cast<size_t>(rows ? rows[r] : r) * ldg + h]));
-    for (int s = lane; s < live; s += 32) {
-      const float m = ml[s].x;
-      wts[hl * nsplit + s] = m != -INFINITY ? __expf(m - M) * inv : 0.f;
-    }
-    for (int s = live + lane; s < nsplit; s += 32) wts[hl * nsplit + s] = 0.f;
-    if (lane == 0) atomicMax(&live_s, live);
-  }
-  __syncthreads();
-  const int L4 = L >> 2;
-  for (int i = threadIdx.x; i < nh * L4; i += blockDim.x) {
-    const int hl = i / L4, d = (i - hl * L4) * 4, h = h0 + hl;
-    const size_t pb = (static_cast<size_t>(r) * H + h) * nsplit;
-    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    const int ns = live_s;
-    for (int s0 = 0; s0 < ns; s0 += 8) {                 // eight partial rows in flight
-      float4 pv[8];
-#pragma unroll
-      for (int u = 0; u < 8; ++u) pv[u] = __ldcg(reinterpret_cast<const float4*>(part_o + (pb + min(s0 + u, ns - 1)) * L + d));
-#pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const float w = s0 + u < ns ? wts[hl * nsplit + s0 + u] : 0.f;
-        const float4 p = pv[u];
-        if (w == 0.f) continue;                         // (an empty split's partial rows are not initialised)
-        o.x = fmaf(w, p.x, o.x); o.y = fmaf(w, p.y, o.y); o.z = fmaf(w, p.z, o.z); o.w = fmaf(w, p.w, o.w);
-      }
-    }
-    const __nv_bfloat162 b0 = __floats2bfloat162_rn(o.x, o.y), b1 = __floats2bfloat162_rn(o.z, o.w);
-    uint2 ov; ov.x = *reinterpret_cast<const uint32_t*>(&b0); ov.y = *reinterpret_cast<const uint32_t*>(&b1);
-    *reinterpret_cast<uint2*>(out + (static_cast<size_t>(r) * H + h) * L + d) = ov;
-  }
-}
-
 }  // namespace spark
 
 using namespace spark;
@@ -524,14 +453,8 @@ static int mla_attn(const void* q_full, const void* lat, const int* pos, const l
   if (splitp) { if (HM == 1) SPARK_MLA_DEC(1, true); else if (HM == 2) SPARK_MLA_DEC(2, true); else SPARK_MLA_DEC(4, true); }
   else { if (HM == 1) SPARK_MLA_DEC(1, false); else if (HM == 2) SPARK_MLA_DEC(2, false); else SPARK_MLA_DEC(4, false); }
 #undef SPARK_MLA_DEC
-  int hpc = H;                                          // heads per merge CTA: enough CTAs for two per SM when rows are few
-  while (hpc > 1 && (R * ((H + hpc - 1) / hpc) < 296 || hpc * nsplit * 4 > 48 * 1024)) hpc = (hpc + 1) / 2;
-  if (hpc * nsplit * 4 > 48 * 1024) return -6;
-  const int L4 = kv_lora >> 2;
-  const int mthreads = hpc * L4 >= 256 ? 256 : ((hpc * L4 + 31) / 32 * 32);   // whole warps
-  mla_merge_kernel<<<dim3(R, (H + hpc - 1) / hpc), mthreads, hpc * nsplit * 4, s>>>(part_o, part_ml, nsplit, sink, H, kv_lora, hpc,
-                                                                                  (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, ldg,
-                                                                                  pg.rows);
+  const int rc = launch_split_merge(part_o, part_ml, nsplit, sink, R, H, kv_lora, out, gate, ldg, pg.rows, 0, s);
+  if (rc) return rc;
   return spark_launch_rc("spark_mla_attn");
 }
 

@@ -15,15 +15,17 @@ namespace spark {
 constexpr int ROUTE_THREADS = 256;
 constexpr int ROUTE_MAXE_PER_THREAD = 4;     // up to 1024 experts
 
-// kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias
+// kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias (the bias enters the choice only).
+// The last n_self of the E router outputs are identity experts: they leave -1 in `ids` and their weight in self_w[row].
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int kind, const float* __restrict__ bias,
                  float scale, int shared_gate, float* __restrict__ wts, int* __restrict__ ids,
-                 int* __restrict__ pair_row, float* __restrict__ sg, int e_lo, int e_hi) {
+                 int* __restrict__ pair_row, float* __restrict__ sg, int e_lo, int e_hi, int n_self, float* __restrict__ self_w) {
   __shared__ float rv[ROUTE_THREADS / 32];
   __shared__ int ri[ROUTE_THREADS / 32];
   __shared__ float bv; __shared__ int bidx;
   __shared__ float sel_p[32];
+  __shared__ int sel_self[32];
   const int r = blockIdx.x, t = threadIdx.x, warp = t >> 5, lane = t & 31;
   const float* x = logits + static_cast<size_t>(r) * ld;
   float p[ROUTE_MAXE_PER_THREAD], s[ROUTE_MAXE_PER_THREAD];
@@ -34,7 +36,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
     p[j] = e < E ? x[e] : -INFINITY;
     mx = fmaxf(mx, p[j]);
   }
-  if (kind == 0) {
+  if (kind == 0 || kind == 3) {
     mx = warp_max(mx);
     if (lane == 0) rv[warp] = mx;
     __syncthreads();
@@ -55,7 +57,11 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
     for (int w = 0; w < ROUTE_THREADS / 32; ++w) sum += rv[w];
     __syncthreads();
 #pragma unroll
-    for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) { p[j] = p[j] / sum; s[j] = p[j]; }
+    for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) {
+      p[j] = p[j] / sum;
+      s[j] = p[j];
+      if (kind == 3 && t + j * ROUTE_THREADS < E) s[j] += bias[t + j * ROUTE_THREADS];
+    }
   } else {
 #pragma unroll
     for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) {
@@ -96,6 +102,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
 #pragma unroll
       for (int jj = 0; jj < ROUTE_MAXE_PER_THREAD; ++jj) if (jj == j) { bp = p[jj]; s[jj] = -INFINITY; }
       sel_p[k] = bp;
+      sel_self[k] = win >= E - n_self;
       // expert-parallel ranks keep only their own experts [e_lo, e_hi): others become -1 (skipped downstream)
       ids[static_cast<size_t>(r) * top_k + k] = (win >= e_lo && win < e_hi) ? win - e_lo : -1;
       if (pair_row) pair_row[static_cast<size_t>(r) * top_k + k] = r;
@@ -106,7 +113,13 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
     float sum = 0.f;
     for (int k = 0; k < top_k; ++k) sum += sel_p[k];
     sum = fmaxf(sum, 1e-20f);
-    for (int k = 0; k < top_k; ++k) wts[static_cast<size_t>(r) * top_k + k] = sel_p[k] / sum * scale;
+    float own = 0.f;
+    for (int k = 0; k < top_k; ++k) {
+      const float w = sel_p[k] / sum * scale;
+      wts[static_cast<size_t>(r) * top_k + k] = w;
+      if (sel_self[k]) own += w;
+    }
+    if (self_w) self_w[r] = own;
     if (shared_gate) sg[r] = 1.f / (1.f + expf(-x[E]));
   }
 }
@@ -123,7 +136,7 @@ struct RouterArgs {
   const __nv_bfloat16* x; int ldx;           // [R, K]
   const __nv_bfloat16* Wg; int ldw;          // [E (+1), K]
   float* logits; int ld;                     // scratch [R, ld]
-  int R, K, E, top_k, kind;                  // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias
+  int R, K, E, top_k, kind;                  // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias
   const float* bias; float scale; int shared_gate;
   int slots;                                 // top_k, or top_k + 1 when the shared expert is a pair
   int shared_expert;                         // index of the shared expert in the local stack (slot top_k)
@@ -131,6 +144,7 @@ struct RouterArgs {
   float* wts; int* ids; int* pair_row;       // [R, slots]
   float* sg;                                 // optional [R]: shared gate (when the shared expert is NOT a pair)
   int* counter;
+  int n_self; float* self_w;                 // identity experts: the last n_self outputs, their weight per row [R]
 };
 
 constexpr int ROUTER_RB = 16;
@@ -254,6 +268,23 @@ moe_router_topk_kernel(const __grid_constant__ RouterArgs a) {
       // softmax -> top-k -> renormalise: the softmax denominator cancels, so experts are ranked by their logits and
       // only the k winners are exponentiated
       mx = warp_max(mx);
+    } else if (a.kind == 3) {
+      // the bias is added to the probabilities, so the ranking needs the denominator
+      mx = warp_max(mx);
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < EPL; ++j) {
+        p[j] = p[j] == -INFINITY ? 0.f : expf(p[j] - mx);
+        sum += p[j];
+      }
+      sum = warp_sum(sum);
+#pragma unroll
+      for (int j = 0; j < EPL; ++j) {
+        const int e = lane + 32 * j;
+        const bool in = j < nj && e < a.E;
+        p[j] = p[j] / sum;
+        s[j] = in ? p[j] + a.bias[e] : -INFINITY;
+      }
     } else {
 #pragma unroll
       for (int j = 0; j < EPL; ++j) {
@@ -289,6 +320,14 @@ moe_router_topk_kernel(const __grid_constant__ RouterArgs a) {
       tot += wp;                                            // slot order, identical on every lane
     }
     tot = fmaxf(tot, 1e-20f);
+    if (a.self_w) {
+      float own = 0.f;
+      for (int k = 0; k < a.top_k; ++k) {                   // slot order, as the combine adds the others
+        const float w = __shfl_sync(0xffffffffu, selp, k) / tot * a.scale;
+        if (__shfl_sync(0xffffffffu, seli, k) >= a.E - a.n_self) own += w;
+      }
+      if (lane == 0) a.self_w[r] = own;
+    }
     const size_t o = static_cast<size_t>(r) * a.slots;
     if (lane < a.top_k) {
       a.wts[o + lane] = selp / tot * a.scale;
@@ -496,10 +535,10 @@ using namespace spark;
 
 extern "C" int spark_moe_route(const float* logits, int ld, int R, int E, int top_k, int kind, const float* bias,
                                float scale, int shared_gate, float* wts, int* ids, int* pair_row, float* sg,
-                               cudaStream_t s, int e_lo, int e_hi) {
+                               cudaStream_t s, int e_lo, int e_hi, int n_self, float* self_w) {
   if (R <= 0) return 0;
-  if (E > ROUTE_THREADS * ROUTE_MAXE_PER_THREAD || top_k > 32) return -5;
-  moe_route_kernel<<<R, ROUTE_THREADS, 0, s>>>(logits, ld, E, top_k, kind, bias, scale, shared_gate, wts, ids, pair_row, sg, e_lo, e_hi);
+  if (E > ROUTE_THREADS * ROUTE_MAXE_PER_THREAD || top_k > 32 || top_k > E || (kind == 3 && !bias)) return -5;
+  moe_route_kernel<<<R, ROUTE_THREADS, 0, s>>>(logits, ld, E, top_k, kind, bias, scale, shared_gate, wts, ids, pair_row, sg, e_lo, e_hi, n_self, self_w);
   return spark_launch_rc(__func__);
 }
 
@@ -537,11 +576,14 @@ extern "C" int spark_moe_combine(float* res, const void* y, int y_f32, const int
 extern "C" int spark_moe_router_topk(const void* x, int ldx, const void* Wg, int ldw, float* logits,
                                      int ld, int R, int K, int E, int top_k, int kind, const float* bias, float scale,
                                      int shared_gate, int slots, int shared_expert, int e_lo, int e_hi, int rank, int world,
-                                     float* wts, int* ids, int* pair_row, float* sg, int* counter, cudaStream_t s) {
+                                     float* wts, int* ids, int* pair_row, float* sg, int* counter, int n_self, float* self_w,
+                                     cudaStream_t s) {
   if (R <= 0) return 0;
-  if (R > ROUTER_RB || E > 1024 || top_k > 32 || (K & 7) || slots < top_k || slots > top_k + 1 || ld < E + (shared_gate ? 1 : 0))
+  if (R > ROUTER_RB || E > 1024 || top_k > 32 || (K & 7) || slots < top_k || slots > top_k + 1 || ld < E + (shared_gate ? 1 : 0) ||
+      top_k > E || (kind == 3 && !bias))
     return -5;
   RouterArgs a;
+  a.n_self = n_self; a.self_w = self_w;
   a.x = (const __nv_bfloat16*)x; a.ldx = ldx;
   a.Wg = (const __nv_bfloat16*)Wg; a.ldw = ldw; a.logits = logits; a.ld = ld;
   a.R = R; a.K = K; a.E = E; a.top_k = top_k; a.kind = kind; a.bias = bias; a.scale = scale; a.shared_gate = shared_gate;

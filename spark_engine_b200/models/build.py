@@ -227,8 +227,13 @@ def decode_step_bytes(W, cfg: ModelConfig, rows: int) -> int:
     total = nbytes(W["lm_head"]) + nbytes(W["final_norm"]) + rows * cfg.hidden * 2
     for i in cfg.layer_runs():
         lw = W["layers"][i]
-        if "post_norm" not in lw:                # parallel block: one norm, everything dense (prompts' up-projection not read)
-            total += nbytes(lw["in_norm"]) + sum(nbytes(t) for k, t in lw["mix"].items() if k != "kv_up")
+        if cfg.layer_specs:                      # everything dense is read (except prompts' up-projection), and the chosen experts
+            total += sum(nbytes(t) for k, t in lw.items() if k not in ("mix", "mlp"))
+            total += sum(nbytes(t) for k, t in lw["mix"].items() if k != "kv_up")
+            c = cfg.layer_specs[i].moe
+            for k, t in lw["mlp"].items():
+                share = min(1.0, rows * c.top_k / c.n_routes) if c is not None and k in ("w_up", "w_down") else 1.0
+                total += int(nbytes(t) * share)
             continue
         total += nbytes(lw["mix"]) + nbytes(lw["in_norm"]) + nbytes(lw["post_norm"])
         m = lw["mlp"]

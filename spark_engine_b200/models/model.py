@@ -617,12 +617,15 @@ class MlaMixer:
 
 # ============================================================================= MLP / MoE
 class MoeBlock:
-    def __init__(self, cfg: ModelConfig, w: dict):
-        self.cfg, self.c, self.w = cfg, cfg.moe, w
+    def __init__(self, cfg: ModelConfig, w: dict, c=None):
+        """`c`: the layer's own MoeConfig (default: the model's)."""
+        self.cfg, self.c, self.w = cfg, c or cfg.moe, w
         self.dense = "dense_gu" in w
 
     def forward(self, h, defer: bool = False):
         c = self.c
+        if "dense_up" in self.w:
+            return ops.linear(ops.linear_relu2(h, self.w["dense_up"]), self.w["dense_down"], out_f32=True)
         if self.dense:
             gu = ops.linear(h, self.w["dense_gu"])
             return ops.linear(ops.swiglu(gu, c.swiglu_limit), self.w["dense_down"])
@@ -665,10 +668,12 @@ class Model:
     def _build_layers(self, lws):
         out = []
         if self.cfg.layer_specs:
-            from .parallel_mixers import build_parallel_mixer
+            from .spec_mixers import build_spec_mixer
             for lw, i in zip(lws, self.cfg.layer_runs()):       # every run of a layer has its own cache or state
-                out.append((lw, build_parallel_mixer(self.cfg, self.cfg.layer_specs[i], lw["mix"], self.n_slots, self.n_pages,
-                                                     self.page, self.page_table, self.device, self.dtype), None))
+                spec = self.cfg.layer_specs[i]
+                mlp = MoeBlock(self.cfg, lw["mlp"], spec.moe) if self.cfg.block == "sequential" and "post_norm" in lw else None
+                out.append((lw, build_spec_mixer(self.cfg, spec, lw["mix"], self.n_slots, self.n_pages, self.page, self.page_table,
+                                                 self.device, self.dtype), mlp))
             return out
         for lw in lws:
             kind = lw["type"]
@@ -723,14 +728,36 @@ class Model:
         return self.page_table[slot, t // self.page].long() * self.page + t % self.page
 
     # -- forward ----------------------------------------------------------------------------
+    def _norm(self, w: dict, name: str) -> ops.RowNorm:
+        """A norm of a model with layer specs."""
+        cfg = self.cfg
+        return ops.RowNorm(w[name], cfg.norm_eps, w[name + "_b"] if cfg.norm_kind == "layer" else None, cfg.norm_one_plus)
+
+    def _spec_block(self, li, lw, mix, mlp, X, pend, plan, commit):
+        """One block of a model with layer specs.  `pend` as in `_block`: every residual update is one launch together with
+        the norm (or the cast) of the rows that its successor reads."""
+        cfg = self.cfg
+        if cfg.block == "parallel":          # `mix` holds the feed-forward too
+            h, X, h32 = ops.add_norm_rows(pend, X, self._norm(lw, "in_norm"), self.dtype, mix.wants_f32_rows)
+            return X, mix.forward(h, plan, self.seqs, commit, h32=h32)
+        h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "in_norm"), self.dtype)
+        pend = ops.Update(mix.forward(h, plan, self.seqs, commit), lw.get("ls1"))
+        if mlp is not None:
+            h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "post_norm"), self.dtype)
+            pend = ops.Update(mlp.forward(h, defer=True), lw.get("ls2"))
+        if "side" in lw:                     # the token's own row of this layer, gated by the residual stream itself
+            s, n = lw["side"], cfg.side_dim
+            x, X, _ = ops.add_norm_rows(pend, X, None, self.dtype)
+            ids = plan.dev["ids32"] if "ids32" in plan.dev else plan.ids
+            g = ops.linear_token_gate(x, s["gate"], self.W["side_embed"], ids, cfg.layer_runs()[li] * n, n)
+            pend = ops.Update(ops.linear(g, s["proj"], out_f32=True), post=ops.RowNorm(s["norm"], cfg.norm_eps))
+        return X, pend
+
     def _block(self, lw, mix, mlp, X, pend, plan, commit):
         """One decoder block.  `pend` is the previous block's MLP output, still to be added to the residual
         (under tensor parallelism it is this rank's partial sum): the add, the all-reduce and this block's
         first RMSNorm happen in one fused op.  Returns (X, new pending output)."""
         cfg, tp = self.cfg, self.tp
-        if cfg.layer_specs:                  # parallel block: `mix` holds the feed-forward too
-            h, X, h32 = ops.add_norm_rows(pend, X, lw["in_norm"], cfg.norm_eps, cfg.norm_one_plus, self.dtype, mix.wants_f32_rows)
-            return X, mix.forward(h, plan, self.seqs, commit, h32=h32)
         if cfg.hc_kind == "none":
             # decode rounds on the device: the MoE combine is deferred into the next residual update (one launch for
             # combine + add + norm; under tensor parallelism the combine happens inside the all-reduce push)
@@ -788,7 +815,10 @@ class Model:
         if taps:
             self.taps = {}
         for li, (lw, mix, mlp) in enumerate(self.layers):
-            X, pend = self._block(lw, mix, mlp, X, pend, plan, commit)
+            if cfg.layer_specs:
+                X, pend = self._spec_block(li, lw, mix, mlp, X, pend, plan, commit)
+            else:
+                X, pend = self._block(lw, mix, mlp, X, pend, plan, commit)
             if taps and li in taps:          # residual stream after layer li (feature taps of a drafter)
                 self.taps[li] = X if (pend is None or cfg.hc_kind != "none") else ops.residual_add(X.clone(), pend)
         if cfg.hc_kind == "gated":
@@ -797,7 +827,7 @@ class Model:
         elif cfg.hc_kind == "mhc":
             X, hn = ops.mhc_final(X, pend, W["final_norm"], cfg.norm_eps, self.tp)
         elif cfg.layer_specs:
-            hn, X, _ = ops.add_norm_rows(pend, X, W["final_norm"], cfg.norm_eps, cfg.norm_one_plus, self.dtype)
+            hn, X, _ = ops.add_norm_rows(pend, X, self._norm(W, "final_norm"), self.dtype)
         else:
             hn, X = ops.add_rmsnorm(pend, X, W["final_norm"], cfg.norm_eps, self.tp)
         if self.tp is not None and getattr(self.tp, "rows_sharded", False):
@@ -872,7 +902,7 @@ class Model:
         block; latent attention: top-k pools x pool), or None when no layer selects.  Up to here dense visibility of the
         committed context (what tree-verification rows use) equals what a decode row sees."""
         lim = None
-        if self.cfg.layer_specs:             # recurrent parallel blocks verify chains only
+        if self.cfg.layer_specs:             # their states and pages verify chains only
             return 0
         for _, mix, _ in self.layers:
             c = getattr(mix, "c", None)

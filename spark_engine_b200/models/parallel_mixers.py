@@ -17,24 +17,14 @@ import torch
 from .. import ops
 from ..config import ModelConfig
 from ..oracle import layers as L
+from .layout import pad
 from .plan import Plan
-from .vabunex import pad
 
 
-class _ParallelMixer:
-    wants_f32_rows = False               # needs the fp32 norm output besides the activation rows
-
-    def __init__(self, cfg: ModelConfig, spec, w: dict, dtype):
-        self.cfg, self.c, self.w, self.dtype, self.eps = cfg, spec.mixer, w, dtype, cfg.norm_eps
-        self.F = spec.ffn
-        self.Fp = pad(spec.ffn, 8)
-        self.pending = None
-
-    def _concat(self, o, n, group, gate, kind, ff, out=None):
-        """cat rows [mixer | feed-forward] for the output product."""
-        off = pad(n, 8)
-        return ops.gate_concat(o, n, group, self.w.get("norm"), self.eps, gate, kind, ff if self.F else None, self.F, off,
-                               off + self.Fp, self.dtype, out)
+class PendingRows:
+    """Slot states that verify rows leave alone: `pending` = (inputs, plan) until the accepted prefix is replayed by
+    `commit_rows(inputs, plan, device row counts)`."""
+    pending = None
 
     def commit(self, accepted: List[List[int]]):
         if self.pending is None:
@@ -42,9 +32,24 @@ class _ParallelMixer:
         args, plan = self.pending
         dev = args[0].device
         for rows in accepted:
-            assert rows == list(range(len(rows))), "recurrent parallel blocks verify chains"
+            assert rows == list(range(len(rows))), "these layers verify chains"
         self.commit_rows(args, plan, torch.tensor([len(r) for r in accepted], dtype=torch.int32, device=dev))
         self.pending = None
+
+
+class _ParallelMixer(PendingRows):
+    wants_f32_rows = False               # needs the fp32 norm output besides the activation rows
+
+    def __init__(self, cfg: ModelConfig, spec, w: dict, dtype):
+        self.cfg, self.c, self.w, self.dtype, self.eps = cfg, spec.mixer, w, dtype, cfg.norm_eps
+        self.F = spec.ffn
+        self.Fp = pad(spec.ffn, 8)
+
+    def _concat(self, o, n, group, gate, kind, ff, out=None):
+        """cat rows [mixer | feed-forward] for the output product."""
+        off = pad(n, 8)
+        return ops.gate_concat(o, n, group, self.w.get("norm"), self.eps, gate, kind, ff if self.F else None, self.F, off,
+                               off + self.Fp, self.dtype, out)
 
 
 class LightningMixer(_ParallelMixer):
@@ -193,13 +198,3 @@ class LatentMixer(_ParallelMixer):
 
     def state_tensors(self):
         return {"lat": self.lat}
-
-
-def build_parallel_mixer(cfg: ModelConfig, spec, w: dict, n_slots: int, n_pages: int, page: int, pages, device, dtype):
-    if spec.kind == "lightning":
-        return LightningMixer(cfg, spec, w, n_slots, device, dtype)
-    if spec.kind == "wkv":
-        return WkvMixer(cfg, spec, w, n_slots, device, dtype)
-    if spec.kind == "latent":
-        return LatentMixer(cfg, spec, w, n_pages, page, pages, device, dtype)
-    raise ValueError(spec.kind)

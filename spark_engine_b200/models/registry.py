@@ -9,8 +9,8 @@ from __future__ import annotations
 
 import importlib
 
-ARCHITECTURES = {"Vabunex": "vabunex"}
-FAMILIES = {"vabunex": "vabunex"}
+ARCHITECTURES = {"Vabunex": "vabunex", "Debisun": "debisun"}
+FAMILIES = {"vabunex": "vabunex", "debisun": "debisun"}
 
 
 def architecture(d: dict):

@@ -21,10 +21,7 @@ from typing import Dict
 import torch
 
 from ..config import LatentConfig, LayerSpec, LightningConfig, LoopConfig, ModelConfig, WkvConfig
-
-
-def pad(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
+from .layout import pad, pad_cols as _cols, stack_rows as _rows, taker
 
 
 # ----------------------------------------------------------------------------- configuration
@@ -61,19 +58,6 @@ def read_config(d: dict) -> ModelConfig:
 
 
 # ----------------------------------------------------------------------------- layout
-def _rows(parts, to: int = 8):
-    """Row blocks stacked, each padded to a multiple of `to` rows."""
-    out = []
-    for t in parts:
-        n = pad(t.shape[0], to) - t.shape[0]
-        out += [t, t.new_zeros(n, t.shape[1])] if n else [t]
-    return torch.cat(out)
-
-
-def _cols(t, n: int):
-    return t if t.shape[-1] == n else torch.cat((t, t.new_zeros(*t.shape[:-1], n - t.shape[-1])), -1)
-
-
 def prepare_layer(raw: Dict[str, torch.Tensor], spec: LayerSpec, hidden: int, dtype) -> dict:
     """`raw`: this layer's tensors by their names behind the layer prefix, on the target device."""
     m = {k[4:]: t for k, t in raw.items() if k.startswith("mix.")}
@@ -150,13 +134,7 @@ def _assemble(cfg: ModelConfig, get, layer, device, dtype) -> dict:
 
 def from_tensors(cfg: ModelConfig, tensors: Dict[str, torch.Tensor], device="cpu", dtype=torch.float32) -> dict:
     """Runner weights from a flat dict of checkpoint tensors (validated against the configuration)."""
-    def get(name, shape=None):
-        if name not in tensors:
-            raise ValueError(f"tensor {name} is missing from the checkpoint")
-        t = tensors[name]
-        if shape is not None and tuple(t.shape) != shape:
-            raise ValueError(f"tensor {name} has shape {tuple(t.shape)}, the configuration says {shape}")
-        return t.to(device)
+    get = taker(tensors, device)
 
     def layer(i):
         spec, p = cfg.layer_specs[i], f"l{i}."

@@ -205,7 +205,7 @@ def count_params(W) -> int:
     return n
 
 
-FP32_KEYS = {"conv", "ape", "norm", "scale", "base", "f_b", "g_b", "mu", "u"}
+FP32_KEYS = {"conv", "conv_t", "dist_bias", "ape", "norm", "scale", "base", "f_b", "g_b", "mu", "u"}
 
 
 def to_device(W, device, dtype=torch.bfloat16):

@@ -68,6 +68,8 @@ def to_tensor(x):
 
 
 def residual_add(res, delta) -> torch.Tensor:
+    if isinstance(delta, Update):
+        return add_norm_rows(delta, res, None, res.dtype)[1]
     res, delta = to_tensor(res), to_tensor(delta)
     if use_kernels(res) and res.dtype == torch.float32 and res.dim() == 2:
         return cuda_ops().residual_add(res, delta)
@@ -120,6 +122,27 @@ def linear(x: torch.Tensor, w, out_f32: bool = False) -> torch.Tensor:
     if use_kernels(x):
         return cuda_ops().dense_linear(x, w)
     return x @ w.to(x.dtype).t()
+
+
+def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """max(x W^T, 0)^2 (the activation is the product's epilogue)."""
+    if use_kernels(x):
+        c = cuda_ops()
+        return c.dense_linear(x, w, act=c.out_act("relu2"))
+    return relu2(x @ w.to(x.dtype).t())
+
+
+def linear_token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, off: int, n: int) -> torch.Tensor:
+    """gelu_tanh(x W^T) * table[ids, off : off + n] (columns from n on are zero; ids outside the table give zero rows)."""
+    if use_kernels(x):
+        c = cuda_ops()
+        return c.dense_linear(x, w, act=c.out_act("token_gate", table, ids.to(torch.int32), off, n))
+    y = gelu_tanh(x @ w.to(x.dtype).t())
+    y[:, n:] = 0
+    inside = (ids >= 0) & (ids < table.shape[0])
+    e = table[torch.where(inside, ids, torch.zeros_like(ids))][:, off: off + n].float() * inside.unsqueeze(1)
+    y[:, :n] *= e
+    return y.to(x.dtype)
 
 
 def linear_pair(x, w_a, w_b):
@@ -188,11 +211,11 @@ def route(h, w, c):
     logits = linear(h, w["gate"]).float()
     sg = None
     if c.shared_gate:
-        sg = torch.sigmoid(logits[:, c.n_experts:])
-        logits = logits[:, : c.n_experts]
-    if c.router == "softmax":
+        sg = torch.sigmoid(logits[:, c.n_routes:])
+        logits = logits[:, : c.n_routes]
+    if c.router in ("softmax", "softmax_bias"):
         p = torch.softmax(logits, -1)
-        sel = p
+        sel = p if c.router == "softmax" else p + w["bias"].float().to(p.device)
     elif c.router == "sigmoid_bias":
         p = torch.sigmoid(logits)
         sel = p + w["bias"].float().to(p.device)
@@ -214,7 +237,8 @@ def moe(h, w, c, defer: bool = False):
     wts, idx, sg = route(h, w, c)
     out = torch.zeros(R, h.shape[1], dtype=torch.float32, device=h.device)
     hf = h.float()
-    wgu, wd = w["w_gu"], w["w_down"]
+    single = c.act == "relu2"                    # one up matrix instead of [gate | up]
+    wgu, wd = w["w_up" if single else "w_gu"], w["w_down"]
     lo, hi = w.get("ep", (0, c.n_experts))       # expert-parallel rank: only its own experts, partial output
     for slot in range(c.top_k):
         for e in idx[:, slot].unique().tolist():
@@ -222,9 +246,14 @@ def moe(h, w, c, defer: bool = False):
                 continue
             rows = (idx[:, slot] == e).nonzero(as_tuple=True)[0]
             gu = hf[rows] @ _expert(wgu, e - lo).t()
-            y = L.swiglu(gu[:, : c.ffn], gu[:, c.ffn:], c.swiglu_limit) @ _expert(wd, e - lo).t()
+            y = (relu2(gu) if single else L.swiglu(gu[:, : c.ffn], gu[:, c.ffn:], c.swiglu_limit)) @ _expert(wd, e - lo).t()
             out[rows] += wts[rows, slot].unsqueeze(1) * y
-    if "s_gu" in w:
+    if c.n_identity:
+        out += (wts * (idx >= c.n_experts)).sum(-1, keepdim=True) * hf
+    if "s_up" in w:
+        sh = linear(relu2(linear(h, w["s_up"])), w["s_down"]).float()
+        out = out + (sg * sh if sg is not None else sh)
+    elif "s_gu" in w:
         gu = linear(h, w["s_gu"]).float()
         Fs = gu.shape[1] // 2
         sh = linear(L.swiglu(gu[:, :Fs], gu[:, Fs:], c.swiglu_limit).to(h.dtype), w["s_down"]).float()
@@ -343,17 +372,63 @@ def ngram_embed(model, X, plan, w):
     return (X.float() + gate * val).to(X.dtype)
 
 
-# ----------------------------------------------------------------------------- parallel block
-def add_norm_rows(delta, res, w, eps, one_plus: bool, dtype, want_f32: bool = False):
-    """res' = res + delta (delta may be None); returns (h = RMSNorm(res') * (w or 1 + w) in `dtype`, res', fp32 h if asked)."""
+# ----------------------------------------------------------------------------- residual updates of models with layer specs
+class RowNorm:
+    """RMS norm (weight w or 1 + w), or with a bias vector a layer norm."""
+
+    def __init__(self, w, eps: float, b=None, one_plus: bool = False):
+        self.w, self.eps, self.b, self.one_plus = w, eps, b, one_plus
+
+    def plain(self, x):
+        return L.rms(x, self.w.float(), self.eps, self.one_plus) if self.b is None else L.layer_norm(x, self.w, self.b, self.eps)
+
+
+class Update:
+    """A block output on its way into the residual stream: `x` (a tensor, or a deferred MoE output), times the per-channel
+    `scale`, or RMS-normed by `post` (a RowNorm) first."""
+
+    def __init__(self, x, scale=None, post: Optional[RowNorm] = None):
+        self.x, self.scale, self.post = x, scale, post
+
+    def plain(self):
+        x = to_tensor(self.x).float()
+        if self.post is not None:
+            x = self.post.plain(x)
+        return x * self.scale if self.scale is not None else x
+
+
+def add_norm_rows(delta, res, norm: Optional[RowNorm], dtype, want_f32: bool = False):
+    """res' = res + delta (None, a tensor or an Update); returns (h = norm(res') in `dtype` (norm None: res' itself), res',
+    fp32 h if asked)."""
     if use_kernels(res):
-        return block_ops().add_norm_rows(delta, res, w, eps, one_plus, dtype, want_f32)
+        return block_ops().add_norm_rows(delta, res, norm, dtype, want_f32)
     if delta is not None:
-        res = res + delta
-    h = L.rms(res.float(), w.float(), eps, one_plus)
+        res = res + (delta.plain() if isinstance(delta, Update) else delta)
+    h = res.float() if norm is None else norm.plain(res.float())
     return h.to(dtype), res, h
 
 
+def relu2(x):
+    return torch.relu(x).square()
+
+
+def paged_gqa(mixer, proj, plan, commit):
+    if use_kernels(proj):
+        from . import paged_attn
+        return paged_attn.mixer(mixer, proj, plan, commit)
+    return None
+
+
+def conv_tail(mixer, proj, plan, n_rows) -> bool:
+    """Advance the convolution tails of the plan's slots by n_rows[i] rows of segment i."""
+    if use_kernels(proj):
+        from . import paged_attn
+        paged_attn.commit_tail(mixer, proj, plan, n_rows)
+        return True
+    return False
+
+
+# ----------------------------------------------------------------------------- parallel block
 def gelu_tanh(x):
     return F.gelu(x.float(), approximate="tanh")
 

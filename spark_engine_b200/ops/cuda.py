@@ -26,15 +26,17 @@ _SIGS = {
     "spark_gemm_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "spark_gemm_bf16_swiglu": [vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp],
     "spark_gemm_grouped_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, i32, f32, i32, vp, vp],
-    "spark_gemm_simt": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, i32, i32, vp],
-    "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, f32, i32, vp],
+    "spark_gemm_bf16_act": [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp],
+    "spark_gemm_simt": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, i32, i32, vp, vp],
+    "spark_gemm_simt_grouped": [vp, i32, vp, i32, i64, vp, i32, i32, i32, vp, vp, i32, vp, i32, i32, i32, vp, vp],
+    "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, f32, i32, vp, vp],
     "spark_gemv_bf16_items": [vp, i32, i64, vp, i64, i32, vp, i32, i64, i32, i32, i32, i32, vp, i32, vp],
     "spark_add_rmsnorm": [vp, i32, vp, vp, vp, i32, i32, f32, i32, vp],
     "spark_rmsnorm_bf16": [vp, vp, vp, i32, i32, f32, i32, vp],
     "spark_embed": [vp, vp, vp, i32, i32, vp, i32, vp],
     "spark_decode_advance": [vp, vp, i32, vp],
     "spark_moe_router_topk": [vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, vp, f32, i32, i32, i32, i32, i32, i32,
-                              i32, vp, vp, vp, vp, vp, vp],
+                              i32, vp, vp, vp, vp, vp, i32, vp, vp],
     "spark_moe_combine_norm": [vp, vp, vp, i32, i32, i32, vp, vp, f32, i32, vp, vp, vp, vp],
     "spark_swiglu": [vp, vp, i32, i32, f32, vp],
     "spark_argmax": [vp, i32, i32, vp, vp, vp, vp, vp],
@@ -67,7 +69,7 @@ _SIGS = {
                         vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp],
     "spark_attn_decode": [vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32,
                           f32, vp, vp, vp, vp, vp, i32],
-    "spark_moe_route": [vp, i32, i32, i32, i32, i32, vp, f32, i32, vp, vp, vp, vp, vp, i32, i32],
+    "spark_moe_route": [vp, i32, i32, i32, i32, i32, vp, f32, i32, vp, vp, vp, vp, vp, i32, i32, i32, vp],
     "spark_moe_sort": [vp, i32, i32, vp, vp, vp, vp, vp, vp, vp],
     "spark_moe_combine": [vp, vp, i32, vp, vp, i32, i32, vp, vp, i32, vp, vp, vp],
     "spark_exl3_gemv": [vp, i32, vp, vp, vp, i64, i64, i64, vp, i32, i32, vp, vp, i32, i32, i32, i32, i32, i32,
@@ -81,7 +83,7 @@ _SIGS = {
 _LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32]
 _SIGS.update({
     "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, i32, vp, vp],
-    "spark_add_norm_rows": [vp, vp, vp, vp, vp, i32, i32, f32, i32, i32, vp],
+    "spark_row_update": [vp, i32, i32, vp],
     "spark_token_shift": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, vp],
     "spark_channel_decay": [vp, i32, vp, i32, i32, vp, vp, i32, i32, i32, vp],
     "spark_neg_exp_bias": [vp, vp, i32, i32, vp],
@@ -96,12 +98,34 @@ _SIGS.update({
     "spark_latent_rows": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
     "spark_latent_prefill": [vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
     "spark_mla_attn_paged": [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
+    "spark_conv_prep": [vp, i32, i32, i32, vp],
+    "spark_paged_rows": [vp, i32, i32, vp],
+    "spark_paged_decode": [vp, i32, vp],
+    "spark_paged_prefill": [vp, i32, i32, vp],
 })
+
+
+class OutAct(C.Structure):
+    """Activation on a product's accumulators (csrc/common/out_act.cuh)."""
+    _fields_ = [(n, i32) for n in ("kind", "ld", "off", "n", "rows", "f32")] + [("table", vp), ("ids", vp)]
+
+
+def out_act(kind: str, table=None, ids32=None, off: int = 0, n: int = 0) -> OutAct:
+    """"relu2": squared relu.  "token_gate": gelu_tanh(v) * table[ids, off + column] (columns from n on: 0)."""
+    if kind == "relu2":
+        return OutAct(kind=1)
+    a = OutAct(2, table.stride(0), off, n, table.shape[0], int(table.dtype == torch.float32), P(table), P(ids32))
+    a.keep = (table, ids32)                      # alive until the launch
+    return a
+
+
+def _act(a):
+    return C.byref(a) if a is not None else None
 
 
 # kernels launched by one call of each entry point (for the launch counter)
 _KERNELS_PER_CALL = {"spark_attn_decode": 2, "spark_moe_sort": 3, "spark_argmax": 2, "spark_hc_gated_site": 2,
-                     "spark_linear_chunked": 3, "spark_mla_attn_paged": 2}
+                     "spark_linear_chunked": 3, "spark_mla_attn_paged": 2, "spark_paged_decode": 2}
 _launches = 0
 
 
@@ -234,8 +258,10 @@ class PendingMoe:
     slot-order combine runs fused with the residual update and the next RMSNorm (`add_rmsnorm`), or on its own
     (`tensor()`)."""
 
-    def __init__(self, y, wts, ids, slots, R, H, shared=None, sg=None):
+    def __init__(self, y, wts, ids, slots, R, H, shared=None, sg=None, inv=None, self_w=None, self_x=None):
+        """`inv` (optional): row of y per pair; `self_w` / `self_x`: weight [R] and rows of identity experts."""
         self.y, self.wts, self.ids, self.slots, self.R, self.H, self.shared, self.sg = y, wts, ids, slots, R, H, shared, sg
+        self.inv, self.self_w, self.self_x = inv, self_w, self_x
 
     def tensor(self) -> torch.Tensor:
         out = torch.empty(self.R, self.H, dtype=torch.bfloat16, device=self.y.device)
@@ -264,7 +290,7 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out_f32: bool = False, fmt: int 
 
 
 def gemv_bf16(x, w, items=1, rows_per_item=None, pair_expert=None, pair_row=None, act=0, limit=0.0, out_f32=False,
-              expert_stride=0, n=None, k=None, out=None, ldx=None):
+              expert_stride=0, n=None, k=None, out=None, ldx=None, oact=None):
     rows_per_item = rows_per_item if rows_per_item is not None else x.shape[0]
     n = n if n is not None else w.shape[-2]
     k = k if k is not None else w.shape[-1]
@@ -279,7 +305,7 @@ def gemv_bf16(x, w, items=1, rows_per_item=None, pair_expert=None, pair_row=None
         dbg.check_index("gemv_bf16 pair_row", pair_row, 0, x.shape[0], count=items)
     rc = lib().spark_gemv_bf16(P(x), ldx if ldx is not None else x.stride(0), P(w), expert_stride, w.stride(-2), P(y), ldy,
                                items, rows_per_item, n, k, P(pair_expert), P(pair_row), act, float(limit), int(out_f32),
-                               stream())
+                               _act(oact), stream())
     check(rc, "spark_gemv_bf16")
     return y
 
@@ -307,15 +333,26 @@ def gemv_rows(K: int, N: int = 0) -> int:
     return r
 
 
-def gemm_simt(a, lda, sa, b, ldb, sb, c, ldc, sc, batch, M, N, K):
+def gemm_simt(a, lda, sa, b, ldb, sb, c, ldc, sc, batch, M, N, K, act=None):
     """Batched C = A B^T on the FP32 units (32-bit mode, unaligned bf16 shapes).  Strides in elements."""
     rc = lib().spark_gemm_simt(P(a), lda, sa, P(b), ldb, sb, P(c), ldc, sc, batch, M, N, K, int(b.dtype == torch.float32),
-                               int(c.dtype == torch.float32), stream())
+                               int(c.dtype == torch.float32), _act(act), stream())
     check(rc, "spark_gemm_simt")
     return c
 
 
-def dense_linear(x: torch.Tensor, w: torch.Tensor, out_f32: bool = False, out=None) -> torch.Tensor:
+def gemm_bf16_act(a: torch.Tensor, b: torch.Tensor, act: OutAct) -> torch.Tensor:
+    """bf16 activation of A[M,K] B[N,K]^T on tcgen05, applied in the epilogue."""
+    M, K = a.shape
+    N = b.shape[0]
+    c = torch.empty(M, N, dtype=torch.bfloat16, device=a.device)
+    check(lib().spark_gemm_bf16_act(P(a), P(b), P(c), M, N, K, a.stride(0), b.stride(0), N, _act(act), P(status_word(a.device)),
+                                    stream()), "spark_gemm_bf16_act")
+    return c
+
+
+def dense_linear(x: torch.Tensor, w: torch.Tensor, out_f32: bool = False, out=None, act: Optional[OutAct] = None) -> torch.Tensor:
+    """`act`: applied to the fp32 accumulators (the result is bf16, or fp32 in the 32-bit mode)."""
     if w.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError("dense weights must be bf16 (or fp32 in the 32-bit mode) on the device")
     R, (N, K) = x.shape[0], w.shape
@@ -323,12 +360,14 @@ def dense_linear(x: torch.Tensor, w: torch.Tensor, out_f32: bool = False, out=No
         x = x.to(w.dtype).contiguous()
         if out is None:
             out = torch.empty(R, N, dtype=torch.float32 if out_f32 else w.dtype, device=x.device)
-        return gemm_simt(x, x.stride(0), 0, w, w.stride(0), 0, out, out.stride(0), 0, 1, R, N, K)
+        return gemm_simt(x, x.stride(0), 0, w, w.stride(0), 0, out, out.stride(0), 0, 1, R, N, K, act)
     x = _as_bf16(x)
     if x.stride(1) != 1 or x.stride(0) % 8 or x.data_ptr() % 16:
         x = x.contiguous()
     if R <= 16 and R <= gemv_rows(K, N):
-        return gemv_bf16(x, w, out_f32=out_f32, out=out)
+        return gemv_bf16(x, w, out_f32=out_f32, out=out, oact=act)
+    if act is not None:
+        return gemm_bf16_act(x, w, act)
     return gemm_bf16(x, w, out_f32, out=out)
 
 
@@ -684,10 +723,11 @@ def gather_rows(src, idx32):
 
 
 # ----------------------------------------------------------------------------- MoE
-ROUTER_KIND = {"softmax": 0, "sigmoid_bias": 1, "sqrt_softplus": 2}
+ROUTER_KIND = {"softmax": 0, "sigmoid_bias": 1, "sqrt_softplus": 2, "softmax_bias": 3}
 
 
-def moe_route(h, w, c, e_lo=0, e_hi=None):
+def moe_route(h, w, c, e_lo=0, e_hi=None, self_w=None):
+    """`self_w` fp32 [R]: gets the weight of a row's identity experts."""
     R = h.shape[0]
     dev = h.device
     logits = dense_linear(h, w["gate"], out_f32=True)
@@ -695,9 +735,9 @@ def moe_route(h, w, c, e_lo=0, e_hi=None):
     ids = torch.empty(R, c.top_k, dtype=torch.int32, device=dev)
     prow = torch.empty(R, c.top_k, dtype=torch.int32, device=dev)
     sg = torch.empty(R, dtype=torch.float32, device=dev) if c.shared_gate else None
-    rc = lib().spark_moe_route(P(logits), logits.stride(0), R, c.n_experts, c.top_k, ROUTER_KIND[c.router],
+    rc = lib().spark_moe_route(P(logits), logits.stride(0), R, c.n_routes, c.top_k, ROUTER_KIND[c.router],
                                P(w.get("bias")), float(c.route_scale), int(c.shared_gate), P(wts), P(ids), P(prow), P(sg),
-                               stream(), e_lo, c.n_experts if e_hi is None else e_hi)
+                               stream(), e_lo, c.n_experts if e_hi is None else e_hi, c.n_identity, P(self_w))
     check(rc, "spark_moe_route")
     return wts, ids, prow, sg
 
@@ -795,7 +835,7 @@ def _moe_decode(h, w, c, defer: bool):
     rc = lib().spark_moe_router_topk(P(h), h.stride(0), P(gate), gate.stride(0), P(logits), ld,
                                      R, H, c.n_experts, c.top_k, ROUTER_KIND[c.router], P(w.get("bias")), float(c.route_scale),
                                      int(c.shared_gate), slots, e_hi - e_lo, e_lo, e_hi, rank, world, P(wts), P(ids), P(prow),
-                                     P(sg), P(counter), stream())
+                                     P(sg), P(counter), 0, None, stream())
     check(rc, "spark_moe_router_topk")
     shared = None
     side = None
@@ -822,6 +862,9 @@ def moe(h, w, c, defer: bool = False):
     outputs of a decode round).  Under expert parallelism (`w["ep"]` = (first local expert, end)) only the local
     experts' pairs are computed and the result is this rank's partial sum; the shared expert is added by the rank
     that holds it."""
+    if c.act == "relu2":
+        from .moe_relu import moe as moe_relu
+        return moe_relu(h, w, c, defer)
     if h.shape[0] * c.top_k <= DECODE_PAIRS_MAX and h.shape[0] <= DECODE_ROWS_MAX and FUSED_DECODE:
         return _moe_decode(h, w, c, defer)
     h = _as_bf16(h).contiguous()

@@ -3,6 +3,8 @@ row ops around the block, the two decayed linear recurrences, latent attention o
 activations; what the mechanisms keep in fp32 (residual, norms, states, decays, scores, softmax weights) is fp32 in both."""
 from __future__ import annotations
 
+import ctypes as C
+
 import torch
 
 from . import cuda as cu
@@ -26,16 +28,40 @@ def embed_scaled(table, ids32, scale: float):
     return out
 
 
-def add_norm_rows(delta, res, w, eps, one_plus, dtype, want_f32):
-    """res (fp32, in place) += delta (fp32); returns (h in `dtype`, res, fp32 copy of h or None)."""
+class RowUpdate(C.Structure):
+    """Arguments of the row update (csrc/kernels/block_rows.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("res", "delta", "y", "inv", "wts", "ids", "shared", "sg", "self_w", "self_x", "scale", "post_w",
+                                          "w", "b", "out", "out32")] \
+        + [(n, C.c_int) for n in ("H", "slots", "norm", "one_plus")] + [("eps", C.c_float), ("post_eps", C.c_float)]
+
+
+def add_norm_rows(delta, res, norm, dtype, want_f32=False):
+    """res (fp32, in place) += delta (None, a tensor, a deferred MoE output, or an ops.Update of one); returns (h in `dtype`, res,
+    fp32 copy of h or None)."""
     R, H = res.shape
     assert res.dtype == torch.float32 and res.is_contiguous()
-    if delta is not None:
-        delta = delta.float().contiguous()
+    u = RowUpdate(res=P(res), H=H)
+    keep = []
+    x = delta
+    if hasattr(delta, "post"):
+        x = delta.x
+        u.scale = P(delta.scale)
+        if delta.post is not None:
+            u.post_w, u.post_eps = P(delta.post.w), delta.post.eps
+    if isinstance(x, cu.PendingMoe):
+        assert x.shared is None or x.shared.dtype == torch.float32
+        u.y, u.inv, u.wts, u.ids, u.slots = P(x.y), P(x.inv), P(x.wts), P(x.ids), x.slots
+        u.shared, u.sg, u.self_w, u.self_x = P(x.shared), P(x.sg), P(x.self_w), P(x.self_x)
+    elif x is not None:
+        x = x.float().contiguous()
+        u.delta = P(x)
+    keep.append(x)
     h = torch.empty(R, H, dtype=dtype, device=res.device)
     h32 = h if dtype == torch.float32 else (torch.empty(R, H, dtype=torch.float32, device=res.device) if want_f32 else None)
-    check(lib().spark_add_norm_rows(P(delta), P(res), P(w), P(h), P(h32) if h32 is not h else None, R, H, float(eps), int(one_plus),
-                                    _is32(dtype), stream()), "spark_add_norm_rows")
+    u.out, u.out32 = P(h), P(h32) if h32 is not h else None
+    if norm is not None:
+        u.norm, u.w, u.b, u.eps, u.one_plus = (1 if norm.b is None else 2), P(norm.w), P(norm.b), norm.eps, int(norm.one_plus)
+    check(lib().spark_row_update(C.byref(u), R, _is32(dtype), stream()), "spark_row_update")
     return h, res, h32
 
 

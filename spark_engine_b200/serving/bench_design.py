@@ -141,8 +141,9 @@ def kernel_figures(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: 
         gu = rnd(rows, 2 * F).bfloat16()
         put(f"swiglu rows, {tag}", "", lambda: ops.swiglu(gu), rows * 3 * F * 2)
         res, d32, d16, nw2 = rnd(rows, 2048), rnd(rows, 2048), rnd(rows, 2048).bfloat16(), torch.ones(2048, device=DEV)
+        rn = ops.RowNorm(nw2, 1e-5, one_plus=True)
         put(f"residual + norm rows, {tag}", f"residual + norm rows (bf16 update), {tag}",
-            lambda: ops.add_norm_rows(d32, res, nw2, 1e-5, True, torch.bfloat16), rows * 2048 * (4 * 3 + 2))
+            lambda: ops.add_norm_rows(d32, res, rn, torch.bfloat16), rows * 2048 * (4 * 3 + 2))
         put(f"residual + norm rows (bf16 update), {tag}", "", lambda: ops.add_rmsnorm(d16, res, nw2, 1e-5), rows * 2048 * (4 * 2 + 2 + 2))
     # latent attention, kernels only
     D, Rr, Vd, L = 128, 64, 128, 512

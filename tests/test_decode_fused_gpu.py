@@ -68,7 +68,7 @@ def test_fused_router_matches_reference(kind, E, k):
             rc = lib.spark_moe_router_topk(h.data_ptr(), h.stride(0), gate.data_ptr(), gate.stride(0), logits.data_ptr(), ld,
                                            R, H, E, k, cu().ROUTER_KIND[kind], bias.data_ptr(), float(c.route_scale),
                                            int(c.shared_gate), slots, e_hi - e_lo, e_lo, e_hi, rank, world, wts.data_ptr(),
-                                           ids.data_ptr(), prow.data_ptr(), sg.data_ptr(), counter.data_ptr(),
+                                           ids.data_ptr(), prow.data_ptr(), sg.data_ptr(), counter.data_ptr(), 0, None,
                                            torch.cuda.current_stream().cuda_stream)
             assert rc == 0
         torch.cuda.synchronize()
