@@ -160,7 +160,7 @@ def main():
     ap.add_argument("--spec", default="none", help="mtp: also time speculative rounds (MTP chain of 3 drafts, 4 rows per "
                                                    "sequence verified) through the captured draft / verify / commit graphs")
     ap.add_argument("--sweep", action="store_true", help="also time 1,2,3 streams")
-    ap.add_argument("--design", default="", help="vabunex: time that architecture at a few layer sizes beside the closest existing "
+    ap.add_argument("--design", default="", help="vabunex | debisun: time that architecture at a few layer sizes beside the closest existing "
                                                  "family at equal size, and its kernels beside their like kernels (one GPU; not the "
                                                  "headline workload)")
     ap.add_argument("--parallel", default="tp", help="N > 1: tp = one model sharded over the GPUs (tensor + expert "
@@ -170,8 +170,8 @@ def main():
         return reference_arm(args)
     if args.design:
         from spark_engine_b200.serving import bench_design
-        if args.design != "vabunex":
-            raise SystemExit(f"unknown --design {args.design!r} (vabunex)")
+        if args.design not in bench_design.DESIGNS:
+            raise SystemExit(f"unknown --design {args.design!r} ({' | '.join(bench_design.DESIGNS)})")
         return bench_design.run(args, ClockSampler(0))
 
     import torch

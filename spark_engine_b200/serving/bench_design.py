@@ -1,7 +1,9 @@
-"""`bench.py --design vabunex`: prefill and decode throughput of a Vabunex model with random weights at a few layer sizes of
-real models, beside the closest existing family at equal size (KDA linear attention + latent attention, sequential
-pre-norm blocks with dense feed-forwards, bf16), and the kernels of the new mechanisms beside their like kernels as
-fractions of the measured copy bandwidth / GEMM throughput.
+"""`bench.py --design NAME`: prefill and decode throughput of a design with random weights at a few layer sizes of real models,
+beside the closest existing family at equal size, and the kernels of its mechanisms beside their like kernels as fractions of
+the measured copy bandwidth / GEMM throughput.
+
+  vabunex   beside KDA linear attention + latent attention in sequential pre-norm blocks with dense feed-forwards
+  debisun   beside grouped-query attention (rotary, no chunks) with softmax-routed SwiGLU experts, as many parameters
 
 Device-timed with CUDA events.  Model figures stream more weights and activations than L2 holds; kernel figures write a
 buffer larger than L2 between iterations (median of the iterations)."""
@@ -13,7 +15,7 @@ import statistics
 
 import torch
 
-from ..config import EngineConfig, KdaConfig, MlaConfig, glm_style, vabunex_style
+from ..config import AttnConfig, EngineConfig, KdaConfig, MlaConfig, ModelConfig, MoeConfig, debisun_style, glm_style, vabunex_style
 from ..models.build import build_random_model, decode_step_bytes
 from ..models.plan import make_plan
 from ..ops import cuda as cu
@@ -87,17 +89,19 @@ def model_figures(cfg, steps: int, warmup: int, prompts=(2048, 8192)) -> dict:
     return out
 
 
-def kernel_figures(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: int = 4) -> dict:
-    """Kernels at hidden size 2048 (16 heads of 128, wkv 32 of 64): {name: (ms, fraction of roofline, bound, like kernel)}."""
-    from .. import ops
-    from ..models.model import KdaMixer
-    hbm, tf = peaks.get("hbm_gbs", 6650.0) * 1e6, peaks.get("bf16_tflops", 1590.0) * 1e9      # bytes, flops per millisecond
-    flush = torch.empty(512 << 20, dtype=torch.uint8, device=DEV)
-    g = torch.Generator(device=DEV).manual_seed(0)
-    rnd = lambda *s: torch.randn(*s, device=DEV, generator=g)
-    out = {}
+class Figures:
+    """Kernel times as fractions of their roofline (bytes over the copy bandwidth or flops over the GEMM throughput)."""
 
-    def put(name, like, fn, nbytes=0, flops=0):
+    def __init__(self, peaks: dict):
+        self.hbm, self.tf = peaks.get("hbm_gbs", 6650.0) * 1e6, peaks.get("bf16_tflops", 1590.0) * 1e9    # bytes, flops per millisecond
+        self.flush = torch.empty(512 << 20, dtype=torch.uint8, device=DEV)
+        self.g = torch.Generator(device=DEV).manual_seed(0)
+        self.out = {}
+
+    def rnd(self, *s):
+        return torch.randn(*s, device=DEV, generator=self.g)
+
+    def put(self, name, like, fn, nbytes=0, flops=0):
         if name.endswith("decode"):              # short kernels: replayed from a graph, no host time between launches
             fn()
             torch.cuda.synchronize()
@@ -105,11 +109,24 @@ def kernel_figures(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: 
             with torch.cuda.graph(graph):
                 fn()
             fn = graph.replay
-        ms = _timed(fn, 7, flush)
-        roof = max(nbytes / hbm, flops / tf)
-        out[name] = {"us": round(ms * 1e3, 1), "of_roofline": round(roof / ms, 3), "bound": "bytes" if nbytes / hbm >= flops / tf else "flops",
-                     "like": like}
+        ms = _timed(fn, 7, self.flush)
+        roof = max(nbytes / self.hbm, flops / self.tf)
+        self.out[name] = {"us": round(ms * 1e3, 1), "of_roofline": round(roof / ms, 3),
+                          "bound": "bytes" if nbytes / self.hbm >= flops / self.tf else "flops", "like": like}
 
+    def done(self) -> dict:
+        for v in self.out.values():
+            if v["like"]:
+                v["distance_ratio"] = round(self.out[v["like"]]["of_roofline"] / v["of_roofline"], 2)    # > 1: farther than the like kernel
+        return self.out
+
+
+def vabunex_kernels(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: int = 4) -> dict:
+    """Kernels at hidden size 2048 (16 heads of 128, wkv 32 of 64)."""
+    from .. import ops
+    from ..models.model import KdaMixer
+    fig = Figures(peaks)
+    rnd, put = fig.rnd, fig.put
     n = H * 128
     pl, pd = make_plan([(0, [1] * T, 0)], device=DEV), make_plan([(s, [1], ctx - 1) for s in range(R)], device=DEV)
     for tag, plan, rows in (("prefill", pl, T), ("decode", pd, R)):
@@ -121,7 +138,7 @@ def kernel_figures(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: 
             lambda: ops.linear_state(x[:, :n], x[:, n: 2 * n], x[:, 2 * n: 3 * n], H, 128, 128, S, plan, True, act=True, log2a=l2),
             rows * n * (3 * 2 + 4) + st)
         S2 = torch.zeros(R, 2 * H, 64, 64, device=DEV)
-        lw, u = -torch.rand(rows, n, device=DEV, generator=g), rnd(2 * H, 64)
+        lw, u = -torch.rand(rows, n, device=DEV, generator=fig.g), rnd(2 * H, 64)
         put(f"wkv recurrence, {tag}", f"kda recurrence, {tag}",
             lambda: ops.linear_state(x[:, :n], x[:, n: 2 * n], x[:, 2 * n: 3 * n], 2 * H, 64, 64, S2, plan, True, logw=lw, u=u),
             rows * n * (3 * 2 + 4 + 4) + st // 2)
@@ -173,10 +190,119 @@ def kernel_figures(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R: 
         put(f"latent attention of the closest model, {tag}", "",
             lambda: lib().spark_mla_attn(P(qf), P(cache), P(pos), P(kvb), None, None, 0, P(po), P(pm), ns, None, rows, H, L, Rr, 0.07, P(ol),
                                          stream(), None, None, None, 0), nb, fl)
-    for v in out.values():
-        if v["like"]:
-            v["distance_ratio"] = round(out[v["like"]]["of_roofline"] / v["of_roofline"], 2)    # > 1: farther than the like kernel
-    return out
+    return fig.done()
+
+
+# ----------------------------------------------------------------------------- debisun
+DEB_SIZES = {"1024": (1024, 4096), "2048": (2048, 8192), "4096": (4096, 16384)}
+DEB_EXPERTS, DEB_TOP = 32, 4
+
+
+def debisun_config(hidden: int, ffn: int):
+    return debisun_style(12, hidden, ffn, VOCAB, experts=DEB_EXPERTS, top=DEB_TOP)
+
+
+def debisun_closest(hidden: int, ffn: int, layers: int):
+    """The same heads and experts; SwiGLU widths are two thirds, so that the three matrices hold as many parameters as two."""
+    w = lambda n: (2 * n // 3 + 127) // 128 * 128
+    h = hidden // 128
+    return ModelConfig(name="gqa + swiglu experts, dense weights", family="hybrid", n_layers=layers, layer_types=["attn"] * layers, hidden=hidden,
+                       vocab=VOCAB, attn=AttnConfig(n_q_heads=h, n_kv_heads=max(1, h // 4), head_dim=128, rope_dim=64),
+                       moe=MoeConfig(n_experts=DEB_EXPERTS, top_k=DEB_TOP, ffn=w(ffn // 4), n_shared=1, shared_ffn=w(ffn // 4), router="softmax",
+                                     shared_gate=True, dense_layers=1, dense_ffn=w(ffn)), weight_format="dense")
+
+
+def debisun_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> dict:
+    """Kernels at hidden size 2048 (16 query and 4 key / value heads of 128, 32 experts of 2048, top 4)."""
+    import dataclasses
+    import types
+    from .. import ops
+    from ..models.layout import pad
+    from ..models.model import AttnMixer
+    from ..models.paged_gqa import PagedGqaMixer
+    from ..ops import moe_relu
+    fig = Figures(peaks)
+    rnd, put = fig.rnd, fig.put
+    N, H, G, D = 2048, 16, 4, 128
+    cfg = debisun_config(N, 8192)
+    near = debisun_closest(N, 8192, 1)
+    spec = dataclasses.replace(cfg.layer_specs[0], mixer=dataclasses.replace(cfg.layer_specs[0].mixer, chunk=ctx))     # one chunk: all keys
+    C = (H + 2 * G) * D
+    w = {"conv_t": rnd(4, C) * 0.5, "dist_bias": rnd(H, 1025), "sink": torch.zeros(H, device=DEV)}
+    pages = torch.arange(R * ctx // 64, dtype=torch.int32, device=DEV).view(R, -1).contiguous()
+    mx = PagedGqaMixer(cfg, spec, w, R, R * ctx // 64, 64, pages, DEV, torch.bfloat16)
+    at = AttnMixer(near, {}, R * ctx, DEV, torch.bfloat16)
+    for t in (mx.k, mx.v, at.k, at.v):
+        t.copy_(rnd(*t.shape))
+    seqs = [types.SimpleNamespace(kv_base=i * ctx, kv_cap=ctx) for i in range(R)]
+    from ..ops import paged_attn as pa
+    lib, P, stream = cu.lib, cu.P, cu.stream
+    for tag, rows in (("prefill", T), ("decode", R)):
+        plan = lambda: make_plan([(0, [1] * T, 0)] if tag == "prefill" else [(s, [1], ctx - 1) for s in range(R)], device=DEV)
+        p1, p2 = plan(), plan()
+        proj = rnd(rows, C).bfloat16()
+        fl = T * T / 2 * H * 2 * D * 2 if tag == "prefill" else R * ctx * H * 2 * D * 2
+        nb = 0 if tag == "prefill" else R * ctx * G * 2 * D * 2
+        # whole mixers (convolution or rotation into the cache, then attention): the attention is nearly all of the time
+        put(f"paged attention with its convolution, {tag}", f"dense attention with its rotation, {tag}",
+            lambda: pa.mixer(mx, proj, p1, True), nb + rows * C * 4, fl)
+        put(f"dense attention with its rotation, {tag}", "", lambda: cu.attn_mixer(at, proj, p2, seqs), nb + rows * C * 4, fl)
+        d, q = cu._plan_dev(p1, DEV), torch.empty(rows, H * D, dtype=torch.bfloat16, device=DEV)
+        put(f"convolution into the cache, {tag}", f"rotation into the cache, {tag}", lambda: pa._conv(mx, proj, p1, d, q, True), rows * C * 4)
+        d2 = cu._plan_dev(p2, DEV)
+        put(f"rotation into the cache, {tag}", "",
+            lambda: lib().spark_attn_prep(P(proj), C, rows, H, G, D, 64, 0, 0, 0, 0, 4, 0, 1e-6, None, None, None, None, P(at.inv), P(d2["pos32"]),
+                                          P(d2["row_kv"]), P(d2["row_j"]), P(q), P(at.k), P(at.v), None, None, None, None, None, stream(), None),
+            rows * C * 4)
+        # residual updates
+        res, d32, d16, one = rnd(rows, N), rnd(rows, N), rnd(rows, N).bfloat16(), torch.ones(N, device=DEV)
+        ln, rn = ops.RowNorm(one, 1e-5, one), ops.RowNorm(one, 1e-5)
+        put(f"scaled update + layer norm, {tag}", f"update + RMS norm, {tag}",
+            lambda: ops.add_norm_rows(ops.Update(d32, one), res, ln, torch.bfloat16), rows * N * 14)
+        put(f"normed update + layer norm, {tag}", f"update + RMS norm, {tag}",
+            lambda: ops.add_norm_rows(ops.Update(d32, post=rn), res, ln, torch.bfloat16), rows * N * 14)
+        put(f"update + RMS norm, {tag}", "", lambda: ops.add_rmsnorm(d16, res, one, 1e-5), rows * N * 12)
+        # token side: gate product with the token rows in its epilogue, and the projection back
+        sd = cfg.side_dim
+        table, ids, gw = rnd(VOCAB, sd).bfloat16(), torch.randint(0, VOCAB, (rows,), device=DEV).int(), rnd(pad(sd, 8), N).bfloat16()
+        nb = rows * (N + 2 * sd) * 2 + sd * N * 2
+        put(f"token gate product, {tag}", f"plain product of its shape, {tag}", lambda: ops.linear_token_gate(d16, gw, table, ids, 0, sd), nb,
+            rows * N * sd * 2)
+        put(f"plain product of its shape, {tag}", "", lambda: cu.dense_linear(d16, gw), nb, rows * N * sd * 2)
+        up = rnd(8192, N).bfloat16()
+        put(f"up product with squared relu, {tag}", f"plain up product, {tag}", lambda: ops.linear_relu2(d16, up), rows * (N + 8192) * 2 + 8192 * N * 2,
+            rows * N * 8192 * 2)
+        put(f"plain up product, {tag}", "", lambda: cu.dense_linear(d16, up), rows * (N + 8192) * 2 + 8192 * N * 2, rows * N * 8192 * 2)
+        # routed feed-forwards: every kernel from the router to the combined rows
+        c, c2 = cfg.layer_specs[1].moe, near.moe
+        F, F2 = c.ffn, c2.ffn
+        w1 = {"gate": rnd(c.n_routes + 1, N).bfloat16() * 0.05, "bias": 0.01 * rnd(c.n_routes), "w_up": (rnd(c.n_experts, F, N) * 0.02).bfloat16(),
+              "w_down": (rnd(c.n_experts, N, F) * 0.02).bfloat16(), "s_up": (rnd(F, N) * 0.02).bfloat16(), "s_down": (rnd(N, F) * 0.02).bfloat16()}
+        w2 = {"gate": rnd(c2.n_experts + 1, N).bfloat16() * 0.05, "w_gu": (rnd(c2.n_experts, 2 * F2, N) * 0.02).bfloat16(),
+              "w_down": (rnd(c2.n_experts, N, F2) * 0.02).bfloat16(), "s_gu": (rnd(2 * F2, N) * 0.02).bfloat16(),
+              "s_down": (rnd(N, F2) * 0.02).bfloat16()}
+
+        def touched(c, ids):                     # bytes of the distinct experts a round reads, and the pairs that have an expert
+            live = ids[(ids >= 0) & (ids < c.n_experts)]
+            return live.unique().numel(), live.numel()
+        e1, pairs1 = touched(c, moe_relu._route(d16, w1, c, torch.empty(rows, device=DEV))[1])
+        e2, pairs2 = touched(c2, cu.moe_route(d16, w2, c2)[1])
+        put(f"routed squared-relu experts + update, {tag}", f"routed SwiGLU experts + update, {tag}",
+            lambda: ops.add_norm_rows(ops.Update(ops.moe(d16, w1, c, True), one), res, None, torch.bfloat16),
+            (e1 + 1) * 2 * F * N * 2 + rows * N * 14, (pairs1 + rows) * 2 * F * N * 2)
+        put(f"routed SwiGLU experts + update, {tag}", "",
+            lambda: ops.add_rmsnorm(ops.moe(d16, w2, c2, True), res, one, 1e-5), (e2 + 1) * 3 * F2 * N * 2 + rows * N * 14,
+            (pairs2 + rows) * 3 * F2 * N * 2)
+        del w1, w2
+    return fig.done()
+
+
+DESIGNS = {
+    "vabunex": (vabunex_config, closest_config, vabunex_kernels, SIZES,
+                "KDA + latent attention (GLM-style layer types), sequential pre-norm blocks, dense feed-forward, bf16"),
+    "debisun": (debisun_config, debisun_closest, debisun_kernels, DEB_SIZES,
+                "grouped-query attention (rotary, whole context), softmax-routed SwiGLU experts of as many parameters, bf16"),
+}
 
 
 def run(args, clocks) -> int:
@@ -186,20 +312,20 @@ def run(args, clocks) -> int:
             peaks = json.load(f)
     except OSError:
         peaks = {}
+    config, closest, kernels, all_sizes, closest_text = DESIGNS[args.design]
     clocks.start()
     sizes = {}
-    for name, (hidden, ffn) in SIZES.items():
-        cv = vabunex_config(hidden, ffn)
+    for name, (hidden, ffn) in all_sizes.items():
+        cv = config(hidden, ffn)
         runs = len(cv.layer_runs())
-        sizes[name] = {"layer_runs": runs, "ffn": ffn, "vabunex": model_figures(cv, args.steps, args.warmup)}
-        torch.cuda.empty_cache()
-        sizes[name]["closest"] = model_figures(closest_config(hidden, ffn, runs), args.steps, args.warmup)
+        sizes[name] = {"layer_runs": runs, "ffn": ffn, args.design: model_figures(cv, args.steps, args.warmup)}
         cu._scratch.clear()
         torch.cuda.empty_cache()
-    out = {"metric": "vabunex prefill / decode throughput beside the closest existing family at equal size", "design": "vabunex",
-           "closest": "KDA + latent attention (GLM-style layer types), sequential pre-norm blocks, dense feed-forward, bf16",
-           "dtype": "bf16", "data": "synthetic", "sizes": sizes, "kernels": kernel_figures(peaks),
-           "clocks": clocks.stop(),
-           "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")}}
+        sizes[name]["closest"] = model_figures(closest(hidden, ffn, runs), args.steps, args.warmup)
+        cu._scratch.clear()
+        torch.cuda.empty_cache()
+    out = {"metric": f"{args.design} prefill / decode throughput beside the closest existing family at equal size", "design": args.design,
+           "closest": closest_text, "dtype": "bf16", "data": "synthetic", "sizes": sizes, "kernels": kernels(peaks),
+           "clocks": clocks.stop(), "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")}}
     print(json.dumps(out))
     return 0
