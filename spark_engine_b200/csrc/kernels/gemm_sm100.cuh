@@ -313,9 +313,25 @@ struct EpiActBf16 {
     if (a.kind == 1) {
 #pragma unroll
       for (int i = 0; i < 32; ++i) y[i] = relu2_f(v[i]);
-    } else {
+    } else if (!a.f32 && ((a.ld | a.off) & 7) == 0 && col + 32 <= a.n) {      // 32 table columns as four 16-byte loads
+      const int id = a.ids[row];
+      const bool ok = id >= 0 && id < a.rows;
+      const uint4* e = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.table) + static_cast<size_t>(ok ? id : 0) * a.ld + a.off + col);
+      uint4 q[4];
 #pragma unroll
-      for (int i = 0; i < 32; ++i) y[i] = out_act(a, v[i], row, col + i);
+      for (int i = 0; i < 4; ++i) q[i] = __ldg(e + i);
+#pragma unroll
+      for (int i = 0; i < 32; i += 2) {
+        const float2 f = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(q)[i >> 1]);
+        y[i] = ok ? gelu_tanh_t<__nv_bfloat16>(v[i]) * f.x : 0.f;
+        y[i + 1] = ok ? gelu_tanh_t<__nv_bfloat16>(v[i + 1]) * f.y : 0.f;
+      }
+    } else {
+      __nv_bfloat16* dst = C + static_cast<size_t>(row) * ldc + col;
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (col + i < N) dst[i] = __float2bfloat16(out_act(a, v[i], row, col + i));
+      return;
     }
     EpiStoreBf16{C, ldc, N}(tc, row, col, y);
   }

@@ -594,11 +594,14 @@ extern "C" int spark_moe_router_topk(const void* x, int ldx, const void* Wg, int
   if (smem > 200 * 1024) return -6;
   static bool attr_set = false;
   if (!attr_set) {
+    cudaFuncSetAttribute(moe_router_topk_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     cudaFuncSetAttribute(moe_router_topk_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     cudaFuncSetAttribute(moe_router_topk_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     attr_set = true;
   }
-  const cudaError_t err = E <= 512
+  const cudaError_t err = E <= 64
+      ? spark_launch_pdl(moe_router_topk_kernel<2>, dim3((NE + 7) / 8), dim3(256), smem, s, dim3(1, 1, 1), a)
+      : E <= 512
       ? spark_launch_pdl(moe_router_topk_kernel<16>, dim3((NE + 7) / 8), dim3(256), smem, s, dim3(1, 1, 1), a)
       : spark_launch_pdl(moe_router_topk_kernel<32>, dim3((NE + 7) / 8), dim3(256), smem, s, dim3(1, 1, 1), a);
   return err == cudaSuccess ? 0 : -4;

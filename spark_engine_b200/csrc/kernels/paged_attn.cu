@@ -34,13 +34,15 @@ struct PagedAttn {
 __device__ __forceinline__ int chunk_first(int p, int chunk) { return chunk > 0 ? p / chunk * chunk : 0; }
 
 // tanh to fp32 accuracy in the sense of the soft cap: the Taylor polynomial near 0 (where the quotient form would cancel),
-// 1 - 2 / (exp(2z) + 1) elsewhere (absolute error of a few 2^-23).
+// 1 - 2 / (exp(2z) + 1) elsewhere (absolute error of a few 2^-23).  The polynomial gives tanh(z) / z.
+constexpr float CAP_NEAR = 0.25f;
+__device__ __forceinline__ float tanh_over_z(float z) {
+  const float s = z * z;
+  return fmaf(s, fmaf(s, fmaf(s, fmaf(s, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
+}
 __device__ __forceinline__ float cap_tanh(float z) {
-  if (fabsf(z) < 0.25f) {
-    const float s = z * z;
-    return z * (1.f + s * (-1.f / 3.f + s * (2.f / 15.f + s * (-17.f / 315.f + s * (62.f / 2835.f)))));
-  }
-  return 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(z, 40.f)));
+  const float near = z * tanh_over_z(z), far = 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(z, 40.f)));
+  return fabsf(z) < CAP_NEAR ? near : far;
 }
 
 // ------------------------------------------------------------------------------------------------ short convolution
@@ -348,7 +350,7 @@ paged_decode_kernel(const __grid_constant__ PagedAttn a) {
 // ------------------------------------------------------------------------------------------------ prompts
 // grid (row tiles, H, segments); NW warps x 16 rows.  VP >= V: compiled value width.  A key tile is one page.
 template <int VP, int NW>
-__global__ void __launch_bounds__(NW * 32)
+__global__ void __launch_bounds__(NW * 32, VP <= 64 ? 2 : 1)      // values of 128: two CTAs per SM spill and are 10 % slower
 paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
   constexpr int BM = NW * 16, BN = PGA_PAGE, LDV = VP + 8, NB = BM + BN;
   extern __shared__ __align__(16) uint8_t smem_pga[];
@@ -406,7 +408,7 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
   const int w0 = pbase + warp * 16, p_lo = w0 + gq, p_hi = p_lo + 8;         // padded rows: positions past the segment, not stored
   const int f_lo = chunk_first(p_lo, a.chunk), f_hi = chunk_first(p_hi, a.chunk);
   const int w_first = chunk_first(w0, a.chunk), w_last = chunk_first(w0 + 15, a.chunk);
-  const float qs = a.cap > 0.f ? a.scale / a.cap : a.scale * PGA_LOG2E, cs = a.cap * PGA_LOG2E;
+  const float qs = a.cap > 0.f ? a.scale / a.cap : a.scale * PGA_LOG2E, cs = a.cap * PGA_LOG2E, csqs = cs * qs;
   for (int j = j0; j < j1; ++j) {
     const int buf = (j - j0) & 1, k0 = j * BN;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -431,6 +433,27 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
       }
     }
     const bool need_mask = k0 + BN - 1 > w0 || k0 < w_last;
+    if (a.cap > 0.f) {                                       // one form for the whole tile: scores far below the cap need no exponential
+      float big = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) big = fmaxf(big, fmaxf(fmaxf(fabsf(s[i][0]), fabsf(s[i][1])), fmaxf(fabsf(s[i][2]), fabsf(s[i][3]))));
+      if (__any_sync(0xffffffffu, big * fabsf(qs) >= CAP_NEAR)) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[i][e] = cs * cap_tanh(s[i][e] * qs);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[i][e] *= csqs * tanh_over_z(s[i][e] * qs);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[i][e] *= qs;
+    }
     float mx_lo = m_lo, mx_hi = m_hi;
     float b_hi[2] = {0.f, 0.f}, b_lo[2] = {0.f, 0.f};
     if (a.bias) { b_lo[0] = bs[0]; b_lo[1] = bs[-1]; }
@@ -440,9 +463,7 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
       if (a.bias) { b_hi[0] = b_lo[0]; b_hi[1] = b_lo[1]; b_lo[0] = bs[-8 * i - 8]; b_lo[1] = bs[-8 * i - 9]; }
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        float v = s[i][e] * qs;
-        if (a.cap > 0.f) v = cs * cap_tanh(v);
-        v += (e >> 1) ? b_hi[e & 1] : b_lo[e & 1];
+        float v = s[i][e] + ((e >> 1) ? b_hi[e & 1] : b_lo[e & 1]);
         if (need_mask) {
           const int key = k0 + i * 8 + 2 * t + (e & 1);
           if (key > ((e >> 1) ? p_hi : p_lo) || key < ((e >> 1) ? f_hi : f_lo)) v = -INFINITY;
