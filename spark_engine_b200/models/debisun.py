@@ -126,12 +126,15 @@ def layer_tensors(cfg: ModelConfig, spec: LayerSpec) -> Dict[str, tuple]:
     return t
 
 
-def _assemble(cfg: ModelConfig, get, layer, dtype) -> dict:
+def _assemble(cfg: ModelConfig, get, layer, dtype, stored: bool) -> dict:
     W = {"embed": get("embed", (cfg.vocab, cfg.hidden)).to(dtype).contiguous(), "final_norm": get("final.norm", (cfg.hidden,)).float().contiguous(),
          "final_norm_b": get("final.norm.b", (cfg.hidden,)).float().contiguous(),
          "lm_head": get("head", (cfg.vocab, cfg.hidden)).to(dtype).contiguous()}
     if cfg.side_dim:
-        W["side_embed"] = get("side.embed", (cfg.vocab, cfg.n_layers * cfg.side_dim)).to(dtype).contiguous()
+        t = get("side.embed", (cfg.vocab, None)) if stored else get("side.embed", (cfg.vocab, cfg.n_layers * cfg.side_dim))
+        if t.shape[1] < cfg.n_layers * cfg.side_dim:
+            raise ValueError(f"tensor side.embed has shape {tuple(t.shape)}, the configuration needs {cfg.n_layers * cfg.side_dim} columns")
+        W["side_embed"] = t.to(dtype).contiguous()
     W["layers"] = [prepare_layer(layer(i, s), s, dtype) for i, s in enumerate(cfg.layer_specs)]
     return W
 
@@ -139,7 +142,8 @@ def _assemble(cfg: ModelConfig, get, layer, dtype) -> dict:
 def from_tensors(cfg: ModelConfig, tensors: Dict[str, torch.Tensor], device="cpu", dtype=torch.float32) -> dict:
     """Runner weights from a flat dict of checkpoint tensors (validated against the configuration)."""
     get = taker(tensors, device)
-    return _assemble(cfg, get, lambda i, spec: {k: get(f"l{i}.{k}", s) for k, s in layer_tensors(cfg, spec).items()}, dtype)
+    return _assemble(cfg, get, lambda i, spec: {k: get(f"l{i}.{k}", s) for k, s in layer_tensors(cfg, spec).items()},
+                     dtype, True)
 
 
 def load_weights(directory: str, cfg: ModelConfig, device="cpu", dtype=torch.bfloat16) -> dict:
@@ -165,4 +169,4 @@ def random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, dtype=torch.bf
     def layer(i, spec):
         spec.mixer.bias_buckets = spec.mixer.bias_buckets or 32
         return {k: tensor(k, s) for k, s in layer_tensors(cfg, spec).items()}
-    return _assemble(cfg, tensor, layer, dtype)
+    return _assemble(cfg, tensor, layer, dtype, False)
