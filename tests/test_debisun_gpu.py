@@ -2,7 +2,7 @@
 portions, mixed batches, page and chunk edges, captured decode rounds, the server.
 
 A routed model in bf16 may take another expert than the plain one where two choice scores are closer than rounding, and a token
-side of width one is +1 or -1 times its weight by the sign of a number that may be close to 0: such models are judged by the ninth
+side of width one is +1 or -1 times its weight by the sign of a number that may be close to 0: such models are compared by the ninth
 decile of their rows in bf16 (and by the worst row in 32-bit); the expert kernels have a test of their own on rows without close
 calls."""
 import json
@@ -42,7 +42,7 @@ SHAPES.update({
 })
 
 
-def judge(got, want, dtype, cfg):
+def agree(got, want, dtype, cfg):
     close_calls = cfg["token_side"]["dim"] == 1 or any(x.get("mlp") and x["mlp"]["kind"] == "moe" for x in cfg["layers"])
     if dtype == torch.float32 or not close_calls:
         assert U.error(got, want) < TOL[dtype] * (len(cfg["layers"]) ** 0.5 if dtype == torch.bfloat16 else 1)
@@ -59,12 +59,12 @@ def test_prompt_then_decoding(name, dtype):
     toks = U.prompt(160, cfg["vocab"])
     want = U.oracle_logits(cfg, T, toks)
     m = U.framework(cfg, T, DEV, dtype)
-    judge(m.forward(make_plan([(0, toks, 0)], device=DEV)), want, dtype, cfg)
+    agree(m.forward(make_plan([(0, toks, 0)], device=DEV)), want, dtype, cfg)
     out, i = [], 0
     for n in (2, 31, 2, 33, 64, *[1] * 28):
         out.append(m.forward(make_plan([(3, toks[i: i + n], i)], device=DEV)))
         i += n
-    judge(torch.cat(out), want, dtype, cfg)
+    agree(torch.cat(out), want, dtype, cfg)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -92,7 +92,7 @@ def test_mixed_batches_equal_each_request_alone(dtype):
     for k, g in got_all.items():
         g = torch.cat(g)
         if len(g) > 10 or dtype == torch.float32:
-            judge(g, want[k][: len(g)], dtype, cfg)
+            agree(g, want[k][: len(g)], dtype, cfg)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
