@@ -76,6 +76,7 @@ class MoeConfig:
     n_shared: int = 1
     shared_ffn: int = 0           # 0 -> ffn * n_shared
     router: str = "softmax"       # softmax | sigmoid_bias | sqrt_softplus | softmax_bias (bias: added to the choice scores only)
+                                  # | sigmoid (the chosen scores are the weights as they are, times route_scale)
     route_scale: float = 1.0
     shared_gate: bool = False     # sigmoid(x . w_sg) on the shared expert
     swiglu_limit: float = 0.0     # clamp-SwiGLU limit (0 = off)
@@ -83,6 +84,7 @@ class MoeConfig:
     dense_ffn: int = 0
     act: str = "swiglu"           # swiglu (gate and up matrices) | relu2 (squared relu of a single up matrix)
     n_identity: int = 0           # router outputs behind the experts' whose "expert" returns its input
+    weight_input: bool = False    # an expert sees its input times the weight (its output is added as it is)
 
     @property
     def n_routes(self) -> int:
@@ -122,21 +124,59 @@ class LatentConfig:
 
 @dataclass
 class PagedGqaConfig:
-    """Grouped-query softmax attention over a paged cache, without rotation: short convolutions on q, k and v, soft-capped
-    scores, a learned bias per distance bucket and head, chunked visibility, a sink in the denominator."""
+    """Grouped-query softmax attention over a paged cache.  Before the cache: short convolutions on q, k and v, or a norm per
+    query / key head, a rotation and a temperature of the queries.  Scores: soft cap, a learned bias per distance bucket and
+    head or a slope per head, chunked or windowed visibility, a sink in the denominator; a gate per head behind them."""
     n_heads: int = 4
     n_kv_heads: int = 2
     head_dim: int = 32
     v_dim: int = 32
-    conv_k: int = 4               # taps of the causal convolutions (1: the current token only)
+    conv_k: int = 4               # taps of the causal convolutions (1: the current token only; 0: none)
     scale: float = 0.125
     softcap: float = 0.0          # 0: none
-    bias_buckets: int = 32        # rows of the bias table
+    bias_buckets: int = 32        # rows of the bias table (without one: unused)
     bias_max: int = 1024          # distance from which on the last row is used
     chunk: int = 0                # tokens see their own aligned chunk of the sequence (0: everything before them)
+    window: int = 0               # tokens see themselves and the window - 1 before them (0: everything before them)
+    qk_norm: bool = False         # RMS norm of every query and key head (weight per dimension, shared by the heads)
+    rope_dims: int = 0            # leading dimensions of a head that rotate, adjacent pairs (0: none)
+    rope_theta: float = 1e4
+    rope_factor: float = 1.0      # every frequency is divided by it
+    temp_coef: float = 0.0        # queries at position p times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
+    temp_every: float = 1.0
+    slopes: bool = False          # scores minus 2^(-8 (h + 1) / heads) times the distance
+    gated: bool = False           # one sigmoid gate per head
+    kv_from: Optional[int] = None  # keys and values are the ones in that layer's cache
 
 
-MIXER_CONFIGS = {"lightning": LightningConfig, "wkv": WkvConfig, "latent": LatentConfig, "gqa": PagedGqaConfig}
+@dataclass
+class GlaConfig:
+    """Linear attention with a decay per token and key channel, sigmoid(low-rank projection + bias)^(1 / tau); an RMS norm per
+    head and a silu gate behind it."""
+    n_heads: int = 2
+    head_dim: int = 32
+    v_dim: int = 32
+    tau: float = 16.0
+    decay_rank: int = 16
+
+
+@dataclass
+class SideBySideConfig:
+    """Grouped-query attention and linear attention on the same rows, outputs scaled and added."""
+    left: PagedGqaConfig = field(default_factory=lambda: PagedGqaConfig(conv_k=0))
+    right: GlaConfig = field(default_factory=GlaConfig)
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+    def __post_init__(self):
+        if isinstance(self.left, dict):
+            self.left = PagedGqaConfig(**self.left)
+        if isinstance(self.right, dict):
+            self.right = GlaConfig(**self.right)
+
+
+MIXER_CONFIGS = {"lightning": LightningConfig, "wkv": WkvConfig, "latent": LatentConfig, "gqa": PagedGqaConfig,
+                 "side_by_side": SideBySideConfig}
 
 
 @dataclass
@@ -159,7 +199,7 @@ class LoopConfig:
 @dataclass
 class ModelConfig:
     name: str = "tiny-hybrid"
-    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex | debisun
+    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex | debisun | zapolorn
     n_layers: int = 4
     layer_types: List[str] = field(default_factory=lambda: ["gdn", "gdn", "gdn", "attn"])
     hidden: int = 256
@@ -188,9 +228,12 @@ class ModelConfig:
     layer_specs: List[LayerSpec] = field(default_factory=list)   # per-layer sizes; else the shared configs above
     loop: Optional[LoopConfig] = None
     block: str = "parallel"       # models with layer_specs: parallel (one norm, mixer + feed-forward) | sequential (pre-norm each)
+                                  # | post (sublayers read the residual itself, their outputs are normed)
     norm_kind: str = "rms"        # models with layer_specs: rms | layer (weight and bias)
     norm_one_plus: bool = False   # norm weights are stored around zero
     embed_scale: float = 1.0
+    logit_scale: float = 1.0
+    tied_head: bool = False       # the logits' matrix is the embedding table (without its scale)
     side_dim: int = 0             # width of the per-layer token input (0 = none)
 
     def layer_runs(self) -> List[int]:
@@ -313,6 +356,28 @@ def debisun_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 8192, vocab
                        weight_format="dense")
 
 
+def zapolorn_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 5632, vocab: int = 65536, experts: int = 64, top: int = 4,
+                   window: int = 1024) -> ModelConfig:
+    """Zapolorn at the layer sizes of a small real model, in periods of four: whole-context attention beside linear attention,
+    window attention, window attention on the keys and values before it, window attention; dense and routed feed-forwards in
+    turn; heads of 128 with four queries per key / value head."""
+    heads = hidden // 128
+    gqa = dict(n_heads=heads, n_kv_heads=max(1, heads // 4), head_dim=128, v_dim=128, conv_k=0, scale=128 ** -0.5, qk_norm=True)
+    moe = MoeConfig(n_experts=experts, top_k=top, ffn=ffn // 4, n_shared=1, shared_ffn=ffn // 4, router="sigmoid", weight_input=True)
+    specs = []
+    for i in range(n_layers):
+        if i % 4 == 0:
+            left = PagedGqaConfig(**gqa, temp_coef=0.1, temp_every=8192, slopes=True)
+            kind, mixer = "side_by_side", SideBySideConfig(left, GlaConfig(n_heads=heads, head_dim=64, v_dim=128, tau=16.0), 0.7, 0.7)
+        else:
+            kind, mixer = "gqa", PagedGqaConfig(**gqa, window=window, rope_dims=128, rope_theta=5e5, rope_factor=4.0, gated=True,
+                                                kv_from=i - 1 if i % 4 == 2 else None)
+        specs.append(LayerSpec(kind, mixer, 0 if i % 2 else ffn, dataclasses.replace(moe) if i % 2 else None))
+    return ModelConfig(name="zapolorn-style", family="zapolorn", n_layers=n_layers, layer_types=[x.kind for x in specs], hidden=hidden,
+                       vocab=vocab, norm_eps=1e-6, layer_specs=specs, block="post", embed_scale=float(hidden) ** 0.5, tied_head=True,
+                       weight_format="dense")
+
+
 def scaled_down(cfg: ModelConfig, hidden: int = 256, n_layers: int = 4, vocab: int = 1024) -> ModelConfig:
     """Same layer types, small dimensions: the CPU test shape of a large config."""
     c = dataclasses.replace(cfg)
@@ -412,6 +477,7 @@ PRESETS = {
     "ds4-style": ds4_style,
     "vabunex-style": vabunex_style,
     "debisun-style": debisun_style,
+    "zapolorn-style": zapolorn_style,
 }
 
 

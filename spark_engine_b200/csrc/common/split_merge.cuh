@@ -12,9 +12,10 @@ namespace spark {
 static __global__ void __launch_bounds__(256)
 split_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int nsplit, const float* __restrict__ sink,
                    int H, int L, int hpc, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gate, int ldg,
-                   const int* __restrict__ rows, int out_by_row) {
+                   const int* __restrict__ rows, int out_by_row, int ldo, float out_scale) {
   // out_by_row: result of launch row r goes to row rows[r] of `out` instead of row r
-  // gate (optional): one logit per head in the row's gate columns, the head's output is scaled by its sigmoid
+  // gate (optional): one logit per head in the row's gate columns, the head's output is scaled by its sigmoid; out_scale: a
+  // constant factor; ldo: row stride of `out` (heads of L columns)
   // The statistics of a head's splits are reduced by one warp (split s in lane s % 32, so empty trailing splits do not
   // change a bit of the result).
   extern __shared__ float wts[];                        // [hpc][nsplit]: exp(m_s - M) / l
@@ -43,7 +44,7 @@ split_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ p
       if (v.x != -INFINITY) l += __expf(v.x - M) * v.y;
     }
     l = warp_sum(l) + (sink ? __expf(sink[h] - M) : 0.f);
-    float inv = 1.f / l;
+    float inv = out_scale / l;
     if (gate) inv /= 1.f + expf(-__bfloat162float(gate[static_cast<size_t>(rows ? rows[r] : r) * ldg + h]));
     for (int s = lane; s < live; s += 32) {
       const float m = ml[s].x;
@@ -73,13 +74,14 @@ split_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ p
     }
     const __nv_bfloat162 b0 = __floats2bfloat162_rn(o.x, o.y), b1 = __floats2bfloat162_rn(o.z, o.w);
     uint2 ov; ov.x = *reinterpret_cast<const uint32_t*>(&b0); ov.y = *reinterpret_cast<const uint32_t*>(&b1);
-    *reinterpret_cast<uint2*>(out + (static_cast<size_t>(out_by_row && rows ? rows[r] : r) * H + h) * L + d) = ov;
+    *reinterpret_cast<uint2*>(out + static_cast<size_t>(out_by_row && rows ? rows[r] : r) * ldo + h * L + d) = ov;
   }
 }
 
 // hpc: heads per CTA -- enough CTAs for two per SM when rows are few.
 static inline int launch_split_merge(const float* part_o, const float* part_ml, int nsplit, const float* sink, int R, int H, int L,
-                                     void* out, const void* gate, int ldg, const int* rows, int out_by_row, cudaStream_t s) {
+                                     void* out, const void* gate, int ldg, const int* rows, int out_by_row, cudaStream_t s, int ldo = 0,
+                                     float out_scale = 1.f) {
   int hpc = H;
   while (hpc > 1 && (R * ((H + hpc - 1) / hpc) < 296 || hpc * nsplit * 4 > 48 * 1024)) hpc = (hpc + 1) / 2;
   if (hpc * nsplit * 4 > 48 * 1024) return -6;
@@ -87,7 +89,7 @@ static inline int launch_split_merge(const float* part_o, const float* part_ml, 
   const int threads = hpc * L4 >= 256 ? 256 : ((hpc * L4 + 31) / 32 * 32);   // whole warps
   split_merge_kernel<<<dim3(R, (H + hpc - 1) / hpc), threads, hpc * nsplit * 4, s>>>(part_o, part_ml, nsplit, sink, H, L, hpc,
                                                                                   (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, ldg,
-                                                                                  rows, out_by_row);
+                                                                                  rows, out_by_row, ldo ? ldo : H * L, out_scale);
   return 0;
 }
 

@@ -5,7 +5,8 @@
 //   row_update        res += an update (plain rows or the slots of a routed feed-forward; per-channel scale, or RMS-normed);
 //                     h = norm of the new residual (RMS, layer norm, or the residual itself), optionally an fp32 copy of h
 //   token_shift       five mixes h + (h' - h) mu_s of the current and the previous row of the sequence
-//   channel_decay     log decay  -exp(W2 tanh(z) + w0)  per channel, fp32 throughout
+//   channel_decay     log decay  -exp(W2 tanh(z) + w0)  or  ln(sigmoid(W2 z + w0)) / tau  per channel, fp32 throughout
+//   swiglu_rows       silu(gate) * up of [gate | up] rows, both times a weight per row if given
 //   gate_concat       [ group-RMSNorm(o) * w * gate(g) | gelu(gate) * up ]: the input row of the block's single output
 //                     product (the mixer's output matrix and the down projection are stored side by side along K)
 #include "../common/rows.cuh"
@@ -26,7 +27,7 @@ embed_scaled_kernel(const TW* __restrict__ table, const int* __restrict__ ids, f
 
 struct RowUpdate {
   float* res;                                   // [R, H], in place
-  // the update: `delta` rows, or sum over slots of wts * y (expert outputs) + sg * shared + self_w * self_x, or nothing
+  // the update: `delta` rows, or sum over slots of wts (null: 1) * y (expert outputs) + sg * shared + self_w * self_x, or nothing
   const float* delta;
   const float* y; const int* inv; const float* wts; const int* ids;      // pair p's row of y: inv[p] (inv null: p); ids[p] < 0: none
   const float* shared; const float* sg; const float* self_w; const void* self_x;
@@ -72,7 +73,7 @@ row_update_kernel(const __grid_constant__ RowUpdate a) {
           for (int q = 0; q < 4; ++q) {
             const int pi = r * a.slots + s0 + q;
             const bool live = s0 + q < a.slots && a.ids[pi] >= 0;
-            w[q] = live ? a.wts[pi] : 0.f;
+            w[q] = live ? (a.wts ? a.wts[pi] : 1.f) : 0.f;
             p[q] = live ? __ldcg(reinterpret_cast<const float4*>(a.y + static_cast<size_t>(a.inv ? a.inv[pi] : pi) * H + i))
                         : make_float4(0.f, 0.f, 0.f, 0.f);
           }
@@ -144,7 +145,7 @@ row_update_kernel(const __grid_constant__ RowUpdate a) {
       float s = 0.f;
       for (int k = 0; k < a.slots; ++k) {
         const int pi = r * a.slots + k;
-        if (a.ids[pi] >= 0) s = fmaf(a.wts[pi], a.y[static_cast<size_t>(a.inv ? a.inv[pi] : pi) * H + i], s);
+        if (a.ids[pi] >= 0) s = fmaf(a.wts ? a.wts[pi] : 1.f, a.y[static_cast<size_t>(a.inv ? a.inv[pi] : pi) * H + i], s);
       }
       if (own != 0.f) s = fmaf(own, ldf(sx + i), s);
       if (a.shared) s = fmaf(sg, a.shared[row + i], s);
@@ -213,18 +214,21 @@ token_shift_kernel(const float* __restrict__ h, const float* __restrict__ carrie
 // log of the decay exp(-exp(x)), bounded where the decay itself is 0 in fp32 (differences of its running sums stay exact)
 __device__ __forceinline__ float log_decay(float x) { return fmaxf(-expf(x), -105.f); }
 
+__device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+
 // grid (ceil(N / 32), ceil(R / RB)); 128 threads: four lanes per channel (eight ranks each in turn), RB rows per CTA.
-// rank is a multiple of 8.
-template <typename TW, int RB>
+// rank is a multiple of 8.  inv_tau 0: -exp(W2 tanh(z) + w0); else ln(sigmoid(W2 z + w0)) * inv_tau.
+template <typename TZ, typename TW, int RB>
 __global__ void __launch_bounds__(128)
-channel_decay_kernel(const float* __restrict__ z, int ldz, const TW* __restrict__ w2, int ldw, int rank,
-                     const float* __restrict__ w0, float* __restrict__ logw, int R, int N) {
+channel_decay_kernel(const TZ* __restrict__ z, int ldz, const TW* __restrict__ w2, int ldw, int rank,
+                     const float* __restrict__ w0, float* __restrict__ logw, int R, int N, float inv_tau) {
   extern __shared__ float t[];                               // [rank][RB]
   const int d = blockIdx.x * 32 + (threadIdx.x >> 2), part = threadIdx.x & 3, r0 = blockIdx.y * RB;
   pdl_wait();
   for (int i = threadIdx.x; i < rank * RB; i += 128) {
     const int k = i / RB, r = r0 + i % RB;
-    t[i] = r < R ? tanhf(z[static_cast<size_t>(r) * ldz + k]) : 0.f;
+    const float x = r < R ? ldf(z + static_cast<size_t>(r) * ldz + k) : 0.f;
+    t[i] = inv_tau > 0.f ? x : tanhf(x);
   }
   __syncthreads();
   float acc[RB];
@@ -245,7 +249,7 @@ channel_decay_kernel(const float* __restrict__ z, int ldz, const TW* __restrict_
     float v = acc[r];
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
-    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = log_decay(v + w0[d]);
+    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = inv_tau > 0.f ? log_sigmoid(v + w0[d]) * inv_tau : log_decay(v + w0[d]);
   }
 }
 
@@ -266,6 +270,24 @@ tanh_split_kernel(const float* __restrict__ z, int ldz, __nv_bfloat16* __restric
     const __nv_bfloat16 hi = __float2bfloat16(v);
     out[static_cast<size_t>(r) * 2 * n + k] = hi;
     out[static_cast<size_t>(r) * 2 * n + n + k] = __float2bfloat16(v - __bfloat162float(hi));
+  }
+}
+
+// grid (ceil(F / 1024), rows); 256 threads x 4 columns of [gate (F) | up (F)].  wts (optional): the weight of row r's pair is
+// wts[perm ? perm[r] : r].
+template <typename T>
+__global__ void __launch_bounds__(256)
+swiglu_rows_kernel(const T* __restrict__ gu, int ldi, int F, const float* __restrict__ wts, const int* __restrict__ perm,
+                   T* __restrict__ out, int ldo, int R) {
+  pdl_wait();
+  const int i = blockIdx.x * 1024 + threadIdx.x * 4;
+  if (i >= F) return;
+  for (int r = blockIdx.y; r < R; r += gridDim.y) {
+    const T* x = gu + static_cast<size_t>(r) * ldi + i;
+    const float4 g = ldf4(x), u = ldf4(x + F);
+    const float w = wts ? wts[perm ? perm[r] : r] : 1.f;
+    stf4(out + static_cast<size_t>(r) * ldo + i, make_float4(silu_t<T>(w * g.x) * (w * u.x), silu_t<T>(w * g.y) * (w * u.y),
+                                                             silu_t<T>(w * g.z) * (w * u.z), silu_t<T>(w * g.w) * (w * u.w)));
   }
 }
 
@@ -374,7 +396,7 @@ extern "C" int spark_embed_scaled(const void* table, const int* ids, float* out,
 
 extern "C" int spark_row_update(const RowUpdate* u, int R, int f32, cudaStream_t s) {
   if (R <= 0) return 0;
-  if (u->y && (u->slots <= 0 || !u->wts || !u->ids)) return -5;
+  if (u->y && (u->slots <= 0 || !u->ids)) return -5;
   if ((u->norm && !u->w) || (u->norm == 2 && !u->b) || (u->self_w && !u->self_x)) return -5;
   const uintptr_t al = reinterpret_cast<uintptr_t>(u->res) | reinterpret_cast<uintptr_t>(u->delta) | reinterpret_cast<uintptr_t>(u->y) |
                        reinterpret_cast<uintptr_t>(u->shared) | reinterpret_cast<uintptr_t>(u->self_x) | reinterpret_cast<uintptr_t>(u->scale) |
@@ -406,11 +428,32 @@ extern "C" int spark_channel_decay(const float* z, int ldz, const void* w2, int 
                                    int R, int N, int f32, cudaStream_t s) {
   if (R <= 0) return 0;
   if (rank <= 0 || (rank & 7) || (ldw & 7) || rank * 64 > 48 * 1024) return -5;
-#define SPARK_CHD(RB)                                                                                                     \
-  spark_launch_pdl(channel_decay_kernel<T, RB>, dim3((N + 31) / 32, (R + RB - 1) / RB), dim3(128), rank * RB * 4, s,      \
-                   dim3(1, 1, 1), z, ldz, (const T*)w2, ldw, rank, w0, logw, R, N)
-  SPARK_BY_TYPE(f32, if (R <= 4) SPARK_CHD(4); else SPARK_CHD(16))
+#define SPARK_CHD(TZ, RB, inv_tau)                                                                                        \
+  spark_launch_pdl(channel_decay_kernel<TZ, T, RB>, dim3((N + 31) / 32, (R + RB - 1) / RB), dim3(128), rank * RB * 4, s,  \
+                   dim3(1, 1, 1), (const TZ*)z, ldz, (const T*)w2, ldw, rank, w0, logw, R, N, inv_tau)
+  SPARK_BY_TYPE(f32, if (R <= 4) SPARK_CHD(float, 4, 0.f); else SPARK_CHD(float, 16, 0.f))
+  return spark_launch_rc(__func__);
+}
+
+// z in the activation type, columns up to the padded rank readable and zero (or w2's columns there zero); tau > 0.
+extern "C" int spark_log_sigmoid_decay(const void* z, int ldz, const void* w2, int ldw, int rank, const float* b, float tau, float* logw,
+                                       int R, int N, int f32, cudaStream_t s) {
+  if (R <= 0) return 0;
+  if (rank <= 0 || (rank & 7) || (ldw & 7) || rank * 64 > 48 * 1024 || !(tau > 0.f)) return -5;
+  const float* w0 = b;
+  const float inv_tau = 1.f / tau;
+  SPARK_BY_TYPE(f32, if (R <= 4) SPARK_CHD(T, 4, inv_tau); else SPARK_CHD(T, 16, inv_tau))
 #undef SPARK_CHD
+  return spark_launch_rc(__func__);
+}
+
+extern "C" int spark_swiglu_rows(const void* gu, int ldi, int F, const float* wts, const int* perm, void* out, int ldo, int R, int f32,
+                                 cudaStream_t s) {
+  if (R <= 0) return 0;
+  if ((F | ldi | ldo) & 7) return -5;
+  const dim3 grid((F + 1023) / 1024, R < 65535 ? R : 65535);
+  SPARK_BY_TYPE(f32, spark_launch_pdl(swiglu_rows_kernel<T>, grid, dim3(256), 0, s, dim3(1, 1, 1), (const T*)gu, ldi, F, wts, perm, (T*)out,
+                                      ldo, R))
   return spark_launch_rc(__func__);
 }
 

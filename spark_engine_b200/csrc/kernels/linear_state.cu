@@ -1,8 +1,11 @@
-// Linear recurrences without a delta rule, one kernel family for two mechanisms.  Per head, with state S [D, V] (fp32):
+// Linear recurrences without a delta rule, one kernel family for three mechanisms.  Per head, with state S [D, V] (fp32):
 //
 //   scalar decay (MODE 0):  S_t = a S_{t-1} + k_t v_t^T,          o_t = S_t^T q_t       (a: one constant per head)
 //   channel decay (MODE 1): o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,   S_t = diag(w_t) S_{t-1} + k_t v_t^T
 //                           (w_t in (0, 1) per key channel and token, u a bonus of the current token)
+//   channel decay (MODE 2): S_t = diag(w_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t
+//
+// Outputs are multiplied by a constant `qscale`.
 //
 // linear_seq_kernel   rows one after the other, state in registers: decode and verify rows, short portions, and the whole
 //                     32-bit mode.  `commit` = 0 leaves the state untouched; a later launch with the accepted row counts
@@ -12,7 +15,7 @@
 //   linear_scan         S <- exp(G_C) S + U_c over the chunks of a segment, element by element; leaves the state ENTERING each
 //                       chunk in place of U_c and the final state in the slot
 //   linear_chunk_o      o = (q exp(E)) S_in + sum_{j < i} (sum_c q_ic k_jc exp(E_ic - G_jc)) v_j + diagonal term
-// G is the running log decay inside the chunk (inclusive), E_i = G_i in MODE 0 and G_{i-1} in MODE 1.  Exponents are
+// G is the running log decay inside the chunk (inclusive), E_i = G_i in MODES 0 and 2, G_{i-1} in MODE 1.  Exponents are
 // only ever taken of differences that are <= 0 (for a pair of 16-row blocks the reference point lies between them, the
 // diagonal blocks are summed pair by pair), so no decay is too strong for fp32.  bf16 enters as operands that are bf16
 // anyway (activations of the projections); every fp32 factor (state, weights, decayed keys) goes to the tensor cores as
@@ -25,7 +28,7 @@ struct LinearArgs {
   const void *q, *k, *v;         // T: row r, head h, channel d at [r * ld + h * hs + d]
   int ldq, ldk, ldv, hsk, hsv;
   const float* log2a;            // MODE 0: log2 of the decay [H]
-  const float* logw;             // MODE 1: natural log of the decay [R, H * D]
+  const float* logw;             // MODES 1, 2: natural log of the decay [R, H * D]
   const float* u;                // MODE 1: [H, D]
   float* S;                      // [slots, H, D, V]
   const int* seg;                // [nseg][4]: slot, first row, rows, first position
@@ -33,6 +36,7 @@ struct LinearArgs {
   float* o;                      // [R, H * V]
   const float* h32; float* carried; int width;   // MODE 1: rows the token shift reads, and the per-slot carried row
   int H, D, V, commit, act;      // act: SiLU on q, k, v
+  float qscale;
 };
 
 // ------------------------------------------------------------------------------------------------ sequential form
@@ -65,7 +69,7 @@ linear_seq_kernel(const __grid_constant__ LinearArgs a) {
   auto fetch = [&](int t, float& x, float& w, float& vv) {
     const size_t r = r0 + t;
     x = c < D ? (tid < DP ? ldf(q + r * a.ldq + c) : ldf(k + r * a.ldk + c)) : 0.f;
-    w = (MODE == 1 && tid < DP && c < D) ? a.logw[r * (static_cast<size_t>(a.H) * D) + h * D + c] : 0.f;
+    w = (MODE >= 1 && tid < DP && c < D) ? a.logw[r * (static_cast<size_t>(a.H) * D) + h * D + c] : 0.f;
     vv = vin ? ldf(v + r * a.ldv + vcol) : 0.f;
   };
   float x, w, vv;
@@ -73,7 +77,7 @@ linear_seq_kernel(const __grid_constant__ LinearArgs a) {
   for (int t = 0; t < n; ++t) {
     const int b = t & 1;
     if (a.act) { x = silu_f(x); vv = silu_f(vv); }
-    if (tid < DP) { sq[b][c] = x; if (MODE == 1) sw[b][c] = c < D ? expf(w) : 0.f; }
+    if (tid < DP) { sq[b][c] = x; if (MODE >= 1) sw[b][c] = c < D ? expf(w) : 0.f; }
     else sk[b][c] = x;
     const float val = vv;
     if (t + 1 < n) fetch(t + 1, x, w, vv);
@@ -82,7 +86,7 @@ linear_seq_kernel(const __grid_constant__ LinearArgs a) {
       float o = 0.f;
 #pragma unroll
       for (int p = 0; p < NP; ++p) o += red[b ^ 1][p][lane];
-      a.o[(static_cast<size_t>(r0) + t - 1) * (static_cast<size_t>(a.H) * V) + h * V + vcol] = o;
+      a.o[(static_cast<size_t>(r0) + t - 1) * (static_cast<size_t>(a.H) * V) + h * V + vcol] = o * a.qscale;
     }
     float o = 0.f;
 #pragma unroll
@@ -91,6 +95,9 @@ linear_seq_kernel(const __grid_constant__ LinearArgs a) {
       const float kv = sk[b][d] * val;
       if (MODE == 0) {
         s[j] = fmaf(lam, s[j], kv);
+        o = fmaf(sq[b][d], s[j], o);
+      } else if (MODE == 2) {
+        s[j] = fmaf(sw[b][d], s[j], kv);
         o = fmaf(sq[b][d], s[j], o);
       } else {
         o = fmaf(sq[b][d], fmaf(su[d], kv, s[j]), o);
@@ -104,7 +111,7 @@ linear_seq_kernel(const __grid_constant__ LinearArgs a) {
     float o = 0.f;
 #pragma unroll
     for (int p = 0; p < NP; ++p) o += red[(n - 1) & 1][p][lane];
-    a.o[(static_cast<size_t>(r0) + n - 1) * (static_cast<size_t>(a.H) * V) + h * V + vcol] = o;
+    a.o[(static_cast<size_t>(r0) + n - 1) * (static_cast<size_t>(a.H) * V) + h * V + vcol] = o * a.qscale;
   }
   if (a.commit) {
 #pragma unroll
@@ -220,7 +227,7 @@ __device__ __forceinline__ void load_decays(float* __restrict__ G, int ldg, cons
   }
 }
 
-// grid (chunks, H, ceil(V / 64)); 128 threads.  ws_u [chunk][H][D][V]; MODE 1 also ws_d [chunk][H][D] = exp(G_C).
+// grid (chunks, H, ceil(V / 64)); 128 threads.  ws_u [chunk][H][D][V]; MODES 1, 2 also ws_d [chunk][H][D] = exp(G_C).
 template <int DP, int MODE>
 __global__ void __launch_bounds__(128)
 linear_chunk_u_kernel(const __grid_constant__ LinearArgs a, const int* __restrict__ chunks, float* __restrict__ ws_u,
@@ -489,7 +496,7 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
       *reinterpret_cast<uint32_t*>(A0 + r * LDK + c) = hi;
       *reinterpret_cast<uint32_t*>(A1 + r * LDK + c) = lo;
     }
-    // diagonal blocks, pair by pair: i > j decayed from j to i - 1, i == j weighted by the bonus
+    // diagonal blocks, pair by pair: i > j decayed from j to i - 1 (MODE 2: to i), i == j weighted by the bonus
     for (int p = lane; p < 136; p += 32) {
       int i = 0;
       while ((i + 1) * (i + 2) / 2 <= p) ++i;
@@ -498,14 +505,14 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
       float s = 0.f;
       if (i == j) {
         for (int c = 0; c < a.D; ++c)
-          s = fmaf(__bfloat162float(Rr[ri * LDR + c]) * a.u[h * a.D + c], __bfloat162float(Kr[rj * LDR + c]), s);
+          s = fmaf(__bfloat162float(Rr[ri * LDR + c]) * (MODE == 1 ? a.u[h * a.D + c] : 1.f), __bfloat162float(Kr[rj * LDR + c]), s);
       } else {
         float s1 = 0.f;
 #pragma unroll 4
         for (int c = 0; c < DP; c += 2) {                                  // (channels past D are zero)
           const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Rr + ri * LDR + c));
           const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Kr + rj * LDR + c));
-          const float2 e = *reinterpret_cast<const float2*>(G + (ri - 1) * LDG + c), f = *reinterpret_cast<const float2*>(G + rj * LDG + c);
+          const float2 e = *reinterpret_cast<const float2*>(G + (MODE == 1 ? ri - 1 : ri) * LDG + c), f = *reinterpret_cast<const float2*>(G + rj * LDG + c);
           s = fmaf(x.x * y.x, ex2(e.x - f.x), s);
           s1 = fmaf(x.y * y.y, ex2(e.y - f.y), s1);
         }
@@ -515,13 +522,14 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
     }
     __syncthreads();
   }
-  // receptance fragment of one 16-channel step: r exp(E - ref), E = G of the previous row
+  // receptance fragment of one 16-channel step: r exp(E - ref), E = G of the previous row (MODE 2: of the row)
   auto rfrag = [&](int ks, int ref_row, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int row = (e & 1) ? row_hi : row_lo, c = ks * 16 + 2 * t + (e >> 1) * 8;
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Rr + row * LDR + c));
-      const float2 E = row > 0 ? *reinterpret_cast<const float2*>(G + (row - 1) * LDG + c) : make_float2(0.f, 0.f);
+      const int er = MODE == 1 ? row - 1 : row;
+      const float2 E = er >= 0 ? *reinterpret_cast<const float2*>(G + er * LDG + c) : make_float2(0.f, 0.f);
       const float2 f = ref_row >= 0 ? *reinterpret_cast<const float2*>(G + ref_row * LDG + c) : make_float2(0.f, 0.f);
       split2(x.x * ex2(E.x - f.x), x.y * ex2(E.y - f.y), hi[e], lo[e]);
     }
@@ -592,7 +600,7 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
         lc_ldsm4t(bl, Sl + off);
         lc_mma(o[2 * np], xh, bh[0], bh[1]); lc_mma(o[2 * np + 1], xh, bh[2], bh[3]);
         lc_mma(o[2 * np], xh, bl[0], bl[1]); lc_mma(o[2 * np + 1], xh, bl[2], bl[3]);
-        if (MODE == 1) { lc_mma(o[2 * np], xl, bh[0], bh[1]); lc_mma(o[2 * np + 1], xl, bh[2], bh[3]); }
+        if (MODE >= 1) { lc_mma(o[2 * np], xl, bh[0], bh[1]); lc_mma(o[2 * np + 1], xl, bh[2], bh[3]); }
       }
     }
     if (MODE == 0) {
@@ -617,10 +625,11 @@ linear_chunk_o_kernel(const __grid_constant__ LinearArgs a, const int* __restric
       for (int e = 0; e < 4; e += 2) {
         const int row = e ? row_hi : row_lo, c = v0 + i * 8 + 2 * t;
         float* p = a.o + (r0 + row) * (static_cast<size_t>(a.H) * a.V) + h * a.V + c;
-        if (row < nv && c + 1 < a.V && (a.V & 1) == 0) *reinterpret_cast<float2*>(p) = make_float2(o[i][e], o[i][e + 1]);
+        const float x = o[i][e] * a.qscale, y = o[i][e + 1] * a.qscale;
+        if (row < nv && c + 1 < a.V && (a.V & 1) == 0) *reinterpret_cast<float2*>(p) = make_float2(x, y);
         else if (row < nv) {
-          if (c < a.V) p[0] = o[i][e];
-          if (c + 1 < a.V) p[1] = o[i][e + 1];
+          if (c < a.V) p[0] = x;
+          if (c + 1 < a.V) p[1] = y;
         }
       }
   }
@@ -661,11 +670,12 @@ static int launch_seq(const LinearArgs& a, int nseg, cudaStream_t s) {
 
 static LinearArgs linear_args(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, int hsk, int hsv,
                               const float* log2a, const float* logw, const float* u, float* S, const int* seg, const int* n_rows,
-                              float* o, const float* h32, float* carried, int width, int H, int D, int V, int commit, int act) {
+                              float* o, const float* h32, float* carried, int width, int H, int D, int V, int commit, int act,
+                              float qscale) {
   LinearArgs a;
   a.q = q; a.k = k; a.v = v; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.hsk = hsk; a.hsv = hsv;
   a.log2a = log2a; a.logw = logw; a.u = u; a.S = S; a.seg = seg; a.n_rows = n_rows; a.o = o;
-  a.h32 = h32; a.carried = carried; a.width = width; a.H = H; a.D = D; a.V = V; a.commit = commit; a.act = act;
+  a.h32 = h32; a.carried = carried; a.width = width; a.H = H; a.D = D; a.V = V; a.commit = commit; a.act = act; a.qscale = qscale;
   return a;
 }
 
@@ -676,16 +686,17 @@ using namespace spark;
 #define SPARK_LINEAR_PARAMS                                                                                              \
   const void *q, int ldq, const void *k, int ldk, const void *v, int ldv, int hsk, int hsv, const float *log2a,          \
       const float *logw, const float *u, float *S, const int *seg, const int *n_rows, float *o, const float *h32,        \
-      float *carried, int width, int H, int D, int V, int commit, int act
+      float *carried, int width, int H, int D, int V, int commit, int act, float qscale
 #define SPARK_LINEAR_ARGS \
-  linear_args(q, ldq, k, ldk, v, ldv, hsk, hsv, log2a, logw, u, S, seg, n_rows, o, h32, carried, width, H, D, V, commit, act)
+  linear_args(q, ldq, k, ldk, v, ldv, hsk, hsv, log2a, logw, u, S, seg, n_rows, o, h32, carried, width, H, D, V, commit, act, qscale)
 
-// log2a != nullptr: scalar decay per head; else channel decay (logw, u).
+// log2a != nullptr: scalar decay per head; else channel decay (logw), with a bonus u or (u null) without.
 extern "C" int spark_linear_seq(SPARK_LINEAR_PARAMS, int nseg, int f32, cudaStream_t s) {
   if (nseg <= 0) return 0;
   const LinearArgs a = SPARK_LINEAR_ARGS;
   if (log2a) return f32 ? launch_seq<float, 0>(a, nseg, s) : launch_seq<__nv_bfloat16, 0>(a, nseg, s);
-  return f32 ? launch_seq<float, 1>(a, nseg, s) : launch_seq<__nv_bfloat16, 1>(a, nseg, s);
+  if (u) return f32 ? launch_seq<float, 1>(a, nseg, s) : launch_seq<__nv_bfloat16, 1>(a, nseg, s);
+  return f32 ? launch_seq<float, 2>(a, nseg, s) : launch_seq<__nv_bfloat16, 2>(a, nseg, s);
 }
 
 // chunks: int [n_chunks][2] = (segment, chunk in segment); chunk0: int [nseg] first chunk of a segment.  D <= 128.
@@ -696,7 +707,8 @@ extern "C" int spark_linear_chunked(SPARK_LINEAR_PARAMS, int nseg, const int* ch
   if (n_rows != nullptr || D > 128) return -5;
   const LinearArgs a = SPARK_LINEAR_ARGS;
 #define SPARK_LCH(DP) (log2a ? launch_chunked<DP, 0>(a, chunks, n_chunks, chunk0, nseg, ws_u, ws_d, s) \
-                             : launch_chunked<DP, 1>(a, chunks, n_chunks, chunk0, nseg, ws_u, ws_d, s))
+         : u  ? launch_chunked<DP, 1>(a, chunks, n_chunks, chunk0, nseg, ws_u, ws_d, s) \
+                             : launch_chunked<DP, 2>(a, chunks, n_chunks, chunk0, nseg, ws_u, ws_d, s))
   if (D <= 32) return SPARK_LCH(32);
   if (D <= 64) return SPARK_LCH(64);
   return SPARK_LCH(128);

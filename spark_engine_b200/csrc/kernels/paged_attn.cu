@@ -1,16 +1,19 @@
-// Grouped-query softmax attention over a paged cache (64-token pages of per-token key / value rows), without rotation, for
-// bf16 and fp32 activations:
+// Grouped-query softmax attention over a paged cache (64-token pages of per-token key / value rows), for bf16 and fp32
+// activations:
 //
 //   conv_prep     short causal convolution over time on the stacked [q | k | v] projections: queries to a buffer, keys and
 //                 values to their pages; the last taps - 1 projected rows of a sequence are its state
+//   head_prep     RMS norm per query / key head, rotation, temperature of the queries; keys and values to their pages (or
+//                 queries alone, for a layer that reads another layer's cache)
 //   paged_prefill prompts: flash-style tiles on tensor cores, one page of keys per step
 //   paged_decode  decode / verify rows: split-KV, a page per split, the query heads of a key / value head as MMA rows
 //   paged_rows    one CTA per (row, head) on the FP32 units: the 32-bit mode, and head sizes the others do not cover
 //
 // Scores are soft-capped (cap * tanh(q.k scale / cap); cap 0: not), get a bias per head and distance (the last entry serves
-// everything farther; null: none), and are visible inside the row's aligned chunk of the sequence (chunk 0: everything before
-// it).  An optional sink per head enters the denominator only.  Scores, softmax and its weights are fp32; the weights enter the
-// tensor-core product as two-term bf16 sums.  Head widths are padded to 16.
+// everything farther; null: none) or lose slope * distance, and are visible inside the row's aligned chunk of the sequence or a
+// window that ends at the row (both 0: everything before it).  An optional sink per head enters the denominator only, an
+// optional sigmoid gate per head and a constant scale the outputs.  Scores, softmax and its weights are fp32; the weights enter
+// the tensor-core product as two-term bf16 sums.  Head widths are padded to 16.
 #include "../common/rows.cuh"
 #include "../common/split_merge.cuh"
 
@@ -21,17 +24,26 @@ constexpr float PGA_LOG2E = 1.4426950408889634f;
 
 struct PagedAttn {
   const void *q, *k, *v;                 // q [rows, ldq]; caches [pages, 64, G * D] / [pages, 64, G * V]
-  void* out;                             // [rows, H * V]
+  void* out;                             // [rows, ldo]: heads of V columns
   const int *pos, *rows, *row_slot;      // per plan row; rows: launch row -> plan row (null: identity)
   const int* pages;                      // [slots, page_ld]
   const float *bias, *sink;              // [H, bias_n] / [H]
   float *part_o, *part_ml;
   const int* segs;                       // prompts: slot, first row, rows, first position (stride seg_ld)
-  int page_ld, H, G, D, V, ldq, bias_n, chunk, seg_ld, nsplit;
-  float scale, cap;
+  const float* slopes;                   // [H]: taken off per token of distance
+  const void* gate;                      // [rows, ldg]: one logit per head
+  int page_ld, H, G, D, V, ldq, bias_n, chunk, seg_ld, nsplit, window, ldg, ldo;
+  float scale, cap, out_scale;
 };
 
-__device__ __forceinline__ int chunk_first(int p, int chunk) { return chunk > 0 ? p / chunk * chunk : 0; }
+__device__ __forceinline__ int first_visible(int p, const PagedAttn& a) {
+  return a.chunk > 0 ? p / a.chunk * a.chunk : (a.window > 0 ? max(p - a.window + 1, 0) : 0);
+}
+// factor of head h's output in plan row pr
+template <typename T>
+__device__ __forceinline__ float head_factor(const PagedAttn& a, int pr, int h) {
+  return a.gate ? a.out_scale * sigmoid_f(ldf(static_cast<const T*>(a.gate) + static_cast<size_t>(pr) * a.ldg + h)) : a.out_scale;
+}
 
 // tanh to fp32 accuracy in the sense of the soft cap: the Taylor polynomial near 0 (where the quotient form would cancel),
 // 1 - 2 / (exp(2z) + 1) elsewhere (absolute error of a few 2^-23).  The polynomial gives tanh(z) / z.
@@ -143,6 +155,76 @@ conv_prep_kernel(const __grid_constant__ ConvPrep a) {
   }
 }
 
+// ------------------------------------------------------------------------------------------------ norm and rotation per head
+struct HeadPrep {
+  const void* proj;                      // [R, ldp]: H query heads, then G key heads (Dp columns each) and G value heads (Vp)
+  const float *q_norm, *k_norm;          // [D] (null: no norm)
+  void *q, *k, *v;                       // q [R, H * Dp]; caches as in PagedAttn
+  const double* inv_freq;                // [rot / 2]
+  const int *pos, *row_slot, *pages;
+  int* status;
+  double temp_every;
+  int ldp, R, H, G, D, Dp, Vp, rot, page_ld;      // G 0: queries only
+  float eps, temp_coef;
+};
+
+// grid (R, head groups); 256 threads: a warp per head, four consecutive channels per lane and step.
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_prep_kernel(const __grid_constant__ HeadPrep a) {
+  extern __shared__ float2 turn[];                           // [rot / 2]: cosine and sine of the row's angles
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x, lane = threadIdx.x & 31, p = a.pos[r];
+  for (int i = threadIdx.x; i < a.rot / 2; i += 256) {
+    float sn, cs;
+    sincosf(static_cast<float>(static_cast<double>(p) * a.inv_freq[i]), &sn, &cs);
+    turn[i] = make_float2(cs, sn);
+  }
+  __syncthreads();
+  const T* row = static_cast<const T*>(a.proj) + static_cast<size_t>(r) * a.ldp;
+  int page = 0;
+  if (a.G > 0) {
+    page = p / PGA_PAGE < a.page_ld ? a.pages[static_cast<size_t>(a.row_slot[r]) * a.page_ld + p / PGA_PAGE] : -1;
+    if (page < 0 && threadIdx.x == 0 && blockIdx.y == 0) set_status(a.status, ST_BOUNDS, r, p, a.row_slot[r]);
+  }
+  const size_t tok = static_cast<size_t>(max(page, 0)) * PGA_PAGE + p % PGA_PAGE;
+  for (int h = blockIdx.y * 8 + (threadIdx.x >> 5); h < a.H + 2 * a.G; h += gridDim.y * 8) {
+    if (h >= a.H && page < 0) break;                         // no page behind this position: nothing is written
+    if (h >= a.H + a.G) {
+      const int g = h - a.H - a.G;
+      const T* x = row + (a.H + a.G) * a.Dp + g * a.Vp;
+      T* d = static_cast<T*>(a.v) + (tok * a.G + g) * a.Vp;
+      for (int i = lane * 4; i < a.Vp; i += 128) stf4(d + i, ldf4(x + i));
+      continue;
+    }
+    const bool isq = h < a.H;
+    const T* x = row + h * a.Dp;
+    T* d = isq ? static_cast<T*>(a.q) + (static_cast<size_t>(r) * a.H + h) * a.Dp : static_cast<T*>(a.k) + (tok * a.G + h - a.H) * a.Dp;
+    const float* w = isq ? a.q_norm : a.k_norm;
+    float4 x0 = make_float4(0.f, 0.f, 0.f, 0.f);             // (padded channels are zero)
+    if (lane * 4 < a.Dp) x0 = ldf4(x + lane * 4);
+    float m = 1.f;
+    if (w) {
+      float ss = x0.x * x0.x + x0.y * x0.y + x0.z * x0.z + x0.w * x0.w;
+      for (int i = lane * 4 + 128; i < a.Dp; i += 128) { const float4 y = ldf4(x + i); ss += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w; }
+      m = 1.f / sqrtf(warp_sum(ss) / a.D + a.eps);
+    }
+    if (isq && a.temp_coef != 0.f) m *= 1.f + a.temp_coef * logf(static_cast<float>(floor((p + 1) / a.temp_every)) + 1.f);
+    for (int i = lane * 4; i < a.Dp; i += 128) {
+      float4 y = i < 128 ? x0 : ldf4(x + i);
+      if (w) {
+        y.x *= i < a.D ? w[i] : 0.f; y.y *= i + 1 < a.D ? w[i + 1] : 0.f;
+        y.z *= i + 2 < a.D ? w[i + 2] : 0.f; y.w *= i + 3 < a.D ? w[i + 3] : 0.f;
+      }
+      y.x *= m; y.y *= m; y.z *= m; y.w *= m;
+      if (i < a.rot) { const float2 t = turn[i >> 1]; y = make_float4(y.x * t.x - y.y * t.y, y.y * t.x + y.x * t.y, y.z, y.w); }
+      if (i + 2 < a.rot) { const float2 t = turn[(i >> 1) + 1]; y = make_float4(y.x, y.y, y.z * t.x - y.w * t.y, y.w * t.x + y.z * t.y); }
+      stf4(d + i, y);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ one row, one head
 // grid (rows, H); 128 threads.  V <= 1024.
 template <typename T>
@@ -162,7 +244,7 @@ paged_rows_kernel(const __grid_constant__ PagedAttn a) {
 #pragma unroll
   for (int c = 0; c < 8; ++c) acc[c] = 0.f;
   float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f;
-  for (int k0 = chunk_first(p, a.chunk); k0 <= p; k0 += 128) {
+  for (int k0 = first_visible(p, a); k0 <= p; k0 += 128) {
     const int tok = k0 + t;
     float s = -INFINITY;
     if (tok <= p) {
@@ -175,6 +257,7 @@ paged_rows_kernel(const __grid_constant__ PagedAttn a) {
       s = x * a.scale;
       if (a.cap > 0.f) s = a.cap * tanhf(s / a.cap);
       if (a.bias) s += a.bias[static_cast<size_t>(h) * a.bias_n + min(p - tok, a.bias_n - 1)];
+      if (a.slopes) s -= a.slopes[h] * static_cast<float>(p - tok);
     }
     float mx = warp_max(s);
     if ((t & 31) == 0) sh[t >> 5] = mx;
@@ -197,10 +280,10 @@ paged_rows_kernel(const __grid_constant__ PagedAttn a) {
     }
     __syncthreads();
   }
-  const float inv = 1.f / l;
+  const float inv = head_factor<T>(a, pr, h) / l;
 #pragma unroll
   for (int c = 0; c < 8; ++c)
-    if (t + c * 128 < a.V) stf(static_cast<T*>(a.out) + (static_cast<size_t>(pr) * a.H + h) * a.V + t + c * 128, acc[c] * inv);
+    if (t + c * 128 < a.V) stf(static_cast<T*>(a.out) + static_cast<size_t>(pr) * a.ldo + h * a.V + t + c * 128, acc[c] * inv);
 }
 
 // ------------------------------------------------------------------------------------------------ tensor-core helpers
@@ -231,7 +314,7 @@ __device__ __forceinline__ void pga_split2(float x, float y, uint32_t& hi, uint3
 // ------------------------------------------------------------------------------------------------ decode rows
 constexpr int PGA_HEADS = 16;            // query heads per CTA (MMA rows)
 
-// grid (rows, G * head groups, splits); 128 threads.  Split s covers page (first page of the row's chunk) + s.
+// grid (rows, G * head groups, splits); 128 threads.  Split s covers page (page of the row's first visible key) + s.
 __global__ void __launch_bounds__(128)
 paged_decode_kernel(const __grid_constant__ PagedAttn a) {
   extern __shared__ __align__(16) uint8_t smem_pga[];
@@ -247,7 +330,7 @@ paged_decode_kernel(const __grid_constant__ PagedAttn a) {
   const int rep = a.H / a.G, groups = (rep + PGA_HEADS - 1) / PGA_HEADS, g = blockIdx.y / groups, hg = blockIdx.y % groups;
   const int h0 = g * rep + hg * PGA_HEADS, nh = min(PGA_HEADS, rep - hg * PGA_HEADS);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gg = lane >> 2, t = lane & 3;
-  const int p = a.pos[pr], first = chunk_first(p, a.chunk), page = first / PGA_PAGE + sp, k0 = page * PGA_PAGE;
+  const int p = a.pos[pr], first = first_visible(p, a), page = first / PGA_PAGE + sp, k0 = page * PGA_PAGE;
   const size_t pb = (static_cast<size_t>(r) * a.H + h0) * a.nsplit + sp;
   if (k0 > p) {                                              // empty split
     if (tid < nh) {
@@ -301,6 +384,7 @@ paged_decode_kernel(const __grid_constant__ PagedAttn a) {
           x = s[j][e] * a.scale;
           if (a.cap > 0.f) x = a.cap * cap_tanh(x * icap);
           if (a.bias) x += __ldg(a.bias + static_cast<size_t>(h0 + row) * a.bias_n + min(p - k0 - tok, a.bias_n - 1));
+          if (a.slopes) x -= __ldg(a.slopes + h0 + row) * static_cast<float>(p - k0 - tok);
         }
         Ss[row * 68 + tok] = x;
       }
@@ -366,7 +450,7 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, t = lane & 3;
   const int rows_valid = min(BM, n - qt * BM), pbase = pos0 + qt * BM;
   const int nkeys = pbase + rows_valid;
-  const int j0 = chunk_first(pbase, a.chunk) / BN, j1 = (nkeys + BN - 1) / BN;
+  const int j0 = first_visible(pbase, a) / BN, j1 = (nkeys + BN - 1) / BN;
   const int vk = D >> 3, vvs = a.V >> 3;
   constexpr int vv = VP >> 3;
   const int* pg = a.pages + static_cast<size_t>(slot) * a.page_ld;
@@ -406,8 +490,9 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
   const float m0 = a.sink ? a.sink[h] * PGA_LOG2E : -INFINITY;
   float m_lo = m0, m_hi = m0, l_lo = a.sink && t == 0 ? 1.f : 0.f, l_hi = l_lo;
   const int w0 = pbase + warp * 16, p_lo = w0 + gq, p_hi = p_lo + 8;         // padded rows: positions past the segment, not stored
-  const int f_lo = chunk_first(p_lo, a.chunk), f_hi = chunk_first(p_hi, a.chunk);
-  const int w_first = chunk_first(w0, a.chunk), w_last = chunk_first(w0 + 15, a.chunk);
+  const int f_lo = first_visible(p_lo, a), f_hi = first_visible(p_hi, a);
+  const int w_first = first_visible(w0, a), w_last = first_visible(w0 + 15, a);
+  const float slope = a.slopes ? a.slopes[h] * PGA_LOG2E : 0.f;
   const float qs = a.cap > 0.f ? a.scale / a.cap : a.scale * PGA_LOG2E, cs = a.cap * PGA_LOG2E, csqs = cs * qs;
   for (int j = j0; j < j1; ++j) {
     const int buf = (j - j0) & 1, k0 = j * BN;
@@ -453,6 +538,13 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
       for (int i = 0; i < 8; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[i][e] *= qs;
+    }
+    if (a.slopes) {
+      const float d = static_cast<float>(k0 + 2 * t - p_lo);
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[i][e] = fmaf(slope, d + static_cast<float>(i * 8 + (e & 1) - (e >> 1) * 8), s[i][e]);
     }
     float mx_lo = m_lo, mx_hi = m_hi;
     float b_hi[2] = {0.f, 0.f}, b_lo[2] = {0.f, 0.f};
@@ -509,8 +601,8 @@ paged_prefill_kernel(const __grid_constant__ PagedAttn a) {
   for (int hh = 0; hh < 2; ++hh) {
     const int rl = warp * 16 + gq + hh * 8;
     if (rl >= rows_valid) continue;
-    const float inv = 1.f / (hh ? l_hi : l_lo);
-    __nv_bfloat16* d = static_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(r0 + qt * BM + rl) * a.H + h) * a.V + 2 * t;
+    const float inv = head_factor<__nv_bfloat16>(a, r0 + qt * BM + rl, h) / (hh ? l_hi : l_lo);
+    __nv_bfloat16* d = static_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(r0 + qt * BM + rl) * a.ldo + h * a.V + 2 * t;
 #pragma unroll
     for (int i = 0; i < VP / 8; ++i)
       if (i * 8 < a.V) *reinterpret_cast<__nv_bfloat162*>(d + i * 8) = __floats2bfloat162_rn(o[i][2 * hh] * inv, o[i][2 * hh + 1] * inv);
@@ -532,7 +624,7 @@ static int launch_paged_prefill(const PagedAttn& a, int nseg, int max_rows, cuda
 
 static bool paged_ok(const PagedAttn* a) {
   return a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->D > 0 && a->V > 0 && ((a->D | a->V) & 15) == 0 && (a->ldq & 7) == 0 &&
-         (!a->bias || a->bias_n > 0);
+         (!a->bias || a->bias_n > 0) && (a->ldo & 3) == 0 && a->ldo >= a->H * a->V;
 }
 
 }  // namespace spark
@@ -560,6 +652,18 @@ extern "C" int spark_conv_prep(const ConvPrep* a, int nseg, int max_rows, int f3
   return spark_launch_rc(__func__);
 }
 
+// Rows of the whole plan: finished queries, and with G > 0 the cache rows.
+extern "C" int spark_head_prep(const HeadPrep* a, int f32, cudaStream_t s) {
+  if (a->R <= 0) return 0;
+  if (a->H <= 0 || ((a->Dp | a->Vp) & 15) || a->D > a->Dp || (a->rot & 1) || a->rot > a->D || (a->ldp & 7) || a->rot > 8192 ||
+      a->ldp < a->H * a->Dp + a->G * (a->Dp + a->Vp) || (a->rot && !a->inv_freq) || !(a->temp_every > 0.0)) return -5;
+  const int groups = (a->H + 2 * a->G + 7) / 8;
+  const dim3 grid(a->R, a->R <= 128 && groups <= 65535 ? groups : 1);    // few rows: a head per warp
+  if (f32) spark_launch_pdl(head_prep_kernel<float>, grid, dim3(256), a->rot * 4, s, dim3(1, 1, 1), *a);
+  else spark_launch_pdl(head_prep_kernel<__nv_bfloat16>, grid, dim3(256), a->rot * 4, s, dim3(1, 1, 1), *a);
+  return spark_launch_rc(__func__);
+}
+
 extern "C" int spark_paged_rows(const PagedAttn* a, int n, int f32, cudaStream_t s) {
   if (n <= 0) return 0;
   if (!paged_ok(a) || a->V > 1024 || a->D > 8192 || a->H > 65535) return -5;
@@ -569,7 +673,7 @@ extern "C" int spark_paged_rows(const PagedAttn* a, int n, int f32, cudaStream_t
   return spark_launch_rc(__func__);
 }
 
-// bf16.  part_o fp32 [n, H, nsplit, V], part_ml fp32 [n, H, nsplit, 2]; nsplit >= pages that a chunk up to any row spans.
+// bf16.  part_o fp32 [n, H, nsplit, V], part_ml fp32 [n, H, nsplit, 2]; nsplit >= pages that any row's visible keys span.
 extern "C" int spark_paged_decode(const PagedAttn* a, int n, cudaStream_t s) {
   if (n <= 0) return 0;
   if (!paged_ok(a) || a->nsplit <= 0 || a->nsplit > 65535) return -5;
@@ -580,7 +684,7 @@ extern "C" int spark_paged_decode(const PagedAttn* a, int n, cudaStream_t s) {
   const int rep = a->H / a->G, groups = (rep + PGA_HEADS - 1) / PGA_HEADS;
   if (a->G * groups > 65535) return -5;
   spark_launch_pdl(paged_decode_kernel, dim3(n, a->G * groups, a->nsplit), dim3(128), smem, s, dim3(1, 1, 1), *a);
-  const int rc = launch_split_merge(a->part_o, a->part_ml, a->nsplit, a->sink, n, a->H, a->V, a->out, nullptr, 0, a->rows, 1, s);
+  const int rc = launch_split_merge(a->part_o, a->part_ml, a->nsplit, a->sink, n, a->H, a->V, a->out, a->gate, a->ldg, a->rows, 1, s, a->ldo, a->out_scale);
   return rc ? rc : spark_launch_rc(__func__);
 }
 

@@ -232,7 +232,7 @@ def decode_step_bytes(W, cfg: ModelConfig, rows: int) -> int:
             total += sum(nbytes(t) for k, t in lw["mix"].items() if k != "kv_up")
             c = cfg.layer_specs[i].moe
             for k, t in lw["mlp"].items():
-                share = min(1.0, rows * c.top_k / c.n_routes) if c is not None and k in ("w_up", "w_down") else 1.0
+                share = min(1.0, rows * c.top_k / c.n_routes) if c is not None and k in ("w_up", "w_gu", "w_down") else 1.0
                 total += int(nbytes(t) * share)
             continue
         total += nbytes(lw["mix"]) + nbytes(lw["in_norm"]) + nbytes(lw["post_norm"])

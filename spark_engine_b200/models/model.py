@@ -626,6 +626,8 @@ class MoeBlock:
         c = self.c
         if "dense_up" in self.w:
             return ops.linear(ops.linear_relu2(h, self.w["dense_up"]), self.w["dense_down"], out_f32=True)
+        if self.dense and self.cfg.layer_specs:
+            return ops.linear(ops.linear_swiglu(h, self.w["dense_gu"]), self.w["dense_down"], out_f32=True)
         if self.dense:
             gu = ops.linear(h, self.w["dense_gu"])
             return ops.linear(ops.swiglu(gu, c.swiglu_limit), self.w["dense_down"])
@@ -671,9 +673,9 @@ class Model:
             from .spec_mixers import build_spec_mixer
             for lw, i in zip(lws, self.cfg.layer_runs()):       # every run of a layer has its own cache or state
                 spec = self.cfg.layer_specs[i]
-                mlp = MoeBlock(self.cfg, lw["mlp"], spec.moe) if self.cfg.block == "sequential" and "post_norm" in lw else None
+                mlp = MoeBlock(self.cfg, lw["mlp"], spec.moe) if self.cfg.block != "parallel" and "post_norm" in lw else None
                 out.append((lw, build_spec_mixer(self.cfg, spec, lw["mix"], self.n_slots, self.n_pages, self.page, self.page_table,
-                                                 self.device, self.dtype), mlp))
+                                                 self.device, self.dtype, [m for _, m, _ in out]), mlp))
             return out
         for lw in lws:
             kind = lw["type"]
@@ -740,6 +742,13 @@ class Model:
         if cfg.block == "parallel":          # `mix` holds the feed-forward too
             h, X, h32 = ops.add_norm_rows(pend, X, self._norm(lw, "in_norm"), self.dtype, mix.wants_f32_rows)
             return X, mix.forward(h, plan, self.seqs, commit, h32=h32)
+        if cfg.block == "post":              # the sublayers read the residual itself, their outputs are normed
+            h, X, _ = ops.add_norm_rows(pend, X, None, self.dtype)
+            pend = ops.Update(mix.forward(h, plan, self.seqs, commit), post=self._norm(lw, "mix_norm"))
+            if mlp is not None:
+                h, X, _ = ops.add_norm_rows(pend, X, None, self.dtype)
+                pend = ops.Update(mlp.forward(h, defer=True), post=self._norm(lw, "post_norm"))
+            return X, pend
         h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "in_norm"), self.dtype)
         pend = ops.Update(mix.forward(h, plan, self.seqs, commit), lw.get("ls1"))
         if mlp is not None:

@@ -9,8 +9,8 @@ from __future__ import annotations
 
 import importlib
 
-ARCHITECTURES = {"Vabunex": "vabunex", "Debisun": "debisun"}
-FAMILIES = {"vabunex": "vabunex", "debisun": "debisun"}
+ARCHITECTURES = {"Vabunex": "vabunex", "Debisun": "debisun", "Zapolorn": "zapolorn"}
+FAMILIES = {"vabunex": "vabunex", "debisun": "debisun", "zapolorn": "zapolorn"}
 
 
 def architecture(d: dict):

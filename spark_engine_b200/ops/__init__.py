@@ -132,6 +132,15 @@ def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return relu2(x @ w.to(x.dtype).t())
 
 
+def linear_swiglu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """silu(x G^T) * (x U^T) for w = [G | U] stacked."""
+    if use_kernels(x):
+        return block_ops().linear_swiglu(x, w)
+    gu = x @ w.to(x.dtype).t()
+    n = gu.shape[1] // 2
+    return L.swiglu(gu[:, :n].float(), gu[:, n:].float()).to(x.dtype)
+
+
 def linear_token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, off: int, n: int) -> torch.Tensor:
     """gelu_tanh(x W^T) * table[ids, off : off + n] (columns from n on are zero; ids outside the table give zero rows)."""
     if use_kernels(x):
@@ -216,6 +225,9 @@ def route(h, w, c):
     if c.router in ("softmax", "softmax_bias"):
         p = torch.softmax(logits, -1)
         sel = p if c.router == "softmax" else p + w["bias"].float().to(p.device)
+    elif c.router == "sigmoid":
+        idx = torch.sort(logits, dim=-1, descending=True, stable=True).indices[:, : c.top_k]
+        return torch.sigmoid(torch.gather(logits, 1, idx)) * c.route_scale, idx, sg
     elif c.router == "sigmoid_bias":
         p = torch.sigmoid(logits)
         sel = p + w["bias"].float().to(p.device)
@@ -245,9 +257,11 @@ def moe(h, w, c, defer: bool = False):
             if not lo <= e < hi:
                 continue
             rows = (idx[:, slot] == e).nonzero(as_tuple=True)[0]
-            gu = hf[rows] @ _expert(wgu, e - lo).t()
-            y = (relu2(gu) if single else L.swiglu(gu[:, : c.ffn], gu[:, c.ffn:], c.swiglu_limit)) @ _expert(wd, e - lo).t()
-            out[rows] += wts[rows, slot].unsqueeze(1) * y
+            a = wts[rows, slot].unsqueeze(1)
+            gu = (hf[rows] * a if c.weight_input else hf[rows]) @ _expert(wgu, e - lo).t()
+            n = gu.shape[1] // 2
+            y = (relu2(gu) if single else L.swiglu(gu[:, :n], gu[:, n:], c.swiglu_limit)) @ _expert(wd, e - lo).t()
+            out[rows] += y if c.weight_input else a * y
     if c.n_identity:
         out += (wts * (idx >= c.n_experts)).sum(-1, keepdim=True) * hf
     if "s_up" in w:
@@ -412,10 +426,10 @@ def relu2(x):
     return torch.relu(x).square()
 
 
-def paged_gqa(mixer, proj, plan, commit):
+def paged_gqa(mixer, proj, plan, commit, out=None):
     if use_kernels(proj):
         from . import paged_attn
-        return paged_attn.mixer(mixer, proj, plan, commit)
+        return paged_attn.mixer(mixer, proj, plan, commit, out)
     return None
 
 
@@ -452,6 +466,7 @@ def gate_concat(o, n, group, w, eps, gate, kind, ff, width_ff, off, width, dtype
         if kind is not None:
             x = x * (torch.sigmoid(gate.float()) if kind == "sigmoid" else F.silu(gate.float()))
         out[:, :n] = x.to(dtype)
+        out[:, n:off] = 0
     if ff is not None:
         up = width - off
         out[:, off: off + width_ff] = (gelu_tanh(ff[:, :width_ff]) * ff[:, up: up + width_ff].float()).to(dtype)
@@ -484,12 +499,20 @@ def channel_decay(z, w2, w0, n: int, w2x2=None):
     return -torch.exp(torch.tanh(z.float()) @ w2.float().t() + w0)
 
 
+def log_sigmoid_decay(z, w2, b, n: int, tau: float):
+    """ln(sigmoid(z w2^T + b)) / tau [R, n] in fp32: the log of sigmoid(..)^(1/tau)."""
+    if use_kernels(z):
+        return block_ops().log_sigmoid_decay(z, w2, b, n, tau)
+    return F.logsigmoid(z.float() @ w2.float().t()[: z.shape[1]] + b) / tau
+
+
 def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=None, u=None, h32=None, carried=None,
-                 n_rows=None):
-    """Decayed linear attention (constant decay per head, or decay per channel and token with a bonus for the current
-    token): o fp32 [R, H * V]; the slots' states advance when `commit` (by n_rows[i] rows of segment i if given)."""
+                 n_rows=None, qscale=1.0):
+    """Decayed linear attention (constant decay per head; or decay per channel and token, with a bonus `u` for the current
+    token, or without one on the state after the current token): o fp32 [R, H * V], times `qscale`; the slots' states advance
+    when `commit` (by n_rows[i] rows of segment i if given)."""
     if use_kernels(q):
-        return block_ops().linear_state(q, k, v, H, D, V, S, plan, commit, act, log2a, logw, u, h32, carried, n_rows)
+        return block_ops().linear_state(q, k, v, H, D, V, S, plan, commit, act, log2a, logw, u, h32, carried, n_rows, qscale)
     R = q.shape[0]
     q, k, v = q.float().view(R, H, D), k.float().view(R, H, D), v.float().view(R, H, V)
     if act:
@@ -501,8 +524,8 @@ def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=
         n = s.n if n_rows is None else min(s.n, int(n_rows[i]))
         for r in range(s.r0, s.r0 + n):
             kv = k[r].unsqueeze(-1) * v[r].unsqueeze(-2)
-            if a is not None:
-                St = a * St + kv
+            if a is not None or u is None:
+                St = (a if a is not None else torch.exp(logw[r]).view(H, D, 1)) * St + kv
                 o[r] = torch.einsum("hd,hdv->hv", q[r], St)
             else:
                 o[r] = torch.einsum("hd,hdv->hv", q[r], St + u.view(H, D, 1) * kv)
@@ -511,7 +534,7 @@ def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=
             S[s.slot] = St
             if carried is not None:
                 carried[s.slot] = h32[s.r0 + n - 1]
-    return o.view(R, H * V)
+    return o.view(R, H * V) * qscale
 
 
 def latent_mixer(mixer, proj, plan, cat):
