@@ -249,7 +249,7 @@ channel_decay_kernel(const TZ* __restrict__ z, int ldz, const TW* __restrict__ w
     float v = acc[r];
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
-    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = inv_tau > 0.f ? log_sigmoid(v + w0[d]) * inv_tau : log_decay(v + w0[d]);
+    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = inv_tau > 0.f ? fmaxf(log_sigmoid(v + w0[d]) * inv_tau, -105.f) : log_decay(v + w0[d]);
   }
 }
 

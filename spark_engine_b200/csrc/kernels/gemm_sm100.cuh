@@ -87,7 +87,7 @@ struct GemmSmem {
 // Epilogue functor contract:
 //   __device__ void operator()(const TileCoord& tc, int row, int col, const float (&v)[32]) const
 // `row` is a valid global row (< tc.row_end), `col` the first of 32 consecutive output columns
-// (col + 32 may exceed N: the functor guards).  In gate-up mode `v` already holds silu(g)*u.
+// (col + 32 may exceed N: the functor guards).  In gate-up mode `v` already holds act(row_weight * g, row_weight * u).
 template <int BN, class Epi, bool GROUPED>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
@@ -200,6 +200,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       const int row = tc.a_row0 + quarter * 32 + lane;
       const uint32_t t_addr = tmem_base + acc * BN + (static_cast<uint32_t>(quarter * 32) << 16);
       if (g.gate_up_F > 0) {
+        const float rw = row < tc.row_end ? epi.row_weight(row) : 0.f;
 #pragma unroll 1
         for (int c = 0; c < BN / 2; c += 32) {
           uint32_t rg[32], ru[32];
@@ -208,7 +209,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
           tmem_ld_wait();
           float v[32];
 #pragma unroll
-          for (int i = 0; i < 32; ++i) v[i] = epi.act(__uint_as_float(rg[i]), __uint_as_float(ru[i]));
+          for (int i = 0; i < 32; ++i) v[i] = epi.act(rw * __uint_as_float(rg[i]), rw * __uint_as_float(ru[i]));
           if (row < tc.row_end) epi(tc, row, tc.out_col0 + c, v);
         }
       } else {
@@ -253,6 +254,7 @@ struct EpiStoreBf16 {
   __nv_bfloat16* C; int ldc; int N;
   __device__ __forceinline__ void cta_done(int) const {}
   __device__ __forceinline__ float act(float g, float u) const { return g; }
+  __device__ __forceinline__ float row_weight(int) const { return 1.f; }
   __device__ __forceinline__ void operator()(const TileCoord&, int row, int col, const float (&v)[32]) const {
     __nv_bfloat16* dst = C + static_cast<size_t>(row) * ldc + col;
     if (col + 32 <= N && (ldc & 7) == 0) {
@@ -276,6 +278,7 @@ struct EpiStoreF32 {
   float* C; int ldc; int N;
   __device__ __forceinline__ void cta_done(int) const {}
   __device__ __forceinline__ float act(float g, float u) const { return g; }
+  __device__ __forceinline__ float row_weight(int) const { return 1.f; }
   __device__ __forceinline__ void operator()(const TileCoord&, int row, int col, const float (&v)[32]) const {
     float* dst = C + static_cast<size_t>(row) * ldc + col;
     if (col + 32 <= N && (ldc & 3) == 0) {
@@ -287,10 +290,13 @@ struct EpiStoreF32 {
   }
 };
 
-// SwiGLU (optionally clamped) over a [gate | up] tile pair -> bf16 [rows, F].
+// SwiGLU (optionally clamped) over a [gate | up] tile pair -> bf16 [rows, F].  With weights, gate and up of sorted row r are
+// multiplied by the weight of its pair first (an expert that sees its input times the weight).
 struct EpiSwigluBf16 {
   static constexpr bool kWarpTile = false;
   __nv_bfloat16* C; int ldc; int N; float limit;
+  const float* wts; const int* perm;
+  __device__ __forceinline__ float row_weight(int row) const { return wts ? wts[perm[row]] : 1.f; }
   __device__ __forceinline__ void cta_done(int) const {}
   __device__ __forceinline__ float act(float g, float u) const {
     if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
@@ -308,6 +314,7 @@ struct EpiActBf16 {
   __nv_bfloat16* C; int ldc; int N; OutAct a;
   __device__ __forceinline__ void cta_done(int) const {}
   __device__ __forceinline__ float act(float g, float u) const { return g; }
+  __device__ __forceinline__ float row_weight(int) const { return 1.f; }
   __device__ __forceinline__ void operator()(const TileCoord& tc, int row, int col, const float (&v)[32]) const {
     float y[32];
     if (a.kind == 1) {
@@ -350,6 +357,7 @@ struct EpiPushRS {
   int* counter;
   const uint32_t* seq_ptr;
   __device__ __forceinline__ float act(float g, float u) const { return g; }
+  __device__ __forceinline__ float row_weight(int) const { return 1.f; }
   __device__ __forceinline__ void operator()(const TileCoord&, int row, int col, const float (&v)[32]) const {
     const int owner = row / rows_per_rank, lr = row - owner * rows_per_rank;
     float* dst = reinterpret_cast<float*>(peers[owner] + slot_off) + (static_cast<size_t>(rank) * rows_per_rank + lr) * N + col;

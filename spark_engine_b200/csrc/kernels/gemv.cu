@@ -19,13 +19,15 @@ __device__ __forceinline__ void unpack8(const uint4& v, float (&f)[8]) {
   for (int i = 0; i < 4; ++i) { float2 t = __bfloat1622float2(p[i]); f[2 * i] = t.x; f[2 * i + 1] = t.y; }
 }
 
-// act: 0 none; 1 = input is [gate | up] (2K wide), x := swiglu(gate, up) computed while staging.
+// act: 0 none; 1 = input is [gate | up] (2K wide), x := swiglu(gate, up) computed while staging; with x_weight (one per item)
+// gate and up are multiplied by the item's weight first.
 template <int RB, typename TO>
 __global__ void __launch_bounds__(GEMV_WARPS * 32)
 gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W,
                  long long expert_stride, int ldw, TO* __restrict__ y, int ldy, int rows_per_item, int N, int K,
                  const int* __restrict__ pair_expert, const int* __restrict__ pair_row, int act, float limit,
-                 long long x_item_stride, long long y_item_stride, int cpc, const OutAct oact) {
+                 long long x_item_stride, long long y_item_stride, int cpc, const float* __restrict__ x_weight,
+                 const OutAct oact) {
   extern __shared__ __align__(16) uint8_t smem_gemv[];
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem_gemv);     // [RB][K]
   const int item = blockIdx.y;
@@ -49,12 +51,13 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
       reinterpret_cast<uint4*>(xs)[i] = v;
     }
   } else {
+    const float xw = x_weight ? x_weight[item] : 1.f;
     for (int i = threadIdx.x; i < RB * K; i += blockDim.x) {
       const int r = i / K, k = i - r * K;
       float v = 0.f;
       if (r < R) {
         const __nv_bfloat16* xr = x + static_cast<size_t>(xr0 + r) * ldx;
-        float g = __bfloat162float(xr[k]), u = __bfloat162float(xr[K + k]);
+        float g = xw * __bfloat162float(xr[k]), u = xw * __bfloat162float(xr[K + k]);
         if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
         v = g / (1.f + __expf(-g)) * u;
       }
@@ -120,7 +123,7 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
 template <int RB, typename TO>
 static int launch_gemv(const void* x, int ldx, const void* W, long long es, int ldw, void* y, int ldy, int items,
                        int rows, int N, int K, const int* pe, const int* pr, int act, float limit, const OutAct& oact, cudaStream_t s,
-                       long long xis = 0, long long yis = 0) {
+                       long long xis = 0, long long yis = 0, const float* xw = nullptr) {
   auto kern = gemv_bf16_kernel<RB, TO>;
   const int smem = RB * K * 2;
   if (smem > 48 * 1024) {
@@ -135,7 +138,7 @@ static int launch_gemv(const void* x, int ldx, const void* W, long long es, int 
   dim3 grid((groups + cpc - 1) / cpc, items);
   const cudaError_t err = spark_launch_pdl(kern, grid, dim3(GEMV_WARPS * 32), smem, s, dim3(1, 1, 1),
                                            (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, es, ldw, (TO*)y, ldy, rows, N, K,
-                                           pe, pr, act, limit, xis, yis, cpc, oact);
+                                           pe, pr, act, limit, xis, yis, cpc, xw, oact);
   return err == cudaSuccess ? 0 : -4;
 }
 
@@ -387,8 +390,9 @@ using namespace spark;
 // items x rows_per_item rows; K % 8 == 0; out_f32 selects fp32 or bf16 output.
 extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long expert_stride, int ldw, void* y, int ldy,
                                int items, int rows_per_item, int N, int K, const int* pair_expert, const int* pair_row,
-                               int act, float limit, int out_f32, const OutAct* out, cudaStream_t s) {
+                               int act, float limit, int out_f32, const OutAct* out, cudaStream_t s, const float* x_weight) {
   if (items <= 0 || rows_per_item <= 0) return 0;
+  if (x_weight && act != 1) return -5;
   const OutAct oact = out ? *out : OutAct{};
   if (K % 8 || rows_per_item > 16) return -5;
   if (gemv_wide_ok(ldx, ldw, items, N, K, pair_expert, pair_row, act) &&
@@ -402,9 +406,9 @@ extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long 
 #define SPARK_GEMV_CASE(RB)                                                                                          \
   if (rows_per_item <= RB)                                                                                           \
     return out_f32 ? launch_gemv<RB, float>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N, K,       \
-                                            pair_expert, pair_row, act, limit, oact, s)                                    \
+                                            pair_expert, pair_row, act, limit, oact, s, 0, 0, x_weight)                    \
                    : launch_gemv<RB, __nv_bfloat16>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N,  \
-                                                    K, pair_expert, pair_row, act, limit, oact, s);
+                                                    K, pair_expert, pair_row, act, limit, oact, s, 0, 0, x_weight);
   SPARK_GEMV_CASE(1)
   SPARK_GEMV_CASE(2)
   SPARK_GEMV_CASE(4)

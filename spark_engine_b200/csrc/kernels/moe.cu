@@ -15,7 +15,8 @@ namespace spark {
 constexpr int ROUTE_THREADS = 256;
 constexpr int ROUTE_MAXE_PER_THREAD = 4;     // up to 1024 experts
 
-// kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias (the bias enters the choice only).
+// kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias (the bias enters the choice only), 4 sigmoid, not
+// renormalised (ranked by the logits, which a saturated sigmoid would tie).
 // The last n_self of the E router outputs are identity experts: they leave -1 in `ids` and their weight in self_w[row].
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int kind, const float* __restrict__ bias,
@@ -62,6 +63,9 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
       s[j] = p[j];
       if (kind == 3 && t + j * ROUTE_THREADS < E) s[j] += bias[t + j * ROUTE_THREADS];
     }
+  } else if (kind == 4) {
+#pragma unroll
+    for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) { s[j] = p[j]; p[j] = 1.f / (1.f + expf(-p[j])); }
   } else {
 #pragma unroll
     for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) {
@@ -112,7 +116,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
   if (t == 0) {
     float sum = 0.f;
     for (int k = 0; k < top_k; ++k) sum += sel_p[k];
-    sum = fmaxf(sum, 1e-20f);
+    sum = kind == 4 ? 1.f : fmaxf(sum, 1e-20f);
     float own = 0.f;
     for (int k = 0; k < top_k; ++k) {
       const float w = sel_p[k] / sum * scale;
@@ -136,7 +140,7 @@ struct RouterArgs {
   const __nv_bfloat16* x; int ldx;           // [R, K]
   const __nv_bfloat16* Wg; int ldw;          // [E (+1), K]
   float* logits; int ld;                     // scratch [R, ld]
-  int R, K, E, top_k, kind;                  // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias
+  int R, K, E, top_k, kind;                  // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias, 4 sigmoid
   const float* bias; float scale; int shared_gate;
   int slots;                                 // top_k, or top_k + 1 when the shared expert is a pair
   int shared_expert;                         // index of the shared expert in the local stack (slot top_k)
@@ -264,7 +268,9 @@ moe_router_topk_kernel(const __grid_constant__ RouterArgs a) {
       s[j] = p[j];
       mx = fmaxf(mx, p[j]);
     }
-    if (a.kind == 0) {
+    if (a.kind == 4) {
+      // ranked by the logits, only the k winners' sigmoids are formed
+    } else if (a.kind == 0) {
       // softmax -> top-k -> renormalise: the softmax denominator cancels, so experts are ranked by their logits and
       // only the k winners are exponentiated
       mx = warp_max(mx);
@@ -313,13 +319,14 @@ moe_router_topk_kernel(const __grid_constant__ RouterArgs a) {
 #pragma unroll
         for (int j = 0; j < EPL; ++j) if (j == bj) { bp = p[j]; s[j] = -INFINITY; }
         if (a.kind == 0) bp = __expf(bp - mx);
+        if (a.kind == 4) bp = 1.f / (1.f + expf(-bp));
         lane_best(s, best, bj);
       }
       const float wp = __shfl_sync(0xffffffffu, bp, wi & 31);
       if (lane == k) { selp = wp; seli = wi; }
       tot += wp;                                            // slot order, identical on every lane
     }
-    tot = fmaxf(tot, 1e-20f);
+    tot = a.kind == 4 ? 1.f : fmaxf(tot, 1e-20f);
     if (a.self_w) {
       float own = 0.f;
       for (int k = 0; k < a.top_k; ++k) {                   // slot order, as the combine adds the others

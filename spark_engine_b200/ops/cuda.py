@@ -25,11 +25,11 @@ vp, i32, i64, f32 = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _SIGS = {
     "spark_gemm_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "spark_gemm_bf16_swiglu": [vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp],
-    "spark_gemm_grouped_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, i32, f32, i32, vp, vp],
+    "spark_gemm_grouped_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, i32, f32, i32, vp, vp, vp, vp],
     "spark_gemm_bf16_act": [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp],
     "spark_gemm_simt": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, i32, i32, vp, vp],
     "spark_gemm_simt_grouped": [vp, i32, vp, i32, i64, vp, i32, i32, i32, vp, vp, i32, vp, i32, i32, i32, vp, vp],
-    "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, f32, i32, vp, vp],
+    "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, f32, i32, vp, vp, vp],
     "spark_gemv_bf16_items": [vp, i32, i64, vp, i64, i32, vp, i32, i64, i32, i32, i32, i32, vp, i32, vp],
     "spark_add_rmsnorm": [vp, i32, vp, vp, vp, i32, i32, f32, i32, vp],
     "spark_rmsnorm_bf16": [vp, vp, vp, i32, i32, f32, i32, vp],
@@ -80,12 +80,15 @@ _SIGS = {
 }
 
 # parallel blocks (ops/parallel_block.py)
-_LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32]
+_LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32]
 _SIGS.update({
     "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, i32, vp, vp],
     "spark_row_update": [vp, i32, i32, vp],
     "spark_token_shift": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, vp],
     "spark_channel_decay": [vp, i32, vp, i32, i32, vp, vp, i32, i32, i32, vp],
+    "spark_log_sigmoid_decay": [vp, i32, vp, i32, i32, vp, f32, vp, i32, i32, i32, vp],
+    "spark_swiglu_rows": [vp, i32, i32, vp, vp, vp, i32, i32, i32, vp],
+    "spark_head_prep": [vp, i32, vp],
     "spark_neg_exp_bias": [vp, vp, i32, i32, vp],
     "spark_tanh_split": [vp, i32, vp, i32, i32, vp],
     "spark_gate_concat": [vp, i32, i32, i32, vp, f32, vp, i32, i32, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp],
@@ -290,7 +293,8 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out_f32: bool = False, fmt: int 
 
 
 def gemv_bf16(x, w, items=1, rows_per_item=None, pair_expert=None, pair_row=None, act=0, limit=0.0, out_f32=False,
-              expert_stride=0, n=None, k=None, out=None, ldx=None, oact=None):
+              expert_stride=0, n=None, k=None, out=None, ldx=None, oact=None, x_weight=None):
+    """`x_weight` (act 1): fp32 weight per item, multiplied into gate and up."""
     rows_per_item = rows_per_item if rows_per_item is not None else x.shape[0]
     n = n if n is not None else w.shape[-2]
     k = k if k is not None else w.shape[-1]
@@ -305,7 +309,7 @@ def gemv_bf16(x, w, items=1, rows_per_item=None, pair_expert=None, pair_row=None
         dbg.check_index("gemv_bf16 pair_row", pair_row, 0, x.shape[0], count=items)
     rc = lib().spark_gemv_bf16(P(x), ldx if ldx is not None else x.stride(0), P(w), expert_stride, w.stride(-2), P(y), ldy,
                                items, rows_per_item, n, k, P(pair_expert), P(pair_row), act, float(limit), int(out_f32),
-                               _act(oact), stream())
+                               _act(oact), stream(), P(x_weight))
     check(rc, "spark_gemv_bf16")
     return y
 
@@ -723,7 +727,7 @@ def gather_rows(src, idx32):
 
 
 # ----------------------------------------------------------------------------- MoE
-ROUTER_KIND = {"softmax": 0, "sigmoid_bias": 1, "sqrt_softplus": 2, "softmax_bias": 3}
+ROUTER_KIND = {"softmax": 0, "sigmoid_bias": 1, "sqrt_softplus": 2, "softmax_bias": 3, "sigmoid": 4}
 
 
 def moe_route(h, w, c, e_lo=0, e_hi=None, self_w=None):
@@ -770,13 +774,14 @@ def moe_sort(ids, E):
     return perm, inv, offs, tiles, ntile, max_tiles
 
 
-def grouped_gemm(a, b, tiles, ntile, max_tiles, n_experts, rows_per_expert, N, mode, limit=0.0, fmt=1):
-    """a [P, K] rows in expert order; b [E*rows_per_expert, K]; mode 0 -> fp32 [P, N]; 1 -> swiglu bf16 [P, N]."""
+def grouped_gemm(a, b, tiles, ntile, max_tiles, n_experts, rows_per_expert, N, mode, limit=0.0, fmt=1, wts=None, perm=None):
+    """a [P, K] rows in expert order; b [E*rows_per_expert, K]; mode 0 -> fp32 [P, N]; 1 -> swiglu bf16 [P, N]; 2 -> squared relu
+    bf16 [P, N].  `wts` (mode 1): row i of `a` counts wts[perm[i]] times."""
     Pn, K = a.shape
-    out = torch.empty(Pn, N, dtype=torch.bfloat16 if mode == 1 else torch.float32, device=a.device)
+    out = torch.empty(Pn, N, dtype=torch.float32 if mode == 0 else torch.bfloat16, device=a.device)
     rc = lib().spark_gemm_grouped_bf16(P(a), P(b), P(out), Pn, N, K, a.stride(0), K, N, n_experts, rows_per_expert,
                                        P(tiles), P(ntile), max_tiles, mode, float(limit), fmt, P(status_word(a.device)),
-                                       stream())
+                                       stream(), P(wts), P(perm))
     check(rc, "spark_gemm_grouped_bf16")
     return out
 
@@ -862,9 +867,9 @@ def moe(h, w, c, defer: bool = False):
     outputs of a decode round).  Under expert parallelism (`w["ep"]` = (first local expert, end)) only the local
     experts' pairs are computed and the result is this rank's partial sum; the shared expert is added by the rank
     that holds it."""
-    if c.act == "relu2":
-        from .moe_relu import moe as moe_relu
-        return moe_relu(h, w, c, defer)
+    if c.act == "relu2" or c.weight_input:
+        from .moe_spec import moe as moe_spec
+        return moe_spec(h, w, c, defer)
     if h.shape[0] * c.top_k <= DECODE_PAIRS_MAX and h.shape[0] <= DECODE_ROWS_MAX and FUSED_DECODE:
         return _moe_decode(h, w, c, defer)
     h = _as_bf16(h).contiguous()

@@ -91,6 +91,35 @@ def channel_decay(z, w2, w0, n: int, w2x2=None):
     return out
 
 
+def log_sigmoid_decay(z, w2, b, n: int, tau: float):
+    """z [R, rank] in the activation type (columns up to w2's padded rank are readable) -> ln(sigmoid(w2 z + b)) / tau fp32."""
+    R, r = z.shape[0], w2.shape[1]
+    out = torch.empty(R, n, dtype=torch.float32, device=z.device)
+    check(lib().spark_log_sigmoid_decay(P(z), z.stride(0), P(w2), w2.stride(0), r, P(b), float(tau), P(out), R, n, _is32(w2.dtype), stream()),
+          "spark_log_sigmoid_decay")
+    return out
+
+
+def swiglu_rows(gu, wts=None, perm=None):
+    """silu(gate) * up of [gate | up] rows; `wts` (fp32): gate and up of row r count wts[perm[r]] times."""
+    R, n = gu.shape[0], gu.shape[1] // 2
+    out = torch.empty(R, n, dtype=gu.dtype, device=gu.device)
+    check(lib().spark_swiglu_rows(P(gu), gu.stride(0), n, P(wts), P(perm), P(out), n, R, _is32(gu.dtype), stream()), "spark_swiglu_rows")
+    return out
+
+
+def linear_swiglu(x, w):
+    """silu(x G^T) * (x U^T) for w = [G | U] (halves of a multiple of 128 rows)."""
+    R, F = x.shape[0], w.shape[0] // 2
+    if w.dtype != torch.bfloat16 or R <= 16 or w.shape[1] % 8 or F % 128:
+        return swiglu_rows(cu.dense_linear(x, w))
+    x = cu._as_bf16(x).contiguous()
+    out = torch.empty(R, F, dtype=torch.bfloat16, device=x.device)
+    check(lib().spark_gemm_bf16_swiglu(P(x), P(w), P(out), R, F, w.shape[1], x.stride(0), w.stride(0), F, 0.0, P(status_word(x.device)),
+                                       stream()), "spark_gemm_bf16_swiglu")
+    return out
+
+
 GATES = {None: 0, "sigmoid": 1, "silu": 2}
 
 
@@ -154,10 +183,11 @@ def _split(plan, dev):
 
 
 def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=None, u=None, h32=None, carried=None,
-                 n_rows=None):
-    """Decayed linear attention of every segment from its slot's state S [slots, H, D, V]; returns o fp32 [R, H * V].
-    `log2a` [H]: constant decay per head; else `logw` [R, H * D] (log decay) and `u` (bonus), with the token-shift row
-    carried along (h32 rows -> carried [slots, width]).  `n_rows`: device counts of accepted rows (commit)."""
+                 n_rows=None, qscale=1.0):
+    """Decayed linear attention of every segment from its slot's state S [slots, H, D, V]; returns o fp32 [R, H * V], times
+    `qscale`.  `log2a` [H]: constant decay per head; else `logw` [R, H * D] (log decay) and `u` (bonus; None: outputs read the
+    state behind the current token), with the token-shift row carried along (h32 rows -> carried [slots, width]).  `n_rows`:
+    device counts of accepted rows (commit)."""
     dev = q.device
     d = cu._plan_dev(plan, dev)
     R = q.shape[0]
@@ -168,7 +198,7 @@ def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=
 
     def args(seg):
         return (P(q), q.stride(0), P(k), k.stride(0), P(v), v.stride(0), D, V, P(log2a), P(logw), P(u), P(S), P(seg), P(n_rows), P(o),
-                P(h32), P(carried), width, H, D, V, int(commit), int(act))
+                P(h32), P(carried), width, H, D, V, int(commit), int(act), float(qscale))
     short, longs = (d["seg"], plan.segs), (None, [])
     if n_rows is None and commit and q.dtype == torch.bfloat16 and D <= 128:
         short, longs = _split(plan, dev)

@@ -221,7 +221,7 @@ def debisun_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> 
     from ..models.layout import pad
     from ..models.model import AttnMixer
     from ..models.paged_gqa import PagedGqaMixer
-    from ..ops import moe_relu
+    from ..ops import moe_spec
     fig = Figures(peaks)
     rnd, put = fig.rnd, fig.put
     N, H, G, D = 2048, 16, 4, 128
@@ -231,7 +231,7 @@ def debisun_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> 
     C = (H + 2 * G) * D
     w = {"conv_t": rnd(4, C) * 0.5, "dist_bias": rnd(H, 1025), "sink": torch.zeros(H, device=DEV)}
     pages = torch.arange(R * ctx // 64, dtype=torch.int32, device=DEV).view(R, -1).contiguous()
-    mx = PagedGqaMixer(cfg, spec, w, R, R * ctx // 64, 64, pages, DEV, torch.bfloat16)
+    mx = PagedGqaMixer(cfg, spec.mixer, w, R, R * ctx // 64, 64, pages, DEV, torch.bfloat16)
     at = AttnMixer(near, {}, R * ctx, DEV, torch.bfloat16)
     for t in (mx.k, mx.v, at.k, at.v):
         t.copy_(rnd(*t.shape))
@@ -286,7 +286,7 @@ def debisun_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> 
         def touched(c, ids):                     # bytes of the distinct experts a round reads, and the pairs that have an expert
             live = ids[(ids >= 0) & (ids < c.n_experts)]
             return live.unique().numel(), live.numel()
-        e1, pairs1 = touched(c, moe_relu._route(d16, w1, c, torch.empty(rows, device=DEV))[1])
+        e1, pairs1 = touched(c, moe_spec._route(d16, w1, c, torch.empty(rows, device=DEV))[1])
         e2, pairs2 = touched(c2, cu.moe_route(d16, w2, c2)[1])
         put(f"routed squared-relu experts + update, {tag}", f"routed SwiGLU experts + update, {tag}",
             lambda: ops.add_norm_rows(ops.Update(ops.moe(d16, w1, c, True), one), res, None, torch.bfloat16),
