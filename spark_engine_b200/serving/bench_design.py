@@ -4,6 +4,7 @@ the measured copy bandwidth / GEMM throughput.
 
   vabunex   beside KDA linear attention + latent attention in sequential pre-norm blocks with dense feed-forwards
   debisun   beside grouped-query attention (rotary, no chunks) with softmax-routed SwiGLU experts, as many parameters
+  zapolorn  beside grouped-query attention (rotary, whole context) with dense and softmax-routed SwiGLU feed-forwards of its sizes
 
 Device-timed with CUDA events.  Model figures stream more weights and activations than L2 holds; kernel figures write a
 buffer larger than L2 between iterations (median of the iterations)."""
@@ -15,7 +16,8 @@ import statistics
 
 import torch
 
-from ..config import AttnConfig, EngineConfig, KdaConfig, MlaConfig, ModelConfig, MoeConfig, debisun_style, glm_style, vabunex_style
+from ..config import AttnConfig, EngineConfig, KdaConfig, MlaConfig, ModelConfig, MoeConfig, debisun_style, glm_style, vabunex_style, \
+    zapolorn_style
 from ..models.build import build_random_model, decode_step_bytes
 from ..models.plan import make_plan
 from ..ops import cuda as cu
@@ -298,11 +300,134 @@ def debisun_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> 
     return fig.done()
 
 
+# ----------------------------------------------------------------------------- zapolorn
+ZAP_SIZES = {"1024": (1024, 3072), "2048": (2048, 6144), "4096": (4096, 12288)}
+ZAP_WINDOW = 1024
+
+
+def zapolorn_config(hidden: int, ffn: int):
+    return zapolorn_style(12, hidden, ffn, VOCAB, experts=DEB_EXPERTS, top=DEB_TOP, window=ZAP_WINDOW)
+
+
+def zapolorn_closest(hidden: int, ffn: int, layers: int):
+    """The same heads, dense and routed feed-forwards (the dense ones first); attention over the whole context in every layer, no
+    linear attention beside it."""
+    h = hidden // 128
+    return ModelConfig(name="gqa + swiglu, dense weights", family="hybrid", n_layers=layers, layer_types=["attn"] * layers, hidden=hidden, vocab=VOCAB,
+                       attn=AttnConfig(n_q_heads=h, n_kv_heads=max(1, h // 4), head_dim=128, rope_dim=128),
+                       moe=MoeConfig(n_experts=DEB_EXPERTS, top_k=DEB_TOP, ffn=ffn // 4, n_shared=1, shared_ffn=ffn // 4, router="softmax",
+                                     dense_layers=layers // 2, dense_ffn=ffn), weight_format="dense")
+
+
+def zapolorn_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> dict:
+    """Kernels at hidden size 2048 (16 query and 4 key / value heads of 128, 32 experts of 1536, top 4; linear attention with 16 heads
+    of 64 x 128).  Like kernels: the closest model's; for windows the chunked attention of Debisun with as many keys per row on
+    average, for the recurrence and its decays those of Vabunex's wkv (and KDA)."""
+    import dataclasses
+    import types
+    from .. import ops
+    from ..models.model import AttnMixer
+    from ..models.paged_gqa import PagedGqaMixer
+    from ..ops import moe_spec
+    from ..ops import paged_attn as pa
+    fig = Figures(peaks)
+    rnd, put = fig.rnd, fig.put
+    N, H, G, D, F = 2048, 16, 4, 128, 6144
+    cfg, near = zapolorn_config(N, F), zapolorn_closest(N, F, 2)
+    C = (H + 2 * G) * D
+    pages = torch.arange(R * ctx // 64, dtype=torch.int32, device=DEV).view(R, -1).contiguous()
+    one_h = torch.ones(D, device=DEV)
+    w = {"q_norm": one_h, "k_norm": one_h, "sink": torch.zeros(H, device=DEV)}
+    mk = lambda c, w: PagedGqaMixer(cfg, c, w, R, R * ctx // 64, 64, pages, DEV, torch.bfloat16)
+    whole, win = cfg.layer_specs[0].mixer.left, cfg.layer_specs[1].mixer
+    chunked = dataclasses.replace(debisun_config(N, 8192).layer_specs[0].mixer, chunk=2 * ZAP_WINDOW)
+    mw, mv = mk(whole, {k: w[k] for k in ("q_norm", "k_norm")}), mk(win, w)
+    mc = mk(chunked, {"conv_t": rnd(4, C) * 0.5, "dist_bias": rnd(H, 1025), "sink": w["sink"]})
+    at = AttnMixer(near, {}, R * ctx, DEV, torch.bfloat16)
+    for t in (mw.k, mw.v, mv.k, mv.v, mc.k, mc.v, at.k, at.v):
+        t.copy_(rnd(*t.shape))
+    seqs = [types.SimpleNamespace(kv_base=i * ctx, kv_cap=ctx) for i in range(R)]
+    lib, P, stream = cu.lib, cu.P, cu.stream
+    for tag, rows in (("prefill", T), ("decode", R)):
+        plan = lambda: make_plan([(0, [1] * T, 0)] if tag == "prefill" else [(s, [1], ctx - 1) for s in range(R)], device=DEV)
+        p1, p2 = plan(), plan()
+        proj = rnd(rows, C + 16).bfloat16()                            # [q | k | v | gate]
+        fl = T * T / 2 * H * 2 * D * 2 if tag == "prefill" else R * ctx * H * 2 * D * 2
+        nb = 0 if tag == "prefill" else R * ctx * G * 2 * D * 2
+        io = rows * C * 4
+        put(f"sloped attention with norms, {tag}", f"dense attention with its rotation, {tag}", lambda: pa.mixer(mw, proj, p1, True), nb + io, fl)
+        put(f"dense attention with its rotation, {tag}", "", lambda: cu.attn_mixer(at, proj[:, :C].contiguous() if tag == "decode" else proj, p2, seqs),
+            nb + io, fl)
+        s = ZAP_WINDOW / (ctx if tag == "decode" else T / 2)
+        put(f"window attention with norms and rotation, {tag}", f"chunked attention with its convolution (Debisun), {tag}",
+            lambda: pa.mixer(mv, proj, p1, True), nb * s + io, fl * s)
+        put(f"chunked attention with its convolution (Debisun), {tag}", "", lambda: pa.mixer(mc, proj[:, :C], p1, True),
+            nb * s * (2 if tag == "decode" else 1) + io, fl * s * (2 if tag == "decode" else 1))
+        d, q = cu._plan_dev(p1, DEV), torch.empty(rows, H * D, dtype=torch.bfloat16, device=DEV)
+        put(f"norms and rotation into the cache, {tag}", f"rotation into the cache, {tag}", lambda: pa._heads(mv, proj, d, q), io)
+        d2 = cu._plan_dev(p2, DEV)
+        put(f"rotation into the cache, {tag}", "",
+            lambda: lib().spark_attn_prep(P(proj), proj.stride(0), rows, H, G, D, 128, 0, 0, 0, 0, 4, 0, 1e-6, None, None, None, None, P(at.inv),
+                                          P(d2["pos32"]), P(d2["row_kv"]), P(d2["row_j"]), P(q), P(at.k), P(at.v), None, None, None, None, None,
+                                          stream(), None), io)
+        # linear attention: 16 heads of 64 x 128 beside 32 wkv heads of 64 x 64
+        st = lambda n: (2 * R if tag == "decode" else 2) * n * 4
+        x, lw = rnd(rows, 2 * H * 64 + 2 * H * 128).bfloat16(), -0.1 * torch.rand(rows, H * 64, device=DEV, generator=fig.g)
+        S = torch.zeros(R, H, 64, 128, device=DEV)
+        put(f"gated linear attention recurrence, {tag}", f"wkv recurrence (Vabunex), {tag}",
+            lambda: ops.linear_state(x[:, :1024], x[:, 1024:2048], x[:, 2048:4096], H, 64, 128, S, p1, True, logw=lw, qscale=0.125),
+            rows * (2 * 1024 * 2 + 2048 * (2 + 4) + 1024 * 4) + st(H * 64 * 128))
+        S2, lw2, u = torch.zeros(R, 32, 64, 64, device=DEV), -torch.rand(rows, N, device=DEV, generator=fig.g), rnd(32, 64)
+        put(f"wkv recurrence (Vabunex), {tag}", "",
+            lambda: ops.linear_state(x[:, :2048], x[:, 1024:3072], x[:, 2048:4096], 32, 64, 64, S2, p1, True, logw=lw2, u=u),
+            rows * N * (3 * 2 + 4 + 4) + st(32 * 64 * 64))
+        a2, b2 = (rnd(1024, 16) * 0.25).bfloat16(), torch.zeros(1024, device=DEV)
+        put(f"decays of the linear attention, {tag}", f"decays of wkv (Vabunex), {tag}",
+            lambda: ops.log_sigmoid_decay(x[:, :16], a2, b2, 1024, 16.0), rows * (16 * 2 + 1024 * 4) + 1024 * 32)
+        z, w2 = rnd(rows, 64), (rnd(N, 64) * 0.1).bfloat16()
+        w22, w0 = torch.cat((w2, w2), 1).contiguous(), torch.zeros(N, device=DEV)
+        put(f"decays of wkv (Vabunex), {tag}", "", lambda: ops.channel_decay(z, w2, w0, N, w22), rows * (64 * 4 + N * 4) + N * 128)
+        o, cat, nw = rnd(rows, N), torch.empty(rows, 2 * N, dtype=torch.bfloat16, device=DEV), torch.ones(N, device=DEV)
+        gate = x[:, 2048:4096]
+        put(f"norm and gate of the linear attention, {tag}", f"SwiGLU rows, {tag}",
+            lambda: ops.gate_concat(o, N, 128, nw, 1e-6, gate, "silu", None, 0, N, 2 * N, torch.bfloat16, cat[:, N:]), rows * N * 8)
+        gu = rnd(rows, 2 * N).bfloat16()
+        put(f"SwiGLU rows, {tag}", "", lambda: ops.swiglu(gu), rows * N * 6)
+        # residual updates
+        res, d32, d16, one = rnd(rows, N), rnd(rows, N), rnd(rows, N).bfloat16(), torch.ones(N, device=DEV)
+        rn = ops.RowNorm(one, 1e-6)
+        put(f"normed update + cast, {tag}", f"update + RMS norm, {tag}",
+            lambda: ops.add_norm_rows(ops.Update(d32, post=rn), res, None, torch.bfloat16), rows * N * 14)
+        put(f"update + RMS norm, {tag}", "", lambda: ops.add_rmsnorm(d16, res, one, 1e-6), rows * N * 12)
+        # dense feed-forward
+        wgu, wd = (rnd(2 * F, N) * 0.02).bfloat16(), (rnd(N, F) * 0.02).bfloat16()
+        nb, fl = 3 * F * N * 2 + rows * N * 6, rows * 3 * F * N * 2
+        put(f"dense feed-forward, {tag}", f"dense feed-forward of the closest model, {tag}",
+            lambda: ops.linear(ops.linear_swiglu(d16, wgu), wd, out_f32=True), nb, fl)
+        put(f"dense feed-forward of the closest model, {tag}", "", lambda: ops.linear(ops.swiglu(ops.linear(d16, wgu)), wd), nb, fl)
+        del wgu, wd
+        # routed feed-forwards: every kernel from the router to the combined rows
+        c, c2 = cfg.layer_specs[1].moe, near.moe
+        Fe = c.ffn
+        w1 = {"gate": rnd(c.n_experts, N).bfloat16() * 0.05, "w_gu": (rnd(c.n_experts, 2 * Fe, N) * 0.02).bfloat16(),
+              "w_down": (rnd(c.n_experts, N, Fe) * 0.02).bfloat16(), "s_gu": (rnd(2 * Fe, N) * 0.02).bfloat16(), "s_down": (rnd(N, Fe) * 0.02).bfloat16()}
+        e = moe_spec._route(d16, w1, c, None)[1].unique().numel()
+        nb, fl = (e + 1) * 3 * Fe * N * 2 + rows * N * 14, rows * (c.top_k + 1) * 3 * Fe * N * 2
+        put(f"routed experts + update, {tag}", f"routed experts of the closest model + update, {tag}",
+            lambda: ops.add_norm_rows(ops.Update(ops.moe(d16, w1, c, True), post=rn), res, None, torch.bfloat16), nb, fl)
+        put(f"routed experts of the closest model + update, {tag}", "", lambda: ops.add_rmsnorm(ops.moe(d16, w1, c2, tag == "decode"), res, one, 1e-6),
+            nb, fl)
+        del w1
+    return fig.done()
+
+
 DESIGNS = {
     "vabunex": (vabunex_config, closest_config, vabunex_kernels, SIZES,
                 "KDA + latent attention (GLM-style layer types), sequential pre-norm blocks, dense feed-forward, bf16"),
     "debisun": (debisun_config, debisun_closest, debisun_kernels, DEB_SIZES,
                 "grouped-query attention (rotary, whole context), softmax-routed SwiGLU experts of as many parameters, bf16"),
+    "zapolorn": (zapolorn_config, zapolorn_closest, zapolorn_kernels, ZAP_SIZES,
+                 "grouped-query attention (rotary, whole context), dense and softmax-routed SwiGLU feed-forwards of its sizes, bf16"),
 }
 
 

@@ -93,7 +93,7 @@ MECHANISMS = {
     "window of a page": dict(layers=[window(size=64, rot=2)]),
     "keys of another layer": dict(layers=[window(dense(), size=9), window(kv_from=0, size=50, scale=0.2), window(size=4), window(kv_from=0, size=9)]),
     "side by side": dict(layers=[pair()]),
-    "side by side, equal sizes and ones": dict(layers=[pair(heads=1, kv_heads=1, dim=16, vdim=16, scale=1.0, coef=1.0, every=1, rheads=1, rdim=16,
+    "side by side, equal sizes and ones": dict(layers=[pair(heads=1, kv_heads=1, dim=16, vdim=16, scale=0.2, coef=1.0, every=1, rheads=1, rdim=16,
                                                             rvdim=16, tau=1.0, left=1.0, right=1.0)]),
     "side by side, heads of no power of two": dict(layers=[pair(heads=6, kv_heads=3, rheads=5, rdim=8, rvdim=12, every=7)]),
     "side by side, nothing on the left": dict(layers=[pair(left=0.0)]),
