@@ -253,6 +253,43 @@ channel_decay_kernel(const TZ* __restrict__ z, int ldz, const TW* __restrict__ w
   }
 }
 
+// The log-sigmoid form for many rows: a channel per thread, 32 rows per CTA.  grid (ceil(N / 128), ceil(R / 32)); 128 threads.
+template <typename T>
+__global__ void __launch_bounds__(128)
+log_sigmoid_decay_rows_kernel(const T* __restrict__ z, int ldz, const T* __restrict__ w2, int ldw, int rank, const float* __restrict__ b,
+                              float inv_tau, float* __restrict__ logw, int R, int N) {
+  constexpr int RB = 32;
+  extern __shared__ __align__(16) float t[];                 // [rank][RB]
+  const int d = blockIdx.x * 128 + threadIdx.x, r0 = blockIdx.y * RB;
+  pdl_wait();
+  for (int i = threadIdx.x; i < rank * RB; i += 128) {
+    const int r = i / rank, k = i - r * rank;
+    t[k * RB + r] = r0 + r < R ? ldf(z + static_cast<size_t>(r0 + r) * ldz + k) : 0.f;
+  }
+  __syncthreads();
+  if (d >= N) return;
+  float acc[RB];
+#pragma unroll
+  for (int r = 0; r < RB; ++r) acc[r] = 0.f;
+  for (int k0 = 0; k0 < rank; k0 += 8) {
+    const T* wr = w2 + static_cast<size_t>(d) * ldw + k0;
+    const float4 p = ldf4(wr), q = ldf4(wr + 4);
+    const float w[8] = {p.x, p.y, p.z, p.w, q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+#pragma unroll
+      for (int r = 0; r < RB; r += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(t + (k0 + k) * RB + r);
+        acc[r] = fmaf(w[k], x.x, acc[r]); acc[r + 1] = fmaf(w[k], x.y, acc[r + 1]);
+        acc[r + 2] = fmaf(w[k], x.z, acc[r + 2]); acc[r + 3] = fmaf(w[k], x.w, acc[r + 3]);
+      }
+  }
+  const float bias = b[d];
+#pragma unroll
+  for (int r = 0; r < RB; ++r)
+    if (r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = fmaxf(log_sigmoid(acc[r] + bias) * inv_tau, -105.f);
+}
+
 // z [R, N] fp32 holds W2 tanh(..) already (prefill: a tensor-core product): z <- -exp(z + w0), in place.
 __global__ void __launch_bounds__(256)
 neg_exp_bias_kernel(float* __restrict__ z, const float* __restrict__ w0, long long n, int N) {
@@ -442,6 +479,11 @@ extern "C" int spark_log_sigmoid_decay(const void* z, int ldz, const void* w2, i
   if (rank <= 0 || (rank & 7) || (ldw & 7) || rank * 64 > 48 * 1024 || !(tau > 0.f)) return -5;
   const float* w0 = b;
   const float inv_tau = 1.f / tau;
+  if (R >= 64 && rank * 128 <= 48 * 1024) {
+    SPARK_BY_TYPE(f32, spark_launch_pdl(log_sigmoid_decay_rows_kernel<T>, dim3((N + 127) / 128, (R + 31) / 32), dim3(128), rank * 128, s,
+                                        dim3(1, 1, 1), (const T*)z, ldz, (const T*)w2, ldw, rank, b, inv_tau, logw, R, N))
+    return spark_launch_rc(__func__);
+  }
   SPARK_BY_TYPE(f32, if (R <= 4) SPARK_CHD(T, 4, inv_tau); else SPARK_CHD(T, 16, inv_tau))
 #undef SPARK_CHD
   return spark_launch_rc(__func__);
