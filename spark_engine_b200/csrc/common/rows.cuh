@@ -41,6 +41,11 @@ template <typename T> __device__ __forceinline__ float gelu_tanh_t(float z) {
   return sizeof(T) == 2 ? __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))) : gelu_tanh_f(z);
 }
 
+// ln(sigmoid(x)) / tau, bounded where the decay sigmoid(x)^(1 / tau) is 0 in fp32
+__device__ __forceinline__ float log_sigmoid_decay(float x, float inv_tau) {
+  return fmaxf((fminf(x, 0.f) - log1pf(expf(-fabsf(x)))) * inv_tau, -105.f);
+}
+
 // Sum over the block in a fixed order; every thread gets the same bits.  sh: >= 32 floats.
 __device__ __forceinline__ float block_sum_all(float v, float* sh) {
   v = warp_sum(v);

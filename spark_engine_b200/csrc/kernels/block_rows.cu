@@ -214,8 +214,6 @@ token_shift_kernel(const float* __restrict__ h, const float* __restrict__ carrie
 // log of the decay exp(-exp(x)), bounded where the decay itself is 0 in fp32 (differences of its running sums stay exact)
 __device__ __forceinline__ float log_decay(float x) { return fmaxf(-expf(x), -105.f); }
 
-__device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
-
 // grid (ceil(N / 32), ceil(R / RB)); 128 threads: four lanes per channel (eight ranks each in turn), RB rows per CTA.
 // rank is a multiple of 8.  inv_tau 0: -exp(W2 tanh(z) + w0); else ln(sigmoid(W2 z + w0)) * inv_tau.
 template <typename TZ, typename TW, int RB>
@@ -249,7 +247,7 @@ channel_decay_kernel(const TZ* __restrict__ z, int ldz, const TW* __restrict__ w
     float v = acc[r];
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
-    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = inv_tau > 0.f ? fmaxf(log_sigmoid(v + w0[d]) * inv_tau, -105.f) : log_decay(v + w0[d]);
+    if (d < N && (r & 3) == part && r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = inv_tau > 0.f ? log_sigmoid_decay(v + w0[d], inv_tau) : log_decay(v + w0[d]);
   }
 }
 
@@ -287,7 +285,7 @@ log_sigmoid_decay_rows_kernel(const T* __restrict__ z, int ldz, const T* __restr
   const float bias = b[d];
 #pragma unroll
   for (int r = 0; r < RB; ++r)
-    if (r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = fmaxf(log_sigmoid(acc[r] + bias) * inv_tau, -105.f);
+    if (r0 + r < R) logw[static_cast<size_t>(r0 + r) * N + d] = log_sigmoid_decay(acc[r] + bias, inv_tau);
 }
 
 // z [R, N] fp32 holds W2 tanh(..) already (prefill: a tensor-core product): z <- -exp(z + w0), in place.

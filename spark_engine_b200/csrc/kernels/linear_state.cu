@@ -39,11 +39,19 @@ struct LinearArgs {
   float qscale;
 };
 
+// Channel decays formed by the sequential kernel itself: ln(sigmoid(w2 z + b)) / tau; z, w2 in the activation type, rank % 8 == 0.
+struct LowRankDecay {
+  const void *z, *w2;
+  const float* b;
+  int ldz, ldw, rank;
+  float inv_tau;
+};
+
 // ------------------------------------------------------------------------------------------------ sequential form
 // grid (ceil(V / 32), H, nseg); 2 * DP threads: lane = value column, warp = 16 key channels
 template <typename T, int DP, int MODE>
 __global__ void __launch_bounds__(2 * DP)
-linear_seq_kernel(const __grid_constant__ LinearArgs a) {
+linear_seq_kernel(const __grid_constant__ LinearArgs a, const __grid_constant__ LowRankDecay lr) {
   constexpr int NP = DP / 16;
   __shared__ float sq[2][DP], sk[2][DP], sw[MODE ? 2 : 1][DP], su[DP], red[2][NP][32];
   pdl_wait();
@@ -69,7 +77,22 @@ linear_seq_kernel(const __grid_constant__ LinearArgs a) {
   auto fetch = [&](int t, float& x, float& w, float& vv) {
     const size_t r = r0 + t;
     x = c < D ? (tid < DP ? ldf(q + r * a.ldq + c) : ldf(k + r * a.ldk + c)) : 0.f;
-    w = (MODE >= 1 && tid < DP && c < D) ? a.logw[r * (static_cast<size_t>(a.H) * D) + h * D + c] : 0.f;
+    w = 0.f;
+    if (MODE >= 1 && tid < DP && c < D) {
+      if (MODE == 2 && lr.z != nullptr) {
+        const T* z = static_cast<const T*>(lr.z) + r * lr.ldz;
+        const T* w2 = static_cast<const T*>(lr.w2) + static_cast<size_t>(h * D + c) * lr.ldw;
+        float e = lr.b[h * D + c];
+        for (int i = 0; i < lr.rank; i += 8) {
+          const float4 z0 = ldf4(z + i), z1 = ldf4(z + i + 4), w0 = ldf4(w2 + i), w1 = ldf4(w2 + i + 4);
+          e = fmaf(z0.x, w0.x, e); e = fmaf(z0.y, w0.y, e); e = fmaf(z0.z, w0.z, e); e = fmaf(z0.w, w0.w, e);
+          e = fmaf(z1.x, w1.x, e); e = fmaf(z1.y, w1.y, e); e = fmaf(z1.z, w1.z, e); e = fmaf(z1.w, w1.w, e);
+        }
+        w = log_sigmoid_decay(e, lr.inv_tau);
+      } else {
+        w = a.logw[r * (static_cast<size_t>(a.H) * D) + h * D + c];
+      }
+    }
     vv = vin ? ldf(v + r * a.ldv + vcol) : 0.f;
   };
   float x, w, vv;
@@ -655,9 +678,9 @@ static int launch_chunked(const LinearArgs& a, const int* chunks, int n_chunks, 
 }
 
 template <typename T, int MODE>
-static int launch_seq(const LinearArgs& a, int nseg, cudaStream_t s) {
+static int launch_seq(const LinearArgs& a, int nseg, cudaStream_t s, const LowRankDecay& lr = LowRankDecay{}) {
   const dim3 grid((a.V + 31) / 32, a.H, nseg);
-#define SPARK_LSEQ(DP) spark_launch_pdl(linear_seq_kernel<T, DP, MODE>, grid, dim3(2 * DP), 0, s, dim3(1, 1, 1), a)
+#define SPARK_LSEQ(DP) spark_launch_pdl(linear_seq_kernel<T, DP, MODE>, grid, dim3(2 * DP), 0, s, dim3(1, 1, 1), a, lr)
   if (a.D <= 32) SPARK_LSEQ(32);
   else if (a.D <= 64) SPARK_LSEQ(64);
   else if (a.D <= 128) SPARK_LSEQ(128);
@@ -697,6 +720,15 @@ extern "C" int spark_linear_seq(SPARK_LINEAR_PARAMS, int nseg, int f32, cudaStre
   if (log2a) return f32 ? launch_seq<float, 0>(a, nseg, s) : launch_seq<__nv_bfloat16, 0>(a, nseg, s);
   if (u) return f32 ? launch_seq<float, 1>(a, nseg, s) : launch_seq<__nv_bfloat16, 1>(a, nseg, s);
   return f32 ? launch_seq<float, 2>(a, nseg, s) : launch_seq<__nv_bfloat16, 2>(a, nseg, s);
+}
+
+// Channel decay without a bonus, the decays from their low-rank rows.
+extern "C" int spark_linear_seq_lowrank(SPARK_LINEAR_PARAMS, int nseg, const LowRankDecay* lr, int f32, cudaStream_t s) {
+  if (nseg <= 0) return 0;
+  if (log2a || u || lr->rank <= 0 || ((lr->rank | lr->ldz | lr->ldw) & 7) || !(lr->inv_tau > 0.f) ||
+      ((reinterpret_cast<uintptr_t>(lr->z) | reinterpret_cast<uintptr_t>(lr->w2)) & 15)) return -5;
+  const LinearArgs a = SPARK_LINEAR_ARGS;
+  return f32 ? launch_seq<float, 2>(a, nseg, s, *lr) : launch_seq<__nv_bfloat16, 2>(a, nseg, s, *lr);
 }
 
 // chunks: int [n_chunks][2] = (segment, chunk in segment); chunk0: int [nseg] first chunk of a segment.  D <= 128.

@@ -27,14 +27,11 @@ class GlaState:
         self.at = at, at + k8, at + 2 * k8, at + 2 * k8 + self.nv8, at + 2 * k8 + 2 * self.nv8
         self.S = torch.zeros(n_slots, c.n_heads, c.head_dim, c.v_dim, device=device, dtype=torch.float32)
 
-    def decays(self, proj):
-        r = self.at[4]
-        return ops.log_sigmoid_decay(proj[:, r: r + self.c.decay_rank], self.w["a2"], self.w["a2_b"], self.nk, self.c.tau)
-
-    def run(self, proj, logw, plan: Plan, commit: bool, n_rows=None):
-        c, (q, k, v, _, _) = self.c, self.at
+    def run(self, proj, plan: Plan, commit: bool, n_rows=None):
+        c, (q, k, v, _, r) = self.c, self.at
+        decays = (proj[:, r: r + c.decay_rank], self.w["a2"], self.w["a2_b"], c.tau)
         return ops.linear_state(proj[:, q: q + self.nk], proj[:, k: k + self.nk], proj[:, v: v + self.nv], c.n_heads, c.head_dim, c.v_dim,
-                                self.S, plan, commit, logw=logw, n_rows=n_rows, qscale=c.head_dim ** -0.5)
+                                self.S, plan, commit, n_rows=n_rows, qscale=c.head_dim ** -0.5, low_rank=decays)
 
     def put(self, o, proj, out):
         """norm per head * silu(gate) -> out (a column range of the output product's rows)."""
@@ -60,9 +57,8 @@ class SideBySideMixer(PendingRows):
         proj = ops.linear(h, self.w["in"])
         cat = torch.empty(h.shape[0], self.nl + self.right.nv8, dtype=self.dtype, device=h.device)
         self.left.attend(proj, plan, commit, cat[:, : self.nl])
-        logw = self.right.decays(proj)
-        self.right.put(self.right.run(proj, logw, plan, commit), proj, cat[:, self.nl:])
-        self.pending = None if commit else ((proj, logw), plan)
+        self.right.put(self.right.run(proj, plan, commit), proj, cat[:, self.nl:])
+        self.pending = None if commit else ((proj,), plan)
         return ops.linear(cat, self.w["out"], out_f32=True)
 
     def commit_rows(self, args, plan, n_rows):

@@ -507,12 +507,15 @@ def log_sigmoid_decay(z, w2, b, n: int, tau: float):
 
 
 def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=None, u=None, h32=None, carried=None,
-                 n_rows=None, qscale=1.0):
+                 n_rows=None, qscale=1.0, low_rank=None):
     """Decayed linear attention (constant decay per head; or decay per channel and token, with a bonus `u` for the current
     token, or without one on the state after the current token): o fp32 [R, H * V], times `qscale`; the slots' states advance
-    when `commit` (by n_rows[i] rows of segment i if given)."""
+    when `commit` (by n_rows[i] rows of segment i if given).  `low_rank` = (z, w2, b, tau): the channel decays are
+    log_sigmoid_decay(z, w2, b, H * D, tau)."""
     if use_kernels(q):
-        return block_ops().linear_state(q, k, v, H, D, V, S, plan, commit, act, log2a, logw, u, h32, carried, n_rows, qscale)
+        return block_ops().linear_state(q, k, v, H, D, V, S, plan, commit, act, log2a, logw, u, h32, carried, n_rows, qscale, low_rank)
+    if low_rank is not None:
+        logw = log_sigmoid_decay(*low_rank[:3], H * D, low_rank[3])
     R = q.shape[0]
     q, k, v = q.float().view(R, H, D), k.float().view(R, H, D), v.float().view(R, H, V)
     if act:

@@ -93,6 +93,7 @@ _SIGS.update({
     "spark_tanh_split": [vp, i32, vp, i32, i32, vp],
     "spark_gate_concat": [vp, i32, i32, i32, vp, f32, vp, i32, i32, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp],
     "spark_linear_seq": _LIN + [i32, i32, vp],
+    "spark_linear_seq_lowrank": _LIN + [i32, vp, i32, vp],
     "spark_linear_chunked": _LIN + [i32, vp, i32, vp, vp, vp, vp],
     "spark_latent_prep": [vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp, i32, vp, vp,
                           i32, vp, vp],

@@ -182,12 +182,18 @@ def _split(plan, dev):
     return d["seg_split"]
 
 
+class LowRankDecay(C.Structure):
+    """Decays formed by the sequential recurrence (csrc/kernels/linear_state.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("z", "w2", "b")] + [(n, C.c_int) for n in ("ldz", "ldw", "rank")] + [("inv_tau", C.c_float)]
+
+
 def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=None, u=None, h32=None, carried=None,
-                 n_rows=None, qscale=1.0):
+                 n_rows=None, qscale=1.0, low_rank=None):
     """Decayed linear attention of every segment from its slot's state S [slots, H, D, V]; returns o fp32 [R, H * V], times
     `qscale`.  `log2a` [H]: constant decay per head; else `logw` [R, H * D] (log decay) and `u` (bonus; None: outputs read the
-    state behind the current token), with the token-shift row carried along (h32 rows -> carried [slots, width]).  `n_rows`:
-    device counts of accepted rows (commit)."""
+    state behind the current token), with the token-shift row carried along (h32 rows -> carried [slots, width]); or `low_rank` =
+    (z, w2, b, tau) of `log_sigmoid_decay`, part of the recurrence's launch for decode rows.  `n_rows`: device counts of
+    accepted rows (commit)."""
     dev = q.device
     d = cu._plan_dev(plan, dev)
     R = q.shape[0]
@@ -195,10 +201,20 @@ def linear_state(q, k, v, H, D, V, S, plan, commit, act=False, log2a=None, logw=
     if cu.dbg.CHECK:
         cu._check_slots("linear_state", plan, S.shape[0])
     width = h32.shape[1] if h32 is not None else 0
+    lr = None
+    if low_rank is not None:
+        z, w2, b, tau = low_rank
+        if R <= cu.DECODE_ROWS_MAX and z.stride(0) % 8 == 0 and z.data_ptr() % 16 == 0:
+            lr = LowRankDecay(P(z), P(w2), P(b), z.stride(0), w2.stride(0), w2.shape[1], 1.0 / tau)
+        else:
+            logw = log_sigmoid_decay(z, w2, b, H * D, tau)
 
     def args(seg):
         return (P(q), q.stride(0), P(k), k.stride(0), P(v), v.stride(0), D, V, P(log2a), P(logw), P(u), P(S), P(seg), P(n_rows), P(o),
                 P(h32), P(carried), width, H, D, V, int(commit), int(act), float(qscale))
+    if lr is not None:
+        check(lib().spark_linear_seq_lowrank(*args(d["seg"]), len(plan.segs), C.byref(lr), _is32(q.dtype), stream()), "spark_linear_seq_lowrank")
+        return o
     short, longs = (d["seg"], plan.segs), (None, [])
     if n_rows is None and commit and q.dtype == torch.bfloat16 and D <= 128:
         short, longs = _split(plan, dev)

@@ -373,20 +373,22 @@ def zapolorn_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) ->
         # linear attention: 16 heads of 64 x 128 beside 32 wkv heads of 64 x 64
         st = lambda n: (2 * R if tag == "decode" else 2) * n * 4
         x, lw = rnd(rows, 2 * H * 64 + 2 * H * 128).bfloat16(), -0.1 * torch.rand(rows, H * 64, device=DEV, generator=fig.g)
+        a2, b2 = (rnd(1024, 16) * 0.25).bfloat16(), torch.zeros(1024, device=DEV)
+        dec = dict(logw=lw) if tag == "prefill" else dict(low_rank=(x[:, :16], a2, b2, 16.0))
         S = torch.zeros(R, H, 64, 128, device=DEV)
         put(f"gated linear attention recurrence, {tag}", f"wkv recurrence (Vabunex), {tag}",
-            lambda: ops.linear_state(x[:, :1024], x[:, 1024:2048], x[:, 2048:4096], H, 64, 128, S, p1, True, logw=lw, qscale=0.125),
+            lambda: ops.linear_state(x[:, :1024], x[:, 1024:2048], x[:, 2048:4096], H, 64, 128, S, p1, True, qscale=0.125, **dec),
             rows * (2 * 1024 * 2 + 2048 * (2 + 4) + 1024 * 4) + st(H * 64 * 128))
         S2, lw2, u = torch.zeros(R, 32, 64, 64, device=DEV), -torch.rand(rows, N, device=DEV, generator=fig.g), rnd(32, 64)
         put(f"wkv recurrence (Vabunex), {tag}", "",
             lambda: ops.linear_state(x[:, :2048], x[:, 1024:3072], x[:, 2048:4096], 32, 64, 64, S2, p1, True, logw=lw2, u=u),
             rows * N * (3 * 2 + 4 + 4) + st(32 * 64 * 64))
-        a2, b2 = (rnd(1024, 16) * 0.25).bfloat16(), torch.zeros(1024, device=DEV)
-        put(f"decays of the linear attention, {tag}", f"decays of wkv (Vabunex), {tag}",
-            lambda: ops.log_sigmoid_decay(x[:, :16], a2, b2, 1024, 16.0), rows * (16 * 2 + 1024 * 4) + 1024 * 32)
-        z, w2 = rnd(rows, 64), (rnd(N, 64) * 0.1).bfloat16()
-        w22, w0 = torch.cat((w2, w2), 1).contiguous(), torch.zeros(N, device=DEV)
-        put(f"decays of wkv (Vabunex), {tag}", "", lambda: ops.channel_decay(z, w2, w0, N, w22), rows * (64 * 4 + N * 4) + N * 128)
+        if tag == "prefill":                             # (decode rows: part of the recurrence's launch)
+            put(f"decays of the linear attention, {tag}", f"decays of wkv (Vabunex), {tag}",
+                lambda: ops.log_sigmoid_decay(x[:, :16], a2, b2, 1024, 16.0), rows * (16 * 2 + 1024 * 4) + 1024 * 32)
+            z, w2 = rnd(rows, 64), (rnd(N, 64) * 0.1).bfloat16()
+            w22, w0 = torch.cat((w2, w2), 1).contiguous(), torch.zeros(N, device=DEV)
+            put(f"decays of wkv (Vabunex), {tag}", "", lambda: ops.channel_decay(z, w2, w0, N, w22), rows * (64 * 4 + N * 4) + N * 128)
         o, cat, nw = rnd(rows, N), torch.empty(rows, 2 * N, dtype=torch.bfloat16, device=DEV), torch.ones(N, device=DEV)
         gate = x[:, 2048:4096]
         put(f"norm and gate of the linear attention, {tag}", f"SwiGLU rows, {tag}",

@@ -227,6 +227,25 @@ def test_channel_decays(R, dtype):
         assert torch.allclose(got, want.clamp(min=-105), atol=3e-5, rtol=3e-6)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,D,V,rank", [(2, 20, 28, 10), (3, 64, 40, 64)])
+def test_decays_inside_the_recurrence(H, D, V, rank, dtype):
+    """Decode rows form their decays in the recurrence's own launch: as with decays computed first, whatever the batch is."""
+    g = torch.Generator().manual_seed(rank)
+    r8, n = (rank + 7) // 8 * 8, 12
+    x = torch.randn(n, H * (2 * D + V), generator=g).to(dtype).to(DEV)
+    z, w2, b = torch.zeros(n, r8 + 8), torch.zeros(H * D, r8), torch.randn(H * D, generator=g).to(DEV)
+    z[:, :rank], w2[:, :rank] = torch.randn(n, rank, generator=g), torch.randn(H * D, rank, generator=g)
+    z, w2 = z.to(dtype).to(DEV), w2.to(dtype).to(DEV)
+    S = torch.randn(4, H, D, V, generator=g).to(DEV)
+    S2 = S.clone()
+    plan = lambda: make_plan([(3, [1] * 7, 50), (0, [1], 9), (1, [1] * 4, 0)], device=DEV)
+    run = lambda S, **kw: ops.linear_state(x[:, : H * D], x[:, H * D: 2 * H * D], x[:, 2 * H * D:], H, D, V, S, plan(), True, qscale=0.5, **kw)
+    a = run(S, low_rank=(z[:, :rank], w2, b, 3.0))
+    c = run(S2, logw=ops.log_sigmoid_decay(z[:, :rank], w2, b, H * D, 3.0))
+    assert torch.allclose(a, c, atol=1e-4, rtol=1e-4) and torch.allclose(S, S2, atol=1e-4, rtol=1e-4) and not torch.equal(S[3], S[2])
+
+
 @pytest.mark.parametrize("R,K,F", [(1, 64, 128), (16, 1024, 512), (17, 264, 128), (300, 96, 384), (3, 75, 128), (40, 75, 256)])
 def test_swiglu_products(R, K, F):
     g = torch.Generator().manual_seed(F)
