@@ -156,7 +156,7 @@ class GlaConfig:
     n_heads: int = 2
     head_dim: int = 32
     v_dim: int = 32
-    tau: float = 16.0
+    tau: float = 8.0
     decay_rank: int = 16
 
 
@@ -368,13 +368,13 @@ def zapolorn_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 5632, voca
     for i in range(n_layers):
         if i % 4 == 0:
             left = PagedGqaConfig(**gqa, temp_coef=0.1, temp_every=8192, slopes=True)
-            kind, mixer = "side_by_side", SideBySideConfig(left, GlaConfig(n_heads=heads, head_dim=64, v_dim=128, tau=16.0), 0.7, 0.7)
+            kind, mixer = "side_by_side", SideBySideConfig(left, GlaConfig(n_heads=heads, head_dim=64, v_dim=128, tau=8.0), 0.7, 0.7)
         else:
-            kind, mixer = "gqa", PagedGqaConfig(**gqa, window=window, rope_dims=128, rope_theta=5e5, rope_factor=4.0, gated=True,
+            kind, mixer = "gqa", PagedGqaConfig(**gqa, window=window, rope_dims=128, rope_theta=1e6, rope_factor=8.0, gated=True,
                                                 kv_from=i - 1 if i % 4 == 2 else None)
         specs.append(LayerSpec(kind, mixer, 0 if i % 2 else ffn, dataclasses.replace(moe) if i % 2 else None))
     return ModelConfig(name="zapolorn-style", family="zapolorn", n_layers=n_layers, layer_types=[x.kind for x in specs], hidden=hidden,
-                       vocab=vocab, norm_eps=1e-6, layer_specs=specs, block="post", embed_scale=float(hidden) ** 0.5, tied_head=True,
+                       vocab=vocab, norm_eps=1e-5, layer_specs=specs, block="post", embed_scale=float(hidden) ** 0.5, tied_head=True,
                        weight_format="dense")
 
 

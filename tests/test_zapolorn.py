@@ -162,6 +162,31 @@ def test_a_key_is_seen_inside_the_window_only(size, at):
         assert U.error(m.forward(make_plan([(1, toks[i: i + 1], i)])), want[i: i + 1]) < 2e-5
 
 
+def slope_case(at):
+    """As far_case for whole-context attention: the planted key stands out for the head with the gentlest slope."""
+    cfg, T = _setup(dict(layers=[U.pair(heads=4, kv_heads=2, coef=0.2, every=64, right=0.3)]), 7)
+    qt, kt, fill = U.planted_pair(cfg, T)
+    toks = [fill[i % len(fill)] for i in range(209)] + [qt]
+    other = list(toks)
+    other[at] = kt
+    return cfg, T, other, toks
+
+
+SLOPED = [0, 1, 63, 64, 127, 128, 192, 207, 208]
+
+
+@pytest.mark.parametrize("at", SLOPED)
+def test_far_keys_under_a_slope(at):
+    cfg, T, toks, without = slope_case(at)
+    want = U.oracle_logits(cfg, T, toks)
+    assert U.error(U.oracle_logits(cfg, T, without)[-1:], want[-1:]) > 0.05
+    m = U.framework(cfg, T)
+    assert U.error(m.forward(make_plan([(0, toks, 0)])), want) < 2e-5
+    m.forward(make_plan([(1, toks[:-3], 0)]))
+    for i in range(207, 210):
+        assert U.error(m.forward(make_plan([(1, toks[i: i + 1], i)])), want[i: i + 1]) < 2e-5
+
+
 def test_a_borrowed_cache_is_the_other_layers():
     """A layer without keys of its own reads the ones the other layer cached, and has no cache of its own."""
     cfg, T = _setup("keys of another layer")

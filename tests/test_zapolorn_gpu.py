@@ -14,7 +14,7 @@ import pytest
 import torch
 import zapolorn_oracle as oracle
 import zapolorn_util as U
-from test_zapolorn import FAR, _serve, _setup, far_case
+from test_zapolorn import FAR, SLOPED, _serve, _setup, far_case, slope_case
 
 from spark_engine_b200 import ops
 from spark_engine_b200.config import EngineConfig, MoeConfig, PagedGqaConfig
@@ -125,6 +125,21 @@ def test_a_key_is_seen_inside_the_window_only(size, at, dtype, borrowed):
         assert torch.equal(same, got)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("at", SLOPED)
+def test_far_keys_under_a_slope(at, dtype):
+    cfg, T, toks, without = slope_case(at)
+    want = U.oracle_logits(cfg, T, toks)
+    moved = U.error(U.oracle_logits(cfg, T, without)[-1:], want[-1:])
+    limit = TOL[dtype] if dtype == torch.float32 else min(0.4 * moved, 0.05)
+    m = U.framework(cfg, T, DEV, dtype)
+    assert U.error(m.forward(make_plan([(0, toks, 0)], device=DEV))[-1:], want[-1:]) < limit
+    m.forward(make_plan([(1, toks[:-3], 0)], device=DEV))
+    for i in range(207, 210):
+        got = m.forward(make_plan([(1, toks[i: i + 1], i)], device=DEV))
+    assert U.error(got, want[-1:]) < limit
+
+
 def attention_case(dtype, n, H, G, D, V, seed=0, **kw):
     """One attention mixer on its own, with the plain result of the projected rows; scores of a spread that makes every key and
     every constant show."""
@@ -217,7 +232,7 @@ def test_decayed_state(H, D, V, strength, dtype):
 @pytest.mark.parametrize("R", [1, 5, 300])
 def test_channel_decays(R, dtype):
     g = torch.Generator().manual_seed(R)
-    for rank, n, tau in ((16, 96, 16.0), (10, 60, 1.0), (64, 33, 0.5)):
+    for rank, n, tau in ((24, 96, 12.0), (10, 60, 1.0), (64, 33, 0.5)):
         r8 = (rank + 7) // 8 * 8
         z, w2, b = torch.zeros(R, r8 + 8), torch.zeros(n, r8), 2 * torch.randn(n, generator=g)
         z[:, :rank], w2[:, :rank] = 4 * torch.randn(R, rank, generator=g), torch.randn(n, rank, generator=g)
@@ -257,7 +272,7 @@ def test_swiglu_products(R, K, F):
         assert torch.allclose(got, oracle.silu(y[:, :F]) * y[:, F:], **tol)
 
 
-@pytest.mark.parametrize("E,top,F", [(6, 2, 40), (1, 1, 8), (12, 1, 96), (60, 8, 136), (500, 30, 16)])
+@pytest.mark.parametrize("E,top,F", [(6, 2, 40), (1, 1, 8), (13, 1, 104), (60, 8, 136), (500, 30, 16)])
 @pytest.mark.parametrize("H", [64, 264, 75])
 def test_experts(E, top, F, H):
     """Fused decode router, pair GEMVs, grouped products and the FP32-unit form against the plain form on rows without close calls."""

@@ -84,12 +84,12 @@ def framework(cfg, T, device="cpu", dtype=torch.float32, slots=4, tokens=1024):
 
 SMALL = dict(heads=4, kv_heads=1, dim=24, vdim=16, size=33, rot=8)
 MIXED = dict(layers=[window(dense()), pair(moe()), window(moe(top=1, shared=0), kv_from=0, size=100), window(None, **SMALL),
-                     pair(None, heads=3, kv_heads=3, dim=16, vdim=8, rheads=2, rdim=12, rvdim=44, tau=16.0), window(moe(), kv_from=3, **SMALL)])
+                     pair(None, heads=3, kv_heads=3, dim=16, vdim=8, rheads=2, rdim=12, rvdim=44, tau=14.0), window(moe(), kv_from=3, **SMALL)])
 MECHANISMS = {
     "window attention": dict(layers=[window()]),
     "window attention, equal sizes and ones": dict(layers=[window(heads=1, kv_heads=1, dim=16, vdim=16, size=1, rot=16, factor=1.0, scale=1.0)]),
     "window attention, no sharing of heads": dict(layers=[window(heads=4, kv_heads=4, rot=20)]),
-    "window beyond the prompt": dict(layers=[window(size=1000, base=5e5)]),
+    "window beyond the prompt": dict(layers=[window(size=1000, base=3e5)]),
     "window of a page": dict(layers=[window(size=64, rot=2)]),
     "keys of another layer": dict(layers=[window(dense(), size=9), window(kv_from=0, size=50, scale=0.2), window(size=4), window(kv_from=0, size=9)]),
     "side by side": dict(layers=[pair()]),
