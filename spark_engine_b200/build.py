@@ -40,7 +40,8 @@ def _run(cmd):
 # kernel sources of families that need only part of the library
 FAMILY_SOURCES = {"vabunex": ("block_rows", "elementwise", "gemm", "gemm_simt", "gemv", "latent", "linear_state", "mla"),
                   "debisun": ("block_rows", "elementwise", "gemm", "gemm_simt", "gemv", "moe", "paged_attn"),
-                  "zapolorn": ("block_rows", "elementwise", "gemm", "gemm_simt", "gemv", "linear_state", "moe", "paged_attn")}
+                  "zapolorn": ("block_rows", "elementwise", "gemm", "gemm_simt", "gemv", "linear_state", "moe", "paged_attn"),
+                  "zakusun": ("block_rows", "elementwise", "gemm", "gemm_simt", "gemv", "latent", "mla", "moe", "row_tiles")}
 
 
 def kernel_library(family: str) -> str:

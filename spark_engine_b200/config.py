@@ -77,9 +77,12 @@ class MoeConfig:
     shared_ffn: int = 0           # 0 -> ffn * n_shared
     router: str = "softmax"       # softmax | sigmoid_bias | sqrt_softplus | softmax_bias (bias: added to the choice scores only)
                                   # | sigmoid (the chosen scores are the weights as they are, times route_scale)
+                                  # | topk_softmax (bias added to the logits, softmax over the chosen logits alone)
     route_scale: float = 1.0
     shared_gate: bool = False     # sigmoid(x . w_sg) on the shared expert
-    swiglu_limit: float = 0.0     # clamp-SwiGLU limit (0 = off)
+    swiglu_limit: float = 0.0     # clamp-SwiGLU limit (0 = off): gate at most the limit, up within +- the limit
+    glu_alpha: float = 1.0        # the gate is gate * sigmoid(glu_alpha * gate)
+    glu_shift: float = 0.0        # added to the (clamped) up half
     dense_layers: int = 0         # first N layers use a dense MLP of width dense_ffn
     dense_ffn: int = 0
     act: str = "swiglu"           # swiglu (gate and up matrices) | relu2 (squared relu of a single up matrix)
@@ -89,6 +92,16 @@ class MoeConfig:
     @property
     def n_routes(self) -> int:
         return self.n_experts + self.n_identity
+
+    @property
+    def glu(self) -> tuple:
+        """(limit, alpha, shift) of the gated activation."""
+        return self.swiglu_limit, self.glu_alpha, self.glu_shift
+
+    @property
+    def plain(self) -> bool:
+        """A router and experts that the quantised and expert-parallel paths know."""
+        return self.act == "swiglu" and not self.weight_input and self.router != "topk_softmax" and self.glu[1:] == (1.0, 0.0)
 
 
 @dataclass
@@ -110,16 +123,19 @@ class WkvConfig:
 
 @dataclass
 class LatentConfig:
-    """Dense causal attention over cached latents, low-rank queries, one shared rotated key part, per-head output gate."""
+    """Dense causal attention over cached latents: low-rank or direct queries, one shared rotated key part (or none), optionally a
+    learned sink per head in the denominator, an output gate per head or per element."""
     n_heads: int = 2
     head_dim: int = 32            # unrotated query / key dimensions per head
     v_dim: int = 32
-    q_rank: int = 64
+    q_rank: int = 64              # 0: queries are projected from the row itself
     kv_rank: int = 48
-    rope_dim: int = 16
+    rope_dim: int = 16            # 0: no rotated part
     rope_theta: float = 1e4
     rope_interleaved: bool = True
     scale: float = 0.125
+    sink: bool = False            # a score per head without key and value
+    gate: str = "head"            # sigmoid gate per head | element (of the concatenated heads)
 
 
 @dataclass
@@ -199,7 +215,7 @@ class LoopConfig:
 @dataclass
 class ModelConfig:
     name: str = "tiny-hybrid"
-    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex | debisun | zapolorn
+    family: str = "hybrid"        # hybrid (Qwen-style) | glm | ds4 | vabunex | debisun | zapolorn | zakusun
     n_layers: int = 4
     layer_types: List[str] = field(default_factory=lambda: ["gdn", "gdn", "gdn", "attn"])
     hidden: int = 256
@@ -231,6 +247,10 @@ class ModelConfig:
                                   # | post (sublayers read the residual itself, their outputs are normed)
     norm_kind: str = "rms"        # models with layer_specs: rms | layer (weight and bias)
     norm_one_plus: bool = False   # norm weights are stored around zero
+    norm_groups: int = 1          # equal parts of the row that are RMS-normed each on its own
+    input_conv: int = 0           # taps of the causal convolution added to every sublayer's normed input (0: none; sequential blocks)
+    depth_average: bool = False   # behind every layer the residual becomes a learned sum of the embedding and all layers' results
+    positions: str = ""           # sinusoidal: added to the embedding ("": nothing is)
     embed_scale: float = 1.0
     logit_scale: float = 1.0
     tied_head: bool = False       # the logits' matrix is the embedding table (without its scale)
@@ -378,6 +398,19 @@ def zapolorn_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 5632, voca
                        weight_format="dense")
 
 
+def zakusun_style(n_layers: int = 12, hidden: int = 2048, ffn: int = 1536, vocab: int = 65536, experts: int = 64, top: int = 4,
+                  taps: int = 4) -> ModelConfig:
+    """Zakusun at the layer sizes of a small real model: latent attention (heads of 128, latents of 512), experts of width `ffn`,
+    two norm groups."""
+    heads = hidden // 128
+    mixer = LatentConfig(n_heads=heads, head_dim=128, v_dim=128, q_rank=0, kv_rank=512, rope_dim=0, scale=128 ** -0.5, sink=True, gate="element")
+    moe = MoeConfig(n_experts=experts, top_k=top, ffn=ffn, n_shared=0, router="topk_softmax", swiglu_limit=7.0, glu_alpha=1.702, glu_shift=1.0)
+    specs = [LayerSpec("latent", dataclasses.replace(mixer), 0, dataclasses.replace(moe)) for _ in range(n_layers)]
+    return ModelConfig(name="zakusun-style", family="zakusun", n_layers=n_layers, layer_types=["latent"] * n_layers, hidden=hidden, vocab=vocab,
+                       norm_eps=1e-5, layer_specs=specs, block="sequential", norm_groups=2, input_conv=taps, depth_average=True,
+                       positions="sinusoidal", tied_head=True, weight_format="dense")
+
+
 def scaled_down(cfg: ModelConfig, hidden: int = 256, n_layers: int = 4, vocab: int = 1024) -> ModelConfig:
     """Same layer types, small dimensions: the CPU test shape of a large config."""
     c = dataclasses.replace(cfg)
@@ -478,6 +511,7 @@ PRESETS = {
     "vabunex-style": vabunex_style,
     "debisun-style": debisun_style,
     "zapolorn-style": zapolorn_style,
+    "zakusun-style": zakusun_style,
 }
 
 

@@ -1,44 +1,42 @@
 // Row kernels of the models whose layers carry their own sizes, for bf16 and fp32 activations.  The residual stream, norms,
 // token-shift state and decays are fp32 in both.
 //
-//   embed_scaled      x = table[id] * scale
+//   embed_scaled      x = table[id] * scale (+ the sines and cosines of the position)
 //   row_update        res += an update (plain rows or the slots of a routed feed-forward; per-channel scale, or RMS-normed);
 //                     h = norm of the new residual (RMS, layer norm, or the residual itself), optionally an fp32 copy of h
 //   token_shift       five mixes h + (h' - h) mu_s of the current and the previous row of the sequence
 //   channel_decay     log decay  -exp(W2 tanh(z) + w0)  or  ln(sigmoid(W2 z + w0)) / tau  per channel, fp32 throughout
-//   swiglu_rows       silu(gate) * up of [gate | up] rows, both times a weight per row if given
+//   swiglu_rows       gated activation (out_act.cuh) of [gate | up] rows, both times a weight per row if given
 //   gate_concat       [ group-RMSNorm(o) * w * gate(g) | gelu(gate) * up ]: the input row of the block's single output
 //                     product (the mixer's output matrix and the down projection are stored side by side along K)
-#include "../common/rows.cuh"
+#include "../common/row_update.cuh"
+#include "../common/out_act.cuh"
 
 namespace spark {
 
+// pos (optional): channel 2i gets the sine of pos * freq[i], channel 2i + 1 its cosine on top.
 template <typename TW>
 __global__ void __launch_bounds__(128)
 embed_scaled_kernel(const TW* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out, int H, int V,
-                    float scale, int* __restrict__ status) {
+                    float scale, const int* __restrict__ pos, const double* __restrict__ freq, int* __restrict__ status) {
   pdl_wait();
   const int r = blockIdx.x, id = ids[r];
   const bool ok = id >= 0 && id < V;                        // an id outside the table: zero row + status word
   if (!ok && threadIdx.x == 0 && status) set_status(status, ST_BOUNDS, r, id, V);
-  for (int i = threadIdx.x; i < H; i += blockDim.x)
-    out[static_cast<size_t>(r) * H + i] = ok ? ldf(table + static_cast<size_t>(id) * H + i) * scale : 0.f;
+  const TW* row = table + static_cast<size_t>(ok ? id : 0) * H;
+  float* o = out + static_cast<size_t>(r) * H;
+  if (pos == nullptr) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = ok ? ldf(row + i) * scale : 0.f;
+    return;
+  }
+  const double p = pos[r];
+  for (int i = threadIdx.x * 2; i < H; i += blockDim.x * 2) {
+    float sn, cs;
+    sincosf(static_cast<float>(p * freq[i >> 1]), &sn, &cs);
+    o[i] = ok ? ldf(row + i) * scale + sn : 0.f;
+    if (i + 1 < H) o[i + 1] = ok ? ldf(row + i + 1) * scale + cs : 0.f;
+  }
 }
-
-struct RowUpdate {
-  float* res;                                   // [R, H], in place
-  // the update: `delta` rows, or sum over slots of wts (null: 1) * y (expert outputs) + sg * shared + self_w * self_x, or nothing
-  const float* delta;
-  const float* y; const int* inv; const float* wts; const int* ids;      // pair p's row of y: inv[p] (inv null: p); ids[p] < 0: none
-  const float* shared; const float* sg; const float* self_w; const void* self_x;
-  const float* scale;                           // [H] (null: 1)
-  const float* post_w;                          // [H]: the update is RMS-normed with this weight (null: it is not)
-  // the new rows
-  const float* w; const float* b;
-  void* out; float* out32;
-  int H, slots, norm, one_plus;                 // norm: 0 none, 1 RMS (w or 1 + w), 2 layer norm (w, b)
-  float eps, post_eps;
-};
 
 // One CTA per row.  NV > 0: every thread keeps NV groups of four channels in registers (blockDim * 4 * NV >= H, H % 4 == 0,
 // 16-byte aligned rows); NV == 0: any width, values are read again.
@@ -313,7 +311,7 @@ tanh_split_kernel(const float* __restrict__ z, int ldz, __nv_bfloat16* __restric
 template <typename T>
 __global__ void __launch_bounds__(256)
 swiglu_rows_kernel(const T* __restrict__ gu, int ldi, int F, const float* __restrict__ wts, const int* __restrict__ perm,
-                   T* __restrict__ out, int ldo, int R) {
+                   T* __restrict__ out, int ldo, int R, GluAct act) {
   pdl_wait();
   const int i = blockIdx.x * 1024 + threadIdx.x * 4;
   if (i >= F) return;
@@ -321,8 +319,8 @@ swiglu_rows_kernel(const T* __restrict__ gu, int ldi, int F, const float* __rest
     const T* x = gu + static_cast<size_t>(r) * ldi + i;
     const float4 g = ldf4(x), u = ldf4(x + F);
     const float w = wts ? wts[perm ? perm[r] : r] : 1.f;
-    stf4(out + static_cast<size_t>(r) * ldo + i, make_float4(silu_t<T>(w * g.x) * (w * u.x), silu_t<T>(w * g.y) * (w * u.y),
-                                                             silu_t<T>(w * g.z) * (w * u.z), silu_t<T>(w * g.w) * (w * u.w)));
+    stf4(out + static_cast<size_t>(r) * ldo + i, make_float4(glu_t<T>(act, w * g.x, w * u.x), glu_t<T>(act, w * g.y, w * u.y),
+                                                             glu_t<T>(act, w * g.z, w * u.z), glu_t<T>(act, w * g.w, w * u.w)));
   }
 }
 
@@ -421,11 +419,12 @@ using namespace spark;
   if (f32) { using T = float; CALL; }     \
   else { using T = __nv_bfloat16; CALL; }
 
-extern "C" int spark_embed_scaled(const void* table, const int* ids, float* out, int R, int H, int V, float scale, int f32,
-                                  int* status, cudaStream_t s) {
+extern "C" int spark_embed_scaled(const void* table, const int* ids, float* out, int R, int H, int V, float scale, const int* pos,
+                                  const double* freq, int f32, int* status, cudaStream_t s) {
   if (R <= 0) return 0;
+  if (pos && !freq) return -5;
   SPARK_BY_TYPE(f32, spark_launch_pdl(embed_scaled_kernel<T>, dim3(R), dim3(128), 0, s, dim3(1, 1, 1), (const T*)table, ids, out,
-                                      H, V, scale, status))
+                                      H, V, scale, pos, freq, status))
   return spark_launch_rc(__func__);
 }
 
@@ -487,13 +486,13 @@ extern "C" int spark_log_sigmoid_decay(const void* z, int ldz, const void* w2, i
   return spark_launch_rc(__func__);
 }
 
-extern "C" int spark_swiglu_rows(const void* gu, int ldi, int F, const float* wts, const int* perm, void* out, int ldo, int R, int f32,
-                                 cudaStream_t s) {
+extern "C" int spark_swiglu_rows(const void* gu, int ldi, int F, const float* wts, const int* perm, void* out, int ldo, int R,
+                                 const GluAct* act, int f32, cudaStream_t s) {
   if (R <= 0) return 0;
   if ((F | ldi | ldo) & 7) return -5;
   const dim3 grid((F + 1023) / 1024, R < 65535 ? R : 65535);
   SPARK_BY_TYPE(f32, spark_launch_pdl(swiglu_rows_kernel<T>, grid, dim3(256), 0, s, dim3(1, 1, 1), (const T*)gu, ldi, F, wts, perm, (T*)out,
-                                      ldo, R))
+                                      ldo, R, act ? *act : GluAct{0.f, 1.f, 0.f}))
   return spark_launch_rc(__func__);
 }
 

@@ -162,9 +162,9 @@ __global__ void f32_to_bf16_kernel(const float* __restrict__ x, __nv_bfloat16* _
 
 // gather rows: out[i, :] = src[idx[i], :]  (bf16, 16-byte vectors; H % 8 == 0)
 __global__ void gather_rows_bf16_kernel(const __nv_bfloat16* __restrict__ src, const int* __restrict__ idx,
-                                        __nv_bfloat16* __restrict__ out, int H) {
+                                        __nv_bfloat16* __restrict__ out, int H, int lds) {
   const int r = blockIdx.x;
-  const uint4* s = reinterpret_cast<const uint4*>(src + static_cast<size_t>(idx[r]) * H);
+  const uint4* s = reinterpret_cast<const uint4*>(src + static_cast<size_t>(idx[r]) * lds);
   uint4* d = reinterpret_cast<uint4*>(out + static_cast<size_t>(r) * H);
   for (int i = threadIdx.x; i < H / 8; i += blockDim.x) d[i] = s[i];
 }
@@ -318,7 +318,7 @@ extern "C" void spark_f32_to_bf16(const float* x, void* y, long n, cudaStream_t 
   if (n <= 0) return;
   f32_to_bf16_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>(x, (__nv_bfloat16*)y, (size_t)n);
 }
-extern "C" void spark_gather_rows_bf16(const void* src, const int* idx, void* out, int R, int H, cudaStream_t s) {
+extern "C" void spark_gather_rows_bf16(const void* src, const int* idx, void* out, int R, int H, cudaStream_t s, int lds) {
   if (R <= 0) return;
-  gather_rows_bf16_kernel<<<R, 256, 0, s>>>((const __nv_bfloat16*)src, idx, (__nv_bfloat16*)out, H);
+  gather_rows_bf16_kernel<<<R, 256, 0, s>>>((const __nv_bfloat16*)src, idx, (__nv_bfloat16*)out, H, lds);
 }

@@ -117,18 +117,18 @@ extern "C" int spark_gemm_bf16_swiglu(const void* A, const void* B, void* C, int
   g.M = M; g.N = F; g.K = K; g.status = status; g.gate_up_F = F; g.ab_fmt = 1;
   g.num_n_tiles = F / 128; g.num_tiles = ((M + GEMM_BM - 1) / GEMM_BM) * g.num_n_tiles;
   int grid = g.num_tiles < num_sms() ? g.num_tiles : num_sms();
-  return launch<256, EpiSwigluBf16, false>(tA, tB, g, EpiSwigluBf16{(__nv_bfloat16*)C, ldc, F, limit, nullptr, nullptr}, grid, stream);
+  return launch<256, EpiSwigluBf16, false>(tA, tB, g, EpiSwigluBf16{(__nv_bfloat16*)C, ldc, F, GluAct{limit, 1.f, 0.f}, nullptr, nullptr}, grid, stream);
 }
 
 // Grouped (MoE) GEMM over a device-side tile list: rows of A are (token, slot) pairs permuted into
 // expert order; tile_list[i] = {a_row0, row_end, expert, 0}; *tile_count m-tiles are valid.
 //   mode 0: C[rows, N] fp32 = A B_e^T          (down projection; combine sums slots later)
-//   mode 1: C[rows, F] bf16 = swiglu(A B_e^T)  (B_e = [gate | up], N = F; with wts, rows of A count wts[perm[row]] times)
+//   mode 1: C[rows, F] bf16 = glu(A B_e^T)  (null: plain SwiGLU; B_e = [gate | up], N = F; with wts, rows of A count wts[perm[row]] times)
 //   mode 2: C[rows, N] bf16 = max(A B_e^T, 0)^2
 extern "C" int spark_gemm_grouped_bf16(const void* A, const void* B, void* C, int total_rows, int N, int K,
                                        int lda, int ldb, int ldc, int n_experts, int b_rows_per_expert,
                                        const void* tile_list, const int* tile_count, int max_m_tiles, int mode,
-                                       float limit, int fmt, int* status, cudaStream_t stream, const float* wts, const int* perm) {
+                                       const GluAct* glu, int fmt, int* status, cudaStream_t stream, const float* wts, const int* perm) {
   if (total_rows <= 0 || max_m_tiles <= 0) return 0;
   CUtensorMap tA, tB;
   int r = make_tmap_bf16(&tA, A, total_rows, K, lda, 128, fmt);
@@ -143,7 +143,7 @@ extern "C" int spark_gemm_grouped_bf16(const void* A, const void* B, void* C, in
   if (mode == 1) {
     if (N % 128) return -5;
     g.gate_up_F = N; g.num_n_tiles = N / 128; g.num_tiles = max_m_tiles * g.num_n_tiles;
-    return launch<256, EpiSwigluBf16, true>(tA, tB, g, EpiSwigluBf16{(__nv_bfloat16*)C, ldc, N, limit, wts, perm}, num_sms(), stream);
+    return launch<256, EpiSwigluBf16, true>(tA, tB, g, EpiSwigluBf16{(__nv_bfloat16*)C, ldc, N, glu ? *glu : GluAct{0.f, 1.f, 0.f}, wts, perm}, num_sms(), stream);
   }
   if (mode == 2) {
     OutAct a{};

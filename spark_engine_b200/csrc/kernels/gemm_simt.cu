@@ -35,6 +35,7 @@ gemm_simt_kernel(const T* __restrict__ A, int lda, long long sa, const T* __rest
     if (grp.perm) r = grp.perm[r] / grp.a_div;
     ar[i] = A + static_cast<size_t>(r) * lda;
   }
+  const int oc = grp.tiles ? 0 : blockIdx.z * act.batch_cols;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
 #pragma unroll
@@ -61,7 +62,7 @@ gemm_simt_kernel(const T* __restrict__ A, int lda, long long sa, const T* __rest
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (m < M && n < N) stf(C + static_cast<size_t>(m) * ldc + n, out_act(act, acc[i][j], m, n));
+      if (m < M && n < N) stf(C + static_cast<size_t>(m) * ldc + n, out_act(act, acc[i][j], m, oc + n));
     }
 }
 

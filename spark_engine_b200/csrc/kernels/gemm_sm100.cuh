@@ -290,18 +290,15 @@ struct EpiStoreF32 {
   }
 };
 
-// SwiGLU (optionally clamped) over a [gate | up] tile pair -> bf16 [rows, F].  With weights, gate and up of sorted row r are
+// Gated activation (out_act.cuh) over a [gate | up] tile pair -> bf16 [rows, F].  With weights, gate and up of sorted row r are
 // multiplied by the weight of its pair first (an expert that sees its input times the weight).
 struct EpiSwigluBf16 {
   static constexpr bool kWarpTile = false;
-  __nv_bfloat16* C; int ldc; int N; float limit;
+  __nv_bfloat16* C; int ldc; int N; GluAct glu;
   const float* wts; const int* perm;
   __device__ __forceinline__ float row_weight(int row) const { return wts ? wts[perm[row]] : 1.f; }
   __device__ __forceinline__ void cta_done(int) const {}
-  __device__ __forceinline__ float act(float g, float u) const {
-    if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
-    return g / (1.f + __expf(-g)) * u;
-  }
+  __device__ __forceinline__ float act(float g, float u) const { return glu_t<__nv_bfloat16>(glu, g, u); }
   __device__ __forceinline__ void operator()(const TileCoord& tc, int row, int col, const float (&v)[32]) const {
     EpiStoreBf16 st{C, ldc, N};
     st(tc, row, col, v);

@@ -19,13 +19,13 @@ __device__ __forceinline__ void unpack8(const uint4& v, float (&f)[8]) {
   for (int i = 0; i < 4; ++i) { float2 t = __bfloat1622float2(p[i]); f[2 * i] = t.x; f[2 * i + 1] = t.y; }
 }
 
-// act: 0 none; 1 = input is [gate | up] (2K wide), x := swiglu(gate, up) computed while staging; with x_weight (one per item)
+// act: 0 none; 1 = input is [gate | up] (2K wide), x := glu(gate, up) computed while staging; with x_weight (one per item)
 // gate and up are multiplied by the item's weight first.
 template <int RB, typename TO>
 __global__ void __launch_bounds__(GEMV_WARPS * 32)
 gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W,
                  long long expert_stride, int ldw, TO* __restrict__ y, int ldy, int rows_per_item, int N, int K,
-                 const int* __restrict__ pair_expert, const int* __restrict__ pair_row, int act, float limit,
+                 const int* __restrict__ pair_expert, const int* __restrict__ pair_row, int act, GluAct glu,
                  long long x_item_stride, long long y_item_stride, int cpc, const float* __restrict__ x_weight,
                  const OutAct oact) {
   extern __shared__ __align__(16) uint8_t smem_gemv[];
@@ -40,7 +40,7 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
   const int xr0 = strided ? 0 : (pair_row ? pair_row[item] : item * rows_per_item);
   const int yr0 = strided ? 0 : item * rows_per_item;
   const __nv_bfloat16* Wb = W + (pair_expert ? static_cast<long long>(pair_expert[item]) * expert_stride : 0);
-  const int R = rows_per_item;
+  const int R = rows_per_item, oc = item * oact.batch_cols;
   // stage activations (zero rows beyond R); plain rows are copied as 16-byte vectors
   if (act == 0) {
     const int KV8 = K >> 3;
@@ -57,9 +57,7 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
       float v = 0.f;
       if (r < R) {
         const __nv_bfloat16* xr = x + static_cast<size_t>(xr0 + r) * ldx;
-        float g = xw * __bfloat162float(xr[k]), u = xw * __bfloat162float(xr[K + k]);
-        if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
-        v = g / (1.f + __expf(-g)) * u;
+        v = glu_t<__nv_bfloat16>(glu, xw * __bfloat162float(xr[k]), xw * __bfloat162float(xr[K + k]));
       }
       xs[i] = __float2bfloat16(v);
     }
@@ -112,8 +110,8 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
     for (int r = 0; r < RB; ++r) {
       if (r < R) {
         TO* yr = y + static_cast<size_t>(yr0 + r) * ldy;
-        yr[n0] = static_cast<TO>(out_act(oact, acc0[r], r, n0));
-        if (two) yr[n0 + 1] = static_cast<TO>(out_act(oact, acc1[r], r, n0 + 1));
+        yr[n0] = static_cast<TO>(out_act(oact, acc0[r], r, oc + n0));
+        if (two) yr[n0 + 1] = static_cast<TO>(out_act(oact, acc1[r], r, oc + n0 + 1));
       }
     }
   }
@@ -122,7 +120,7 @@ gemv_bf16_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat
 
 template <int RB, typename TO>
 static int launch_gemv(const void* x, int ldx, const void* W, long long es, int ldw, void* y, int ldy, int items,
-                       int rows, int N, int K, const int* pe, const int* pr, int act, float limit, const OutAct& oact, cudaStream_t s,
+                       int rows, int N, int K, const int* pe, const int* pr, int act, const GluAct& glu, const OutAct& oact, cudaStream_t s,
                        long long xis = 0, long long yis = 0, const float* xw = nullptr) {
   auto kern = gemv_bf16_kernel<RB, TO>;
   const int smem = RB * K * 2;
@@ -138,7 +136,7 @@ static int launch_gemv(const void* x, int ldx, const void* W, long long es, int 
   dim3 grid((groups + cpc - 1) / cpc, items);
   const cudaError_t err = spark_launch_pdl(kern, grid, dim3(GEMV_WARPS * 32), smem, s, dim3(1, 1, 1),
                                            (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, es, ldw, (TO*)y, ldy, rows, N, K,
-                                           pe, pr, act, limit, xis, yis, cpc, xw, oact);
+                                           pe, pr, act, glu, xis, yis, cpc, xw, oact);
   return err == cudaSuccess ? 0 : -4;
 }
 
@@ -390,7 +388,8 @@ using namespace spark;
 // items x rows_per_item rows; K % 8 == 0; out_f32 selects fp32 or bf16 output.
 extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long expert_stride, int ldw, void* y, int ldy,
                                int items, int rows_per_item, int N, int K, const int* pair_expert, const int* pair_row,
-                               int act, float limit, int out_f32, const OutAct* out, cudaStream_t s, const float* x_weight) {
+                               int act, const GluAct* act_glu, int out_f32, const OutAct* out, cudaStream_t s, const float* x_weight) {
+  const GluAct glu = act_glu ? *act_glu : GluAct{0.f, 1.f, 0.f};
   if (items <= 0 || rows_per_item <= 0) return 0;
   if (x_weight && act != 1) return -5;
   const OutAct oact = out ? *out : OutAct{};
@@ -406,9 +405,9 @@ extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long 
 #define SPARK_GEMV_CASE(RB)                                                                                          \
   if (rows_per_item <= RB)                                                                                           \
     return out_f32 ? launch_gemv<RB, float>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N, K,       \
-                                            pair_expert, pair_row, act, limit, oact, s, 0, 0, x_weight)                    \
+                                            pair_expert, pair_row, act, glu, oact, s, 0, 0, x_weight)                    \
                    : launch_gemv<RB, __nv_bfloat16>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N,  \
-                                                    K, pair_expert, pair_row, act, limit, oact, s, 0, 0, x_weight);
+                                                    K, pair_expert, pair_row, act, glu, oact, s, 0, 0, x_weight);
   SPARK_GEMV_CASE(1)
   SPARK_GEMV_CASE(2)
   SPARK_GEMV_CASE(4)
@@ -424,15 +423,16 @@ extern "C" int spark_gemv_bf16(const void* x, int ldx, const void* W, long long 
 // offsets must keep x 16-byte aligned.
 extern "C" int spark_gemv_bf16_items(const void* x, int ldx, long long x_item_stride, const void* W, long long expert_stride,
                                      int ldw, void* y, int ldy, long long y_item_stride, int items, int rows_per_item, int N,
-                                     int K, const int* pair_expert, int out_f32, cudaStream_t s) {
+                                     int K, const int* pair_expert, int out_f32, const OutAct* out, cudaStream_t s) {
+  const OutAct oact = out ? *out : OutAct{};
   if (items <= 0 || rows_per_item <= 0) return 0;
   if (K % 8 || rows_per_item > 16 || (x_item_stride & 7) || (ldx & 7) || (x_item_stride | y_item_stride) == 0) return -5;
 #define SPARK_GEMV_ITEMS(RB)                                                                                         \
   if (rows_per_item <= RB)                                                                                           \
     return out_f32 ? launch_gemv<RB, float>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N, K,       \
-                                            pair_expert, nullptr, 0, 0.f, OutAct{}, s, x_item_stride, y_item_stride)           \
+                                            pair_expert, nullptr, 0, GluAct{}, oact, s, x_item_stride, y_item_stride)           \
                    : launch_gemv<RB, __nv_bfloat16>(x, ldx, W, expert_stride, ldw, y, ldy, items, rows_per_item, N,  \
-                                                    K, pair_expert, nullptr, 0, 0.f, OutAct{}, s, x_item_stride, y_item_stride);
+                                                    K, pair_expert, nullptr, 0, GluAct{}, oact, s, x_item_stride, y_item_stride);
   SPARK_GEMV_ITEMS(1)
   SPARK_GEMV_ITEMS(2)
   SPARK_GEMV_ITEMS(4)

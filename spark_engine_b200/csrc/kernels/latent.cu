@@ -9,7 +9,9 @@
 //                    fp32 (the weights enter the second product as two-term bf16 sums)
 //   latent_rows      one CTA per (row, head) in the absorbed form on the FP32 units: the 32-bit mode, and shapes the
 //                    tensor-core kernels do not cover
-// Rotary pairs are (2i, 2i + 1) when `interleaved`, else (i, i + rope/2).
+// Rotary pairs are (2i, 2i + 1) when `interleaved`, else (i, i + rope/2).  Queries may come straight from the projected row (no
+// query latent) and rows may have no rotated part.  An optional sink per head enters the denominator only; the output gate is one
+// sigmoid per head, or per element of the concatenated heads (prompts here; absorbed rows: in the product behind the attention).
 #include "../common/rows.cuh"
 
 namespace spark {
@@ -41,12 +43,14 @@ latent_prep_kernel(const T* __restrict__ proj, int ldp, int oq, int okv, int okr
   pdl_wait();
   const int r = blockIdx.x, t = threadIdx.x, p = pos[r];
   const T* a = proj + static_cast<size_t>(r) * ldp;
-  float ss = 0.f;
-  for (int i = t; i < d.q_rank; i += 128) { const float x = ldf(a + oq + i); ss = fmaf(x, x, ss); }
-  float rs = 1.f / sqrtf(block_sum_all(ss, sh) / d.q_rank + d.eps);
-  for (int i = t; i < d.ldcq; i += 128)
-    stf(cq + static_cast<size_t>(r) * d.ldcq + i, i < d.q_rank ? ldf(a + oq + i) * rs * q_norm[i] : 0.f);
-  ss = 0.f;
+  float ss = 0.f, rs;
+  if (d.q_rank > 0) {
+    for (int i = t; i < d.q_rank; i += 128) { const float x = ldf(a + oq + i); ss = fmaf(x, x, ss); }
+    rs = 1.f / sqrtf(block_sum_all(ss, sh) / d.q_rank + d.eps);
+    for (int i = t; i < d.ldcq; i += 128)
+      stf(cq + static_cast<size_t>(r) * d.ldcq + i, i < d.q_rank ? ldf(a + oq + i) * rs * q_norm[i] : 0.f);
+    ss = 0.f;
+  }
   for (int i = t; i < d.L; i += 128) { const float x = ldf(a + okv + i); ss = fmaf(x, x, ss); }
   rs = 1.f / sqrtf(block_sum_all(ss, sh) / d.L + d.eps);
   const int page = p / LAT_PAGE < page_ld ? pages[static_cast<size_t>(row_slot[r]) * page_ld + p / LAT_PAGE] : -1;
@@ -109,7 +113,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 latent_rows_kernel(const T* __restrict__ q_full, const T* __restrict__ cache, const int* __restrict__ pos, const int* __restrict__ rows,
                    const int* __restrict__ row_slot, const int* __restrict__ pages, int page_ld, int H, int Lp, int Rp, float scale,
-                   const T* __restrict__ gate, int ldg, T* __restrict__ out) {
+                   const T* __restrict__ gate, int ldg, const float* __restrict__ sink, T* __restrict__ out) {
   extern __shared__ float sq[];                              // [KW] query, then [128] weights
   __shared__ float sh[32];
   pdl_wait();
@@ -122,7 +126,7 @@ latent_rows_kernel(const T* __restrict__ q_full, const T* __restrict__ cache, co
   float acc[8];
 #pragma unroll
   for (int c = 0; c < 8; ++c) acc[c] = 0.f;
-  float m = -INFINITY, l = 0.f;
+  float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f;
   for (int k0 = 0; k0 < n; k0 += 128) {
     const int tok = k0 + t;
     float s = -INFINITY;
@@ -195,7 +199,8 @@ struct LatentPrefill {
   const __nv_bfloat16 *q, *kv, *lat, *gate;
   __nv_bfloat16* out;
   const int* segs;                 // [n][5]
-  int ldq, ldkv, ldlat, ldg, ldo, H, Dp, Rp, V, Vp, Lp;
+  const float* sink;               // [H]
+  int ldq, ldkv, ldlat, ldg, ldo, H, Dp, Rp, V, Vp, Lp, gate_all;      // gate_all: a gate column per output column, else per head
   float scale_log2;
 };
 
@@ -245,7 +250,9 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefill a) {
   float o[VP / 8][4];
 #pragma unroll
   for (int i = 0; i < VP / 8; ++i) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
-  float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+  // the sink is a key seen first: maximum = its score, sum = 1 (once per row: the quad's lane 0), output 0
+  const float m0 = a.sink ? a.sink[h] * 1.4426950408889634f : -INFINITY;
+  float m_lo = m0, m_hi = m0, l_lo = a.sink && t == 0 ? 1.f : 0.f, l_hi = l_lo;
   const int p_lo = pos0 + qt * BM + min(warp * 16 + g, rows_valid - 1);
   const int p_hi = pos0 + qt * BM + min(warp * 16 + g + 8, rows_valid - 1);
   const int p_first = pos0 + qt * BM + min(warp * 16, rows_valid - 1);
@@ -322,13 +329,32 @@ latent_prefill_kernel(const __grid_constant__ LatentPrefill a) {
     if (rl >= rows_valid) continue;
     const size_t r = static_cast<size_t>(r0 + qt * BM + rl);
     float inv = 1.f / (hh ? l_hi : l_lo);
-    if (a.gate) inv *= sigmoid_f(__bfloat162float(a.gate[r * a.ldg + h]));
+    const __nv_bfloat16* gate = a.gate ? a.gate + r * a.ldg + (a.gate_all ? h * a.V : h) : nullptr;
+    if (gate && !a.gate_all) inv *= sigmoid_f(__bfloat162float(*gate));
+    const bool each = gate && a.gate_all;
+    __nv_bfloat16* o_row = a.out + r * a.ldo + h * a.V;
+    if (((a.V | a.ldo | (each ? a.ldg : 0)) & 1) == 0) {       // column pairs are 4-byte aligned
+#pragma unroll
+      for (int i = 0; i < VP / 8; ++i) {
+        const int d = i * 8 + 2 * t;
+        if (d >= a.V) continue;
+        float x = o[i][2 * hh] * inv, y = o[i][2 * hh + 1] * inv;
+        if (each) {
+          const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + d));
+          x *= sigmoid_t<__nv_bfloat16>(g.x); y *= sigmoid_t<__nv_bfloat16>(g.y);
+        }
+        *reinterpret_cast<__nv_bfloat162*>(o_row + d) = __floats2bfloat162_rn(x, y);
+      }
+      continue;
+    }
 #pragma unroll
     for (int i = 0; i < VP / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int d = i * 8 + 2 * t + e;
-        if (d < a.V) a.out[r * a.ldo + h * a.V + d] = __float2bfloat16(o[i][2 * hh + e] * inv);
+        if (d >= a.V) continue;
+        const float x = o[i][2 * hh + e] * inv;
+        o_row[d] = __float2bfloat16(each ? x * sigmoid_t<__nv_bfloat16>(__bfloat162float(gate[d])) : x);
       }
   }
 }
@@ -368,7 +394,7 @@ extern "C" int spark_latent_prep(const void* proj, int ldp, int oq, int okv, int
 extern "C" int spark_latent_qrope(const void* src, int lds, int hss, void* dst, int ldd, int hsd, int n, int H, int rope, int Rp,
                                   int interleaved, const double* inv_freq, const int* pos, const int* rows, int src_compact, int f32,
                                   cudaStream_t s) {
-  if (n <= 0) return 0;
+  if (n <= 0 || Rp <= 0) return 0;
   SPARK_BY_TYPE(f32, spark_launch_pdl(latent_qrope_kernel<T>, dim3(n, (H * (Rp / 2) + 127) / 128), dim3(128), 0, s, dim3(1, 1, 1),
                                       (const T*)src, lds, hss, (T*)dst, ldd, hsd, H, rope, Rp, interleaved, inv_freq, pos, rows,
                                       src_compact))
@@ -386,25 +412,27 @@ extern "C" int spark_latent_gather(const void* cache, int width, const int* segs
 
 extern "C" int spark_latent_rows(const void* q_full, const void* cache, const int* pos, const int* rows, const int* row_slot,
                                  const int* pages, int page_ld, int n, int H, int Lp, int Rp, float scale, const void* gate, int ldg,
-                                 void* out, int f32, cudaStream_t s) {
+                                 const float* sink, void* out, int f32, cudaStream_t s) {
   if (n <= 0) return 0;
   if (Lp > 1024 || H > 65535 || ((Lp + Rp) & 3)) return -5;
   SPARK_BY_TYPE(f32, spark_launch_pdl(latent_rows_kernel<T>, dim3(n, H), dim3(128), (Lp + Rp + 128) * 4, s, dim3(1, 1, 1),
                                       (const T*)q_full, (const T*)cache, pos, rows, row_slot, pages, page_ld, H, Lp, Rp, scale,
-                                      (const T*)gate, ldg, (T*)out))
+                                      (const T*)gate, ldg, sink, (T*)out))
   return spark_launch_rc(__func__);
 }
 
-// bf16.  -6: the shape does not fit shared memory (the caller uses spark_latent_rows).
+// bf16.  gate (optional): at column 0 of its rows, one logit per head or (gate_all) one per output column.  -6: the shape does not fit shared memory (the caller uses spark_latent_rows).
 extern "C" int spark_latent_prefill(const void* q, int ldq, const void* kv, int ldkv, const void* lat, int ldlat, const int* segs,
                                     int nseg, int max_rows, int H, int Dp, int Rp, int V, int Vp, int Lp, float scale,
-                                    const void* gate, int ldg, void* out, int ldo, cudaStream_t s) {
+                                    const void* gate, int ldg, int gate_all, const float* sink, void* out, int ldo, cudaStream_t s) {
   if (nseg <= 0) return 0;
+  if ((gate_all && (reinterpret_cast<uintptr_t>(gate) & 3)) || (reinterpret_cast<uintptr_t>(out) & 3)) return -5;
   if ((Dp | Rp | Vp | Lp) & 15 || Vp < V || (ldq | ldkv | ldlat) & 7) return -5;
   LatentPrefill a;
   a.q = (const __nv_bfloat16*)q; a.kv = (const __nv_bfloat16*)kv; a.lat = (const __nv_bfloat16*)lat; a.gate = (const __nv_bfloat16*)gate;
   a.out = (__nv_bfloat16*)out; a.segs = segs; a.ldq = ldq; a.ldkv = ldkv; a.ldlat = ldlat; a.ldg = ldg; a.ldo = ldo;
   a.H = H; a.Dp = Dp; a.Rp = Rp; a.V = V; a.Vp = Vp; a.Lp = Lp; a.scale_log2 = scale * 1.4426950408889634f;
+  a.sink = sink; a.gate_all = gate_all;
   if (Vp <= 32) return launch_latent_prefill<32, 8>(a, nseg, max_rows, s);
   if (Vp <= 64) return launch_latent_prefill<64, 8>(a, nseg, max_rows, s);
   if (Vp <= 128) return launch_latent_prefill<128, 8>(a, nseg, max_rows, s);

@@ -469,11 +469,12 @@ extern "C" int spark_mla_attn(const void* q_full, const void* lat, const int* po
                   row_pos0, row_j, anc, lat_fp8, MlaPages{nullptr, 0, nullptr, nullptr}, false, nullptr, 0);
 }
 
-// Rows over a paged latent cache (dense causal context), fp32-grade softmax weights, optional per-head sigmoid gate.
+// Rows over a paged latent cache (dense causal context), fp32-grade softmax weights, optional per-head sigmoid gate and sink.
 // Query row i of the launch is plan row rows[i] (rows == nullptr: i); pos and row_slot are indexed by plan row.
 extern "C" int spark_mla_attn_paged(const void* q_full, const void* lat, const int* pos, const int* rows, const int* row_slot,
                                     const int* page_table, int page_ld, float* part_o, float* part_ml, int nsplit, int R, int H,
-                                    int kv_lora, int rope, float scale, const void* gate, int ldg, void* out, cudaStream_t s) {
-  return mla_attn(q_full, lat, pos, nullptr, nullptr, nullptr, 0, part_o, part_ml, nsplit, nullptr, R, H, kv_lora, rope, scale, out,
+                                    int kv_lora, int rope, float scale, const void* gate, int ldg, const float* sink, void* out,
+                                    cudaStream_t s) {
+  return mla_attn(q_full, lat, pos, nullptr, nullptr, nullptr, 0, part_o, part_ml, nsplit, sink, R, H, kv_lora, rope, scale, out,
                   s, nullptr, nullptr, nullptr, 0, MlaPages{page_table, page_ld, row_slot, rows}, true, gate, ldg);
 }

@@ -16,7 +16,8 @@ constexpr int ROUTE_THREADS = 256;
 constexpr int ROUTE_MAXE_PER_THREAD = 4;     // up to 1024 experts
 
 // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias (the bias enters the choice only), 4 sigmoid, not
-// renormalised (ranked by the logits, which a saturated sigmoid would tie).
+// renormalised (ranked by the logits, which a saturated sigmoid would tie), 5 softmax over the chosen logits alone (bias, if any,
+// added to the logits; ranked by them, and only the chosen ones are exponentiated, against the largest).
 // The last n_self of the E router outputs are identity experts: they leave -1 in `ids` and their weight in self_w[row].
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int kind, const float* __restrict__ bias,
@@ -35,6 +36,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
   for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) {
     const int e = t + j * ROUTE_THREADS;
     p[j] = e < E ? x[e] : -INFINITY;
+    if (kind == 5 && bias && e < E) p[j] += bias[e];
     mx = fmaxf(mx, p[j]);
   }
   if (kind == 0 || kind == 3) {
@@ -66,6 +68,9 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
   } else if (kind == 4) {
 #pragma unroll
     for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) { s[j] = p[j]; p[j] = 1.f / (1.f + expf(-p[j])); }
+  } else if (kind == 5) {
+#pragma unroll
+    for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) s[j] = p[j];
   } else {
 #pragma unroll
     for (int j = 0; j < ROUTE_MAXE_PER_THREAD; ++j) {
@@ -115,6 +120,10 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int E, int top_k, int
   }
   if (t == 0) {
     float sum = 0.f;
+    if (kind == 5) {                                         // the first one chosen is the largest
+      const float top = sel_p[0];
+      for (int k = 0; k < top_k; ++k) sel_p[k] = expf(sel_p[k] - top);
+    }
     for (int k = 0; k < top_k; ++k) sum += sel_p[k];
     sum = kind == 4 ? 1.f : fmaxf(sum, 1e-20f);
     float own = 0.f;
@@ -140,7 +149,7 @@ struct RouterArgs {
   const __nv_bfloat16* x; int ldx;           // [R, K]
   const __nv_bfloat16* Wg; int ldw;          // [E (+1), K]
   float* logits; int ld;                     // scratch [R, ld]
-  int R, K, E, top_k, kind;                  // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias, 4 sigmoid
+  int R, K, E, top_k, kind;                  // kind: 0 softmax, 1 sigmoid+bias, 2 sqrt(softplus)+bias, 3 softmax+bias, 4 sigmoid, 5 softmax of the chosen
   const float* bias; float scale; int shared_gate;
   int slots;                                 // top_k, or top_k + 1 when the shared expert is a pair
   int shared_expert;                         // index of the shared expert in the local stack (slot top_k)
@@ -265,11 +274,14 @@ moe_router_topk_kernel(const __grid_constant__ RouterArgs a) {
     for (int j = 0; j < EPL; ++j) {
       const int e = lane + 32 * j;
       p[j] = (j < nj && e < a.E) ? __ldcg(lg + e) : -INFINITY;
+      if (a.kind == 5 && a.bias && j < nj && e < a.E) p[j] += a.bias[e];
       s[j] = p[j];
       mx = fmaxf(mx, p[j]);
     }
     if (a.kind == 4) {
       // ranked by the logits, only the k winners' sigmoids are formed
+    } else if (a.kind == 5) {
+      mx = warp_max(mx);
     } else if (a.kind == 0) {
       // softmax -> top-k -> renormalise: the softmax denominator cancels, so experts are ranked by their logits and
       // only the k winners are exponentiated
@@ -319,6 +331,7 @@ moe_router_topk_kernel(const __grid_constant__ RouterArgs a) {
 #pragma unroll
         for (int j = 0; j < EPL; ++j) if (j == bj) { bp = p[j]; s[j] = -INFINITY; }
         if (a.kind == 0) bp = __expf(bp - mx);
+        if (a.kind == 5) bp = expf(bp - mx);
         if (a.kind == 4) bp = 1.f / (1.f + expf(-bp));
         lane_best(s, best, bj);
       }

@@ -40,6 +40,18 @@ def pad_head_cols(t: torch.Tensor, heads: int, to: int) -> torch.Tensor:
     return pad_cols(t.view(m, heads, d), to).reshape(m, heads * to)
 
 
+def latent_up(uk: torch.Tensor, uv: torch.Tensor, c, dtype) -> Dict[str, torch.Tensor]:
+    """Key and value matrices over the latents, [heads * dim | heads * v, latent], as the runner uses them: uk_t [heads, latent, dim]
+    and uv [heads, v, latent] for absorbed rows, kv_up (per head [key | value], padded to 16) for prompts."""
+    H, D, V, Lp = c.n_heads, c.head_dim, c.v_dim, pad(c.kv_rank, 16)
+    Dp, Vp = pad(D, 16), pad(V, 16)
+    uk, uv = pad_cols(uk, Lp).view(H, D, Lp), pad_cols(uv, Lp).view(H, V, Lp)
+    up = uk.new_zeros(H, Dp + Vp, Lp)
+    up[:, :D], up[:, Dp: Dp + V] = uk, uv
+    wd = lambda t: t.to(dtype).contiguous()
+    return {"uk_t": wd(pad_cols(uk.transpose(1, 2), Dp)), "uv": wd(uv), "kv_up": wd(up.view(H * (Dp + Vp), Lp))}
+
+
 def taker(tensors: Dict[str, torch.Tensor], device):
     """get(name, shape=None): the tensor on `device`; its shape must be the given one (None entries: any)."""
     def get(name: str, shape: Optional[tuple] = None) -> torch.Tensor:

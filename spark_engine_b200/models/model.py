@@ -656,6 +656,12 @@ class Model:
         if not self.page:
             self.seqs = [SeqInfo(i * per, per) if kv_backing is None else SeqInfo(0, 0) for i in range(n_slots)]
         self.layers = self._build_layers([W["layers"][i] for i in cfg.layer_runs()])
+        self.convs = self._build_convs()     # per layer run: input convolutions of the two sublayers
+        self.pos_freq = None                 # angle per position of the pairs of a sinusoidal position vector
+        if cfg.positions:
+            if cfg.positions != "sinusoidal":
+                raise ValueError(f"unknown positions {cfg.positions!r}")
+            self.pos_freq = (1e4 ** (-torch.arange((cfg.hidden + 1) // 2, dtype=torch.float64) * 2 / cfg.hidden)).to(self.device)
         self.mtp_layers = self._build_layers(W["mtp"]["layers"]) if "mtp" in W else []
         self.hidden_out = None
         # a hashed n-gram table that stays on the host is read through asynchronous gathers into a pinned ring
@@ -695,11 +701,22 @@ class Model:
             out.append((lw, mix, MoeBlock(self.cfg, lw["mlp"])))
         return out
 
+    def _build_convs(self):
+        from .input_conv import InputConv
+        if not self.cfg.input_conv:
+            return []
+        return [tuple(InputConv(lw[k], self.n_slots, self.device) if k in lw else None for k in ("conv1", "conv2")) for lw, _, _ in self.layers]
+
     # -- sequence bookkeeping ---------------------------------------------------------------
+    def stateful(self, drafter: bool = True) -> list:
+        """Everything that holds state or cache rows of the slots, in a fixed order (`drafter`: the draft layers' too)."""
+        mixers = [mix for _, mix, _ in self.layers + (self.mtp_layers if drafter else [])]
+        return mixers + [c for pair in self.convs for c in pair if c is not None]
+
     def reset_slot(self, slot: int):
         self.seqs[slot].length = 0
-        for _, mix, _ in self.layers + self.mtp_layers:
-            mix.reset(slot)
+        for x in self.stateful():
+            x.reset(slot)
 
     def set_kv_region(self, slot: int, base: int, cap: int):
         self.seqs[slot].kv_base, self.seqs[slot].kv_cap = base, cap
@@ -733,9 +750,9 @@ class Model:
     def _norm(self, w: dict, name: str) -> ops.RowNorm:
         """A norm of a model with layer specs."""
         cfg = self.cfg
-        return ops.RowNorm(w[name], cfg.norm_eps, w[name + "_b"] if cfg.norm_kind == "layer" else None, cfg.norm_one_plus)
+        return ops.RowNorm(w[name], cfg.norm_eps, w[name + "_b"] if cfg.norm_kind == "layer" else None, cfg.norm_one_plus, cfg.norm_groups)
 
-    def _spec_block(self, li, lw, mix, mlp, X, pend, plan, commit):
+    def _spec_block(self, li, lw, mix, mlp, X, pend, plan, commit, depth=None):
         """One block of a model with layer specs.  `pend` as in `_block`: every residual update is one launch together with
         the norm (or the cast) of the rows that its successor reads."""
         cfg = self.cfg
@@ -749,10 +766,12 @@ class Model:
                 h, X, _ = ops.add_norm_rows(pend, X, None, self.dtype)
                 pend = ops.Update(mlp.forward(h, defer=True), post=self._norm(lw, "post_norm"))
             return X, pend
-        h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "in_norm"), self.dtype)
+        rows = ops.RowContext(plan, commit, depth is not None)
+        convs = self.convs[li] if self.convs else (None, None)
+        h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "in_norm"), self.dtype, conv=convs[0], ctx=rows)
         pend = ops.Update(mix.forward(h, plan, self.seqs, commit), lw.get("ls1"))
         if mlp is not None:
-            h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "post_norm"), self.dtype)
+            h, X, _ = ops.add_norm_rows(pend, X, self._norm(lw, "post_norm"), self.dtype, conv=convs[1], ctx=rows)
             pend = ops.Update(mlp.forward(h, defer=True), lw.get("ls2"))
         if "side" in lw:                     # the token's own row of this layer, gated by the residual stream itself
             s, n = lw["side"], cfg.side_dim
@@ -760,6 +779,8 @@ class Model:
             ids = plan.dev["ids32"] if "ids32" in plan.dev else plan.ids
             g = ops.linear_token_gate(x, s["gate"], self.W["side_embed"], ids, cfg.layer_runs()[li] * n, n)
             pend = ops.Update(ops.linear(g, s["proj"], out_f32=True), post=ops.RowNorm(s["norm"], cfg.norm_eps))
+        if depth is not None:
+            pend.depth = ops.DepthAverage(depth, li + 1, lw["depth"])
         return X, pend
 
     def _block(self, lw, mix, mlp, X, pend, plan, commit):
@@ -803,6 +824,7 @@ class Model:
                 if sg.pos0 + sg.n > self.seqs[sg.slot].kv_cap:
                     raise RuntimeError(f"slot {sg.slot}: rows up to position {sg.pos0 + sg.n} exceed its KV region of "
                                        f"{self.seqs[sg.slot].kv_cap} tokens")
+        depth = None
         if plan.mm_rows:
             # salted placeholder ids are outside the vocabulary: look up row 0 for them, then write the encoded media
             # rows over those positions (engine-rs/src/weights.rs:536-569)
@@ -812,7 +834,10 @@ class Model:
             X[salted.to(X.device)] = 0
             X = inject_rows(X, plan.ids, plan.mm_rows)
         else:
-            X = ops.embed(W["embed"], plan.ids, self.dtype, cfg.embed_scale)
+            if cfg.depth_average:            # the embedding's rows and every layer's result, fp32
+                depth = torch.empty(len(self.layers) + 1, plan.rows, cfg.hidden, dtype=torch.float32, device=self.device)
+            pos = (plan.dev.get("pos32", plan.pos), self.pos_freq) if cfg.positions else None
+            X = ops.embed(W["embed"], plan.ids, self.dtype, cfg.embed_scale, pos, depth[0] if depth is not None else None)
         if cfg.hc_kind != "none":
             X = X.unsqueeze(1).repeat(1, cfg.hc_streams, 1).contiguous()
         self._ids_for_ngram = plan
@@ -825,7 +850,7 @@ class Model:
             self.taps = {}
         for li, (lw, mix, mlp) in enumerate(self.layers):
             if cfg.layer_specs:
-                X, pend = self._spec_block(li, lw, mix, mlp, X, pend, plan, commit)
+                X, pend = self._spec_block(li, lw, mix, mlp, X, pend, plan, commit, depth)
             else:
                 X, pend = self._block(lw, mix, mlp, X, pend, plan, commit)
             if taps and li in taps:          # residual stream after layer li (feature taps of a drafter)
@@ -836,7 +861,7 @@ class Model:
         elif cfg.hc_kind == "mhc":
             X, hn = ops.mhc_final(X, pend, W["final_norm"], cfg.norm_eps, self.tp)
         elif cfg.layer_specs:
-            hn, X, _ = ops.add_norm_rows(pend, X, self._norm(W, "final_norm"), self.dtype)
+            hn, X, _ = ops.add_norm_rows(pend, X, self._norm(W, "final_norm"), self.dtype, ctx=ops.RowContext(plan, commit, depth is not None))
         else:
             hn, X = ops.add_rmsnorm(pend, X, W["final_norm"], cfg.norm_eps, self.tp)
         if self.tp is not None and getattr(self.tp, "rows_sharded", False):
@@ -895,7 +920,7 @@ class Model:
         from the segment's first row (always accepted: it is the last sampled token)."""
         plan = self._pending_plan
         assert plan is not None, "commit() without a pending verify"
-        for _, mix, _ in self.layers:
+        for mix in self.stateful(drafter=False):
             mix.commit(accepted)
             if plan.is_tree and hasattr(mix, "compact"):
                 for s, rows in zip(plan.segs, accepted):
@@ -962,7 +987,7 @@ class Model:
         (reference: spec_probe.rs:1420-1444 ckpt_save/restore/clone)."""
         si = self.seqs[slot]
         snap = {"length": si.length, "layers": []}
-        for _, mix, _ in self.layers + self.mtp_layers:
+        for mix in self.stateful():
             d = {}
             for name, t in mix.state_tensors().items():
                 if name in ("S", "tail", "carried"):
@@ -981,7 +1006,7 @@ class Model:
         si = self.seqs[slot]
         n = snap["length"]
         assert n <= si.kv_cap, "sequence capacity exceeded"
-        for (_, mix, _), d in zip(self.layers + self.mtp_layers, snap["layers"]):
+        for mix, d in zip(self.stateful(), snap["layers"]):
             for name, t in mix.state_tensors().items():
                 if name in ("S", "tail", "carried"):
                     t[slot] = d[name]

@@ -126,7 +126,8 @@ class WkvMixer(_ParallelMixer):
 class LatentMixer(_ParallelMixer):
     """The cache holds one row per token, [normed latent | rotated key part] with both parts padded to 16, in pages shared by
     all slots (`pages`: the model's page table).  Decode rows attend in the absorbed form, prompts on up-projected keys
-    and values."""
+    and values.  Queries come from their own latent (`q_rank`) or from the row; without `rope_dim` nothing is rotated; in a
+    sequential block (no feed-forward here) the output product is the mixer's alone."""
     paged = True
 
     def __init__(self, cfg, spec, w, n_pages, page, pages, device, dtype):
@@ -134,10 +135,11 @@ class LatentMixer(_ParallelMixer):
         c = self.c
         self.Dp, self.Rp, self.Vp, self.Lp = pad(c.head_dim, 16), pad(c.rope_dim, 16), pad(c.v_dim, 16), pad(c.kv_rank, 16)
         self.nv = c.n_heads * c.v_dim
-        o = {"dq": 0, "lat": pad(c.q_rank, 8)}
+        self.nq = c.n_heads * (self.Dp + self.Rp)                # query columns, behind uq or in the projected row itself
+        o = {"dq": 0, "lat": pad(c.q_rank, 8) if c.q_rank else self.nq}
         o["rot"] = o["lat"] + self.Lp
         o["g"] = o["rot"] + self.Rp
-        o["ff"] = o["g"] + pad(c.n_heads, 8)
+        o["ff"] = o["g"] + pad(self.nv if c.gate == "element" else c.n_heads, 8)
         self.off, self.page, self.pages = o, page, pages
         self.lat = torch.zeros(n_pages, page, self.Lp + self.Rp, device=device, dtype=dtype)
         # shapes of the tensor-core kernels (heads as MMA rows, rows staged in shared memory); else one CTA per row and head
@@ -167,9 +169,12 @@ class LatentMixer(_ParallelMixer):
         c, w, off = self.c, self.w, self.off
         R, H, D, Ro, V = proj.shape[0], c.n_heads, c.head_dim, c.rope_dim, c.v_dim
         rope = L.rope_interleaved if c.rope_interleaved else L.rope_neox
-        cq = L.rms(proj[:, : c.q_rank].float(), w["dq_norm"], self.eps)
-        cq = torch.cat((cq, cq.new_zeros(R, w["uq"].shape[1] - c.q_rank)), 1)
-        q = (cq @ w["uq"].float().t()).view(R, H, self.Dp + self.Rp)
+        if c.q_rank:
+            cq = L.rms(proj[:, : c.q_rank].float(), w["dq_norm"], self.eps)
+            cq = torch.cat((cq, cq.new_zeros(R, w["uq"].shape[1] - c.q_rank)), 1)
+            q = (cq @ w["uq"].float().t()).view(R, H, self.Dp + self.Rp)
+        else:
+            q = proj[:, : self.nq].float().reshape(R, H, self.Dp + self.Rp)
         qr = rope(q[..., self.Dp: self.Dp + Ro], plan.pos, Ro, c.rope_theta)
         lat = L.rms(proj[:, off["lat"]: off["lat"] + c.kv_rank].float(), w["kv_norm"], self.eps)
         kr = rope(proj[:, off["rot"]: off["rot"] + Ro].float().view(R, 1, Ro), plan.pos, Ro, c.rope_theta)[:, 0]
@@ -186,8 +191,11 @@ class LatentMixer(_ParallelMixer):
             kv = torch.einsum("sl,hdl->shd", ctx[:, : c.kv_rank], up)
             sc = torch.einsum("thd,shd->hts", q[sl, :, :D], kv[..., :D]) + torch.einsum("thd,sd->hts", qr[sl], ctx[:, self.Lp: self.Lp + Ro])
             sc = (sc * c.scale).masked_fill(t.view(1, 1, n) > plan.pos[sl].view(1, -1, 1), float("-inf"))
-            o = torch.einsum("hts,shd->thd", torch.softmax(sc, -1), kv[..., self.Dp: self.Dp + V])
-            o = o * torch.sigmoid(proj[sl, off["g"]: off["g"] + H].float()).unsqueeze(-1)
+            if c.sink:                           # one more score, without a value
+                sc = torch.cat((sc, w["sink"].view(H, 1, 1).expand(H, s.n, 1)), -1)
+            o = torch.einsum("hts,shd->thd", torch.softmax(sc, -1)[..., :n], kv[..., self.Dp: self.Dp + V])
+            gate = proj[sl, off["g"]: off["g"] + (self.nv if c.gate == "element" else H)].float()
+            o = o * torch.sigmoid(gate).view(s.n, H, -1)
             cat[sl, : self.nv] = o.reshape(s.n, self.nv).to(cat.dtype)
 
     def commit(self, accepted):

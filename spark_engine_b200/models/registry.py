@@ -9,8 +9,8 @@ from __future__ import annotations
 
 import importlib
 
-ARCHITECTURES = {"Vabunex": "vabunex", "Debisun": "debisun", "Zapolorn": "zapolorn"}
-FAMILIES = {"vabunex": "vabunex", "debisun": "debisun", "zapolorn": "zapolorn"}
+ARCHITECTURES = {"Vabunex": "vabunex", "Debisun": "debisun", "Zapolorn": "zapolorn", "Zakusun": "zakusun"}
+FAMILIES = {"vabunex": "vabunex", "debisun": "debisun", "zapolorn": "zapolorn", "zakusun": "zakusun"}
 
 
 def architecture(d: dict):

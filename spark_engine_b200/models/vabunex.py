@@ -21,7 +21,7 @@ from typing import Dict
 import torch
 
 from ..config import LatentConfig, LayerSpec, LightningConfig, LoopConfig, ModelConfig, WkvConfig
-from .layout import pad, pad_cols as _cols, stack_rows as _rows, taker
+from .layout import latent_up, pad, pad_cols as _cols, stack_rows as _rows, taker
 
 
 # ----------------------------------------------------------------------------- configuration
@@ -84,8 +84,8 @@ def prepare_layer(raw: Dict[str, torch.Tensor], spec: LayerSpec, hidden: int, dt
         if F:
             w["ff"] = wd(_rows(ff))
     else:
-        H, D, R, V, L = c.n_heads, c.head_dim, c.rope_dim, c.v_dim, c.kv_rank
-        Dp, Rp, Vp, Lp = pad(D, 16), pad(R, 16), pad(V, 16), pad(L, 16)
+        H, D, R, L = c.n_heads, c.head_dim, c.rope_dim, c.kv_rank
+        Dp, Rp = pad(D, 16), pad(R, 16)
         dkv = m["dkv"]
         w["in"] = wd(torch.cat((_rows([m["dq"]]), _rows([dkv[:L]], 16), _rows([dkv[L:]], 16), _rows([m["g"]] + ff))))
         w["dq_norm"], w["kv_norm"] = f32(m["dq.norm"]), f32(m["dkv.norm"])
@@ -93,12 +93,7 @@ def prepare_layer(raw: Dict[str, torch.Tensor], spec: LayerSpec, hidden: int, dt
         q = uq.new_zeros(H, Dp + Rp, uq.shape[-1])
         q[:, :D], q[:, Dp: Dp + R] = uq[:, :D], uq[:, D:]
         w["uq"] = wd(q.view(H * (Dp + Rp), -1))
-        uk, uv = _cols(m["uk"], Lp).view(H, D, Lp), _cols(m["uv"], Lp).view(H, V, Lp)
-        w["uk_t"] = wd(_cols(uk.transpose(1, 2), Dp))
-        w["uv"] = wd(uv)
-        up = uk.new_zeros(H, Dp + Vp, Lp)
-        up[:, :D], up[:, Dp: Dp + V] = uk, uv
-        w["kv_up"] = wd(up.view(H * (Dp + Vp), Lp))
+        w.update(latent_up(m["uk"], m["uv"], c, dtype))
     return {"type": spec.kind, "in_norm": f32(raw["norm1"]), "mix": w, "mlp": {"ffn": F}}
 
 

@@ -47,14 +47,21 @@ def set_fallback(on: bool):
 
 
 # ----------------------------------------------------------------------------- basic ops
-def embed(table: torch.Tensor, ids: torch.Tensor, dtype, scale: float = 1.0) -> torch.Tensor:
-    """Token embedding rows (times `scale`).  On the device the residual stream is fp32 (activations bf16)."""
+def embed(table: torch.Tensor, ids: torch.Tensor, dtype, scale: float = 1.0, pos=None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Token embedding rows (times `scale`), into `out` if given.  `pos` = (positions, angle per position of every channel pair): the
+    sines (even channels) and cosines (odd ones) of the row's position are added.  On the device the residual stream is fp32
+    (activations bf16)."""
     if use_kernels(table):
-        if scale != 1.0 or table.dtype == torch.float32:
-            return block_ops().embed_scaled(table, ids.to(torch.int32), scale)
+        if scale != 1.0 or table.dtype == torch.float32 or pos is not None or out is not None:
+            return block_ops().embed_scaled(table, ids.to(torch.int32), scale, pos, out)
         return cuda_ops().embed(table, ids.to(torch.int32))
     x = table[ids].to(dtype)
-    return x * scale if scale != 1.0 else x
+    if scale != 1.0:
+        x = x * scale
+    if pos is not None:
+        a = (pos[0].double().unsqueeze(1) * pos[1]).to(x.dtype)
+        x = x + torch.stack((a.sin(), a.cos()), -1).flatten(1)[:, : x.shape[1]]
+    return x if out is None else out.copy_(x)
 
 
 def to_tensor(x):
@@ -222,6 +229,10 @@ def route(h, w, c):
     if c.shared_gate:
         sg = torch.sigmoid(logits[:, c.n_routes:])
         logits = logits[:, : c.n_routes]
+    if c.router == "topk_softmax":
+        z = logits + w["bias"].float().to(logits.device) if "bias" in w else logits
+        idx = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, : c.top_k]
+        return torch.softmax(torch.gather(z, 1, idx), -1) * c.route_scale, idx, sg
     if c.router in ("softmax", "softmax_bias"):
         p = torch.softmax(logits, -1)
         sel = p if c.router == "softmax" else p + w["bias"].float().to(p.device)
@@ -260,7 +271,7 @@ def moe(h, w, c, defer: bool = False):
             a = wts[rows, slot].unsqueeze(1)
             gu = (hf[rows] * a if c.weight_input else hf[rows]) @ _expert(wgu, e - lo).t()
             n = gu.shape[1] // 2
-            y = (relu2(gu) if single else L.swiglu(gu[:, :n], gu[:, n:], c.swiglu_limit)) @ _expert(wd, e - lo).t()
+            y = (relu2(gu) if single else L.swiglu(gu[:, :n], gu[:, n:], *c.glu)) @ _expert(wd, e - lo).t()
             out[rows] += y if c.weight_input else a * y
     if c.n_identity:
         out += (wts * (idx >= c.n_experts)).sum(-1, keepdim=True) * hf
@@ -270,7 +281,7 @@ def moe(h, w, c, defer: bool = False):
     elif "s_gu" in w:
         gu = linear(h, w["s_gu"]).float()
         Fs = gu.shape[1] // 2
-        sh = linear(L.swiglu(gu[:, :Fs], gu[:, Fs:], c.swiglu_limit).to(h.dtype), w["s_down"]).float()
+        sh = linear(L.swiglu(gu[:, :Fs], gu[:, Fs:], *c.glu).to(h.dtype), w["s_down"]).float()
         out = out + (sg * sh if sg is not None else sh)
     return out.to(h.dtype)
 
@@ -388,18 +399,43 @@ def ngram_embed(model, X, plan, w):
 
 # ----------------------------------------------------------------------------- residual updates of models with layer specs
 class RowNorm:
-    """RMS norm (weight w or 1 + w), or with a bias vector a layer norm."""
+    """RMS norm (weight w or 1 + w) over each of `groups` equal parts of the row, or with a bias vector a layer norm."""
 
-    def __init__(self, w, eps: float, b=None, one_plus: bool = False):
-        self.w, self.eps, self.b, self.one_plus = w, eps, b, one_plus
+    def __init__(self, w, eps: float, b=None, one_plus: bool = False, groups: int = 1):
+        assert b is None or groups == 1
+        self.w, self.eps, self.b, self.one_plus, self.groups = w, eps, b, one_plus, groups
 
     def plain(self, x):
+        if self.groups > 1:
+            y = L.rms(x.view(*x.shape[:-1], self.groups, -1), None, self.eps).view(x.shape)
+            return y * (1 + self.w if self.one_plus else self.w)
         return L.rms(x, self.w.float(), self.eps, self.one_plus) if self.b is None else L.layer_norm(x, self.w, self.b, self.eps)
+
+
+class DepthAverage:
+    """Result number `k` of the layers: it is put into `stack` [results + 1, R, H] (0: the embedding), and the sum of a[j] * stack[j]
+    over j <= k goes on in its place."""
+
+    def __init__(self, stack, k: int, a):
+        self.stack, self.k, self.a = stack, k, a
+
+    def plain(self, x):
+        self.stack[self.k] = x
+        return torch.einsum("j,jrh->rh", self.a, self.stack[: self.k + 1])
+
+
+class RowContext:
+    """What a row update needs to know of its pass: the plan (an input convolution looks at the sequence's earlier rows), whether
+    states advance, and whether the residual must be left as it is (`fresh`: the new one is another tensor)."""
+
+    def __init__(self, plan, commit: bool = True, fresh: bool = False):
+        self.plan, self.commit, self.fresh = plan, commit, fresh
 
 
 class Update:
     """A block output on its way into the residual stream: `x` (a tensor, or a deferred MoE output), times the per-channel
-    `scale`, or RMS-normed by `post` (a RowNorm) first."""
+    `scale`, or RMS-normed by `post` (a RowNorm) first; `depth`: a DepthAverage of the sum."""
+    depth: Optional[DepthAverage] = None
 
     def __init__(self, x, scale=None, post: Optional[RowNorm] = None):
         self.x, self.scale, self.post = x, scale, post
@@ -411,15 +447,35 @@ class Update:
         return x * self.scale if self.scale is not None else x
 
 
-def add_norm_rows(delta, res, norm: Optional[RowNorm], dtype, want_f32: bool = False):
+def add_norm_rows(delta, res, norm: Optional[RowNorm], dtype, want_f32: bool = False, conv=None, ctx: Optional[RowContext] = None):
     """res' = res + delta (None, a tensor or an Update); returns (h = norm(res') in `dtype` (norm None: res' itself), res',
-    fp32 h if asked)."""
+    fp32 h if asked).  `conv` (an InputConv): h + conv(h) over the sequences of `ctx.plan` instead of h."""
     if use_kernels(res):
-        return block_ops().add_norm_rows(delta, res, norm, dtype, want_f32)
+        return block_ops().add_norm_rows(delta, res, norm, dtype, want_f32, conv, ctx)
     if delta is not None:
         res = res + (delta.plain() if isinstance(delta, Update) else delta)
+        if isinstance(delta, Update) and delta.depth is not None:
+            res = delta.depth.plain(res)
     h = res.float() if norm is None else norm.plain(res.float())
+    if conv is not None:
+        rows, h = h, h.clone()
+        for s in ctx.plan.segs:
+            y = rows[s.r0: s.r0 + s.n]
+            h[s.r0: s.r0 + s.n] += L.causal_conv(y, conv.w.t(), tail=conv.tail[s.slot])
+        if ctx.commit:
+            advance_tail(conv.tail, rows, ctx.plan, None)
+        conv.keep(rows, ctx.plan, ctx.commit)
     return h.to(dtype), res, h
+
+
+def advance_tail(tail, rows, plan, n_rows):
+    """The last rows of every segment's sequence behind n_rows[i] more rows (None: all of segment i's): `tail` [slots, kept, H]."""
+    if use_kernels(tail):
+        return block_ops().advance_tail(tail, rows, plan, n_rows)
+    kept = tail.shape[1]
+    for i, s in enumerate(plan.segs):
+        n = s.n if n_rows is None else int(n_rows[i])
+        tail[s.slot] = torch.cat((tail[s.slot], rows[s.r0: s.r0 + n]))[n: n + kept]
 
 
 def relu2(x):

@@ -25,12 +25,12 @@ vp, i32, i64, f32 = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _SIGS = {
     "spark_gemm_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "spark_gemm_bf16_swiglu": [vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp],
-    "spark_gemm_grouped_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, i32, f32, i32, vp, vp, vp, vp],
+    "spark_gemm_grouped_bf16": [vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, i32, vp, i32, vp, vp, vp, vp],
     "spark_gemm_bf16_act": [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp],
     "spark_gemm_simt": [vp, i32, i64, vp, i32, i64, vp, i32, i64, i32, i32, i32, i32, i32, i32, vp, vp],
     "spark_gemm_simt_grouped": [vp, i32, vp, i32, i64, vp, i32, i32, i32, vp, vp, i32, vp, i32, i32, i32, vp, vp],
-    "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, f32, i32, vp, vp, vp],
-    "spark_gemv_bf16_items": [vp, i32, i64, vp, i64, i32, vp, i32, i64, i32, i32, i32, i32, vp, i32, vp],
+    "spark_gemv_bf16": [vp, i32, vp, i64, i32, vp, i32, i32, i32, i32, i32, vp, vp, i32, vp, i32, vp, vp, vp],
+    "spark_gemv_bf16_items": [vp, i32, i64, vp, i64, i32, vp, i32, i64, i32, i32, i32, i32, vp, i32, vp, vp],
     "spark_add_rmsnorm": [vp, i32, vp, vp, vp, i32, i32, f32, i32, vp],
     "spark_rmsnorm_bf16": [vp, vp, vp, i32, i32, f32, i32, vp],
     "spark_embed": [vp, vp, vp, i32, i32, vp, i32, vp],
@@ -50,7 +50,7 @@ _SIGS = {
     "spark_draft_path": [vp, vp, vp, vp, i32, i32, i32, vp, vp, vp, vp, vp],
     "spark_add": [vp, i32, vp, C.c_long, vp],
     "spark_f32_to_bf16": [vp, vp, C.c_long, vp],
-    "spark_gather_rows_bf16": [vp, vp, vp, i32, i32, vp],
+    "spark_gather_rows_bf16": [vp, vp, vp, i32, i32, vp, i32],
     "spark_gdn_seq": [vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, f32, i32, vp, vp, i32, i32],
     "spark_mla_prep": [vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp,
                        vp, vp, vp, i32],
@@ -82,12 +82,12 @@ _SIGS = {
 # parallel blocks (ops/parallel_block.py)
 _LIN = [vp, i32, vp, i32, vp, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32]
 _SIGS.update({
-    "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, i32, vp, vp],
+    "spark_embed_scaled": [vp, vp, vp, i32, i32, i32, f32, vp, vp, i32, vp, vp],
     "spark_row_update": [vp, i32, i32, vp],
     "spark_token_shift": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, vp],
     "spark_channel_decay": [vp, i32, vp, i32, i32, vp, vp, i32, i32, i32, vp],
     "spark_log_sigmoid_decay": [vp, i32, vp, i32, i32, vp, f32, vp, i32, i32, i32, vp],
-    "spark_swiglu_rows": [vp, i32, i32, vp, vp, vp, i32, i32, i32, vp],
+    "spark_swiglu_rows": [vp, i32, i32, vp, vp, vp, i32, i32, vp, i32, vp],
     "spark_head_prep": [vp, i32, vp],
     "spark_neg_exp_bias": [vp, vp, i32, i32, vp],
     "spark_tanh_split": [vp, i32, vp, i32, i32, vp],
@@ -99,9 +99,11 @@ _SIGS.update({
                           i32, vp, vp],
     "spark_latent_qrope": [vp, i32, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp, i32, i32, vp],
     "spark_latent_gather": [vp, i32, vp, i32, i32, vp, i32, vp, vp],
-    "spark_latent_rows": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
-    "spark_latent_prefill": [vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp],
-    "spark_mla_attn_paged": [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp],
+    "spark_latent_rows": [vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp, i32, vp],
+    "spark_latent_prefill": [vp, i32, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, i32, vp, vp, i32, vp],
+    "spark_mla_attn_paged": [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, vp, vp],
+    "spark_row_tiles": [vp, i32, i32, i32, i32, vp],
+    "spark_tail_advance": [vp, vp, vp, i32, vp, i32, i32, vp],
     "spark_conv_prep": [vp, i32, i32, i32, vp],
     "spark_paged_rows": [vp, i32, i32, vp],
     "spark_paged_decode": [vp, i32, vp],
@@ -111,16 +113,28 @@ _SIGS.update({
 
 class OutAct(C.Structure):
     """Activation on a product's accumulators (csrc/common/out_act.cuh)."""
-    _fields_ = [(n, i32) for n in ("kind", "ld", "off", "n", "rows", "f32")] + [("table", vp), ("ids", vp)]
+    _fields_ = [(n, i32) for n in ("kind", "ld", "off", "n", "rows", "f32")] + [("table", vp), ("ids", vp), ("batch_cols", i32)]
 
 
-def out_act(kind: str, table=None, ids32=None, off: int = 0, n: int = 0) -> OutAct:
-    """"relu2": squared relu.  "token_gate": gelu_tanh(v) * table[ids, off + column] (columns from n on: 0)."""
+def out_act(kind: str, table=None, ids32=None, off: int = 0, n: int = 0, batch_cols: int = 0) -> OutAct:
+    """"relu2": squared relu.  "token_gate": gelu_tanh(v) * table[ids, off + column] (columns from n on: 0).  "gate":
+    v * sigmoid(table[ids or row, item * batch_cols + column])."""
     if kind == "relu2":
         return OutAct(kind=1)
-    a = OutAct(2, table.stride(0), off, n, table.shape[0], int(table.dtype == torch.float32), P(table), P(ids32))
+    a = OutAct(2 if kind == "token_gate" else 3, table.stride(0), off, n, table.shape[0], int(table.dtype == torch.float32), P(table), P(ids32),
+               batch_cols)
     a.keep = (table, ids32)                      # alive until the launch
     return a
+
+
+class GluAct(C.Structure):
+    """Gated activation (csrc/common/out_act.cuh): g sigmoid(alpha g) (u + shift), g and u limited first if limit > 0."""
+    _fields_ = [("limit", f32), ("alpha", f32), ("shift", f32)]
+
+
+def _glu(g):
+    """`g`: a limit, or (limit, alpha, shift)."""
+    return C.byref(GluAct(*g) if isinstance(g, tuple) else GluAct(float(g), 1.0, 0.0))
 
 
 def _act(a):
@@ -295,7 +309,7 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out_f32: bool = False, fmt: int 
 
 def gemv_bf16(x, w, items=1, rows_per_item=None, pair_expert=None, pair_row=None, act=0, limit=0.0, out_f32=False,
               expert_stride=0, n=None, k=None, out=None, ldx=None, oact=None, x_weight=None):
-    """`x_weight` (act 1): fp32 weight per item, multiplied into gate and up."""
+    """`x_weight` (act 1): fp32 weight per item, multiplied into gate and up; `limit` (act 1): see `_glu`."""
     rows_per_item = rows_per_item if rows_per_item is not None else x.shape[0]
     n = n if n is not None else w.shape[-2]
     k = k if k is not None else w.shape[-1]
@@ -309,20 +323,20 @@ def gemv_bf16(x, w, items=1, rows_per_item=None, pair_expert=None, pair_row=None
         dbg.check_index("gemv_bf16 pair_expert", pair_expert, 0, w.shape[0] if w.dim() == 3 else 1, allow=-1, count=items)
         dbg.check_index("gemv_bf16 pair_row", pair_row, 0, x.shape[0], count=items)
     rc = lib().spark_gemv_bf16(P(x), ldx if ldx is not None else x.stride(0), P(w), expert_stride, w.stride(-2), P(y), ldy,
-                               items, rows_per_item, n, k, P(pair_expert), P(pair_row), act, float(limit), int(out_f32),
+                               items, rows_per_item, n, k, P(pair_expert), P(pair_row), act, _glu(limit), int(out_f32),
                                _act(oact), stream(), P(x_weight))
     check(rc, "spark_gemv_bf16")
     return y
 
 
 def gemv_bf16_items(x, ldx, x_item_stride, w, expert_stride, ldw, y, ldy, y_item_stride, items, rows_per_item, n, k,
-                    pair_expert):
+                    pair_expert, oact=None):
     """Per-item GEMV over strided slices: item i multiplies rows x[i * x_item_stride + r * ldx] (r < rows_per_item) by
     matrix pair_expert[i] of `w` and writes y[i * y_item_stride + r * ldy].  Strides in elements."""
     if dbg.CHECK:
         dbg.check_index("gemv_bf16_items pair_expert", pair_expert, 0, w.shape[0], count=items)
     rc = lib().spark_gemv_bf16_items(P(x), ldx, x_item_stride, P(w), expert_stride, ldw, P(y), ldy, y_item_stride, items,
-                                     rows_per_item, n, k, P(pair_expert), int(y.dtype == torch.float32), stream())
+                                     rows_per_item, n, k, P(pair_expert), int(y.dtype == torch.float32), _act(oact), stream())
     check(rc, "spark_gemv_bf16_items")
     return y
 
@@ -720,15 +734,16 @@ def draft_path(unary, ids, eu, ev):
 
 
 def gather_rows(src, idx32):
+    """Rows idx32 of `src` (rows may be slices of wider ones; 16-byte aligned)."""
     R, H = idx32.shape[0], src.shape[1]
     dbg.check_index("gather_rows indices", idx32, 0, src.shape[0])
     out = torch.empty(R, H, dtype=torch.bfloat16, device=src.device)
-    lib().spark_gather_rows_bf16(P(src), P(idx32), P(out), R, H, stream())
+    lib().spark_gather_rows_bf16(P(src), P(idx32), P(out), R, H, stream(), src.stride(0))
     return out
 
 
 # ----------------------------------------------------------------------------- MoE
-ROUTER_KIND = {"softmax": 0, "sigmoid_bias": 1, "sqrt_softplus": 2, "softmax_bias": 3, "sigmoid": 4}
+ROUTER_KIND = {"softmax": 0, "sigmoid_bias": 1, "sqrt_softplus": 2, "softmax_bias": 3, "sigmoid": 4, "topk_softmax": 5}
 
 
 def moe_route(h, w, c, e_lo=0, e_hi=None, self_w=None):
@@ -776,12 +791,12 @@ def moe_sort(ids, E):
 
 
 def grouped_gemm(a, b, tiles, ntile, max_tiles, n_experts, rows_per_expert, N, mode, limit=0.0, fmt=1, wts=None, perm=None):
-    """a [P, K] rows in expert order; b [E*rows_per_expert, K]; mode 0 -> fp32 [P, N]; 1 -> swiglu bf16 [P, N]; 2 -> squared relu
-    bf16 [P, N].  `wts` (mode 1): row i of `a` counts wts[perm[i]] times."""
+    """a [P, K] rows in expert order; b [E*rows_per_expert, K]; mode 0 -> fp32 [P, N]; 1 -> gated bf16 [P, N] (`limit`: see `_glu`);
+    2 -> squared relu bf16 [P, N].  `wts` (mode 1): row i of `a` counts wts[perm[i]] times."""
     Pn, K = a.shape
     out = torch.empty(Pn, N, dtype=torch.float32 if mode == 0 else torch.bfloat16, device=a.device)
     rc = lib().spark_gemm_grouped_bf16(P(a), P(b), P(out), Pn, N, K, a.stride(0), K, N, n_experts, rows_per_expert,
-                                       P(tiles), P(ntile), max_tiles, mode, float(limit), fmt, P(status_word(a.device)),
+                                       P(tiles), P(ntile), max_tiles, mode, _glu(limit), fmt, P(status_word(a.device)),
                                        stream(), P(wts), P(perm))
     check(rc, "spark_gemm_grouped_bf16")
     return out
@@ -868,7 +883,7 @@ def moe(h, w, c, defer: bool = False):
     outputs of a decode round).  Under expert parallelism (`w["ep"]` = (first local expert, end)) only the local
     experts' pairs are computed and the result is this rank's partial sum; the shared expert is added by the rank
     that holds it."""
-    if c.act == "relu2" or c.weight_input:
+    if not c.plain:
         from .moe_spec import moe as moe_spec
         return moe_spec(h, w, c, defer)
     if h.shape[0] * c.top_k <= DECODE_PAIRS_MAX and h.shape[0] <= DECODE_ROWS_MAX and FUSED_DECODE:

@@ -1,6 +1,6 @@
 """Routed feed-forwards of models whose layers carry their own sizes (dense bf16 weights, or fp32 in the 32-bit mode): experts with
-one up matrix and a squared relu, or SwiGLU experts whose input is multiplied by the routing weight; identity experts, a shared
-expert with or without a gate.  Routing, sorting and the products are the engine's MoE kernels: decode rows take the fused router
+one up matrix and a squared relu, or gated experts (SwiGLU, or with a limit, a slope of the sigmoid and a shift of the up half) whose
+input or output is multiplied by the routing weight; identity experts, a shared expert with or without a gate.  Routing, sorting and the products are the engine's MoE kernels: decode rows take the fused router
 and one GEMV item per (row, expert) pair, prompts the grouped tcgen05 GEMM over the sorted pairs, the 32-bit mode (and widths
 that are no multiple of 8) the grouped FP32-unit product.  Activation and input weight are part of the products (the experts
 have no biases, so weighting the input is weighting gate and up); the combine (slot order, identity weight times the input row,
@@ -34,10 +34,10 @@ def _route(h, w, c, self_w):
     return wts, ids, prow, sg
 
 
-def _shared(h, w, relu2):
-    if relu2:
+def _shared(h, w, c):
+    if c.act == "relu2":
         return cu.dense_linear(cu.dense_linear(h, w["s_up"], act=cu.out_act("relu2")), w["s_down"], out_f32=True)
-    return cu.dense_linear(linear_swiglu(h, w["s_gu"]), w["s_down"], out_f32=True)
+    return cu.dense_linear(linear_swiglu(h, w["s_gu"], c.glu), w["s_down"], out_f32=True)
 
 
 def _grouped_simt(h, w, c, wts, perm, tiles, ntile, max_tiles):
@@ -53,7 +53,7 @@ def _grouped_simt(h, w, c, wts, perm, tiles, ntile, max_tiles):
     check(lib().spark_gemm_simt_grouped(P(h), H, P(wu), H, Nu * H, P(act), Nu, Nu, H, P(tiles), P(ntile), max_tiles, P(perm), c.top_k,
                                         f32, f32, cu._act(oact), stream()), "spark_gemm_simt_grouped")
     if not relu2:
-        act = swiglu_rows(act, wts, perm)
+        act = swiglu_rows(act, wts, perm, c.glu)
     check(lib().spark_gemm_simt_grouped(P(act), Fp, P(wd), Fp, H * Fp, P(y), H, H, Fp, P(tiles), P(ntile), max_tiles, None, 1, f32, 1, None,
                                         stream()), "spark_gemm_simt_grouped")
     return y
@@ -80,14 +80,14 @@ def moe(h, w, c, defer: bool = False):
         if side is not None:
             side.wait_stream(main)
         with torch.cuda.stream(side if side is not None else main):
-            shared = _shared(h, w, relu2)
+            shared = _shared(h, w, c)
     wts, ids, prow, sg = _route(h, w, c, self_w)
     inv, xw = None, wts if c.weight_input else None
     if pairs:
         n, pe = R * c.top_k, ids.view(-1)
         a = cu.gemv_bf16(h, wu, items=n, rows_per_item=1, pair_expert=pe, pair_row=prow.view(-1), expert_stride=Nu * H, n=Nu, k=H,
                          oact=cu.out_act("relu2") if relu2 else None)
-        y = cu.gemv_bf16(a, wd, items=n, rows_per_item=1, pair_expert=pe, act=0 if relu2 else 1, out_f32=True, expert_stride=H * Fp, n=H,
+        y = cu.gemv_bf16(a, wd, items=n, rows_per_item=1, pair_expert=pe, act=0 if relu2 else 1, limit=c.glu, out_f32=True, expert_stride=H * Fp, n=H,
                          k=Fp, x_weight=xw)
     else:
         perm, inv, _, tiles, ntile, max_tiles = cu.moe_sort(ids.view(-1), E)
@@ -95,7 +95,7 @@ def moe(h, w, c, defer: bool = False):
             y = _grouped_simt(h, w, c, xw, perm, tiles, ntile, max_tiles)
         else:
             a = cu.gather_rows(h, torch.div(perm, c.top_k, rounding_mode="floor").to(torch.int32))
-            a = cu.grouped_gemm(a, wu.view(E * Nu, H), tiles, ntile, max_tiles, E, Nu, Fp, 2 if relu2 else 1, wts=xw, perm=perm)
+            a = cu.grouped_gemm(a, wu.view(E * Nu, H), tiles, ntile, max_tiles, E, Nu, Fp, 2 if relu2 else 1, c.glu, wts=xw, perm=perm)
             y = cu.grouped_gemm(a, wd.view(E * H, Fp), tiles, ntile, max_tiles, E, H, H, 0)
     if side is not None:
         torch.cuda.current_stream().wait_stream(side)

@@ -1,5 +1,6 @@
-"""CUDA implementations of the parallel-block ops (`csrc/kernels/block_rows.cu`, `linear_state.cu`, `latent.cu`, `mla.cu`):
-row ops around the block, the two decayed linear recurrences, latent attention over a paged cache.  bf16 and fp32
+"""CUDA implementations of the ops of models whose layers carry their own sizes (`csrc/kernels/block_rows.cu`, `row_tiles.cu`,
+`linear_state.cu`, `latent.cu`, `mla.cu`): row ops around the block, the decayed linear recurrences, latent attention over a paged
+cache.  bf16 and fp32
 activations; what the mechanisms keep in fp32 (residual, norms, states, decays, scores, softmax weights) is fp32 in both."""
 from __future__ import annotations
 
@@ -19,11 +20,13 @@ def _is32(dtype) -> int:
 
 
 # ----------------------------------------------------------------------------- rows
-def embed_scaled(table, ids32, scale: float):
+def embed_scaled(table, ids32, scale: float, pos=None, out=None):
     R, H = ids32.shape[0], table.shape[1]
     cu.dbg.check_index("embed token ids", ids32, 0, table.shape[0])
-    out = torch.empty(R, H, dtype=torch.float32, device=table.device)
-    check(lib().spark_embed_scaled(P(table), P(ids32), P(out), R, H, table.shape[0], float(scale), _is32(table.dtype),
+    if out is None:
+        out = torch.empty(R, H, dtype=torch.float32, device=table.device)
+    p32, freq = (pos[0].to(torch.int32), pos[1]) if pos is not None else (None, None)
+    check(lib().spark_embed_scaled(P(table), P(ids32), P(out), R, H, table.shape[0], float(scale), P(p32), P(freq), _is32(table.dtype),
                                    P(status_word(table.device)), stream()), "spark_embed_scaled")
     return out
 
@@ -35,11 +38,23 @@ class RowUpdate(C.Structure):
         + [(n, C.c_int) for n in ("H", "slots", "norm", "one_plus")] + [("eps", C.c_float), ("post_eps", C.c_float)]
 
 
-def add_norm_rows(delta, res, norm, dtype, want_f32=False):
-    """res (fp32, in place) += delta (None, a tensor, a deferred MoE output, or an ops.Update of one); returns (h in `dtype`, res,
-    fp32 copy of h or None)."""
+class RowTiles(C.Structure):
+    """Arguments of the row update over tiles of a sequence (csrc/kernels/row_tiles.cu)."""
+    _fields_ = [("u", RowUpdate)] + [(n, C.c_void_p) for n in ("res_out", "stack", "avg", "conv_w", "tail", "rows", "segs")] \
+        + [(n, C.c_int) for n in ("k", "groups", "taps", "tile", "commit", "R")]
+
+
+def add_norm_rows(delta, res, norm, dtype, want_f32=False, conv=None, ctx=None):
+    """res (fp32) += delta (None, a tensor, a deferred MoE output, or an ops.Update of one), in place unless `ctx` says otherwise;
+    returns (h in `dtype`, res, fp32 copy of h or None).  Grouped norms, depth averages and input convolutions (`conv`) run in the
+    tiled form, which leaves the old residual as it is."""
     R, H = res.shape
     assert res.dtype == torch.float32 and res.is_contiguous()
+    depth = getattr(delta, "depth", None)
+    tiled = conv is not None or depth is not None or (ctx is not None and ctx.fresh) or (norm is not None and norm.groups > 1)
+    if tiled and getattr(delta, "post", None) is not None:      # (the tiled form does not norm updates)
+        assert depth is None
+        res, delta = add_norm_rows(delta, res.clone(), None, dtype)[1], None
     u = RowUpdate(res=P(res), H=H)
     keep = []
     x = delta
@@ -61,8 +76,48 @@ def add_norm_rows(delta, res, norm, dtype, want_f32=False):
     u.out, u.out32 = P(h), P(h32) if h32 is not h else None
     if norm is not None:
         u.norm, u.w, u.b, u.eps, u.one_plus = (1 if norm.b is None else 2), P(norm.w), P(norm.b), norm.eps, int(norm.one_plus)
+    if tiled:
+        if x is not None or depth is not None:
+            new = torch.empty_like(res)
+            _row_tiles(u, R, new, norm, depth, conv, ctx, _is32(dtype))
+            res = new
+        else:
+            _row_tiles(u, R, None, norm, None, conv, ctx, _is32(dtype))
+        return h, res, h32
     check(lib().spark_row_update(C.byref(u), R, _is32(dtype), stream()), "spark_row_update")
     return h, res, h32
+
+
+TILE_THREADS = 1024          # threads of a CTA at most
+TILE_CTAS = 592              # CTAs a launch aims at: rows per tile grow beyond
+
+
+def _row_tiles(u, R, new, norm, depth, conv, ctx, f32):
+    a = RowTiles(u=u, res_out=P(new), groups=norm.groups if norm is not None else 1, R=R, tile=max(1, -(-R // TILE_CTAS)), commit=1)
+    nseg, longest = 1, R
+    if depth is not None:
+        assert depth.stack.is_contiguous() and depth.stack.shape[1] == R and depth.stack.dtype == torch.float32
+        a.stack, a.avg, a.k = P(depth.stack), P(depth.a), depth.k
+    if conv is not None:
+        plan = ctx.plan
+        d = cu._plan_dev(plan, conv.tail.device)
+        if cu.dbg.CHECK:
+            cu._check_slots("row_tiles", plan, conv.tail.shape[0])
+        nseg, longest = len(plan.segs), max(s.n for s in plan.segs)
+        a.conv_w, a.tail, a.segs, a.taps, a.commit = P(conv.w), P(conv.tail), P(d["seg"]), conv.taps, int(ctx.commit)
+        a.tile = max(a.tile, conv.taps - 1)
+        rows = None
+        if not ctx.commit:
+            rows = torch.empty(R, u.H, dtype=torch.float32, device=conv.tail.device)
+            a.rows = P(rows)
+        conv.keep(rows, plan, ctx.commit)
+    check(lib().spark_row_tiles(C.byref(a), nseg, longest, TILE_THREADS, f32, stream()), "spark_row_tiles")
+
+
+def advance_tail(tail, rows, plan, n_rows):
+    d = cu._plan_dev(plan, tail.device)
+    check(lib().spark_tail_advance(P(tail), P(rows), P(d["seg"]), len(plan.segs), P(n_rows), tail.shape[1], tail.shape[2], stream()),
+          "spark_tail_advance")
 
 
 def token_shift(h32, carried, mu, plan, dtype):
@@ -100,22 +155,24 @@ def log_sigmoid_decay(z, w2, b, n: int, tau: float):
     return out
 
 
-def swiglu_rows(gu, wts=None, perm=None):
-    """silu(gate) * up of [gate | up] rows; `wts` (fp32): gate and up of row r count wts[perm[r]] times."""
+def swiglu_rows(gu, wts=None, perm=None, glu=0.0):
+    """silu(gate) * up of [gate | up] rows (`glu`: see `cuda._glu`); `wts` (fp32): gate and up of row r count wts[perm[r]] times."""
     R, n = gu.shape[0], gu.shape[1] // 2
     out = torch.empty(R, n, dtype=gu.dtype, device=gu.device)
-    check(lib().spark_swiglu_rows(P(gu), gu.stride(0), n, P(wts), P(perm), P(out), n, R, _is32(gu.dtype), stream()), "spark_swiglu_rows")
+    check(lib().spark_swiglu_rows(P(gu), gu.stride(0), n, P(wts), P(perm), P(out), n, R, cu._glu(glu), _is32(gu.dtype), stream()),
+          "spark_swiglu_rows")
     return out
 
 
-def linear_swiglu(x, w):
-    """silu(x G^T) * (x U^T) for w = [G | U] (halves of a multiple of 128 rows)."""
+def linear_swiglu(x, w, glu=0.0):
+    """silu(x G^T) * (x U^T) for w = [G | U] (halves of a multiple of 128 rows); `glu`: see `cuda._glu`."""
     R, F = x.shape[0], w.shape[0] // 2
-    if w.dtype != torch.bfloat16 or R <= 16 or w.shape[1] % 8 or F % 128:
-        return swiglu_rows(cu.dense_linear(x, w))
+    if w.dtype != torch.bfloat16 or R <= 16 or w.shape[1] % 8 or F % 128 or (isinstance(glu, tuple) and glu[1:] != (1.0, 0.0)):
+        return swiglu_rows(cu.dense_linear(x, w), glu=glu)
     x = cu._as_bf16(x).contiguous()
     out = torch.empty(R, F, dtype=torch.bfloat16, device=x.device)
-    check(lib().spark_gemm_bf16_swiglu(P(x), P(w), P(out), R, F, w.shape[1], x.stride(0), w.stride(0), F, 0.0, P(status_word(x.device)),
+    check(lib().spark_gemm_bf16_swiglu(P(x), P(w), P(out), R, F, w.shape[1], x.stride(0), w.stride(0), F,
+                                       float(glu[0] if isinstance(glu, tuple) else glu), P(status_word(x.device)),
                                        stream()), "spark_gemm_bf16_swiglu")
     return out
 
@@ -262,14 +319,20 @@ def _max_ctx(plan, d):
     return d["max_ctx"]
 
 
-def _heads_product(x, ldx, xh, w, y, ldy, yh, R):
-    """y[r, h] = x[r, h] w[h]^T over heads: x at r * ldx + h * xh, w [H, N, K], y at r * ldy + h * yh."""
+def _heads_product(x, ldx, xh, w, y, ldy, yh, R, gate=None, rows=None):
+    """y[r, h] = x[r, h] w[h]^T over heads: x at r * ldx + h * xh, w [H, N, K], y at r * ldy + h * yh.  `gate` [plan rows, H * N]:
+    outputs times its sigmoid (row r's gate is row rows[r], or r)."""
     H, N, K = w.shape
+
+    def act(r):
+        if gate is None:
+            return None
+        return cu.out_act("gate", gate[r:] if rows is None else gate, rows[r:] if rows is not None else None, batch_cols=N)
     if w.dtype == torch.float32 or R > 64 or K % 8 or xh % 8 or ldx % 8 or x.data_ptr() % 16:
-        return cu.gemm_simt(x, ldx, xh, w, K, N * K, y, ldy, yh, H, R, N, K)
+        return cu.gemm_simt(x, ldx, xh, w, K, N * K, y, ldy, yh, H, R, N, K, act(0))
     step = min(16, cu.gemv_rows(K))
     for r in range(0, R, step):                         # every head's matrix is streamed once per 16 rows
-        cu.gemv_bf16_items(x[r:], ldx, xh, w, N * K, K, y[r:], ldy, yh, H, min(step, R - r), N, K, _iota(H, x.device))
+        cu.gemv_bf16_items(x[r:], ldx, xh, w, N * K, K, y[r:], ldy, yh, H, min(step, R - r), N, K, _iota(H, x.device), act(r))
     return y
 
 
@@ -283,21 +346,23 @@ def latent_mixer(mx, proj, plan, cat):
     is32 = _is32(dt)
     if not hasattr(mx, "_inv"):
         mx._inv = (c.rope_theta ** (-torch.arange(c.rope_dim // 2, dtype=torch.float64) * 2 / c.rope_dim)).to(dev)
-    cq = torch.empty(R, w["uq"].shape[1], dtype=dt, device=dev)
-    check(lib().spark_latent_prep(P(proj), proj.stride(0), mx.off["dq"], mx.off["lat"], mx.off["rot"], R, c.q_rank, cq.shape[1], c.kv_rank,
-                                  Lp, c.rope_dim, Rp, int(c.rope_interleaved), float(mx.eps), P(w["dq_norm"]), P(w["kv_norm"]), P(mx._inv),
-                                  P(d["pos32"]), P(d["row_slot"]), P(pages), pld, P(cq), P(mx.lat), is32, P(status_word(dev)), stream()),
-          "spark_latent_prep")
-    q = cu.dense_linear(cq, w["uq"])                      # [R, H * (Dp + Rp)]
+    cq = torch.empty(R, w["uq"].shape[1], dtype=dt, device=dev) if c.q_rank else None
+    check(lib().spark_latent_prep(P(proj), proj.stride(0), mx.off["dq"], mx.off["lat"], mx.off["rot"], R, c.q_rank, cq.shape[1] if c.q_rank else 0,
+                                  c.kv_rank, Lp, c.rope_dim, Rp, int(c.rope_interleaved), float(mx.eps), P(w.get("dq_norm")), P(w["kv_norm"]),
+                                  P(mx._inv), P(d["pos32"]), P(d["row_slot"]), P(pages), pld, P(cq), P(mx.lat), is32, P(status_word(dev)),
+                                  stream()), "spark_latent_prep")
+    q = cu.dense_linear(cq, w["uq"]) if c.q_rank else proj[:, : mx.nq]       # [R, H * (Dp + Rp)]
     gate = proj[:, mx.off["g"]:]
+    each = gate if c.gate == "element" else None
+    sink = w["sink"] if c.sink else None
     rows, ns, tab, longs, ctx = (None, R, None, [], 0) if is32 else _short_long(plan, dev)
     if longs and not mx.prefill_ok:
         rows, ns, longs = None, R, []
     if ns:
         qs = q if rows is None else cu.gather_rows(q, rows)
-        o = _latent_absorbed(mx, qs, rows, ns, gate, d, plan, is32)
+        o = _latent_absorbed(mx, qs, rows, ns, gate if each is None else None, sink, d, plan, is32)
         dst = cat if rows is None else torch.empty(ns, H * V, dtype=dt, device=dev)
-        _heads_product(o, H * Lp, Lp, w["uv"], dst, dst.stride(0), V, ns)
+        _heads_product(o, H * Lp, Lp, w["uv"], dst, dst.stride(0), V, ns, each, rows)
         if rows is not None:
             cat[:, : H * V].index_copy_(0, rows.long(), dst)
     if longs:
@@ -309,13 +374,14 @@ def latent_mixer(mx, proj, plan, cat):
         check(lib().spark_latent_qrope(P(qr), q.stride(0), Dp + Rp, P(qr), q.stride(0), Dp + Rp, R, H, c.rope_dim, Rp,
                                        int(c.rope_interleaved), P(mx._inv), P(d["pos32"]), None, 0, 0, stream()), "spark_latent_qrope")
         check(lib().spark_latent_prefill(P(q), q.stride(0), P(kv), kv.stride(0), P(lat), KW, P(tab), len(longs), max(s.n for s in longs),
-                                         H, Dp, Rp, V, Vp, Lp, float(c.scale), P(gate), proj.stride(0), P(cat), cat.stride(0), stream()),
-              "spark_latent_prefill")
+                                         H, Dp, Rp, V, Vp, Lp, float(c.scale), P(gate), proj.stride(0), int(each is not None), P(sink), P(cat),
+                                         cat.stride(0), stream()), "spark_latent_prefill")
     return cat
 
 
-def _latent_absorbed(mx, q, rows, n, gate, d, plan, is32):
-    """Absorbed attention rows [n, H, Lp] (gated): q [n, H * (Dp + Rp)] before rotation."""
+def _latent_absorbed(mx, q, rows, n, gate, sink, d, plan, is32):
+    """Absorbed attention rows [n, H, Lp] (gated per head if `gate`): q [n, H * (Dp + Rp)] before rotation."""
+    ldg = gate.stride(0) if gate is not None else 0
     c, w, dev = mx.c, mx.w, q.device
     H, Dp, Rp, Lp = c.n_heads, mx.Dp, mx.Rp, mx.Lp
     KW = Lp + Rp
@@ -328,7 +394,7 @@ def _latent_absorbed(mx, q, rows, n, gate, d, plan, is32):
     o = torch.empty(n, H * Lp, dtype=q.dtype, device=dev)
     if is32 or not mx.decode_tc_ok:
         check(lib().spark_latent_rows(P(qf), P(mx.lat), P(d["pos32"]), P(rows), P(d["row_slot"]), P(pages), pld, n, H, Lp, Rp, float(c.scale),
-                                      P(gate), gate.stride(0), P(o), is32, stream()), "spark_latent_rows")
+                                      P(gate), ldg, P(sink), P(o), is32, stream()), "spark_latent_rows")
         return o
     nsplit = (_max_ctx(plan, d) + 63) // 64
     step = n if n <= 16 else 16                            # bounds the partial results of long contexts
@@ -339,6 +405,6 @@ def _latent_absorbed(mx, q, rows, n, gate, d, plan, is32):
     for r in range(0, n, step):
         m = min(step, n - r)
         check(lib().spark_mla_attn_paged(P(qf[r:]), P(mx.lat), P(d["pos32"]), P(rows[r:]) if rows is not None else None, P(d["row_slot"]),
-                                         P(pages), pld, P(part_o), P(part_ml), nsplit, m, H, Lp, Rp, float(c.scale), P(gate),
-                                         gate.stride(0), P(o[r:]), stream()), "spark_mla_attn_paged")
+                                         P(pages), pld, P(part_o), P(part_ml), nsplit, m, H, Lp, Rp, float(c.scale), P(gate), ldg,
+                                         P(sink), P(o[r:]), stream()), "spark_mla_attn_paged")
     return o

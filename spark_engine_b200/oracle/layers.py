@@ -307,10 +307,11 @@ def route(x, w_gate, top_k: int, kind: str = "softmax", bias: Optional[torch.Ten
     return wts, idx
 
 
-def swiglu(g, u, limit: float = 0.0):
+def swiglu(g, u, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0):
+    """g sigmoid(alpha g) (u + shift), with a limit > 0 on g from above and on u from both sides."""
     if limit > 0:
-        return F.silu(g.clamp(max=limit)) * u.clamp(-limit, limit)
-    return F.silu(g) * u
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return F.silu(g) * u if alpha == 1.0 and shift == 0.0 else g * torch.sigmoid(alpha * g) * (u + shift)
 
 
 def moe_layer(x, w: dict, top_k: int, kind: str = "softmax", scale: float = 1.0, limit: float = 0.0,

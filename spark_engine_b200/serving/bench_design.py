@@ -174,7 +174,7 @@ def vabunex_kernels(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R:
     flops = T * T / 2 * H * (D + Rr + Vd) * 2
     put("latent attention, prefill", "latent attention of the closest model, prefill",
         lambda: lib().spark_latent_prefill(P(q), q.stride(0), P(kv), kv.stride(0), P(lat), L + Rr, P(tab), 1, T, H, D, Rr, Vd, Vd, L, 0.07,
-                                           None, 0, P(dst), H * Vd, stream()), flops=flops)
+                                           None, 0, 0, None, P(dst), H * Vd, stream()), flops=flops)
     for tag, rows, c in (("prefill", 2048, 2048), ("decode", R, ctx)):
         qf, ol = rnd(rows, H, L + Rr).bfloat16(), torch.empty(rows, H, L, dtype=torch.bfloat16, device=DEV)
         cache = rnd(R * c, L + Rr).bfloat16()
@@ -189,7 +189,7 @@ def vabunex_kernels(peaks: dict, T: int = 8192, H: int = 16, ctx: int = 8192, R:
             pages = torch.arange(R * ns, dtype=torch.int32, device=DEV).view(R, ns)
             put("latent attention, decode", "latent attention of the closest model, decode",
                 lambda: lib().spark_mla_attn_paged(P(qf), P(cache), P(pos), None, P(slot), P(pages), ns, P(po), P(pm), ns, rows, H, L, Rr,
-                                                   0.07, None, 0, P(ol), stream()), nb, fl)
+                                                   0.07, None, 0, None, P(ol), stream()), nb, fl)
         put(f"latent attention of the closest model, {tag}", "",
             lambda: lib().spark_mla_attn(P(qf), P(cache), P(pos), P(kvb), None, None, 0, P(po), P(pm), ns, None, rows, H, L, Rr, 0.07, P(ol),
                                          stream(), None, None, None, 0), nb, fl)

@@ -209,7 +209,7 @@ class RoundGraph:
             m._pending_plan = None
             self.graph = g
             if not commit:
-                self.pendings = [(mix, mix.pending) for _, mix, _ in m.layers if getattr(mix, "pending", None) is not None]
+                self.pendings = [(x, x.pending) for x in m.stateful(drafter=False) if getattr(x, "pending", None) is not None]
         self.replay()
         self.out_host.copy_(self.out_ids, non_blocking=True)
 
