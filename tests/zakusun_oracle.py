@@ -2,6 +2,7 @@
 framework: the tests compare the product path against it.
 
 Weights are a flat dict name -> tensor ("l<i>.mix.q", "embed", ...), the configuration is the parsed config.json."""
+import functools
 import math
 
 import torch
@@ -22,6 +23,7 @@ def grouped_rms_norm(x, w, eps, groups):
     return torch.cat([p / torch.sqrt((p * p).mean(-1, keepdim=True) + eps) for p in parts], -1) * w
 
 
+@functools.lru_cache(maxsize=4096)
 def position_vector(p, width):
     v = torch.zeros(width, dtype=torch.float64)
     for i in range((width + 1) // 2):
@@ -41,11 +43,8 @@ def input_convolution(h, w):
     """h + conv(h): every channel's own taps over the last inputs, the last tap on the token itself; w [width, taps]."""
     T, taps = h.shape[0], w.shape[1]
     out = h.clone()
-    for t in range(T):
-        for j in range(taps):
-            s = t - (taps - 1) + j
-            if s >= 0:
-                out[t] = out[t] + w[:, j] * h[s]
+    for back in range(min(taps, T)):                             # the input of `back` tokens before
+        out[back:] += w[:, taps - 1 - back] * h[: T - back]
     return out
 
 
@@ -94,9 +93,9 @@ def routed(h, W, p, top):
 def experts(h, W, p, mlp):
     w, ids = routed(h, W, p, mlp["router"]["top"])
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for a, e in zip(w[t], ids[t].tolist()):
-            out[t] += a * expert(h[t], W, f"{p}e{e}.", mlp["expert"]["limit"])
+    for e in range(mlp["router"]["experts"]):
+        share = (w * (ids == e)).sum(-1, keepdim=True)           # 0 for the tokens that did not choose it
+        out += share * expert(h, W, f"{p}e{e}.", mlp["expert"]["limit"])
     return out
 
 
