@@ -160,7 +160,7 @@ def main():
     ap.add_argument("--spec", default="none", help="mtp: also time speculative rounds (MTP chain of 3 drafts, 4 rows per "
                                                    "sequence verified) through the captured draft / verify / commit graphs")
     ap.add_argument("--sweep", action="store_true", help="also time 1,2,3 streams")
-    ap.add_argument("--design", default="", help="vabunex | debisun | zapolorn: time that architecture at a few layer sizes beside the closest existing "
+    ap.add_argument("--design", default="", help="vabunex | debisun | zapolorn | zakusun: time that architecture at a few layer sizes beside the closest existing "
                                                  "family at equal size, and its kernels beside their like kernels (one GPU; not the "
                                                  "headline workload)")
     ap.add_argument("--parallel", default="tp", help="N > 1: tp = one model sharded over the GPUs (tensor + expert "

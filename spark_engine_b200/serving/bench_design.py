@@ -5,6 +5,7 @@ the measured copy bandwidth / GEMM throughput.
   vabunex   beside KDA linear attention + latent attention in sequential pre-norm blocks with dense feed-forwards
   debisun   beside grouped-query attention (rotary, no chunks) with softmax-routed SwiGLU experts, as many parameters
   zapolorn  beside grouped-query attention (rotary, whole context) with dense and softmax-routed SwiGLU feed-forwards of its sizes
+  zakusun   beside latent attention (low-rank queries, a rotated part) with softmax-routed SwiGLU experts of its sizes
 
 Device-timed with CUDA events.  Model figures stream more weights and activations than L2 holds; kernel figures write a
 buffer larger than L2 between iterations (median of the iterations)."""
@@ -17,7 +18,7 @@ import statistics
 import torch
 
 from ..config import AttnConfig, EngineConfig, KdaConfig, MlaConfig, ModelConfig, MoeConfig, debisun_style, glm_style, vabunex_style, \
-    zapolorn_style
+    zakusun_style, zapolorn_style
 from ..models.build import build_random_model, decode_step_bytes
 from ..models.plan import make_plan
 from ..ops import cuda as cu
@@ -423,6 +424,97 @@ def zapolorn_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) ->
     return fig.done()
 
 
+# ----------------------------------------------------------------------------- zakusun
+ZAK_SIZES = {"1024": (1024, 768), "2048": (2048, 1536), "4096": (4096, 3072)}
+
+
+def zakusun_config(hidden: int, ffn: int):
+    return zakusun_style(12, hidden, ffn, VOCAB, experts=DEB_EXPERTS, top=DEB_TOP)
+
+
+def zakusun_closest(hidden: int, ffn: int, layers: int):
+    """Latent attention in every layer (the same heads, values and latents; low-rank queries, a rotated part of 64), the same experts."""
+    c = closest_config(hidden, ffn, layers)
+    c.name, c.layer_types = "latent attention + swiglu experts, dense weights", ["mla"] * layers
+    c.moe = MoeConfig(n_experts=DEB_EXPERTS, top_k=DEB_TOP, ffn=ffn, n_shared=0, router="softmax")
+    return c
+
+
+def zakusun_kernels(peaks: dict, T: int = 8192, ctx: int = 8192, R: int = 4) -> dict:
+    """Kernels at hidden size 2048 (16 heads of 128, latents of 512, 32 experts of 1536, top 4, two norm groups, four taps).  Like
+    kernels: Vabunex's latent attention (low-rank queries, a rotated part, a gate per head), the closest model's experts and row
+    updates."""
+    import dataclasses
+    from .. import ops
+    from ..models.input_conv import InputConv
+    from ..models.model import Model
+    from ..ops import moe_spec
+    from ..ops import parallel_block as pb
+    fig = Figures(peaks)
+    rnd, put = fig.rnd, fig.put
+    N, H, F, L = 2048, 16, 1536, 512
+    P, lib, stream = pb.P, pb.lib, pb.stream
+    cfg, near = zakusun_config(N, F), zakusun_closest(N, F, 1)
+    cut = lambda c, kind: dataclasses.replace(c, n_layers=1, layer_types=[kind], layer_specs=[x for x in c.layer_specs if x.kind == kind][:1], loop=None)
+    vab = cut(vabunex_config(N, 5632), "latent")
+    vab.layer_specs = [dataclasses.replace(vab.layer_specs[0], ffn=0)]
+    mixers = {}
+    for name, c in (("latent attention with sink and element gate", cut(cfg, "latent")), ("latent attention (Vabunex)", vab)):
+        m = Model(c, build_random_model(c, DEV, seed=0), device=DEV, dtype=torch.bfloat16, n_slots=R, kv_tokens=R * ctx)
+        mixers[name] = m.layers[0][1]
+        mixers[name].lat.copy_(rnd(*mixers[name].lat.shape))
+    ours, like = mixers
+    for tag, rows in (("prefill", T), ("decode", R)):
+        plan = lambda: make_plan([(0, [1] * T, 0)] if tag == "prefill" else [(s, [1], ctx - 1) for s in range(R)], device=DEV)
+        for name, mx in mixers.items():
+            w, proj, p1 = mx.w, rnd(rows, mx.off["ff"]).bfloat16(), plan()
+            cat = torch.empty(rows, H * 128, dtype=torch.bfloat16, device=DEV)
+            up = 2 * 128 * H * L * 2                                            # flops (prompts) / bytes (decode rows) of both up matrices
+            qc = sum(w[k].numel() for k in ("uq",) if k in w) * 2
+            dq = 128 + mx.Rp
+            fl = T * T / 2 * H * (dq + 128) * 2 + T * (up + qc) if tag == "prefill" else R * ctx * H * (2 * L + mx.Rp) * 2 + R * up
+            nb = 0 if tag == "prefill" else R * ctx * (L + mx.Rp) * 2 + up + qc
+            put(f"{name}, whole mixer, {tag}", f"{like}, whole mixer, {tag}" if name == ours else "",
+                lambda mx=mx, proj=proj, p1=p1, cat=cat: pb.latent_mixer(mx, proj, p1, cat), nb + rows * (proj.shape[1] + H * 128) * 2, fl)
+            if tag == "prefill":                                                # the attention kernel alone
+                q, kv, lat = rnd(T, H * dq).bfloat16(), rnd(T, H * 256).bfloat16(), rnd(T, L + mx.Rp).bfloat16()
+                tab = torch.tensor([[0, 0, T, 0, 0]], dtype=torch.int32, device=DEV)
+                gate = proj[:, mx.off["g"]:]
+                put(f"{name}, {tag}", f"{like}, {tag}" if name == ours else "",
+                    lambda mx=mx, q=q, kv=kv, lat=lat, cat=cat, gate=gate: lib().spark_latent_prefill(
+                        P(q), q.stride(0), P(kv), kv.stride(0), P(lat), lat.shape[1], P(tab), 1, T, H, 128, mx.Rp, 128, 128, L, 0.07, P(gate),
+                        gate.stride(0), int(mx.c.gate == "element"), P(mx.w.get("sink")), P(cat), H * 128, stream()),
+                    flops=T * T / 2 * H * (dq + 128) * 2)
+        # residual updates: a plain one, and one behind the sixth layer
+        res, d32, d16, one = rnd(rows, N), rnd(rows, N), rnd(rows, N).bfloat16(), torch.ones(N, device=DEV)
+        cv = InputConv(rnd(4, N), R, DEV)
+        ctx1, rn = ops.RowContext(plan(), True, True), ops.RowNorm(one, 1e-5, groups=2)
+        put(f"update + grouped norm + convolution, {tag}", f"update + RMS norm, {tag}",
+            lambda: ops.add_norm_rows(d32, res, rn, torch.bfloat16, conv=cv, ctx=ctx1), rows * N * 14)
+        up = ops.Update(d32)
+        up.depth = ops.DepthAverage(rnd(7, rows, N), 6, rnd(7))
+        put(f"update + depth average of seven + grouped norm + convolution, {tag}", f"update + RMS norm, {tag}",
+            lambda: ops.add_norm_rows(up, res, rn, torch.bfloat16, conv=cv, ctx=ctx1), rows * N * 42)
+        put(f"update + RMS norm, {tag}", "", lambda: ops.add_rmsnorm(d16, res, one, 1e-5), rows * N * 12)
+        table, ids = rnd(VOCAB, N).bfloat16(), torch.randint(0, VOCAB, (rows,), device=DEV).int()
+        pos, freq = ctx1.plan.dev["pos32"], 1e4 ** (-torch.arange(N // 2, dtype=torch.float64, device=DEV) * 2 / N)
+        put(f"embedding with positions, {tag}", f"embedding, {tag}", lambda: ops.embed(table, ids, torch.bfloat16, 1.0, (pos, freq)), rows * N * 6)
+        put(f"embedding, {tag}", "", lambda: ops.embed(table, ids, torch.bfloat16), rows * N * 6)
+        # routed feed-forwards: every kernel from the router to the combined rows
+        c, c2 = cfg.layer_specs[0].moe, near.moe
+        w1 = {"gate": rnd(c.n_experts, N).bfloat16() * 0.05, "bias": torch.zeros(c.n_experts, device=DEV),
+              "w_gu": (rnd(c.n_experts, 2 * F, N) * 0.02).bfloat16(), "w_down": (rnd(c.n_experts, N, F) * 0.02).bfloat16()}
+        e = moe_spec._route(d16, w1, c, None)[1].unique().numel()
+        nb, fl = e * 3 * F * N * 2 + rows * N * 14, rows * c.top_k * 3 * F * N * 2
+        ctx2 = ops.RowContext(ctx1.plan, True, True)
+        put(f"routed experts + update, {tag}", f"routed experts of the closest model + update, {tag}",
+            lambda: ops.add_norm_rows(ops.Update(ops.moe(d16, w1, c, True)), res, rn, torch.bfloat16, conv=cv, ctx=ctx2), nb, fl)
+        put(f"routed experts of the closest model + update, {tag}", "", lambda: ops.add_rmsnorm(ops.moe(d16, w1, c2, tag == "decode"), res, one, 1e-6),
+            nb, fl)
+        del w1
+    return fig.done()
+
+
 DESIGNS = {
     "vabunex": (vabunex_config, closest_config, vabunex_kernels, SIZES,
                 "KDA + latent attention (GLM-style layer types), sequential pre-norm blocks, dense feed-forward, bf16"),
@@ -430,6 +522,8 @@ DESIGNS = {
                 "grouped-query attention (rotary, whole context), softmax-routed SwiGLU experts of as many parameters, bf16"),
     "zapolorn": (zapolorn_config, zapolorn_closest, zapolorn_kernels, ZAP_SIZES,
                  "grouped-query attention (rotary, whole context), dense and softmax-routed SwiGLU feed-forwards of its sizes, bf16"),
+    "zakusun": (zakusun_config, zakusun_closest, zakusun_kernels, ZAK_SIZES,
+                "latent attention (low-rank queries, a rotated part, absorbed prompts), softmax-routed SwiGLU experts of its sizes, bf16"),
 }
 
 
