@@ -47,7 +47,8 @@ template <int N, typename T> __device__ __forceinline__ void stc(T* p, const Ch<
 }
 
 // grid (tiles, segments); whole warps, N channels per thread and step.  WIDE: groups are multiples of a warp's 128 channels.
-// Shared memory: [taps - 1][H] ring | [H] row | WIDE: [2][H / 128] partial sums, else [H / N] squares and [groups] factors.
+// Shared memory: [taps - 1][H] ring | [H] row | WIDE: [2][H / 128] partial sums, [H / 128] first piece of a piece's group; else
+// [H / N] squares and [groups] factors.
 template <typename T, int N, bool WIDE>
 __global__ void __launch_bounds__(1024)
 row_tiles_kernel(const __grid_constant__ RowTiles a) {
@@ -62,8 +63,14 @@ row_tiles_kernel(const __grid_constant__ RowTiles a) {
   float* ring = sm;
   float* xs = ring + static_cast<size_t>(past) * H;
   float* red = xs + H;
+  int* first = reinterpret_cast<int*>(red + 2 * (H >> 7));    // WIDE
+  if (WIDE) {
+    const int per = (H / a.groups) >> 7;
+    for (int c = t; c < H >> 7; c += nt) first[c] = c / per * per;      // (read behind the first row's barrier)
+  }
   const size_t plane = static_cast<size_t>(a.R) * H;
   const int gs = H / a.groups;
+  const float inv_gs = 1.f / gs;
   const bool has = a.u.delta != nullptr || a.u.y != nullptr;
   const float one = a.u.one_plus ? 1.f : 0.f;
   T* out = static_cast<T*>(a.u.out);
@@ -164,7 +171,7 @@ row_tiles_kernel(const __grid_constant__ RowTiles a) {
           float s = 0.f;
           for (int c = lane; c < gs / N; c += 32) s += part[g * (gs / N) + c];
           s = warp_sum(s);
-          if (lane == 0) fac[g] = 1.f / sqrtf(s / gs + a.u.eps);
+          if (lane == 0) fac[g] = rsqrtf(s * inv_gs + a.u.eps);
         }
         __syncthreads();
       }
@@ -174,10 +181,10 @@ row_tiles_kernel(const __grid_constant__ RowTiles a) {
       if (a.u.norm) {
         float rs;
         if (WIDE) {                                           // a warp's channels are of one group
-          const int g = i / gs;
+          const int c0 = first[i >> 7];
           float s = 0.f;
-          for (int c = lane; c < gs >> 7; c += 32) s += part[g * (gs >> 7) + c];
-          rs = 1.f / sqrtf(warp_sum(s) / gs + a.u.eps);
+          for (int c = lane; c < gs >> 7; c += 32) s += part[c0 + c];
+          rs = rsqrtf(warp_sum(s) * inv_gs + a.u.eps);
         } else rs = fac[i / gs];
         const Ch<N> w = ldc<N>(a.u.w + i);
 #pragma unroll
@@ -286,7 +293,7 @@ extern "C" int spark_row_tiles(const RowTiles* p, int nseg, int max_rows, int th
                        reinterpret_cast<uintptr_t>(a.tail) | reinterpret_cast<uintptr_t>(a.rows);
   const int gs = H / a.groups, n = (al & 15) == 0 && (gs & 3) == 0 ? 4 : 1;
   const bool wide = n == 4 && (gs & 127) == 0;
-  const int red = wide ? 2 * (H / 128) : H / n + a.groups;
+  const int red = wide ? 3 * (H / 128) : H / n + a.groups;
   const size_t smem = (static_cast<size_t>(past + 1) * H + red) * 4;
   if (smem > RT_SMEM) return -6;
   const int want = (H / n + 31) / 32 * 32, most = threads < 32 ? 32 : (threads > 1024 ? 1024 : threads / 32 * 32);

@@ -88,12 +88,18 @@ def add_norm_rows(delta, res, norm, dtype, want_f32=False, conv=None, ctx=None):
     return h, res, h32
 
 
-TILE_THREADS = 1024          # threads of a CTA at most
-TILE_CTAS = 592              # CTAs a launch aims at: rows per tile grow beyond
+TILE_THREADS = 512           # threads of a CTA at most
+SM_THREADS = 1024            # resident threads per SM (registers); a launch of many rows is one wave of tiles
+
+
+def tile_rows(R: int, H: int, taps: int) -> int:
+    """Rows per CTA of the tiled row update: tiles cover the rows before them anew, so they are as long as one wave allows."""
+    threads = min(TILE_THREADS, -(-H // 128) * 32)
+    return max(1, taps - 1, -(-R // (148 * (SM_THREADS // threads))))
 
 
 def _row_tiles(u, R, new, norm, depth, conv, ctx, f32):
-    a = RowTiles(u=u, res_out=P(new), groups=norm.groups if norm is not None else 1, R=R, tile=max(1, -(-R // TILE_CTAS)), commit=1)
+    a = RowTiles(u=u, res_out=P(new), groups=norm.groups if norm is not None else 1, R=R, tile=tile_rows(R, u.H, 0), commit=1)
     nseg, longest = 1, R
     if depth is not None:
         assert depth.stack.is_contiguous() and depth.stack.shape[1] == R and depth.stack.dtype == torch.float32
@@ -105,7 +111,7 @@ def _row_tiles(u, R, new, norm, depth, conv, ctx, f32):
             cu._check_slots("row_tiles", plan, conv.tail.shape[0])
         nseg, longest = len(plan.segs), max(s.n for s in plan.segs)
         a.conv_w, a.tail, a.segs, a.taps, a.commit = P(conv.w), P(conv.tail), P(d["seg"]), conv.taps, int(ctx.commit)
-        a.tile = max(a.tile, conv.taps - 1)
+        a.tile = tile_rows(R, u.H, conv.taps)
         rows = None
         if not ctx.commit:
             rows = torch.empty(R, u.H, dtype=torch.float32, device=conv.tail.device)
