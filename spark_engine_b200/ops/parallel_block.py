@@ -88,13 +88,17 @@ def add_norm_rows(delta, res, norm, dtype, want_f32=False, conv=None, ctx=None):
     return h, res, h32
 
 
-TILE_THREADS = 512           # threads of a CTA at most
 SM_THREADS = 1024            # resident threads per SM (registers); a launch of many rows is one wave of tiles
+
+
+def tile_threads(R: int) -> int:
+    """Threads of a CTA at most (a row's bits do not depend on it): few rows are one step of the whole CTA."""
+    return 1024 if R <= 148 else 512
 
 
 def tile_rows(R: int, H: int, taps: int) -> int:
     """Rows per CTA of the tiled row update: tiles cover the rows before them anew, so they are as long as one wave allows."""
-    threads = min(TILE_THREADS, -(-H // 128) * 32)
+    threads = min(tile_threads(R), -(-H // 128) * 32)
     return max(1, taps - 1, -(-R // (148 * (SM_THREADS // threads))))
 
 
@@ -117,7 +121,7 @@ def _row_tiles(u, R, new, norm, depth, conv, ctx, f32):
             rows = torch.empty(R, u.H, dtype=torch.float32, device=conv.tail.device)
             a.rows = P(rows)
         conv.keep(rows, plan, ctx.commit)
-    check(lib().spark_row_tiles(C.byref(a), nseg, longest, TILE_THREADS, f32, stream()), "spark_row_tiles")
+    check(lib().spark_row_tiles(C.byref(a), nseg, longest, tile_threads(R), f32, stream()), "spark_row_tiles")
 
 
 def advance_tail(tail, rows, plan, n_rows):
