@@ -126,7 +126,7 @@ def row_case(H, taps, groups, k, R, seed=0):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,groups", [(192, 2), (256, 2), (2048, 2), (72, 3), (75, 5), (50, 2), (1024, 1), (4608, 3), (640, 5), (24, 24)])
+@pytest.mark.parametrize("H,groups", [(320, 2), (256, 2), (2048, 2), (72, 3), (75, 5), (50, 2), (1024, 1), (4608, 3), (640, 5), (24, 24)])
 @pytest.mark.parametrize("taps", [1, 2, 4, 7])
 def test_row_updates(H, groups, taps, dtype):
     """Update, depth average, grouped norm and convolution of several sequences in one launch; a sequence in portions down to one
